@@ -63,6 +63,8 @@ class LayerSpec:
     token_input: Optional[PartSpec] = None      # a sublayer that reads the token ids again (arrangements that take one)
     out_norm: Optional[PartSpec] = None         # a norm on every sublayer's output before it joins the stream (arrangements that take one)
     layer_scale: bool = False                   # a learned vector per sublayer multiplies what joins the stream
+    residual_scale: float = 1.0                 # a constant on what joins the stream (arrangements that take one)
+    input_conv: int = 0                         # taps of a causal convolution on what the mixer reads (arrangements that take one)
 
     def name_of(self, role: str) -> str:
         for key, value in self.names:

@@ -438,7 +438,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                                         v_lane, v_xor, m_row, l_row, o,
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min(lane >> 2, group - 1)) * (fused.score_bias_last + 1),
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min((lane >> 2) + 8, group - 1)) * (fused.score_bias_last + 1),
-                                        fused.score_bias_last);
+                                        fused.score_bias_last, fused.softcap);
       __syncwarp();                                  // every lane is done with this slot: refill it
       if (edge) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       if (requested < tiles) {
@@ -814,19 +814,21 @@ VOSTI_API int vosti_attention_decode(const void* q, const void* k_cache, const v
 }
 
 // The same with a distance bias (float32 [nq][bias_last + 1], base-2 units, by min(distance,
-// bias_last); or null) added to the scaled scores and a sink logit per head (float32 [nq], natural
-// units; or null) in the denominator: see attention_sink.cu for their meaning.
+// bias_last); or null) added to the scaled scores, a sink logit per head (float32 [nq], natural
+// units; or null) in the denominator and a soft cap on the scores (natural units; 0: none): see attention_sink.cu for their meaning.
 VOSTI_API int vosti_attention_decode_biased(const void* q, const void* k_cache, const void* v_cache, void* out, float* scratch,
                                             int64_t scratch_elems, int* arrivals, const int* token_list, int count,
                                             int tokens_total, const int* positions, const int* request_of,
                                             const int* block_table, int max_pages, int page_size, int num_pages, int nq,
                                             int nkv, int d, int max_kv_len, float scale, int window, const float* bias,
-                                            int bias_last, const float* sink, unsigned* status, cudaStream_t stream) {
+                                            int bias_last, const float* sink, float softcap, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(bias == nullptr || bias_last >= 0, "attention_decode: bad bias table");
+  VOSTI_REQUIRE(softcap >= 0.f, "attention_decode: the soft cap is positive, or 0 for none");
   FusedProjection extras = {};
   extras.score_bias = bias;
   extras.score_bias_last = bias_last;
   extras.sink = sink;
+  extras.softcap = softcap * LOG2E;
   return launch_decode(q, k_cache, v_cache, out, scratch, scratch_elems, arrivals, token_list, count, tokens_total, positions,
                        request_of, block_table, max_pages, page_size, num_pages, nq, nkv, d, max_kv_len, scale, window,
                        status, stream, extras);

@@ -134,8 +134,9 @@ __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint
                                             float scale_log2, bool upper_rows_live, uint32_t k_lane, uint32_t k_xor,
                                             uint32_t v_lane, uint32_t v_xor, float (&m_row)[2], float (&l_row)[2],
                                             float (&o)[DMAX / 8][4], const float* __restrict__ bias0 = nullptr,
-                                            const float* __restrict__ bias1 = nullptr, int bias_last = 0) {
-  // bias0 / bias1 (or null): the rows of a distance-bias table (base-2 units) of this lane's two
+                                            const float* __restrict__ bias1 = nullptr, int bias_last = 0,
+                                            float softcap = 0.f) {
+  // softcap (base-2 units; 0: none) caps the scaled score; bias0 / bias1 (or null): the rows of a distance-bias table (base-2 units) of this lane's two
   // query heads, indexed by min(pos - key, bias_last) and added to the scaled score
   const int lane = threadIdx.x & 31;
   // ---- S = Q K^T for 16 keys: two 8-key column tiles
@@ -164,7 +165,11 @@ __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint
     for (int e = 0; e < 4; ++e) {
       const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
       const bool visible = key >= kstart && key <= pos;
-      if (bias0 != nullptr) {
+      if (softcap > 0.f) {
+        s[nt][e] = soft_capped(s[nt][e] * scale_log2, softcap, 2.f * LOG2E / softcap);
+        if (bias0 != nullptr) s[nt][e] += ((e >> 1) ? bias1 : bias0)[min(max(pos - key, 0), bias_last)];
+        if (!visible) s[nt][e] = -INFINITY;
+      } else if (bias0 != nullptr) {
         const int back = min(max(pos - key, 0), bias_last);
         s[nt][e] = visible ? fmaf(s[nt][e], scale_log2, (e >> 1) ? bias1[back] : bias0[back]) : -INFINITY;
       } else
@@ -231,6 +236,7 @@ struct FusedProjection {
   const float* score_bias;     // [nq][score_bias_last + 1] float32, base-2 units, by min(distance, last)
   int score_bias_last;
   const float* sink;           // [nq] float32, natural units: a logit in the denominator without key or value
+  float softcap;               // base-2 units: the scaled scores' soft cap
 };
 
 constexpr int ONCE_MAX_SEGMENTS = 16;     // CTAs per cluster of that kernel (above 8 it opts in to non-portable sizes)

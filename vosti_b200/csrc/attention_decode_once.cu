@@ -327,7 +327,7 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
                                         v_lane, v_xor, m_row, l_row, o,
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min(lane >> 2, group - 1)) * (fused.score_bias_last + 1),
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min((lane >> 2) + 8, group - 1)) * (fused.score_bias_last + 1),
-                                        fused.score_bias_last);
+                                        fused.score_bias_last, fused.softcap);
       __syncwarp();                                    // every lane is done with this slot: refill it
       if (edge) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       if (requested < tiles) request_tile();

@@ -16,14 +16,19 @@
 //                   every query head (the last `rot` elements of a head) is turned and written
 //                   behind the place of the query's latent form; the first `rank` elements of the
 //                   down projection are divided by their root mean square, weighted and stored as
-//                   c; the last `rot`, turned, as r; the gates pass a sigmoid.
-//   head_project    y[t, h, :] = g[t, h] * (x[t, h, :] @ M_h), M_h a strided view, on the CUDA cores.
+//                   c; the last `rot`, turned, as r; per-head gates, if any, pass a sigmoid. A layer
+//                   that reads another layer's latents has no down projection: only queries are turned.
+//   head_project    y[t, h, :] = g[t, h] * (x[t, h, :] @ M_h), M_h a strided view, on the CUDA cores; or
+//                   with a gate per element, sigmoid(z[t, h, :]) times the product.
 //   latent_attend   one warp per (token, head), 32 keys at a time aligned to the absolute key index
 //                   (a row's arithmetic does not depend on the cut or the batch); with few rows the
-//                   keys are cut into segments and merged in order by latent_merge.
-// Rotation: element i of the rotated part pairs with i + rot/2, angle = position * freq[i] in
-// float32, cos and sin multiplied by `magnitude`.
+//                   keys are cut into segments and merged in order by latent_merge. Under a window a
+//                   row's segments are counted from the one that holds its first key. A sink (one logit
+//                   per head) joins the denominator once, at the end or at the merge.
+// Rotation: element i of the rotated part pairs with i + rot/2 (or 2i with 2i + 1), angle = position *
+// freq[i] in float32, cos and sin multiplied by `magnitude`.
 #include "common.cuh"
+#include "latent.cuh"
 
 namespace {
 constexpr int WARPS = 16;            // warps of a block: the heads of one token share their keys through L1
@@ -34,7 +39,8 @@ __global__ void __launch_bounds__(256)
 latent_prep_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __restrict__ qk, float* __restrict__ gate,
                    T* __restrict__ c_cache, T* __restrict__ r_cache, const void* __restrict__ norm_w, int norm_f32, float eps,
                    const int* __restrict__ positions, const int* __restrict__ slot_mapping, int64_t num_slots, int heads,
-                   int dim, int rot, int rank, const float* __restrict__ freq, float magnitude, unsigned* status) {
+                   int dim, int rot, int rank, const float* __restrict__ freq, int interleaved, float magnitude,
+                   unsigned* status) {
   extern __shared__ float turn[];            // [rot]: cosines, then sines
   __shared__ float scratch[32];
   pdl_wait();
@@ -50,6 +56,10 @@ latent_prep_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __restric
   __syncthreads();
   auto turned = [&](const T* src, int i) {          // element i of a rotated part that starts at src
     const float x = to_f32(src[i]);
+    if (interleaved) {
+      const int pair = i >> 1;
+      return (i & 1) == 0 ? x * turn[pair] - to_f32(src[i + 1]) * turn[half + pair] : x * turn[pair] + to_f32(src[i - 1]) * turn[half + pair];
+    }
     if (i < half) return x * turn[i] - to_f32(src[i + half]) * turn[half + i];
     return x * turn[i - half] + to_f32(src[i - half]) * turn[i];
   };
@@ -60,7 +70,8 @@ latent_prep_kernel(const T* __restrict__ proj, int64_t proj_stride, T* __restric
   }
   const T* down = row + heads * qw;
   const T* graw = down + kw;
-  for (int i = threadIdx.x; i < heads; i += blockDim.x) gate[(int64_t)t * heads + i] = 1.f / (1.f + expf(-to_f32(graw[i])));
+  if (gate != nullptr)
+    for (int i = threadIdx.x; i < heads; i += blockDim.x) gate[(int64_t)t * heads + i] = 1.f / (1.f + expf(-to_f32(graw[i])));
   if (c_cache == nullptr) return;
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
@@ -85,7 +96,7 @@ constexpr int HP_TOKENS = 16, HP_OUT = 128, HP_IN = 32;
 template <typename TX, typename TM, typename TY>
 __global__ void __launch_bounds__(HP_OUT)
 head_project_kernel(const TX* __restrict__ x, int64_t x_row, int64_t x_head, const TM* __restrict__ m, int64_t m_head,
-                    int64_t m_in, int64_t m_out, const float* __restrict__ gate, TY* __restrict__ y, int64_t y_row,
+                    int64_t m_in, int64_t m_out, const HeadGate gate, TY* __restrict__ y, int64_t y_row,
                     int64_t y_head, int tokens, int heads, int in, int out) {
   __shared__ float xs[HP_TOKENS][HP_IN];
   __shared__ float ms[HP_IN][HP_OUT + 1];
@@ -126,7 +137,7 @@ head_project_kernel(const TX* __restrict__ x, int64_t x_row, int64_t x_head, con
 #pragma unroll
   for (int u = 0; u < HP_TOKENS; ++u) {
     if (t0 + u >= tokens) break;
-    const float g = gate != nullptr ? gate[(int64_t)(t0 + u) * heads + h] : 1.f;
+    const float g = gate.at(t0 + u, h, o0 + tid, heads, out);
     y[(int64_t)(t0 + u) * y_row + (int64_t)h * y_head + o0 + tid] = from_f32<TY>(acc[u] * g);
   }
 }
@@ -175,7 +186,7 @@ latent_attend_kernel(const T* __restrict__ qk, const T* __restrict__ c_cache, co
                      float* __restrict__ out, const int* __restrict__ positions, const int* __restrict__ request_of,
                      const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
                      const int* __restrict__ token_list, int tokens, int heads, int rank, int rot, float scale_log2,
-                     int window, float* __restrict__ partial, int segment, unsigned* status) {
+                     int window, const float* __restrict__ sink, float* __restrict__ partial, int segment, unsigned* status) {
   extern __shared__ float q_smem[];
   pdl_wait();
   pdl_launch_dependents();
@@ -194,8 +205,9 @@ latent_attend_kernel(const T* __restrict__ qk, const T* __restrict__ c_cache, co
   int kstart = first_visible_key(pos, window);
   int kend = pos;                                   // inclusive
   if (partial != nullptr) {                         // this warp's segment of the keys (a multiple of 32)
-    kstart = max(kstart, (int)blockIdx.y * segment);
-    kend = min(kend, (int)(blockIdx.y + 1) * segment - 1);
+    const int seg = (window > 0 ? kstart / segment : 0) + (int)blockIdx.y;
+    kstart = max(kstart, seg * segment);
+    kend = min(kend, (seg + 1) * segment - 1);
   }
   const int* table = block_table + (int64_t)b * max_pages;
   float m = -INFINITY, l = 0.f;
@@ -263,7 +275,7 @@ latent_attend_kernel(const T* __restrict__ qk, const T* __restrict__ c_cache, co
     }
     return;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = sink_inverse(m, l, sink != nullptr ? sink[h] * LOG2E : -INFINITY);
   float* orow = out + ((int64_t)t * heads + h) * rank;
 #pragma unroll
   for (int i = 0; i < RW; ++i) {
@@ -280,7 +292,7 @@ latent_attend_kernel(const T* __restrict__ qk, const T* __restrict__ c_cache, co
 template <int MERGE_SLICE>
 __global__ void __launch_bounds__(WARPS * 32)
 latent_merge_kernel(const float* __restrict__ partial, int segments, float* __restrict__ out,
-                    const int* __restrict__ token_list, int tokens, int heads, int rank) {
+                    const int* __restrict__ token_list, int tokens, int heads, int rank, const float* __restrict__ sink) {
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -322,7 +334,7 @@ latent_merge_kernel(const float* __restrict__ partial, int segments, float* __re
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = sink_inverse(top, l, sink != nullptr ? sink[h] * LOG2E : -INFINITY);
   float* orow = out + ((int64_t)t * heads + h) * rank;
 #pragma unroll
   for (int i = 0; i < MERGE_SLICE / 32; ++i) {
@@ -332,67 +344,73 @@ latent_merge_kernel(const float* __restrict__ partial, int segments, float* __re
 }
 
 void launch_merge(int64_t blocks, cudaStream_t stream, const float* partial, int segments, float* out, const int* token_list,
-                  int tokens, int heads, int rank) {
+                  int tokens, int heads, int rank, const float* sink) {
   if (blocks * ((rank + 127) / 128) >= 2 * 148)
     vosti_launch(latent_merge_kernel<128>, dim3((unsigned)blocks, (rank + 127) / 128), dim3(WARPS * 32), 0, stream, partial,
-                 segments, out, token_list, tokens, heads, rank);
+                 segments, out, token_list, tokens, heads, rank, sink);
   else
     vosti_launch(latent_merge_kernel<32>, dim3((unsigned)blocks, (rank + 31) / 32), dim3(WARPS * 32), 0, stream, partial,
-                 segments, out, token_list, tokens, heads, rank);
+                 segments, out, token_list, tokens, heads, rank, sink);
 }
 
 template <typename T, int RW>
 void launch_attend(dim3 grid, size_t smem, cudaStream_t stream, const void* qk, const void* c_cache, const void* r_cache,
                    float* out, const int* positions, const int* request_of, const int* block_table, int max_pages,
                    int page_size, int num_pages, const int* token_list, int tokens, int heads, int rank, int rot,
-                   float scale_log2, int window, float* partial, int segment, unsigned* status) {
+                   float scale_log2, int window, const float* sink, float* partial, int segment, unsigned* status) {
   vosti_launch(latent_attend_kernel<T, RW>, grid, dim3(WARPS * 32), smem, stream, (const T*)qk, (const T*)c_cache,
                (const T*)r_cache, out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list,
-               tokens, heads, rank, rot, scale_log2, window, partial, segment, status);
+               tokens, heads, rank, rot, scale_log2, window, sink, partial, segment, status);
 }
 
 }  // namespace
 
 constexpr int LATENT_MAX_RANK = 1024;
 
-// proj [tokens, heads * (dim + rot) + rank + rot + heads] = q | down | gate; qk [tokens, heads, rank + rot]
-// (the last rot columns of every head are written); gate float32 [tokens, heads]; caches
+// proj rows (proj_stride elements apart) start with heads * (dim + rot) query elements, then `down` (rank + rot), then a
+// gate per head; the last two are read only where c_cache and `gate` are given. qk [tokens, heads, rank + rot]
+// (the last rot columns of every head are written); gate float32 [tokens, heads] or null; caches
 // [pages, 1, page_size, rank | rot] or null (a run that reads another layer's cache).
-VOSTI_API int vosti_latent_prep(const void* proj, void* qk, float* gate, void* c_cache, void* r_cache, const void* norm_w,
+VOSTI_API int vosti_latent_prep(const void* proj, int64_t proj_stride, void* qk, float* gate, void* c_cache, void* r_cache, const void* norm_w,
                                 int norm_f32, float eps, const int* positions, const int* slot_mapping, int64_t num_slots,
-                                int tokens, int heads, int dim, int rot, int rank, const float* freq, float magnitude,
+                                int tokens, int heads, int dim, int rot, int rank, const float* freq, int interleaved, float magnitude,
                                 int is_f32, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && heads > 0 && dim > 0 && rank > 0 && rot >= 0 && rot % 2 == 0, "latent_prep: bad sizes");
   VOSTI_REQUIRE(rot == 0 || freq != nullptr, "latent_prep: a rotation needs frequencies");
   VOSTI_REQUIRE(c_cache == nullptr || (r_cache != nullptr && slot_mapping != nullptr && norm_w != nullptr), "latent_prep: a cache needs slots and the norm's weight");
   if (tokens == 0) return VOSTI_OK;
-  const int64_t stride = (int64_t)heads * (dim + rot) + rank + rot + heads;
+  VOSTI_REQUIRE(proj_stride >= (int64_t)heads * (dim + rot) + (c_cache != nullptr || gate != nullptr ? rank + rot : 0) + (gate != nullptr ? heads : 0),
+                "latent_prep: the projection's rows are too narrow");
   const size_t smem = (size_t)(rot > 0 ? rot : 1) * sizeof(float);
   if (is_f32)
-    vosti_launch(latent_prep_kernel<float>, dim3(tokens), dim3(256), smem, stream, (const float*)proj, stride, (float*)qk, gate,
+    vosti_launch(latent_prep_kernel<float>, dim3(tokens), dim3(256), smem, stream, (const float*)proj, proj_stride, (float*)qk, gate,
                  (float*)c_cache, (float*)r_cache, norm_w, norm_f32, eps, positions, slot_mapping, num_slots, heads, dim, rot, rank,
-                 freq, magnitude, status);
+                 freq, interleaved, magnitude, status);
   else
-    vosti_launch(latent_prep_kernel<bf16>, dim3(tokens), dim3(256), smem, stream, (const bf16*)proj, stride, (bf16*)qk, gate,
+    vosti_launch(latent_prep_kernel<bf16>, dim3(tokens), dim3(256), smem, stream, (const bf16*)proj, proj_stride, (bf16*)qk, gate,
                  (bf16*)c_cache, (bf16*)r_cache, norm_w, norm_f32, eps, positions, slot_mapping, num_slots, heads, dim, rot, rank,
-                 freq, magnitude, status);
+                 freq, interleaved, magnitude, status);
   VOSTI_LAUNCH_CHECK();
 }
 
-// y[t, h, o] = gate[t, h] * sum_i x[t, h, i] * m[h * m_head + i * m_in + o * m_out]; strides in elements.
+// y[t, h, o] = gate[t, h] * sum_i x[t, h, i] * m[h * m_head + i * m_in + o * m_out]; strides in elements. Instead of
+// `gate`, `element_gate` (float32 or bfloat16, rows of at least heads * out elements element_gate_row apart) multiplies
+// by sigmoid(element_gate[t, h * out + o]).
 // Types: x and y float32 or bfloat16 (x_f32, y_f32), m float32 or bfloat16 (m_f32).
 VOSTI_API int vosti_head_project(const void* x, int x_f32, int64_t x_row, int64_t x_head, const void* m, int m_f32,
-                                 int64_t m_head, int64_t m_in, int64_t m_out, const float* gate, void* y, int y_f32,
+                                 int64_t m_head, int64_t m_in, int64_t m_out, const float* gate, const void* element_gate,
+                                 int element_gate_f32, int64_t element_gate_row, void* y, int y_f32,
                                  int64_t y_row, int64_t y_head, int tokens, int heads, int in, int out,
                                  cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && heads > 0 && heads <= 65535 && in > 0 && out > 0, "head_project: bad sizes");
+  VOSTI_REQUIRE(element_gate == nullptr || (gate == nullptr && element_gate_row >= (int64_t)heads * out), "head_project: one gate, with whole rows");
   if (tokens == 0) return VOSTI_OK;
   const int token_tiles = (tokens + HP_TOKENS - 1) / HP_TOKENS;
   VOSTI_REQUIRE(token_tiles <= 65535, "head_project: too many tokens for one launch");
   const dim3 grid((out + HP_OUT - 1) / HP_OUT, heads, token_tiles), block(HP_OUT);
 #define VOSTI_HP(TX, TM, TY)                                                                                          \
   vosti_launch(head_project_kernel<TX, TM, TY>, grid, block, 0, stream, (const TX*)x, x_row, x_head, (const TM*)m, m_head, \
-               m_in, m_out, gate, (TY*)y, y_row, y_head, tokens, heads, in, out)
+               m_in, m_out, HeadGate{gate, element_gate, element_gate_f32, element_gate_row}, (TY*)y, y_row, y_head, tokens, heads, in, out)
   if (x_f32 && m_f32 && y_f32) VOSTI_HP(float, float, float);
   else if (x_f32 && !m_f32 && y_f32) VOSTI_HP(float, bf16, float);
   else if (x_f32 && !m_f32 && !y_f32) VOSTI_HP(float, bf16, bf16);
@@ -410,12 +428,13 @@ VOSTI_API int vosti_head_project(const void* x, int x_f32, int64_t x_row, int64_
 // qk [rows, heads, rank + rot]; caches [pages, 1, page_size, rank | rot]; out float32 [rows, heads, rank].
 // `token_list` (or null: all) names the `tokens` rows to compute. With `segments` > 1 the keys
 // are cut into pieces of `segment` keys (a multiple of 32) and `scratch` holds
-// tokens * heads * segments * (rank + 2) floats.
+// tokens * heads * segments * (rank + 2) floats; with a window a row's pieces are counted from the one that
+// holds its first key. `sink` float32 [heads] in natural units, or null.
 VOSTI_API int vosti_latent_attend(const void* qk, const void* c_cache, const void* r_cache, float* out, const int* positions,
                                   const int* request_of, const int* block_table, int max_pages, int page_size,
                                   int num_pages, const int* token_list, int tokens, int heads, int rank, int rot,
-                                  float scale, int window, float* scratch, int segment, int segments, int is_f32,
-                                  unsigned* status, cudaStream_t stream) {
+                                  float scale, int window, const float* sink, float* scratch, int segment, int segments,
+                                  int is_f32, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && heads > 0 && rank > 0 && rank <= LATENT_MAX_RANK && rot >= 0,
                 "latent_attend: bad sizes heads=%d rank=%d (at most %d) rot=%d", heads, rank, LATENT_MAX_RANK, rot);
   VOSTI_REQUIRE(page_size > 0 && max_pages > 0 && num_pages > 0, "latent_attend: bad cache geometry");
@@ -445,15 +464,15 @@ VOSTI_API int vosti_latent_attend(const void* qk, const void* c_cache, const voi
     if (is_f32)                                                                                                         \
       launch_attend<float, RW>(grid, smem, stream, qk, c_cache, r_cache, out, positions, request_of, block_table,       \
                                max_pages, page_size, num_pages, token_list, tokens, heads, rank, rot, scale * LOG2E,    \
-                               window, partial, segment, status);                                                       \
+                               window, sink, partial, segment, status);                                                 \
     else                                                                                                                \
       launch_attend<bf16, RW>(grid, smem, stream, qk, c_cache, r_cache, out, positions, request_of, block_table,        \
                               max_pages, page_size, num_pages, token_list, tokens, heads, rank, rot, scale * LOG2E,     \
-                              window, partial, segment, status);                                                        \
+                              window, sink, partial, segment, status);                                                  \
     if (segments > 1) {                                                                                                 \
       cudaError_t e = cudaGetLastError();                                                                               \
       if (e != cudaSuccess) { vosti_set_error("%s", cudaGetErrorString(e)); return (int)e; }                            \
-      launch_merge(blocks, stream, partial, segments, out, token_list, tokens, heads, rank);                           \
+      launch_merge(blocks, stream, partial, segments, out, token_list, tokens, heads, rank, sink);                     \
     }                                                                                                                   \
   } while (0)
   if (rw == 4) VOSTI_LA(4);
@@ -467,12 +486,12 @@ VOSTI_API int vosti_latent_attend(const void* qk, const void* c_cache, const voi
 // The merge alone, for a kernel that left the (m, l, sum) records itself: partial float32
 // [tokens * heads, segments, rank + 2]; out float32 [tokens, heads, rank].
 VOSTI_API int vosti_latent_merge(const float* partial, int segments, float* out, int tokens, int heads, int rank,
-                                 cudaStream_t stream) {
+                                 const float* sink, cudaStream_t stream) {
   VOSTI_REQUIRE(partial != nullptr && segments >= 1 && tokens >= 0 && heads > 0 && rank > 0 && rank <= LATENT_MAX_RANK,
                 "latent_merge: bad sizes");
   if (tokens == 0) return VOSTI_OK;
   const int64_t blocks = ((int64_t)tokens * heads + WARPS - 1) / WARPS;
   VOSTI_REQUIRE(blocks <= 0x7fffffffLL, "latent_merge: too many (token, head) pairs");
-  launch_merge(blocks, stream, partial, segments, out, nullptr, tokens, heads, rank);
+  launch_merge(blocks, stream, partial, segments, out, nullptr, tokens, heads, rank, sink);
   VOSTI_LAUNCH_CHECK();
 }

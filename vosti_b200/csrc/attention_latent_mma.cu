@@ -15,10 +15,13 @@
 //            O += (P_hi + P_lo) C, the tile's first `rank` columns read transposed by ldmatrix
 //
 // With few rows (decode steps) the keys are cut into segments over grid.z and every (row,
-// segment) leaves (m, l, unnormalised sum) for latent_merge_kernel, like the CUDA-core kernel.
+// segment) leaves (m, l, unnormalised sum) for latent_merge_kernel, like the CUDA-core kernel. Under a
+// window a CTA's segments are counted from the one that holds its rows' first key. A sink (one logit per
+// head) joins a row's denominator once, at the end or at the merge.
 // Sizes: rank 128, 256 or 512; rot a multiple of 32; bfloat16 only. Everything else takes the
 // CUDA-core kernel.
 #include "common.cuh"
+#include "latent.cuh"
 #include "mma_util.cuh"
 
 namespace {
@@ -33,8 +36,8 @@ __global__ void __launch_bounds__(LW * HALVES * 32, 1)
 latent_attend_mma_kernel(const bf16* __restrict__ qk, const bf16* __restrict__ c_cache, const bf16* __restrict__ r_cache,
                          float* __restrict__ out, const int* __restrict__ positions, const int* __restrict__ cu_q,
                          const int* __restrict__ block_table, int max_pages, int page_size, int num_pages, int heads,
-                         int rot, float scale_log2, int window, float* __restrict__ partial, int segment,
-                         unsigned* status) {
+                         int rot, float scale_log2, int window, const float* __restrict__ sink, float* __restrict__ partial,
+                         int segment, unsigned* status) {
   extern __shared__ __align__(16) uint8_t smem[];
   pdl_wait();
   pdl_launch_dependents();
@@ -78,8 +81,9 @@ latent_attend_mma_kernel(const bf16* __restrict__ qk, const bf16* __restrict__ c
   const int pos_lo = positions[q_start + token_lo], pos_hi = positions[q_start + token_hi];
   int first_key = first_visible_key(pos_lo, window), key_end = pos_hi + 1;   // [first_key, key_end)
   if (partial != nullptr) {
-    first_key = max(first_key, (int)blockIdx.z * segment);
-    key_end = min(key_end, (int)(blockIdx.z + 1) * segment);
+    const int seg = (window > 0 ? first_key / segment : 0) + (int)blockIdx.z;
+    first_key = max(first_key, seg * segment);
+    key_end = min(key_end, (seg + 1) * segment);
   }
   const int segments = gridDim.z;
   if (first_key >= key_end) {                    // nothing of this segment is visible: empty records
@@ -298,7 +302,7 @@ latent_attend_mma_kernel(const bf16* __restrict__ qk, const bf16* __restrict__ c
         dst = rec + 2;
       } else {
         dst = out + (first_row + row) * RANK;
-        inv = l > 0.f ? 1.f / l : 0.f;
+        inv = sink_inverse(m_row[mt][r], l, sink != nullptr ? sink[(row0 + row) % heads] * LOG2E : -INFINITY);
       }
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt)
@@ -321,7 +325,7 @@ constexpr int HPK = 64;
 template <bool XF32, bool KMAJOR, int WM, int WN, int NT, typename TY>
 __global__ void __launch_bounds__(WM * WN * 32)
 head_project_mma_kernel(const void* __restrict__ x_, int64_t x_row, int64_t x_head, const bf16* __restrict__ m,
-                        int64_t m_head, int64_t m_stride, const float* __restrict__ gate, TY* __restrict__ y,
+                        int64_t m_head, int64_t m_stride, const HeadGate gate, TY* __restrict__ y,
                         int64_t y_row, int64_t y_head, int tokens, int heads, int in, int out) {
   constexpr int THREADS = WM * WN * 32, TM = 16 * WM, TN = 8 * NT * WN;
   constexpr int A_PITCH = HPK + 8;
@@ -442,13 +446,12 @@ head_project_mma_kernel(const void* __restrict__ x_, int64_t x_row, int64_t x_he
   for (int r = 0; r < 2; ++r) {
     const int t = t0 + wm * 16 + (lane >> 2) + 8 * r;
     if (t >= tokens) continue;
-    const float g = gate != nullptr ? gate[(int64_t)t * heads + h] : 1.f;
     TY* dst = y + (int64_t)t * y_row + (int64_t)h * y_head;
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       const int o = o0 + n_warp + nt * 8 + (lane & 3) * 2;
       if (o >= out) continue;
-      store_pair(dst + o, acc[nt][2 * r] * g, acc[nt][2 * r + 1] * g);
+      store_pair(dst + o, acc[nt][2 * r] * gate.at(t, h, o, heads, out), acc[nt][2 * r + 1] * gate.at(t, h, o + 1, heads, out));
     }
   }
 }
@@ -468,11 +471,12 @@ VOSTI_API int vosti_latent_attend_mma_fits(int rank, int rot) {
 // qk bf16 [tokens, heads, rank + rot]; caches bf16 [pages, 1, page_size, rank | rot]; out float32
 // [tokens, heads, rank]. Serves requests 0 .. requests - 1 of cu_q, the longest portion having
 // max_q_len tokens. With `segments` > 1 the keys are cut into pieces of `segment` keys (a multiple
-// of 64) and `scratch` holds tokens * heads * segments * (rank + 2) floats for latent_merge.
+// of 64) and `scratch` holds tokens * heads * segments * (rank + 2) floats for latent_merge (which then
+// takes the sink, float32 [heads] in natural units or null, in this kernel's place).
 VOSTI_API int vosti_latent_attend_mma(const void* qk, const void* c_cache, const void* r_cache, float* out,
                                       const int* positions, const int* cu_q, const int* block_table, int max_pages,
                                       int page_size, int num_pages, int requests, int max_q_len, int heads, int rank,
-                                      int rot, float scale, int window, float* scratch, int segment, int segments,
+                                      int rot, float scale, int window, const float* sink, float* scratch, int segment, int segments,
                                       unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(vosti_latent_attend_mma_fits(rank, rot), "latent_attend_mma: rank %d, rot %d are not sizes this kernel takes", rank, rot);
   VOSTI_REQUIRE(requests >= 0 && requests <= 65535 && heads > 0 && max_q_len >= 0, "latent_attend_mma: bad sizes");
@@ -497,7 +501,7 @@ VOSTI_API int vosti_latent_attend_mma(const void* qk, const void* c_cache, const
     }                                                                                                                   \
     vosti_launch(latent_attend_mma_kernel<RANK, 1, HALVES>, grid, dim3(LW * HALVES * 32), smem, stream, (const bf16*)qk, \
                  (const bf16*)c_cache, (const bf16*)r_cache, out, positions, cu_q, block_table, max_pages, page_size,   \
-                 num_pages, heads, rot, scale * LOG2E, window, partial, segment, status);                               \
+                 num_pages, heads, rot, scale * LOG2E, window, sink, partial, segment, status);                               \
   } while (0)
   if (rank == 512) { if (halves == 2) VOSTI_LM(512, 2); else VOSTI_LM(512, 1); }
   else if (rank == 256) { if (halves == 2) VOSTI_LM(256, 2); else VOSTI_LM(256, 1); }
@@ -508,7 +512,7 @@ VOSTI_API int vosti_latent_attend_mma(const void* qk, const void* c_cache, const
 
 // y[t, h, o] = gate[t, h] * sum_i x[t, h, i] * m[h * m_head + i * m_in + o * m_out] with a bfloat16 m
 // whose inner or output index is contiguous (m_in == 1 or m_out == 1), on the tensor cores. The
-// caller has checked vosti_head_project_mma_fits. x and y float32 or bfloat16; strides in elements.
+// caller has checked vosti_head_project_mma_fits. `element_gate` as for vosti_head_project. x and y float32 or bfloat16; strides in elements.
 VOSTI_API int vosti_head_project_mma_fits(int64_t x_row, int64_t x_head, int x_f32, int64_t m_head, int64_t m_in,
                                           int64_t m_out, int64_t y_row, int64_t y_head, int in, int out) {
   const int xv = x_f32 ? 4 : 8;
@@ -518,7 +522,8 @@ VOSTI_API int vosti_head_project_mma_fits(int64_t x_row, int64_t x_head, int x_f
 }
 
 VOSTI_API int vosti_head_project_mma(const void* x, int x_f32, int64_t x_row, int64_t x_head, const void* m,
-                                     int64_t m_head, int64_t m_in, int64_t m_out, const float* gate, void* y, int y_f32,
+                                     int64_t m_head, int64_t m_in, int64_t m_out, const float* gate, const void* element_gate,
+                                     int element_gate_f32, int64_t element_gate_row, void* y, int y_f32,
                                      int64_t y_row, int64_t y_head, int tokens, int heads, int in, int out,
                                      cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && heads > 0 && heads <= 65535 && in > 0 && out > 0, "head_project_mma: bad sizes");
@@ -526,7 +531,9 @@ VOSTI_API int vosti_head_project_mma(const void* x, int x_f32, int64_t x_row, in
                 "head_project_mma: strides or sizes this kernel does not take");
   VOSTI_REQUIRE((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(m)) % 16 == 0 &&
                 reinterpret_cast<uintptr_t>(y) % 8 == 0, "head_project_mma: operands are not aligned");
+  VOSTI_REQUIRE(element_gate == nullptr || (gate == nullptr && element_gate_row >= (int64_t)heads * out), "head_project_mma: one gate, with whole rows");
   if (tokens == 0) return VOSTI_OK;
+  const HeadGate head_gate = {gate, element_gate, element_gate_f32, element_gate_row};
   const bool kmajor = m_in == 1;
   const int64_t m_stride = kmajor ? m_out : m_in;
   const bool few = tokens <= 16;
@@ -536,7 +543,7 @@ VOSTI_API int vosti_head_project_mma(const void* x, int x_f32, int64_t x_row, in
   const dim3 grid((out + tn - 1) / tn, heads, token_tiles);
 #define VOSTI_HPM(XF, KM, WM, WN, NT, TY)                                                                          \
   vosti_launch(head_project_mma_kernel<XF, KM, WM, WN, NT, TY>, grid, dim3(WM * WN * 32), 0, stream, x, x_row,     \
-               x_head, (const bf16*)m, m_head, m_stride, gate, (TY*)y, y_row, y_head, tokens, heads, in, out)
+               x_head, (const bf16*)m, m_head, m_stride, head_gate, (TY*)y, y_row, y_head, tokens, heads, in, out)
 #define VOSTI_HPM_SHAPE(XF, KM, TY)                                                                                \
   do {                                                                                                             \
     if (few) VOSTI_HPM(XF, KM, 1, 4, 2, TY);                                                                       \

@@ -56,7 +56,8 @@ __device__ __forceinline__ uint32_t swizzled(int row, int chunk) { return row * 
 
 // BIASED: the scaled score also gets bias[head][min(distance, bias_last)] (base-2 units; the
 // table's last column serves every larger distance, so a tile that lies wholly beyond it adds a
-// constant), and exp(sink[head]) joins the denominator once at the end (either may be null).
+// constant), and exp(sink[head]) joins the denominator once at the end (either may be null); softcap
+// (base-2 units) > 0 caps the scaled score before the bias.
 // Without BIASED the arithmetic is what it was before the flag existed, bit for bit.
 template <int D, bool BIASED>
 __global__ void __launch_bounds__(THREADS, 1)
@@ -66,7 +67,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ kv_len, const int* __restrict__ block_table, int max_pages,
                             int page_size, int page_shift, int num_pages, int nq, int nkv, float scale_log2_in,
                             int window, const float* __restrict__ bias, int bias_last,
-                            const float* __restrict__ sink, unsigned* status) {
+                            const float* __restrict__ sink, float softcap, unsigned* status) {
   const float scale_log2 = BIASED ? 1.f : scale_log2_in;      // BIASED: scores are scaled where the bias is added
   constexpr int NB = D / 64;                          // 64-element blocks of the head size
   constexpr int STAGES = kv_stages<D>();
@@ -171,18 +172,26 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&s_empty[wg]));       // the scores are in registers
-      if (BIASED && valid) {
+      if (BIASED && valid && softcap > 0.f) {
+        // the capped score; a bias, if there is one, is added to it below with a factor of one
+        const float rate = 2.f * LOG2E / softcap;
+#pragma unroll
+        for (int i = 0; i < KT; ++i)
+          raw[i >> 5][i & 31] = __float_as_uint(soft_capped(__uint_as_float(raw[i >> 5][i & 31]) * scale_log2_in, softcap, rate));
+      }
+      const float scale_here = BIASED && softcap > 0.f ? 1.f : scale_log2_in;
+      if (BIASED && valid && (softcap <= 0.f || bias_h != nullptr)) {
         const int d0 = pos - key0;                               // key i of the tile is d0 - i positions back
         if (bias_h == nullptr || d0 - (KT - 1) >= bias_last) {
           const float far = bias_h != nullptr ? bias_h[bias_last] : 0.f;
 #pragma unroll
           for (int i = 0; i < KT; ++i)
-            raw[i >> 5][i & 31] = __float_as_uint(fmaf(__uint_as_float(raw[i >> 5][i & 31]), scale_log2_in, far));
+            raw[i >> 5][i & 31] = __float_as_uint(fmaf(__uint_as_float(raw[i >> 5][i & 31]), scale_here, far));
         } else {
 #pragma unroll
           for (int i = 0; i < KT; ++i) {
             const int back = min(max(d0 - i, 0), bias_last);     // (keys ahead of the row are masked below)
-            raw[i >> 5][i & 31] = __float_as_uint(fmaf(__uint_as_float(raw[i >> 5][i & 31]), scale_log2_in, __ldg(bias_h + back)));
+            raw[i >> 5][i & 31] = __float_as_uint(fmaf(__uint_as_float(raw[i >> 5][i & 31]), scale_here, __ldg(bias_h + back)));
           }
         }
       }
@@ -442,7 +451,7 @@ int launch_prefill_tc(const void* q, const void* k_cache, const void* v_cache, v
                                          const int* row_list, int count, const int* cu_q, const int* kv_len,
                                          const int* block_table, int max_pages, int page_size, int num_pages, int nq,
                                          int nkv, int d, int max_q_len, int tokens_total, float scale, int window,
-                                         bool biased, const float* bias, int bias_last, const float* sink,
+                                         bool biased, const float* bias, int bias_last, const float* sink, float softcap,
                                          unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(count >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "attention_prefill_tc: bad head counts nq=%d nkv=%d", nq, nkv);
   VOSTI_REQUIRE(nq / nkv <= 16, "attention_prefill_tc: at most 16 query heads per kv head, got %d", nq / nkv);
@@ -480,7 +489,7 @@ int launch_prefill_tc(const void* q, const void* k_cache, const void* v_cache, v
     }                                                                                                                \
     vosti_launch(attention_prefill_tc_kernel<D, B>, grid, dim3(THREADS), prefill_tc_smem_bytes<D>(), stream, map_q,  \
         map_k, map_v, (bf16*)out, row_list, cu_q, kv_len, block_table, max_pages, page_size, page_shift, num_pages,   \
-        nq, nkv, scale * LOG2E, window, bias, bias_last, sink, status);                                               \
+        nq, nkv, scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, status);                                               \
   } while (0)
   if (biased) {
     if (d == 64) LAUNCH_PREFILL_TC(64, true);
@@ -502,20 +511,22 @@ VOSTI_API int vosti_attention_prefill_tc(const void* q, const void* k_cache, con
                                          int nkv, int d, int max_q_len, int tokens_total, float scale, int window,
                                          unsigned* status, cudaStream_t stream) {
   return launch_prefill_tc(q, k_cache, v_cache, out, row_list, count, cu_q, kv_len, block_table, max_pages, page_size,
-                           num_pages, nq, nkv, d, max_q_len, tokens_total, scale, window, false, nullptr, 0, nullptr,
+                           num_pages, nq, nkv, d, max_q_len, tokens_total, scale, window, false, nullptr, 0, nullptr, 0.f,
                            status, stream);
 }
 
-// The same with a distance bias (float32 [nq, bias_last + 1], base-2 units, or null) and a sink
-// logit per head (float32 [nq], natural units, or null): see attention_sink.cu for their meaning.
+// The same with a distance bias (float32 [nq, bias_last + 1], base-2 units, or null), a sink
+// logit per head (float32 [nq], natural units, or null) and a soft cap on the scores (natural units, 0: none):
+// see attention_sink.cu for their meaning.
 VOSTI_API int vosti_attention_prefill_tc_biased(const void* q, const void* k_cache, const void* v_cache, void* out,
                                                 const int* row_list, int count, const int* cu_q, const int* kv_len,
                                                 const int* block_table, int max_pages, int page_size, int num_pages,
                                                 int nq, int nkv, int d, int max_q_len, int tokens_total, float scale,
                                                 int window, const float* bias, int bias_last, const float* sink,
-                                                unsigned* status, cudaStream_t stream) {
+                                                float softcap, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(bias == nullptr || bias_last >= 0, "attention_prefill_tc: bad bias table");
+  VOSTI_REQUIRE(softcap >= 0.f, "attention_prefill_tc: the soft cap is positive, or 0 for none");
   return launch_prefill_tc(q, k_cache, v_cache, out, row_list, count, cu_q, kv_len, block_table, max_pages, page_size,
-                           num_pages, nq, nkv, d, max_q_len, tokens_total, scale, window, true, bias, bias_last, sink,
+                           num_pages, nq, nkv, d, max_q_len, tokens_total, scale, window, true, bias, bias_last, sink, softcap,
                            status, stream);
 }

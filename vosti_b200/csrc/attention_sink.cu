@@ -9,6 +9,7 @@
 //   * a learned bias per (distance, head) added to the scaled score. The host hands a table
 //     bias[head][min(distance, last)] (already in base-2 units): beyond `last` the bias no
 //     longer changes, so the table is as long as the distances that differ;
+//   * a soft cap c on the scaled score, c tanh(score / c), before the bias;
 //   * a sink: one more term exp(sink[head]) in the softmax denominator, with no key or value;
 //   * two score maps a head over the same values (differential attention), combined after the
 //     softmax, and a finish of the head's output: unit root mean square, a sigmoid gate (HeadFinish);
@@ -20,7 +21,8 @@
 // arithmetic for both storage types. A tile is 32 keys aligned to the absolute key index, so a
 // row's order of arithmetic depends on its position only, not on how the prompt was cut or
 // what else is in the batch. With few query rows (decoding) the keys are cut into segments of
-// a fixed length, one warp per (token, head, segment), and a second kernel merges a row's
+// a fixed length (their borders at its multiples; under a window, counted from the one that holds the
+// row's first key), one warp per (token, head, segment), and a second kernel merges a row's
 // segments in order; the sink joins at the merge. (Head sizes 64 and 128 in bfloat16 take the
 // tensor-memory kernel of attention_prefill_tc.cu for their long rows instead.)
 #include "common.cuh"
@@ -585,7 +587,7 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
                       const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
                       const int* __restrict__ token_list, int tokens,
                       int nq, int nkv, int dk, int dv, float scale_log2, int window, const float* __restrict__ bias,
-                      int bias_last, const float* __restrict__ sink, float* __restrict__ partial, int segment,
+                      int bias_last, const float* __restrict__ sink, float softcap, float* __restrict__ partial, int segment,
                       unsigned* status, HeadFinish finish) {
   // MAPS score maps a head: the query row holds MAPS queries, a key entry MAPS keys side by side,
   // every map has a softmax of its own over the same values (a value row is loaded once for all).
@@ -607,8 +609,9 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
   int kstart = first_visible_key(pos, window);
   int kend = pos;                                   // inclusive
   if (partial != nullptr) {                         // this warp's segment of the keys (segment: a multiple of 32)
-    kstart = max(kstart, (int)blockIdx.y * segment);
-    kend = min(kend, (int)(blockIdx.y + 1) * segment - 1);
+    const int seg = (window > 0 ? kstart / segment : 0) + (int)blockIdx.y;
+    kstart = max(kstart, seg * segment);
+    kend = min(kend, (seg + 1) * segment - 1);
   }
   const int* table = block_table + (int64_t)b * max_pages;
   const float* bias_h = bias != nullptr ? bias + (int64_t)h * (bias_last + 1) : nullptr;
@@ -641,6 +644,7 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
 #pragma unroll
         for (int a = 0; a < MAPS; ++a) {
           s[a] = dot_key(qs + a * dk, k_cache + (slot * MAPS + a) * dk, dk) * scale_log2;
+          if (softcap > 0.f) s[a] = softcap * tanhf(s[a] / softcap);       // softcap in base-2 units like the scores
           if (bias_h != nullptr) s[a] += bias_h[min(pos - j, bias_last)];
         }
       }
@@ -799,14 +803,14 @@ template <typename T, int MAPS>
 static cudaError_t attention_sink_launch(const void* q, const void* k_cache, const void* v_cache, void* out, const int* positions,
                                          const int* request_of, const int* block_table, int max_pages, int page_size, int num_pages,
                                          const int* token_list, int tokens, int nq, int nkv, int dk, int dv, float scale, int window,
-                                         const float* bias, int bias_last, const float* sink, float* partial, int segment,
+                                         const float* bias, int bias_last, const float* sink, float softcap, float* partial, int segment,
                                          int segments, unsigned* status, const HeadFinish& finish, cudaStream_t stream) {
   const int64_t blocks = ((int64_t)tokens * nq + WARPS - 1) / WARPS;
   const size_t smem = (size_t)WARPS * MAPS * dk * sizeof(float);
   const dim3 grid((unsigned)blocks, segments > 1 ? segments : 1);
   vosti_launch(attention_sink_kernel<T, MAPS>, grid, dim3(WARPS * 32), smem, stream, (const T*)q, (const T*)k_cache, (const T*)v_cache,
                (T*)out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list, tokens, nq, nkv, dk, dv,
-               scale * LOG2E, window, bias, bias_last, sink, partial, segment, status, finish);
+               scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, partial, segment, status, finish);
   if (segments > 1) {
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
@@ -821,12 +825,13 @@ static cudaError_t attention_sink_launch(const void* q, const void* k_cache, con
 // times log2(e), or null; sink: float32 [nq] in natural-log units, or null. `token_list` (or
 // null: all of them) names the `tokens` rows to compute. With `segments` > 1 the keys are cut
 // into pieces of `segment` keys (a multiple of 32) and `scratch` holds tokens * nq * segments * maps *
-// (dv + 2) floats. maps is 1 or 2 (see HeadFinish for what follows the softmax: lambda, the unit norm
+// (dv + 2) floats; with a window a row's pieces are counted from the one that holds its first key, so
+// (window - 1) / segment + 2 of them reach every key. `softcap` (natural units) > 0 caps the scores. maps is 1 or 2 (see HeadFinish for what follows the softmax: lambda, the unit norm
 // with eps and out_scale, the gate).
 VOSTI_API int vosti_attention_maps(const void* q, const void* k_cache, const void* v_cache, void* out, const int* positions,
                                    const int* request_of, const int* block_table, int max_pages, int page_size,
                                    int num_pages, const int* token_list, int tokens, int nq, int nkv, int maps, int dk, int dv,
-                                   float scale, int window, const float* bias, int bias_last, const float* sink,
+                                   float scale, int window, const float* bias, int bias_last, const float* sink, float softcap,
                                    float* scratch, int segment, int segments, float lambda, int unit_norm, float eps,
                                    float out_scale, const void* gate, int gate_f32, long long gate_stride, int is_f32,
                                    unsigned* status, cudaStream_t stream) {
@@ -835,6 +840,7 @@ VOSTI_API int vosti_attention_maps(const void* q, const void* k_cache, const voi
   VOSTI_REQUIRE(dk > 0 && dv > 0 && dk <= MAX_W && dv <= MAX_W, "attention: head widths %d / %d must be at most %d", dk, dv, MAX_W);
   VOSTI_REQUIRE(page_size > 0 && max_pages > 0 && num_pages > 0, "attention: bad cache geometry");
   VOSTI_REQUIRE(bias == nullptr || bias_last >= 0, "attention: bad bias table");       // (window < 0: a chunk)
+  VOSTI_REQUIRE(softcap >= 0.f, "attention: the soft cap is positive, or 0 for none");
   VOSTI_REQUIRE(segments >= 1 && segments <= 65535 && (segments == 1 || (scratch != nullptr && segment > 0 && segment % 32 == 0)),
                 "attention: key segments need scratch and a length that is a multiple of 32");
   VOSTI_REQUIRE(gate == nullptr || gate_stride >= (long long)nq * dv, "attention: the gate's rows are narrower than the heads");
@@ -844,7 +850,7 @@ VOSTI_API int vosti_attention_maps(const void* q, const void* k_cache, const voi
   float* partial = segments > 1 ? scratch : nullptr;
   cudaError_t e;
 #define VOSTI_SINK_ARGS q, k_cache, v_cache, out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list, \
-                        tokens, nq, nkv, dk, dv, scale, window, bias, bias_last, sink, partial, segment, segments, status, finish, stream
+                        tokens, nq, nkv, dk, dv, scale, window, bias, bias_last, sink, softcap, partial, segment, segments, status, finish, stream
   if (is_f32) e = maps == 2 ? attention_sink_launch<float, 2>(VOSTI_SINK_ARGS) : attention_sink_launch<float, 1>(VOSTI_SINK_ARGS);
   else e = maps == 2 ? attention_sink_launch<bf16, 2>(VOSTI_SINK_ARGS) : attention_sink_launch<bf16, 1>(VOSTI_SINK_ARGS);
 #undef VOSTI_SINK_ARGS
@@ -859,7 +865,7 @@ VOSTI_API int vosti_attention_sink(const void* q, const void* k_cache, const voi
                                    float* scratch, int segment, int segments, int is_f32, unsigned* status,
                                    cudaStream_t stream) {
   return vosti_attention_maps(q, k_cache, v_cache, out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list,
-                              tokens, nq, nkv, 1, dk, dv, scale, window, bias, bias_last, sink, scratch, segment, segments,
+                              tokens, nq, nkv, 1, dk, dv, scale, window, bias, bias_last, sink, 0.f, scratch, segment, segments,
                               NO_FINISH.lambda, 0, 0.f, 1.f, nullptr, 0, 0, is_f32, status, stream);
 }
 

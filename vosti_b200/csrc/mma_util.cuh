@@ -38,6 +38,15 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// A soft cap on a score, cap * tanh(x / cap), with x and cap in base-2 units and rate = 2 / (cap in natural
+// units), through tanh(v) = 1 - 2 / (1 + e^(2v)) on the special-function unit: the error is about
+// cap * 2^-22, whatever the size of x.
+__device__ __forceinline__ float soft_capped(float x, float cap, float rate) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + fast_exp2(x * rate)));
+  return fmaf(-2.f * cap, r, cap);
+}
+
 // ---- bulk copies (TMA, untiled) with mbarrier completion, for whole cache rows
 __device__ __forceinline__ void mb_init(uint32_t bar, uint32_t count) {
   asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count));

@@ -12,6 +12,9 @@
 // that stand for experts returning their input, and one more router row whose sigmoid gates a
 // shared expert. moe_identity adds the input-returning experts' share of the input.
 //
+// moe_table: no router at all: a table [vocab, top] names the experts of every token id, which all
+// weigh 1 / top; it writes the same lists and dense matrix. moe_scale can read the table itself.
+//
 // moe_scale: multiplies each expert's slice of the stacked activation [tokens, experts * ff] by
 // the token's weight for that expert (zero for experts it did not choose), after an optional
 // activation of its own (the exact GELU, for experts without a gate), so that one product
@@ -276,11 +279,46 @@ __device__ __forceinline__ float moe_activation(float x, int mode) {
   return x;
 }
 
-template <typename T>
-__global__ void moe_scale_kernel(T* __restrict__ act, const float* __restrict__ dense, int64_t tokens, int experts, int ff,
-                                 int gelu, int tail) {
+// Experts by token id: table [vocab, top] (entries of a row differ), every listed expert with weight `share`.
+struct TokenTable {
+  const int* ids;          // [tokens], or null: the weights are in `dense`
+  const int* table;
+  int top, vocab;
+  float share;
+};
+__device__ __forceinline__ const int* table_row(const TokenTable& by, int64_t t) {
+  const int id = by.ids[t];
+  return by.table + (int64_t)(id < 0 || id >= by.vocab ? 0 : id) * by.top;
+}
+__device__ __forceinline__ float table_weight(const TokenTable& by, int64_t t, int e) {
+  const int* row = table_row(by, t);
+  for (int k = 0; k < by.top; ++k)
+    if (row[k] == e) return by.share;
+  return 0.f;
+}
+
+__global__ void __launch_bounds__(128)
+moe_table_kernel(const TokenTable by, int tokens, int experts, int* __restrict__ chosen, float* __restrict__ weights,
+                 float* __restrict__ dense) {
   pdl_wait();
   pdl_launch_dependents();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= tokens) return;
+  const int* row = table_row(by, t);
+  for (int k = lane; k < by.top; k += 32) {
+    chosen[(int64_t)t * by.top + k] = row[k];
+    weights[(int64_t)t * by.top + k] = by.share;
+  }
+  if (dense != nullptr)
+    for (int e = lane; e < experts; e += 32) dense[(int64_t)t * experts + e] = table_weight(by, t, e);
+}
+
+template <typename T>
+__global__ void moe_scale_kernel(T* __restrict__ act, const float* __restrict__ dense, int64_t tokens, int experts, int ff,
+                                 int gelu, int tail, const TokenTable table) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const bool weighted = dense != nullptr || table.ids != nullptr;
   const int64_t width = (int64_t)experts * ff + tail, n = tokens * width;
   const int cols = experts + (tail > 0 ? 1 : 0);
   if (sizeof(T) == 2 && ff % 8 == 0 && tail % 8 == 0 && (reinterpret_cast<uintptr_t>(act) & 15) == 0) {
@@ -290,14 +328,14 @@ __global__ void moe_scale_kernel(T* __restrict__ act, const float* __restrict__ 
       const int64_t t = w / per_row;
       const int64_t c = (w - t * per_row) * 8;
       const int e = c < (int64_t)experts * ff ? (int)(c / ff) : experts;
-      const float by = dense != nullptr ? dense[t * cols + e] : 1.f;
+      const float by = table.ids != nullptr ? table_weight(table, t, e) : dense != nullptr ? dense[t * cols + e] : 1.f;
       uint4 raw = reinterpret_cast<uint4*>(act)[w];
       __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&raw);
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float2 f = __bfloat1622float2(p[k]);
         float a = moe_activation(f.x, gelu), b = moe_activation(f.y, gelu);
-        if (dense != nullptr) { a *= by; b *= by; }
+        if (weighted) { a *= by; b *= by; }
         p[k] = __floats2bfloat162_rn(a, b);
       }
       reinterpret_cast<uint4*>(act)[w] = raw;
@@ -309,7 +347,7 @@ __global__ void moe_scale_kernel(T* __restrict__ act, const float* __restrict__ 
     const int64_t c = i - t * width;
     const int e = c < (int64_t)experts * ff ? (int)(c / ff) : experts;
     float x = moe_activation(to_f32(act[i]), gelu);
-    if (dense != nullptr) x *= dense[t * cols + e];
+    if (weighted) x *= table.ids != nullptr ? table_weight(table, t, e) : dense[t * cols + e];
     act[i] = from_f32<T>(x);
   }
 }
@@ -409,28 +447,47 @@ VOSTI_API int vosti_moe_route(const float* logits, int tokens, int experts, int 
 }
 
 static int moe_scale_launch(void* act, const float* dense, int tokens, int experts, int ff, int is_f32, int gelu, int tail,
-                            cudaStream_t stream) {
+                            const TokenTable& table, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && experts >= 0 && ff > 0 && tail >= 0 && (experts > 0 || tail > 0) && gelu >= 0 && gelu <= 2,
                 "moe_scale: bad sizes");
   if (tokens == 0) return VOSTI_OK;
   const int64_t n = (int64_t)tokens * ((int64_t)experts * ff + tail);
   const int64_t items = (!is_f32 && ff % 8 == 0 && tail % 8 == 0) ? n / 8 : n;      // 16-byte words where the slices allow them
   const int blocks = (int)((items + 255) / 256 < 148 * 16 ? (items + 255) / 256 : 148 * 16);
-  if (is_f32) vosti_launch(moe_scale_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)act, dense, (int64_t)tokens, experts, ff, gelu, tail);
-  else vosti_launch(moe_scale_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)act, dense, (int64_t)tokens, experts, ff, gelu, tail);
+  if (is_f32) vosti_launch(moe_scale_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)act, dense, (int64_t)tokens, experts, ff, gelu, tail, table);
+  else vosti_launch(moe_scale_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (bf16*)act, dense, (int64_t)tokens, experts, ff, gelu, tail, table);
   VOSTI_LAUNCH_CHECK();
 }
 
 VOSTI_API int vosti_moe_scale(void* act, const float* dense, int tokens, int experts, int ff, int is_f32, int gelu,
                               cudaStream_t stream) {
-  return moe_scale_launch(act, dense, tokens, experts, ff, is_f32, gelu, 0, stream);
+  return moe_scale_launch(act, dense, tokens, experts, ff, is_f32, gelu, 0, TokenTable{}, stream);
+}
+
+// The same with weights by token id: ids int32 [tokens], table int32 [vocab, top]; an expert listed in the
+// row of a token's id weighs `share`, the others nothing. No activation of its own.
+VOSTI_API int vosti_moe_scale_table(void* act, const int* ids, const int* table, int vocab, int top, float share, int tokens,
+                                    int experts, int ff, int is_f32, cudaStream_t stream) {
+  VOSTI_REQUIRE(ids != nullptr && table != nullptr && vocab > 0 && top > 0, "moe_scale: bad table");
+  return moe_scale_launch(act, nullptr, tokens, experts, ff, is_f32, 0, 0, TokenTable{ids, table, top, vocab, share}, stream);
+}
+
+// The choice by token id as lists (chosen, weights [tokens, top]) and, if `dense` is given, as a matrix [tokens, experts].
+VOSTI_API int vosti_moe_table(const int* ids, const int* table, int vocab, int top, float share, int tokens, int experts,
+                              int* chosen, float* weights, float* dense, cudaStream_t stream) {
+  VOSTI_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && top <= experts && vocab > 0, "moe_table: bad sizes experts=%d top=%d", experts, top);
+  VOSTI_REQUIRE(ids != nullptr && table != nullptr && chosen != nullptr && weights != nullptr, "moe_table: missing arrays");
+  if (tokens == 0) return VOSTI_OK;
+  vosti_launch(moe_table_kernel, dim3((tokens + 3) / 4), dim3(128), 0, stream, TokenTable{ids, table, top, vocab, share}, tokens, experts,
+               chosen, weights, dense);
+  VOSTI_LAUNCH_CHECK();
 }
 
 // The same with an activation mode (0 none, 1 exact GELU, 2 squared relu) and a tail slice of `tail`
 // columns whose weight is dense's last column (dense: [tokens, experts + (tail > 0)]).
 VOSTI_API int vosti_moe_scale_tail(void* act, const float* dense, int tokens, int experts, int ff, int tail, int is_f32,
                                    int activation, cudaStream_t stream) {
-  return moe_scale_launch(act, dense, tokens, experts, ff, is_f32, activation, tail, stream);
+  return moe_scale_launch(act, dense, tokens, experts, ff, is_f32, activation, tail, TokenTable{}, stream);
 }
 
 VOSTI_API int vosti_moe_identity(float* y, const float* coeff, const void* x, int x_f32, int tokens, int width, cudaStream_t stream) {

@@ -9,12 +9,12 @@
 // With `source`, row t takes its id from values[source[t]] where source[t] >= 0: a token the
 // sampler of the step before left on the device, which the host has not read yet.
 // `scale` multiplies the row in float32 (1: a plain copy), for architectures that scale
-// their embeddings.
+// their embeddings. `resolved` (or null) receives the id every row was taken for.
 template <typename T, typename TO = T>
 __global__ void embedding_kernel(const int* __restrict__ ids, const int* __restrict__ source,
                                  const int* __restrict__ values, const T* __restrict__ table,
                                  TO* __restrict__ out, int hidden, int vocab, float scale, unsigned* status,
-                                 bf16* __restrict__ rounded = nullptr) {
+                                 bf16* __restrict__ rounded, int* __restrict__ resolved) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
@@ -27,6 +27,7 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const int* __restr
   }
   const T* src = table + (int64_t)id * hidden;
   TO* dst = out + (int64_t)t * hidden;
+  if (resolved != nullptr && threadIdx.x == 0) resolved[t] = id;
   const int bytes = hidden * (int)sizeof(T);
   if (sizeof(TO) == 4 && sizeof(T) == 2 && hidden % 8 == 0) {
     // a float32 stream from a bfloat16 table: 16-byte words in, two out, and the row's rounding beside it if asked for
@@ -68,15 +69,15 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const int* __restr
 }
 
 VOSTI_API int vosti_embedding(const int* ids, const int* source, const int* values, const void* table, void* out,
-                              int tokens, int hidden, int vocab, int is_f32, float scale, unsigned* status,
+                              int tokens, int hidden, int vocab, int is_f32, float scale, int* resolved, unsigned* status,
                               cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0, "embedding: bad sizes T=%d H=%d V=%d",
                 tokens, hidden, vocab);
   if (tokens == 0) return VOSTI_OK;
   if (is_f32)
-    vosti_launch(embedding_kernel<float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const float*)table, (float*)out, hidden, vocab, scale, status, (bf16*)nullptr);
+    vosti_launch(embedding_kernel<float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const float*)table, (float*)out, hidden, vocab, scale, status, (bf16*)nullptr, resolved);
   else
-    vosti_launch(embedding_kernel<bf16>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const bf16*)table, (bf16*)out, hidden, vocab, scale, status, (bf16*)nullptr);
+    vosti_launch(embedding_kernel<bf16>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const bf16*)table, (bf16*)out, hidden, vocab, scale, status, (bf16*)nullptr, resolved);
   VOSTI_LAUNCH_CHECK();
 }
 
@@ -84,14 +85,14 @@ VOSTI_API int vosti_embedding(const int* ids, const int* source, const int* valu
 // (a bfloat16 entry times the scale is not rounded again).
 // `rounded` (or null): the same rows rounded to bfloat16, for products that read the stream's rounding.
 VOSTI_API int vosti_embedding_stream(const int* ids, const int* source, const int* values, const void* table, float* out,
-                                     void* rounded, int tokens, int hidden, int vocab, int is_f32, float scale, unsigned* status,
-                                     cudaStream_t stream) {
+                                     void* rounded, int tokens, int hidden, int vocab, int is_f32, float scale, int* resolved,
+                                     unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0, "embedding: bad sizes T=%d H=%d V=%d", tokens, hidden, vocab);
   if (tokens == 0) return VOSTI_OK;
   if (is_f32)
-    vosti_launch(embedding_kernel<float, float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const float*)table, out, hidden, vocab, scale, status, (bf16*)rounded);
+    vosti_launch(embedding_kernel<float, float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const float*)table, out, hidden, vocab, scale, status, (bf16*)rounded, resolved);
   else
-    vosti_launch(embedding_kernel<bf16, float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const bf16*)table, out, hidden, vocab, scale, status, (bf16*)rounded);
+    vosti_launch(embedding_kernel<bf16, float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, (const bf16*)table, out, hidden, vocab, scale, status, (bf16*)rounded, resolved);
   VOSTI_LAUNCH_CHECK();
 }
 
@@ -359,30 +360,39 @@ __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ o
   }
 }
 
-// act(gate) * up with act = relu (1) or the square of relu (2); same layout as silu_mul.
+// act(gate) * up with act = relu (1) or the square of relu (2), or the clamped form (3): with a limit L and a constant
+// c, g sigmoid(c g) (u + 1) of g = min(gate, L), u = up clamped to [-L, L]; same layout as silu_mul.
 template <typename T>
-__global__ void glu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int64_t rows, int inter, int act) {
+__global__ void glu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int64_t rows, int inter, int act,
+                               float limit, float sigmoid_scale) {
   pdl_wait();
   pdl_launch_dependents();
   const int64_t n = rows * inter;
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
     const int64_t r = i / inter;
     const int c = (int)(i - r * inter);
+    if (act == 3) {
+      const float g = fminf(to_f32(gate_up[r * 2 * inter + c]), limit);
+      const float u = fminf(fmaxf(to_f32(gate_up[r * 2 * inter + inter + c]), -limit), limit);
+      out[i] = from_f32<T>(g * (1.f / (1.f + expf(-sigmoid_scale * g))) * (u + 1.f));
+      continue;
+    }
     float g = fmaxf(to_f32(gate_up[r * 2 * inter + c]), 0.f);
     if (act == 2) g *= g;
     out[i] = from_f32<T>(g * to_f32(gate_up[r * 2 * inter + inter + c]));
   }
 }
 
-VOSTI_API int vosti_glu_mul(const void* gate_up, void* out, int rows, int inter, int act, int is_f32, cudaStream_t stream) {
-  VOSTI_REQUIRE(rows >= 0 && inter > 0 && (act == 1 || act == 2), "glu_mul: bad sizes rows=%d inter=%d or activation %d", rows, inter, act);
+VOSTI_API int vosti_glu_mul(const void* gate_up, void* out, int rows, int inter, int act, float limit, float sigmoid_scale, int is_f32,
+                            cudaStream_t stream) {
+  VOSTI_REQUIRE(rows >= 0 && inter > 0 && act >= 1 && act <= 3, "glu_mul: bad sizes rows=%d inter=%d or activation %d", rows, inter, act);
   if (rows == 0) return VOSTI_OK;
   const int64_t n = (int64_t)rows * inter;
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
   if (is_f32)
-    vosti_launch(glu_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, (int64_t)rows, inter, act);
+    vosti_launch(glu_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, (int64_t)rows, inter, act, limit, sigmoid_scale);
   else
-    vosti_launch(glu_mul_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, (int64_t)rows, inter, act);
+    vosti_launch(glu_mul_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, (int64_t)rows, inter, act, limit, sigmoid_scale);
   VOSTI_LAUNCH_CHECK();
 }
 

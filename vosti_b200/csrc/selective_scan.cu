@@ -11,6 +11,7 @@
 // Kernels:
 //   scan_conv   convolution + SiLU for every token of the step (block per token); a token near the start
 //               of its request's portion takes the inputs before the portion from the slot's tail.
+//               Its plain form adds the convolution to its input, h + conv(h), without SiLU or bias.
 //   scan_tail   the tail after this step, one thread per (request, channel); it runs after
 //               scan_conv has read the old tail.
 //   scan_run    the recurrence: a block per (request, 32 channels, chunk of tokens), LANES lanes share a
@@ -34,7 +35,7 @@ __global__ void __launch_bounds__(256)
 scan_conv_kernel(const T* __restrict__ xz, int64_t xz_stride, const void* __restrict__ conv_w, const void* __restrict__ conv_b,
                  int w_f32, const float* state, int64_t state_stride, int64_t tail_offset, const int* __restrict__ request_of,
                  const int* __restrict__ cu_q, const int* __restrict__ state_slots, int num_slots, int inner, int taps,
-                 int tokens, int per_block, T* __restrict__ out, unsigned* status) {
+                 int tokens, int per_block, int plain, T* __restrict__ out, unsigned* status) {
   pdl_wait();
   pdl_launch_dependents();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
@@ -82,7 +83,7 @@ scan_conv_kernel(const T* __restrict__ xz, int64_t xz_stride, const void* __rest
 #pragma unroll
       for (int k = CONV_WINDOW - 1; k >= 0; --k)
         if (k < taps) acc = fmaf(w[CONV_WINDOW - 1 - k], win[CONV_WINDOW - 1 - k], acc);
-      out[(int64_t)t * inner + c] = from_f32<T>(silu_f(acc));
+      out[(int64_t)t * inner + c] = from_f32<T>(plain ? win[CONV_WINDOW - 1] + acc : silu_f(acc));
     }
     return;
   }
@@ -100,7 +101,7 @@ scan_conv_kernel(const T* __restrict__ xz, int64_t xz_stride, const void* __rest
     float acc = bias;
     for (int j = 0; j < taps; ++j)                                                      // tap j reads the input taps - 1 - j tokens back
       acc = fmaf(load_flex(conv_w, w_f32, (int64_t)c * taps + j), input(t, taps - 1 - j, first, tail), acc);
-    out[(int64_t)t * inner + c] = from_f32<T>(silu_f(acc));
+    out[(int64_t)t * inner + c] = from_f32<T>(plain ? to_f32(xz[(int64_t)t * xz_stride + c]) + acc : silu_f(acc));
   }
 }
 
@@ -270,12 +271,13 @@ scan_carry_kernel(const void* __restrict__ a_log, int w_f32, const float* state,
 
 // xz [tokens, xz_stride] holds the convolution's inputs in its first `inner` columns; out [tokens, inner].
 // The state slot's tail [taps - 1, inner] starts tail_offset floats into the slot. Two launches
-// when taps > 1.
+// when taps > 1. `plain`: out = input + convolution, no SiLU (conv_b must be null).
 VOSTI_API int vosti_scan_conv(const void* xz, int64_t xz_stride, const void* conv_w, const void* conv_b, int w_f32, float* state,
                               int64_t state_stride, int64_t tail_offset, const int* request_of, const int* cu_q,
-                              const int* state_slots, int num_slots, int requests, int tokens, int inner, int taps, void* out,
+                              const int* state_slots, int num_slots, int requests, int tokens, int inner, int taps, int plain, void* out,
                               int is_f32, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && requests >= 0 && inner > 0 && taps >= 1 && taps <= 64, "scan_conv: bad sizes");
+  VOSTI_REQUIRE(!plain || conv_b == nullptr, "scan_conv: the plain form has no bias");
   if (tokens == 0) return VOSTI_OK;
   const int across_c = (inner + 255) / 256;
   int per_block = 1;                      // tokens a block takes: more once the grid fills the GPU several times over
@@ -286,11 +288,11 @@ VOSTI_API int vosti_scan_conv(const void* xz, int64_t xz_stride, const void* con
   if (is_f32)
     vosti_launch(scan_conv_kernel<float>, grid, dim3(256), 0, stream, (const float*)xz, xz_stride, conv_w, conv_b, w_f32,
                  (const float*)state, state_stride, tail_offset, request_of, cu_q, state_slots, num_slots, inner, taps,
-                 tokens, per_block, (float*)out, status);
+                 tokens, per_block, plain, (float*)out, status);
   else
     vosti_launch(scan_conv_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)xz, xz_stride, conv_w, conv_b, w_f32,
                  (const float*)state, state_stride, tail_offset, request_of, cu_q, state_slots, num_slots, inner, taps,
-                 tokens, per_block, (bf16*)out, status);
+                 tokens, per_block, plain, (bf16*)out, status);
   if (taps > 1) {
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) { vosti_set_error("%s", cudaGetErrorString(e)); return (int)e; }

@@ -8,6 +8,7 @@ embeddings are tied. Logits are float32.
 """
 from __future__ import annotations
 
+import dataclasses
 from typing import Dict, List, Optional
 
 import torch
@@ -29,10 +30,13 @@ class DecoderModel:
         self.reentry = build_reentry(spec.reentry, spec.hidden_size)
         # One cache (pages and state slot storage) per (layer, instance) that owns one. Cache i
         # belongs to layer i's first run; further runs of a layer get caches after those.
+        # A run that reads another layer's pages keeps its own state, and no pages if that is all its
+        # layer does.
         self.cache_index = {(i, 0): i for i in range(len(self.blocks))}
         self.cache_layers = list(range(len(self.blocks)))
         for entry in spec.run_order:
-            if entry.cache_from is None and (entry.layer, entry.instance) not in self.cache_index:
+            wanted = entry.cache_from is None or self.blocks[entry.layer].state_spec() is not None
+            if wanted and (entry.layer, entry.instance) not in self.cache_index:
                 self.cache_index[(entry.layer, entry.instance)] = len(self.cache_layers)
                 self.cache_layers.append(entry.layer)
         # an embedding that keeps something per request gets state slots of its own, after the blocks' caches
@@ -57,8 +61,23 @@ class DecoderModel:
     def cache_specs(self):
         """(paged cache spec, state spec) of every cache in `cache_layers` order."""
         own = self.embedding_cache is not None
-        return ([self.blocks[i].mixer.cache_spec() for i in self.cache_layers] + ([None] if own else []),
-                [self.blocks[i].mixer.state_spec() for i in self.cache_layers] + ([self.embedding.state_spec()] if own else []))
+        pages = [self.blocks[i].mixer.cache_spec() for i in self.cache_layers]
+        owned, readers = set(), {}
+        for entry in self.spec.run_order:
+            if entry.cache_from is None:
+                owned.add(self.cache_index[(entry.layer, entry.instance)])
+            else:
+                readers.setdefault(self.cache_index[(entry.cache_from, entry.instance)], []).append(entry.layer)
+        for index, layers in readers.items():
+            # pages live as long as any run that reads them needs them
+            owned.add(index)
+            for spec in (self.blocks[i].mixer.cache_spec() for i in layers):
+                if pages[index] is not None and spec is not None and pages[index].window:
+                    wider = max(pages[index].window, spec.window) if spec.window else 0
+                    pages[index] = dataclasses.replace(pages[index], window=wider)
+        pages = [spec if i in owned else None for i, spec in enumerate(pages)]
+        return (pages + ([None] if own else []),
+                [self.blocks[i].state_spec() for i in self.cache_layers] + ([self.embedding.state_spec()] if own else []))
 
     @property
     def capture_safe(self) -> bool:
@@ -168,6 +187,11 @@ class DecoderModel:
         for block in self.blocks:
             for _, part in block._children():
                 visit(part)
+            for weight in getattr(block, "extra_weights", list)():
+                data = weight.data if isinstance(weight, ops.PackedWeight) else weight
+                if data.untyped_storage().data_ptr() not in seen:
+                    seen.add(data.untyped_storage().data_ptr())
+                    total += data.untyped_storage().nbytes()
         visit(self.final_norm)
         if self.reentry is not None:
             visit(self.reentry)
@@ -190,9 +214,12 @@ class DecoderModel:
             owner = entry.layer if entry.cache_from is None else entry.cache_from
             if entry.reenter:
                 hidden, residual = self.reentry.forward(ctx, hidden, residual, first)
-            hidden, residual = self.blocks[entry.layer].forward(
-                ctx, hidden, residual, layer_caches[self.cache_index[(owner, entry.instance)]],
-                writes_cache=entry.cache_from is None)
+            cache = layer_caches[self.cache_index[(owner, entry.instance)]]
+            if entry.cache_from is not None:
+                # another layer's pages beside this run's own state
+                mine = self.cache_index.get((entry.layer, entry.instance))
+                cache = dataclasses.replace(cache, state=None if mine is None else layer_caches[mine].state)
+            hidden, residual = self.blocks[entry.layer].forward(ctx, hidden, residual, cache, writes_cache=entry.cache_from is None)
         return hidden, residual
 
     def logits(self, ctx, hidden: torch.Tensor, residual: Optional[torch.Tensor], rows: torch.Tensor) -> torch.Tensor:
@@ -202,6 +229,9 @@ class DecoderModel:
             # a sublayer output still to be normed, scaled and added: only the wanted rows are
             hidden = hidden.rows(rows, ctx.status)
             return self.head.forward(ctx, self.final_norm.forward_add(ctx, hidden, ops.gather_rows(residual, rows, ctx.status))[0])
+        if isinstance(hidden, ops.DeferredGated):
+            # a sublayer output that joins through its gate: gather, gate, add and norm in one kernel
+            return self.head.forward(ctx, self.final_norm.forward_gated(ctx, hidden, residual, rows=rows))
         if isinstance(hidden, ops.DeferredSum):
             # a float32 stream with sublayer outputs still to be added: add, then gather
             hidden, residual = ops.stream_sum(residual, hidden), None

@@ -89,12 +89,13 @@ def _contig(*tensors):
 
 def embedding(ids: torch.Tensor, table: torch.Tensor, status: torch.Tensor,
               feedback: Optional[tuple] = None, scale: float = 1.0, out_dtype: Optional[torch.dtype] = None,
-              rounded: bool = False):
+              rounded: bool = False, resolved: Optional[torch.Tensor] = None):
     """table[ids] * scale. `feedback` = (source, values), int32: row t takes values[source[t]] as
     its id where source[t] >= 0 (a token sampled on the device that the host has not read yet).
     `out_dtype` float32 gives float32 rows from a bfloat16 table (the scaled entry is not rounded
     again): the start of a float32 residual stream; with `rounded` the call returns a `StreamPair` of
-    those rows and their rounding to bfloat16, written by the same kernel."""
+    those rows and their rounding to bfloat16, written by the same kernel. `resolved` (int32, a slot per
+    row) receives the ids the rows were taken for."""
     _contig(ids, table)
     source, values = feedback if feedback is not None else (None, None)
     if source is not None:
@@ -104,14 +105,14 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, status: torch.Tensor,
         out = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
         low = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.bfloat16, device=table.device) if rounded else None
         _check(library().vosti_embedding_stream(_p(ids), _p(source), _p(values), _p(table), _p(out), _p(low), ids.shape[0],
-                                                table.shape[1], table.shape[0], _is_f32(table), ctypes.c_float(scale), _p(status),
-                                                _stream()), "embedding")
+                                                table.shape[1], table.shape[0], _is_f32(table), ctypes.c_float(scale), _p(resolved),
+                                                _p(status), _stream()), "embedding")
         return StreamPair(low, out) if rounded else out
     if out_dtype is not None and out_dtype != table.dtype:
         raise KernelError("embedding: rows come in the table's type or in float32")
     out = torch.empty((ids.shape[0], table.shape[1]), dtype=table.dtype, device=table.device)
     _check(library().vosti_embedding(_p(ids), _p(source), _p(values), _p(table), _p(out), ids.shape[0], table.shape[1],
-                                     table.shape[0], _is_f32(table), ctypes.c_float(scale), _p(status), _stream()),
+                                     table.shape[0], _is_f32(table), ctypes.c_float(scale), _p(resolved), _p(status), _stream()),
            "embedding")
     return out
 
@@ -173,20 +174,21 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return out
 
 
-GLU_ACTIVATIONS = {"silu": 0, "relu": 1, "relu2": 2}
-FUSED_GLU_ACTIVATIONS = {"silu": 2, "relu": 4, "relu2": 5}         # the tensor-core product's gated epilogues
+GLU_ACTIVATIONS = {"silu": 0, "relu": 1, "relu2": 2, "clamped": 3}
+FUSED_GLU_ACTIVATIONS = {"silu": 2, "relu": 4, "relu2": 5, "clamped": 6}         # the tensor-core product's gated epilogues
 
 
-def glu_mul(gate_up: torch.Tensor, activation: str) -> torch.Tensor:
+def glu_mul(gate_up: torch.Tensor, activation: str, limit: float = 0.0, sigmoid_scale: float = 0.0) -> torch.Tensor:
     """act(gate) * up of a [rows, 2 * inter] product with the gate half first; `activation` is
-    "silu", "relu" or "relu2" (the square of relu)."""
+    "silu", "relu" or "relu2" (the square of relu), or "clamped": g sigmoid(sigmoid_scale g) (u + 1) of
+    g = min(gate, limit) and u = up clamped to [-limit, limit]."""
     if activation == "silu":
         return silu_mul(gate_up)
     _contig(gate_up)
     inter = gate_up.shape[-1] // 2
     out = torch.empty((gate_up.shape[0], inter), dtype=gate_up.dtype, device=gate_up.device)
-    _check(library().vosti_glu_mul(_p(gate_up), _p(out), gate_up.shape[0], inter, GLU_ACTIVATIONS[activation], _is_f32(gate_up),
-                                   _stream()), "glu_mul")
+    _check(library().vosti_glu_mul(_p(gate_up), _p(out), gate_up.shape[0], inter, GLU_ACTIVATIONS[activation],
+                                   ctypes.c_float(limit), ctypes.c_float(sigmoid_scale), _is_f32(gate_up), _stream()), "glu_mul")
     return out
 
 
@@ -341,27 +343,27 @@ def _counters(device: torch.device, count: int) -> torch.Tensor:
 
 
 EPI_BF16, EPI_F32, EPI_SWIGLU = 0, 1, 2
-_SPLIT_GENERATION = 0   # counts split-K products: a PartialSum is valid until the next one runs
+_SPLIT_GENERATION = {}   # per scratch: counts its split-K products; a PartialSum is valid until the next one runs
 
 
 class PartialSum:
     """The result of a split-K product whose splits have not been summed yet: float32
     [splits, rows, width] in the split-K scratch. A consumer that can add the splits itself
     (the fused add + RMSNorm, the head norm / rotation kernel) takes it as it is; anything else
-    calls `materialize`. It must be consumed before the next split-K product runs."""
+    calls `materialize`. It must be consumed before the next split-K product into the same scratch runs."""
 
     def __init__(self, partial: torch.Tensor, splits: int, rows: int, width: int, dtype: torch.dtype,
-                 status: torch.Tensor):
+                 status: torch.Tensor, scratch: str = "split_k"):
         self.partial, self.splits, self.rows, self.width, self.dtype = partial, splits, rows, width, dtype
         self.status = status
-        self.generation = _SPLIT_GENERATION
+        self.scratch, self.generation = scratch, _SPLIT_GENERATION.get(scratch, 0)
 
     @property
     def shape(self):
         return (self.rows, self.width)
 
     def check(self) -> None:
-        if self.generation != _SPLIT_GENERATION:
+        if self.generation != _SPLIT_GENERATION.get(self.scratch, 0):
             raise KernelError("a deferred split-K result was used after a later split-K product overwrote it")
 
     def materialize(self) -> torch.Tensor:
@@ -409,11 +411,14 @@ class PackedWeight:
 
 
 def gemm_tc(x: torch.Tensor, w, status: torch.Tensor, *, out_dtype: Optional[torch.dtype] = None,
-            swiglu: bool = False, allow_partial: bool = False, activation: str = "silu"):
+            swiglu: bool = False, allow_partial: bool = False, activation: str = "silu", glu=(0.0, 0.0),
+            scratch: str = "split_k"):
     """y = x @ w.T on the tensor cores (bfloat16 operands, float32 accumulation); w is a
     [features, k] tensor or a `PackedWeight`. With `swiglu` the rows of w are blocks of 16 gate
     rows followed by their 16 up rows and y = act(gate) * up has half as many columns, act being
-    `activation`: "silu", "relu" or "relu2" (the square of relu)."""
+    `activation`: "silu", "relu" or "relu2" (the square of relu), or the pair goes through the "clamped"
+    form (see glu_mul; `glu` = (limit, sigmoid_scale)). `scratch` names the buffer of the K splits: two
+    results that stay unsummed at the same time need buffers of their own."""
     packed = isinstance(w, PackedWeight)
     w_data = w.data if packed else w
     _contig(x, w_data)
@@ -432,21 +437,20 @@ def gemm_tc(x: torch.Tensor, w, status: torch.Tensor, *, out_dtype: Optional[tor
             raise KernelError("gemm_tc: the fused SiLU*up epilogue writes bfloat16")
     else:
         epilogue, width = (EPI_F32 if out_dtype == torch.float32 else EPI_BF16), features
-    global _SPLIT_GENERATION
     lib = library()
     splits = lib.vosti_gemm_tc_splits(tokens, features, k)
     elems = splits * tokens * features if splits > 1 else 0
-    ws = _workspace(x.device, elems, "split_k") if elems else None
+    ws = _workspace(x.device, elems, scratch) if elems else None
     defer = bool(allow_partial and splits > 1 and epilogue in (EPI_BF16, EPI_F32))
     out = None if defer else torch.empty((tokens, width), dtype=out_dtype, device=x.device)
     if splits > 1:
-        _SPLIT_GENERATION += 1
+        _SPLIT_GENERATION[scratch] = _SPLIT_GENERATION.get(scratch, 0) + 1
     _check(lib.vosti_gemm_tc(_p(x), _p(w_data), _p(out), tokens, features, k, epilogue, _p(ws),
-                             ctypes.c_int64(ws.numel() if ws is not None else 0), int(defer), int(packed), _p(status),
-                             _stream()),
+                             ctypes.c_int64(ws.numel() if ws is not None else 0), int(defer), int(packed), ctypes.c_float(glu[0]),
+                             ctypes.c_float(glu[1]), _p(status), _stream()),
            "gemm_tc", kernels=2 if splits > 1 and not defer else 1)
     if defer:
-        return PartialSum(ws, splits, tokens, features, out_dtype, status)
+        return PartialSum(ws, splits, tokens, features, out_dtype, status, scratch)
     return out
 
 
@@ -793,6 +797,89 @@ def rms_stream(x, weight: Optional[torch.Tensor], eps: float, out_dtype: Optiona
     return out
 
 
+class DeferredGated:
+    """A sublayer's output y [rows, width] on its way into the float32 stream through a gate: what joins is
+    scale * sigmoid(z + bias) * y, z a float32 product of the sublayer's input. The kernel that next reads
+    the stream (`gated_rms_stream`) does it; y and z may be unsummed K splits (`PartialSum`, each in a
+    scratch of its own)."""
+
+    def __init__(self, y, z, bias: Optional[torch.Tensor], scale: float):
+        for t in (y, z):
+            if isinstance(t, PartialSum) and t.dtype != torch.float32:
+                raise KernelError("deferred gate: unsummed products are float32")
+        if isinstance(y, PartialSum) and isinstance(z, PartialSum) and y.scratch == z.scratch:
+            raise KernelError("deferred gate: two unsummed products need a scratch each")
+        self.y, self.z, self.bias, self.scale = y, z, bias, float(scale)
+        self.shape = tuple(y.shape)
+
+
+def _splits_of(x):
+    """(pointer, is_f32, splits) of a tensor or of unsummed K splits."""
+    if x is None:
+        return None, 0, 1
+    if isinstance(x, PartialSum):
+        x.check()
+        return _p(x.partial), 1, x.splits
+    _contig(x)
+    return _p(x), _is_f32(x), 1
+
+
+class StreamConv:
+    """A causal convolution over time on the normed rows, h + conv(h), for `gated_rms_stream`: weights float32
+    [taps, width] (oldest tap first) and the state slots [slots, size] whose first (taps - 1) * width
+    floats are a request's last inputs."""
+
+    def __init__(self, weight: torch.Tensor, state: torch.Tensor):
+        _contig(weight, state)
+        if weight.dtype != torch.float32 or state.dtype != torch.float32:
+            raise KernelError("stream convolution: taps and state are float32")
+        self.weight, self.state = weight, state
+
+
+def gated_rms_stream(stream: torch.Tensor, x: Optional[DeferredGated], eps: float, out_dtype: torch.dtype, *,
+                     weight: Optional[torch.Tensor] = None, offset: float = 0.0, gain: float = 1.0, store: bool = True,
+                     rows: Optional[torch.Tensor] = None, conv: Optional[StreamConv] = None, ctx=None,
+                     status: Optional[torch.Tensor] = None):
+    """The boundary between two gated sublayers (csrc/gated_stream.cu): s = stream + scale * sigmoid(z + bias) * y
+    (x a `DeferredGated`; None: s = stream), stored over the stream with `store`; returns
+    s / sqrt(mean(s^2) + eps) * (offset + weight), or * gain without a weight, rounded to `out_dtype`. `rows`
+    (int32) asks for those rows only and stores nothing. With `conv` (a step of one token a request, `ctx`
+    its context) returns (h, h + conv(h)) and moves the requests' tails on."""
+    _contig(stream, weight, rows)
+    if stream.dtype != torch.float32:
+        raise KernelError("gated_rms_stream: the residual stream is float32")
+    source, width = stream.shape
+    if x is not None and tuple(x.shape) != (source, width):
+        raise KernelError("gated_rms_stream: the sublayer's output does not match the stream")
+    yp, y_f32, y_splits = _splits_of(x.y if x is not None else None)
+    zp, z_f32, z_splits = _splits_of(x.z if x is not None else None)
+    bias = x.bias if x is not None else None
+    _contig(bias)
+    if zp is not None and not z_f32:
+        raise KernelError("gated_rms_stream: the gate's product is float32")
+    count = source if rows is None else rows.shape[0]
+    store = store and rows is None and x is not None
+    out = torch.empty((count, width), dtype=out_dtype, device=stream.device)
+    u = None
+    cw = cs = slots = None
+    taps, stride, num_slots = 0, 0, 0
+    if conv is not None:
+        if count != ctx.num_requests or rows is not None or conv.weight.shape[1] != width:
+            raise KernelError("gated_rms_stream: the convolution needs a step of one token a request")
+        u = torch.empty_like(out)
+        cw, cs, slots, taps = conv.weight, conv.state, ctx.state_slots, conv.weight.shape[0]
+        stride, num_slots = cs.shape[1], cs.shape[0]
+        if stride < (taps - 1) * width:
+            raise KernelError("gated_rms_stream: the state slots are too small for the convolution's tail")
+    _check(library().vosti_gated_rms_stream(
+        _p(stream), yp, y_f32, y_splits, zp, z_splits, _p(bias), 0 if bias is None else _is_f32(bias),
+        ctypes.c_float(x.scale if x is not None else 1.0), _p(rows), count, source, _p(stream) if store else None, _p(weight),
+        0 if weight is None else _is_f32(weight), ctypes.c_float(offset), ctypes.c_float(gain), ctypes.c_float(eps), _p(cw),
+        taps, _p(cs), ctypes.c_int64(stride), ctypes.c_int64(0), _p(slots), num_slots, _p(out), _p(u), _is_f32(out), width,
+        _p(status if status is not None else getattr(ctx, "status", None)), _stream()), "gated_rms_stream")
+    return out if conv is None else (out, u)
+
+
 # ---------------------------------------------------------------- token inputs
 class StreamPair:
     """A float32 residual stream [rows, width] together with its rounding to the serving type: what a
@@ -905,6 +992,16 @@ SINK_SEGMENT = int(_os.environ.get("VOSTI_SINK_SEGMENT", "256"))          # keys
 SINK_SPLIT_MAX_ROWS = 2048  # (token, head) rows up to which the keys are cut into segments
 
 
+def key_segments(max_kv_len: int, window: int, segment: int, tokens: int = 1) -> int:
+    """How many key segments of `segment` keys (borders at its multiples) reach every key that `tokens`
+    neighbouring positions see: all of the context, or with a window those from the segment of the
+    first position's first key on. 1: not worth cutting."""
+    if max_kv_len <= segment or (window > 0 and window + tokens - 1 <= segment):
+        return 1
+    whole = -(-max_kv_len // segment)
+    return whole if window <= 0 else min(whole, (window + tokens - 2) // segment + 2)
+
+
 class HeadFinish:
     """What follows a head's softmax-weighted sum before the output projection, in float32 (the
     kernels' HeadFinish): with two score maps a head o = a1 - `lam` * a2; with `unit_norm`
@@ -1004,30 +1101,32 @@ def qkv_heads(proj: torch.Tensor, k_cache: Optional[torch.Tensor], v_cache: Opti
 
 
 def _attention_sink_rows(ctx, q, k_cache, v_cache, out, group, *, token_list, count, nq, nkv, dk, dv, scale, window,
-                         bias, sink, maps=1, finish=None) -> None:
+                         bias, sink, softcap=0.0, maps=1, finish=None) -> None:
     """The CUDA-core kernel over `count` rows of the step (all of them if `token_list` is None)."""
     flag = _same_dtype(q, k_cache, v_cache)
     num_pages = k_cache.numel() // (group.page_size * nkv * maps * dk)
     segments, scratch = 1, None
-    if count * nq <= SINK_SPLIT_MAX_ROWS and ctx.max_kv_len > SINK_SEGMENT:
-        segments = -(-ctx.max_kv_len // SINK_SEGMENT)
+    if count * nq <= SINK_SPLIT_MAX_ROWS:
+        segments = key_segments(ctx.max_kv_len, window, SINK_SEGMENT)
+    if segments > 1:
         scratch = _workspace(q.device, count * nq * segments * maps * (dv + 2))
     _check(library().vosti_attention_maps(
         _p(q), _p(k_cache), _p(v_cache), _p(out), _p(ctx.positions), _p(ctx.request_of), _p(group.block_table),
         group.block_table.shape[1], group.page_size, num_pages, _p(token_list), count, nq, nkv, maps, dk, dv,
-        ctypes.c_float(scale), window, _p(bias), 0 if bias is None else bias.shape[1] - 1, _p(sink), _p(scratch),
+        ctypes.c_float(scale), window, _p(bias), 0 if bias is None else bias.shape[1] - 1, _p(sink), ctypes.c_float(softcap), _p(scratch),
         SINK_SEGMENT, segments, *(finish or _NO_FINISH).args(), flag, _p(ctx.status), _stream()), "attention_sink",
         kernels=2 if segments > 1 else 1)
 
 
 def attention_sink(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, group, *, nq: int, nkv: int,
                    dk: int, dv: int, scale: float, window: int, bias: Optional[torch.Tensor],
-                   sink: Optional[torch.Tensor], chunk: int = 0, maps: int = 1,
+                   sink: Optional[torch.Tensor], chunk: int = 0, softcap: float = 0.0, maps: int = 1,
                    finish: Optional["HeadFinish"] = None) -> torch.Tensor:
     """Causal attention of every query row over its request's cached keys (the last `window` of
     them, or with `chunk` those of the query's own chunk of positions), with an optional bias
     table float32 [nq, distances] (base-2 units, the last column serving every larger distance)
-    and an optional sink logit per head (float32 [nq], natural units). Returns [tokens, nq * dv].
+    and an optional sink logit per head (float32 [nq], natural units); `softcap` c > 0 makes the scaled
+    scores c tanh(score / c). Returns [tokens, nq * dv].
     With `maps` = 2 a head has two score maps (queries [tokens, nq, 2, dk], the key cache's entries
     2 * dk wide) over the same values; `finish` (a `HeadFinish`) says how they are combined and what
     else follows the softmax (unit norm, gate).
@@ -1043,7 +1142,7 @@ def attention_sink(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
     if chunk < 0 or window < 0 or (chunk and window):
         raise KernelError("attention_sink: a window or a chunk, not both, and neither negative")
     window = -chunk if chunk else window            # the kernels take a chunk as a negative window
-    common = dict(nq=nq, nkv=nkv, dk=dk, dv=dv, scale=scale, window=window, bias=bias, sink=sink)
+    common = dict(nq=nq, nkv=nkv, dk=dk, dv=dv, scale=scale, window=window, bias=bias, sink=sink, softcap=softcap)
     lib = library()
     tensor_memory = (q.dtype == torch.bfloat16 and dk == dv and nq // nkv <= 16 and maps == 1
                      and lib.vosti_attention_prefill_tc_supported(dk, group.page_size))
@@ -1064,14 +1163,14 @@ def attention_sink(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
             _p(q), _p(k_cache), _p(v_cache), _p(out), _p(scratch), ctypes.c_int64(scratch.numel()), _p(arrivals),
             _p(ctx.extras.get("attention.short_tokens")), count, tokens, _p(ctx.positions), _p(ctx.request_of),
             _p(group.block_table), group.block_table.shape[1], group.page_size, num_pages, nq, nkv, dk, ctx.max_kv_len,
-            ctypes.c_float(scale), window, _p(bias), bias_last, _p(sink), _p(ctx.status), _stream()),
+            ctypes.c_float(scale), window, _p(bias), bias_last, _p(sink), ctypes.c_float(softcap), _p(ctx.status), _stream()),
             "attention_decode_biased")
     if lists["num_long_rows"]:
         _check(lib.vosti_attention_prefill_tc_biased(
             _p(q), _p(k_cache), _p(v_cache), _p(out), _p(ctx.extras.get("attention.long_rows")), lists["num_long_rows"],
             _p(ctx.cu_q), _p(ctx.kv_len), _p(group.block_table), group.block_table.shape[1], group.page_size, num_pages,
             nq, nkv, dk, lists["max_long_q_len"], tokens, ctypes.c_float(scale), window, _p(bias), bias_last, _p(sink),
-            _p(ctx.status), _stream()), "attention_prefill_tc_biased")
+            ctypes.c_float(softcap), _p(ctx.status), _stream()), "attention_prefill_tc_biased")
     if finish is not None:
         return head_finish(out, finish, nq=nq, maps=1, dv=dv)
     return out
@@ -1132,29 +1231,35 @@ def layer_norm_stream(x, weight: Optional[torch.Tensor], bias: Optional[torch.Te
 
 # ---------------------------------------------------------------- latent attention
 def latent_prep(proj: torch.Tensor, qk: torch.Tensor, c_cache: Optional[torch.Tensor], r_cache: Optional[torch.Tensor],
-                norm_w: torch.Tensor, eps: float, ctx, slot_mapping: Optional[torch.Tensor], *, heads: int, dim: int, rot: int,
-                rank: int, freq: Optional[torch.Tensor], magnitude: float) -> torch.Tensor:
+                norm_w: Optional[torch.Tensor], eps: float, ctx, slot_mapping: Optional[torch.Tensor], *, heads: int, dim: int,
+                rot: int, rank: int, freq: Optional[torch.Tensor], magnitude: float, interleaved: bool = False,
+                head_gate: bool = True) -> Optional[torch.Tensor]:
     """After the q | down | gate projection (csrc/attention_latent.cu): the rotated part of every
     query head goes to the last `rot` columns of qk [tokens, heads, rank + rot]; the latent
     (root-mean-square normed with `norm_w`) and the rotated shared key part go to their cache
-    slots; returns sigmoid(gate) float32 [tokens, heads]."""
+    slots; with `head_gate` returns sigmoid of the columns after `down`, float32 [tokens, heads]. Without
+    caches (a run that reads another layer's) and head gate the projection needs query columns only;
+    further columns may follow what is read."""
     proj = materialize(proj)
     _contig(proj, qk, c_cache, r_cache, norm_w, slot_mapping, freq)
     flag = _same_dtype(proj, qk, c_cache, r_cache)
     tokens = proj.shape[0]
-    if proj.shape[1] != heads * (dim + rot) + rank + rot + heads or tuple(qk.shape) != (tokens, heads, rank + rot):
+    if tuple(qk.shape) != (tokens, heads, rank + rot):
         raise KernelError("latent_prep: widths do not match the head sizes")
-    gate = torch.empty((tokens, heads), dtype=torch.float32, device=proj.device)
+    gate = torch.empty((tokens, heads), dtype=torch.float32, device=proj.device) if head_gate else None
     num_slots = 0 if c_cache is None else c_cache.numel() // rank
-    _check(library().vosti_latent_prep(_p(proj), _p(qk), _p(gate), _p(c_cache), _p(r_cache), _p(norm_w), _is_f32(norm_w),
+    _check(library().vosti_latent_prep(_p(proj), ctypes.c_int64(proj.shape[1]), _p(qk), _p(gate), _p(c_cache), _p(r_cache),
+                                       _p(norm_w), 0 if norm_w is None else _is_f32(norm_w),
                                        ctypes.c_float(eps), _p(ctx.positions), _p(slot_mapping), ctypes.c_int64(num_slots),
-                                       tokens, heads, dim, rot, rank, _p(freq), ctypes.c_float(magnitude), flag,
+                                       tokens, heads, dim, rot, rank, _p(freq), int(bool(interleaved)), ctypes.c_float(magnitude), flag,
                                        _p(ctx.status), _stream()), "latent_prep")
     return gate
 
 
-def head_project(x: torch.Tensor, m: torch.Tensor, y: torch.Tensor, *, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """y[t, h, :] = gate[t, h] * (x[t, h, :] @ m[h]) with float32 sums. x [tokens, heads, in],
+def head_project(x: torch.Tensor, m: torch.Tensor, y: torch.Tensor, *, gate: Optional[torch.Tensor] = None,
+                 element_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y[t, h, :] = gate[t, h] * (x[t, h, :] @ m[h]) with float32 sums, or sigmoid(element_gate[t, h, :]) times
+    the product (element_gate [tokens, heads * out], rows may be strided). x [tokens, heads, in],
     m [heads, in, out] and y [tokens, heads, out] may be strided views (unit stride along x's and
     y's last axis); gate float32 [tokens, heads]. A bfloat16 m with a contiguous inner or output
     axis and strides in multiples of 8 runs on the tensor cores (a float32 x as two bfloat16
@@ -1165,6 +1270,11 @@ def head_project(x: torch.Tensor, m: torch.Tensor, y: torch.Tensor, *, gate: Opt
     if tokens and (x.stride(2) != 1 or y.stride(2) != 1):
         raise KernelError("head_project: the last axis of x and y must be contiguous")
     _contig(gate)
+    if element_gate is not None and (gate is not None or tuple(element_gate.shape) != (tokens, heads * m.shape[2])
+                                     or (tokens and element_gate.stride(1) != 1)):
+        raise KernelError("head_project: the element gate is [tokens, heads * out] with contiguous rows, and the only gate")
+    eg = (_p(element_gate), 0 if element_gate is None else _is_f32(element_gate),
+          ctypes.c_int64(0 if element_gate is None else element_gate.stride(0)))
     lib = library()
     if (tokens and m.dtype == torch.bfloat16 and x.dtype in (torch.bfloat16, torch.float32)
             and y.dtype in (torch.bfloat16, torch.float32) and x.data_ptr() % 16 == 0 and m.data_ptr() % 16 == 0
@@ -1175,12 +1285,12 @@ def head_project(x: torch.Tensor, m: torch.Tensor, y: torch.Tensor, *, gate: Opt
                                                 ctypes.c_int64(y.stride(1)), inner, m.shape[2])):
         _check(lib.vosti_head_project_mma(
             _p(x), _is_f32(x), ctypes.c_int64(x.stride(0)), ctypes.c_int64(x.stride(1)), _p(m), ctypes.c_int64(m.stride(0)),
-            ctypes.c_int64(m.stride(1)), ctypes.c_int64(m.stride(2)), _p(gate), _p(y), _is_f32(y), ctypes.c_int64(y.stride(0)),
+            ctypes.c_int64(m.stride(1)), ctypes.c_int64(m.stride(2)), _p(gate), *eg, _p(y), _is_f32(y), ctypes.c_int64(y.stride(0)),
             ctypes.c_int64(y.stride(1)), tokens, heads, inner, m.shape[2], _stream()), "head_project_mma")
         return y
     _check(lib.vosti_head_project(
         _p(x), _is_f32(x), ctypes.c_int64(x.stride(0)), ctypes.c_int64(x.stride(1)), _p(m), _is_f32(m),
-        ctypes.c_int64(m.stride(0)), ctypes.c_int64(m.stride(1)), ctypes.c_int64(m.stride(2)), _p(gate), _p(y), _is_f32(y),
+        ctypes.c_int64(m.stride(0)), ctypes.c_int64(m.stride(1)), ctypes.c_int64(m.stride(2)), _p(gate), *eg, _p(y), _is_f32(y),
         ctypes.c_int64(y.stride(0)), ctypes.c_int64(y.stride(1)), tokens, heads, inner, m.shape[2], _stream()), "head_project")
     return y
 
@@ -1192,15 +1302,19 @@ LATENT_MMA_SPLIT_BELOW = 296   # CTAs (two per SM) below which it cuts the keys
 
 
 def latent_attend(ctx, qk: torch.Tensor, c_cache: torch.Tensor, r_cache: torch.Tensor, group, *, scale: float,
-                  window: int = 0) -> torch.Tensor:
+                  window: int = 0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal softmax attention of every (token, head) row of qk [tokens, heads, rank + rot] over the
     cached latents [pages, 1, page_size, rank] and shared rotated key parts [.., rot] of its
-    request; returns the weighted latents, float32 [tokens, heads, rank]. bfloat16 with a rank of
+    request (the last `window` of them if it is positive); `sink` (float32 [heads], natural units) adds a
+    logit without key or value to every softmax denominator. Returns the weighted latents, float32
+    [tokens, heads, rank]. bfloat16 with a rank of
     128, 256 or 512 and a rotated part in multiples of 32 runs on the tensor cores
     (csrc/attention_latent_mma.cu), everything else on the CUDA cores (csrc/attention_latent.cu)."""
-    _contig(qk, c_cache, r_cache)
+    _contig(qk, c_cache, r_cache, sink)
     flag = _same_dtype(qk, c_cache, r_cache)
     tokens, heads = qk.shape[0], qk.shape[1]
+    if sink is not None and (sink.dtype != torch.float32 or sink.shape[0] != heads):
+        raise KernelError("latent_attend: the sink is float32 [heads]")
     rank, rot = c_cache.shape[-1], r_cache.shape[-1]
     out = torch.empty((tokens, heads, rank), dtype=torch.float32, device=qk.device)
     num_pages = c_cache.shape[0]
@@ -1208,34 +1322,37 @@ def latent_attend(ctx, qk: torch.Tensor, c_cache: torch.Tensor, r_cache: torch.T
     segments, scratch = 1, None
     if not flag and window >= 0 and lib.vosti_latent_attend_mma_fits(rank, rot):
         rows = ctx.max_q_len * heads
-        ctas = -(-rows // (32 if rows > 16 else 16)) * ctx.num_requests
-        if ctas < LATENT_MMA_SPLIT_BELOW and ctx.max_kv_len > LATENT_MMA_SEGMENT:
-            segments = -(-ctx.max_kv_len // LATENT_MMA_SEGMENT)
+        tile = 32 if rows > 16 else 16
+        ctas = -(-rows // tile) * ctx.num_requests
+        if ctas < LATENT_MMA_SPLIT_BELOW:
+            segments = key_segments(ctx.max_kv_len, window, LATENT_MMA_SEGMENT, min(ctx.max_q_len, -(-tile // heads) + 1))
+        if segments > 1:
             scratch = _workspace(qk.device, tokens * heads * segments * (rank + 2))
         _check(lib.vosti_latent_attend_mma(
             _p(qk), _p(c_cache), _p(r_cache), _p(out), _p(ctx.positions), _p(ctx.cu_q), _p(group.block_table),
             group.block_table.shape[1], group.page_size, num_pages, ctx.num_requests, ctx.max_q_len, heads, rank, rot,
-            ctypes.c_float(scale), window, _p(scratch), LATENT_MMA_SEGMENT, segments, _p(ctx.status), _stream()),
+            ctypes.c_float(scale), window, _p(sink), _p(scratch), LATENT_MMA_SEGMENT, segments, _p(ctx.status), _stream()),
             "latent_attend_mma")
         if segments > 1:
-            _check(lib.vosti_latent_merge(_p(scratch), segments, _p(out), tokens, heads, rank, _stream()), "latent_merge")
+            _check(lib.vosti_latent_merge(_p(scratch), segments, _p(out), tokens, heads, rank, _p(sink), _stream()), "latent_merge")
         return out
-    if tokens * heads <= LATENT_SPLIT_MAX_ROWS and ctx.max_kv_len > LATENT_SEGMENT:
-        segments = -(-ctx.max_kv_len // LATENT_SEGMENT)
+    if tokens * heads <= LATENT_SPLIT_MAX_ROWS:
+        segments = key_segments(ctx.max_kv_len, window, LATENT_SEGMENT)
+    if segments > 1:
         scratch = _workspace(qk.device, tokens * heads * segments * (rank + 2))
     _check(lib.vosti_latent_attend(
         _p(qk), _p(c_cache), _p(r_cache), _p(out), _p(ctx.positions), _p(ctx.request_of), _p(group.block_table),
         group.block_table.shape[1], group.page_size, num_pages, None, tokens, heads, rank, rot, ctypes.c_float(scale),
-        window, _p(scratch), LATENT_SEGMENT, segments, flag, _p(ctx.status), _stream()), "latent_attend",
+        window, _p(sink), _p(scratch), LATENT_SEGMENT, segments, flag, _p(ctx.status), _stream()), "latent_attend",
         kernels=2 if segments > 1 else 1)
     return out
 
 
 # ---------------------------------------------------------------- selective scan
 def scan_conv(xz: torch.Tensor, conv_w: torch.Tensor, conv_b: Optional[torch.Tensor], state: torch.Tensor, tail_offset: int,
-              ctx, *, inner: int, taps: int) -> torch.Tensor:
-    """silu(causal convolution) of the first `inner` columns of xz [tokens, >= inner] per channel
-    (csrc/selective_scan.cu); the inputs before a portion come from the tail [taps - 1, inner] kept
+              ctx, *, inner: int, taps: int, plain: bool = False) -> torch.Tensor:
+    """silu(causal convolution) of the first `inner` columns of xz [tokens, >= inner] per channel, or with
+    `plain` the columns plus their convolution, without SiLU or bias (csrc/selective_scan.cu); the inputs before a portion come from the tail [taps - 1, inner] kept
     `tail_offset` floats into the request's state slot, which is then moved on."""
     xz = materialize(xz)
     _contig(xz, conv_w, conv_b, state)
@@ -1246,7 +1363,7 @@ def scan_conv(xz: torch.Tensor, conv_w: torch.Tensor, conv_b: Optional[torch.Ten
     _check(library().vosti_scan_conv(
         _p(xz), ctypes.c_int64(xz.shape[1]), _p(conv_w), _p(conv_b), _is_f32(conv_w), _p(state), ctypes.c_int64(state.shape[1]),
         ctypes.c_int64(tail_offset), _p(ctx.request_of), _p(ctx.cu_q), _p(ctx.state_slots), state.shape[0], ctx.num_requests,
-        tokens, inner, taps, _p(out), _is_f32(xz), _p(ctx.status), _stream()), "scan_conv", kernels=2 if taps > 1 else 1)
+        tokens, inner, taps, int(bool(plain)), _p(out), _is_f32(xz), _p(ctx.status), _stream()), "scan_conv", kernels=2 if taps > 1 else 1)
     return out
 
 
@@ -1436,6 +1553,36 @@ def moe_router_scored(x: torch.Tensor, router: torch.Tensor, top: int, *, identi
                                              _p(correction), groups, keep, int(gate_row), ctypes.c_float(scale), _p(chosen),
                                              _p(weights), _p(dense), _p(ident), _p(logits), _stream()), "moe_router_scored")
     return (chosen, weights, dense, ident, logits) if want_logits else (chosen, weights, dense, ident)
+
+
+def _table_args(ids: torch.Tensor, table: torch.Tensor):
+    _contig(ids, table)
+    if ids.dtype != torch.int32 or table.dtype != torch.int32 or table.dim() != 2:
+        raise KernelError("moe: token ids and the table [vocab, top] are int32")
+    return _p(ids), _p(table), table.shape[0], table.shape[1], ctypes.c_float(1.0 / table.shape[1])
+
+
+def moe_table(ids: torch.Tensor, table: torch.Tensor, experts: int, want_dense: bool = False):
+    """Experts by token id: (chosen int32 [tokens, top] = table[ids], weights float32 [tokens, top], all
+    1 / top, and with `want_dense` the same as a matrix [tokens, experts], else None)."""
+    args = _table_args(ids, table)
+    tokens, top = ids.shape[0], table.shape[1]
+    chosen = torch.empty((tokens, top), dtype=torch.int32, device=ids.device)
+    weights = torch.empty((tokens, top), dtype=torch.float32, device=ids.device)
+    dense = torch.empty((tokens, experts), dtype=torch.float32, device=ids.device) if want_dense else None
+    _check(library().vosti_moe_table(*args, tokens, experts, _p(chosen), _p(weights), _p(dense), _stream()), "moe_table")
+    return chosen, weights, dense
+
+
+def moe_scale_table(act: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, ff: int) -> torch.Tensor:
+    """act[t, e * ff + i] <- act[t, e * ff + i] / top where the row of t's id lists expert e, else 0, in place."""
+    args = _table_args(ids, table)
+    _contig(act)
+    if act.shape[1] % ff or ids.shape[0] != act.shape[0]:
+        raise KernelError("moe_scale: the activation's width does not match the experts' width")
+    _check(library().vosti_moe_scale_table(_p(act), *args, act.shape[0], act.shape[1] // ff, ff, _is_f32(act), _stream()),
+           "moe_scale")
+    return act
 
 
 MOE_ACTIVATIONS = {None: 0, "gelu": 1, "relu2": 2}

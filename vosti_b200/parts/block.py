@@ -8,14 +8,16 @@ returns (feed_forward_out, residual); the model's final norm does the last add.
 """
 from __future__ import annotations
 
-from typing import Dict
+import dataclasses
+from typing import Dict, Optional
 
 import torch
 
 from .. import ops
 from ..config.schema import ConfigError, LayerSpec
 from ..weights.loader import WeightSpec
-from .base import Norm, build_feed_forward, build_mixer, build_norm, build_token_input, part_factory, register_part
+from .base import (Norm, StateSpec, build_feed_forward, build_mixer, build_norm, build_token_input, part_factory, register_part)
+from .linear import linear, prepare_weight
 
 
 class PreNormBlock:
@@ -46,6 +48,9 @@ class PreNormBlock:
     def setup(self, device, dtype):
         for _, part in self._children():
             part.setup(device, dtype)
+
+    def state_spec(self):
+        return self.mixer.state_spec()
 
     def forward(self, ctx, hidden, residual, cache, writes_cache=True):
         # In a step of few tokens a norm leaves HBM idle: it is told which weight the product
@@ -132,6 +137,9 @@ class ParallelBlock:
         for _, part in self._children():
             part.setup(device, dtype)
 
+    def state_spec(self):
+        return self.mixer.state_spec()
+
     def forward(self, ctx, hidden, residual, cache, writes_cache=True):
         normed, residual = self.norm.forward_add(ctx, hidden, residual)
         mixed = self.mixer.forward(ctx, normed, cache, writes_cache)
@@ -200,6 +208,9 @@ class StreamPreNormBlock:
         for _, part in self._children():
             part.setup(device, dtype)
 
+    def state_spec(self):
+        return self.mixer.state_spec()
+
     def forward(self, ctx, hidden, residual, cache, writes_cache=True):
         if residual is None and isinstance(hidden, torch.Tensor) and hidden.dtype == torch.float32:
             residual, normed = hidden, self.input_norm.forward(ctx, hidden)      # float32 embedding rows are the stream
@@ -267,7 +278,6 @@ class SandwichStreamBlock(StreamPreNormBlock):
             yield n("ff_scale"), "ff_scale", self.feed_forward is None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        import dataclasses
         specs = super().weight_specs()
         for name, _, unused in self._scales():
             specs[name] = WeightSpec((self.mixer.hidden_size,), init="norm", std=0.1, optional=unused)
@@ -325,7 +335,6 @@ class PostNormStreamBlock(StreamPreNormBlock):
                 raise ConfigError("post_norm_stream block: the norm must be a root-mean-square norm over the stream (rms_stream)")
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        import dataclasses
         specs = super().weight_specs()
         if self.feed_forward is None:
             fragment = self.spec.name_of("post_norm")
@@ -355,3 +364,103 @@ class PostNormStreamBlock(StreamPreNormBlock):
 
 
 register_part("arrangement", "post_norm_stream", PostNormStreamBlock, replace=True)
+
+
+class GatedStreamBlock(StreamPreNormBlock):
+    """'gated_pre_norm_stream': pre-norm over a float32 residual stream whose sublayers join it through
+    gates made of their own normed input, and an optional causal convolution on what the mixer reads,
+
+        h = norm1(x),  x <- x + m s(R1 h + r1) * mixer(h + conv(h))
+        h = norm2(x),  x <- x + m s(R2 h + r2) * ff(h)
+
+    s the logistic function, m = `LayerSpec.residual_scale`; `LayerSpec.input_conv` taps (0: no
+    convolution). The convolution's last inputs are per-request state of the block, so the mixer
+    keeps none. The norm is a root-mean-square norm over the stream (`rms_stream`). One kernel per sublayer boundary
+    applies the gate to the output before it, adds it, norms, and, in steps of one token a request,
+    convolves (`ops.gated_rms_stream`); longer portions convolve in a kernel of their own (`ops.scan_conv`).
+    The gate's product runs before the sublayer, and both leave their K splits to that kernel.
+
+    Checkpoint names: `LayerSpec.names` maps the roles "input_norm", "post_norm", "mixer",
+    "feed_forward", "input_conv" ([width, taps]), "mixer_gate" and "ff_gate" ([width, width], their
+    biases `<fragment>.b`) to name fragments; a norm's `weight` and those are called by the fragment
+    itself, every other tensor `<fragment>.<key>`. Of a layer without a feed-forward a checkpoint may
+    carry the second norm and gate all the same."""
+
+    def __init__(self, spec: LayerSpec, hidden_size: int):
+        super().__init__(spec, hidden_size)
+        if spec.token_input is not None or spec.out_norm is not None or spec.layer_scale:
+            raise ConfigError("gated_pre_norm_stream block: it takes no token input, output norm or layer scale")
+        self.width, self.scale, self.taps = hidden_size, float(spec.residual_scale), int(spec.input_conv)
+        if not 0 <= self.taps <= 64:
+            raise ConfigError("gated_pre_norm_stream block: input_conv is between 0 and 64 taps")
+        if self.taps and self.mixer.state_spec() is not None:
+            raise ConfigError("gated_pre_norm_stream block: the state slot holds the convolution's inputs; the mixer keeps none")
+        self.unused_post_norm = build_norm(spec.norm, hidden_size) if self.post_norm is None else None
+        for norm in (self.input_norm, self.post_norm):
+            if norm is not None and not hasattr(norm, "forward_gated"):
+                raise ConfigError("gated_pre_norm_stream block: the norm must be a root-mean-square norm over the stream (rms_stream)")
+        self.conv_w = self.conv = None
+        self.gates = {}
+
+    def state_spec(self) -> Optional[StateSpec]:
+        if self.taps == 0:
+            return self.mixer.state_spec()
+        return StateSpec((max(4, ((self.taps - 1) * self.width + 3) // 4 * 4),), torch.float32)
+
+    def _gates(self):
+        """(role, whether the layer reads it)."""
+        return (("mixer_gate", True), ("ff_gate", self.feed_forward is not None))
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        specs, n, w = super().weight_specs(), self.spec.name_of, self.width
+        if self.taps:
+            specs[n("input_conv")] = WeightSpec((w, self.taps), std=0.3)
+        for role, used in self._gates():
+            specs[n(role)] = WeightSpec((w, w), optional=not used)
+            specs[n(role) + ".b"] = WeightSpec((w,), std=0.1, optional=not used)
+        if self.unused_post_norm is not None:
+            for key, s in self.unused_post_norm.weight_specs().items():
+                specs[n("post_norm") if key == "weight" else f"{n('post_norm')}.{key}"] = dataclasses.replace(s, optional=True)
+        return specs
+
+    def load(self, tensors, dtype):
+        super().load(tensors, dtype)
+        n = self.spec.name_of
+        for role, used in self._gates():
+            if used:
+                self.gates[role] = (prepare_weight(tensors[n(role)], dtype), tensors[n(role) + ".b"])
+        if self.taps:
+            self.conv_w = tensors[n("input_conv")].contiguous()
+            self.conv = self.conv_w.float().t().contiguous()            # [taps, width]: a thread's channels lie side by side
+
+    def extra_weights(self):
+        """Weights a step reads whole that are not a part's (for the count of bytes)."""
+        return [w for w, _ in self.gates.values()]
+
+    def _gated(self, ctx, role, h, run):
+        weight, bias = self.gates[role]
+        z = linear(ctx, h, weight, out_dtype=torch.float32, allow_partial=True, scratch="split_k_gate")
+        return ops.DeferredGated(run(), z, bias, self.scale)
+
+    def forward(self, ctx, hidden, residual, cache, writes_cache=True):
+        if residual is None:
+            hidden = ops.materialize(hidden)                            # the embedding's rows start the stream
+            residual, pending = (hidden if hidden.dtype == torch.float32 else ops.stream_sum(None, hidden)), None
+        elif isinstance(hidden, ops.DeferredGated):
+            pending = hidden
+        else:
+            residual, pending = ops.stream_sum(residual, hidden), None
+        if self.taps and ctx.all_decode:
+            h, u = self.input_norm.forward_gated(ctx, pending, residual, conv=ops.StreamConv(self.conv, cache.state))
+        else:
+            h = u = self.input_norm.forward_gated(ctx, pending, residual)
+            if self.taps:
+                u = ops.scan_conv(h, self.conv_w, None, cache.state, 0, ctx, inner=self.width, taps=self.taps, plain=True)
+        out = self._gated(ctx, "mixer_gate", h, lambda: self.mixer.forward(ctx, u, cache, writes_cache))
+        if self.feed_forward is not None:
+            h = self.post_norm.forward_gated(ctx, out, residual)
+            out = self._gated(ctx, "ff_gate", h, lambda: self.feed_forward.forward(ctx, h))
+        return out, residual
+
+
+register_part("arrangement", "gated_pre_norm_stream", GatedStreamBlock, replace=True)

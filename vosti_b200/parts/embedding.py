@@ -3,7 +3,9 @@ optionally multiplied by a constant `scale` in float32 (Qwen3 has none; architec
 scale their embeddings by sqrt(hidden) name it in their spec). `out_dtype` "float32" gives float32
 rows whatever the table's type: the start of a float32 residual stream (in bfloat16 serving the
 same kernel writes the rows' rounding beside them and the part returns both, an `ops.StreamPair`,
-for arrangements whose sublayers read the rounded stream).
+for arrangements whose sublayers read the rounded stream; `rounded` false leaves the rounding out).
+With `publish_ids` the step's token ids, those a sampler left on the device filled in, appear in
+`ctx.extras["token_ids"]` for parts that read them again.
 """
 from __future__ import annotations
 
@@ -24,6 +26,8 @@ class TableEmbedding(Embedding):
         if not self.scale == self.scale or self.scale in (float("inf"), float("-inf")):
             raise ConfigError("embedding: scale must be a finite number")
         self.out_dtype = torch.float32 if spec.get("out_dtype") == "float32" else None
+        self.rounded = bool(spec.get("rounded", True))
+        self.publish_ids = bool(spec.get("publish_ids", False))
         self.weight = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -36,9 +40,14 @@ class TableEmbedding(Embedding):
         return self.weight
 
     def forward(self, ctx, tokens, feedback=None):
-        pair = self.out_dtype == torch.float32 and ctx.dtype == torch.bfloat16 and self.weight.dtype == torch.bfloat16
+        pair = (self.rounded and self.out_dtype == torch.float32 and ctx.dtype == torch.bfloat16
+                and self.weight.dtype == torch.bfloat16)
+        resolved = None
+        if self.publish_ids:
+            resolved = torch.empty((tokens.shape[0],), dtype=torch.int32, device=self.weight.device)
+            ctx.extras["token_ids"] = resolved
         return ops.embedding(tokens, self.weight, ctx.status, feedback=feedback, scale=self.scale, out_dtype=self.out_dtype,
-                             rounded=pair)
+                             rounded=pair, resolved=resolved)
 
 
 register_part("embedding", "table", TableEmbedding, replace=True)

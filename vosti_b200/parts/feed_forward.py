@@ -48,10 +48,10 @@ def stack_gate_up(gate: torch.Tensor, up: torch.Tensor, dtype: torch.dtype, acti
     return prepare_weight(blocks.reshape(2 * inter, h).contiguous(), dtype), True
 
 
-def gated_activation(ctx, x, w_gate_up, fused: bool, activation: str = "silu"):
+def gated_activation(ctx, x, w_gate_up, fused: bool, activation: str = "silu", glu=(0.0, 0.0)):
     if fused:
-        return ops.gemm_tc(ops.materialize(x), w_gate_up, ctx.status, swiglu=True, activation=activation)
-    return ops.glu_mul(ops.materialize(linear(ctx, x, w_gate_up)), activation)
+        return ops.gemm_tc(ops.materialize(x), w_gate_up, ctx.status, swiglu=True, activation=activation, glu=glu)
+    return ops.glu_mul(ops.materialize(linear(ctx, x, w_gate_up)), activation, *glu)
 
 
 class SwiGLU(FeedForward):
@@ -115,6 +115,12 @@ class ExpertMixture(FeedForward):
     one pass that adds their share of the input. Long portions take the sorted way described below
     too: identity rows are runs that are copied, the shared expert runs over all tokens afterwards.
 
+    With `route` "table" there is no router: `table` [vocab, top] (integers, the entries of a row differ)
+    names the experts of every token id, each with weight 1 / top; the step's ids come from the
+    model's embedding part (`ctx.extras["token_ids"]`; `vocab`). Experts with a gate may be "clamped"
+    (`activation`): g sigmoid(`sigmoid_scale` g) (u + 1) of g = min(gate x, `limit`) and u = up x clamped to
+    [-limit, limit].
+
     The router's logits are float32. The experts' gate and up matrices stand side by side as one
     [2 * experts * I, hidden] matrix and their down matrices as one [hidden, experts * I]: every
     token's activation is computed for all experts by one product, each expert's slice is
@@ -149,11 +155,20 @@ class ExpertMixture(FeedForward):
         self.shared = int(spec.get("shared", 0) or 0)
         self.partial_out = bool(spec.get("partial_out", False))
         self.activation = spec.get("activation") or ("gelu" if not self.gated else None)
+        self.glu, self.gate_activation = (0.0, 0.0), "silu"
+        self.table, self.vocab = None, int(spec.get("vocab", 0) or 0)
+        if self.gated and self.activation == "clamped":
+            self.gate_activation, self.activation = "clamped", None
+            self.glu = (float(spec["limit"]), float(spec["sigmoid_scale"]))
+            if not self.glu[0] > 0:
+                raise ConfigError("moe: the clamped activation's limit must be positive")
         self.correction = None
         if self.experts <= 0 or not 0 < self.top <= self.experts + self.identity or self.inter <= 0:
             raise ConfigError("moe: experts, top (at most experts) and intermediate_size must be positive")
-        if self.route not in ("top_softmax", "softmax_renorm", "scored") or self.scale != self.scale:
-            raise ConfigError("moe: route is 'top_softmax', 'softmax_renorm' or 'scored' and scale a number")
+        if self.route not in ("top_softmax", "softmax_renorm", "scored", "table") or self.scale != self.scale:
+            raise ConfigError("moe: route is 'top_softmax', 'softmax_renorm', 'scored' or 'table' and scale a number")
+        if self.route == "table" and (not self.gated or self.scale != 1.0 or self.vocab <= 0):
+            raise ConfigError("moe: route 'table' takes gated experts, no scale, and the size of the vocabulary")
         if self.route != "scored" and (self.identity or self.has_correction or self.groups != 1 or self.shared
                                        or self.activation not in (None, "gelu")):
             raise ConfigError("moe: identity experts, a correction, groups, a shared expert and other activations need route 'scored'")
@@ -170,7 +185,10 @@ class ExpertMixture(FeedForward):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         h, i = self.hidden_size, self.inter
-        specs = {"router": WeightSpec((self.experts + self.identity, h), std=0.5)}
+        if self.route == "table":
+            specs = {"table": WeightSpec((self.vocab, self.top), integer=True, distinct_below=self.experts)}
+        else:
+            specs = {"router": WeightSpec((self.experts + self.identity, h), std=0.5)}
         if self.has_correction:
             specs["correction"] = WeightSpec((self.experts + self.identity,), std=0.05)
         if self.shared:
@@ -183,13 +201,18 @@ class ExpertMixture(FeedForward):
         return specs
 
     def load(self, tensors, dtype):
-        self.router = tensors["router"].float().contiguous()        # 32-bit logits from exact 32-bit products
+        if self.route == "table":
+            self.table = tensors["table"].to(torch.int32).contiguous()
+            if self.table.numel() and (int(self.table.min()) < 0 or int(self.table.max()) >= self.experts):
+                raise ConfigError(f"moe: the table names experts outside 0 .. {self.experts - 1}")
+        else:
+            self.router = tensors["router"].float().contiguous()        # 32-bit logits from exact 32-bit products
         if self.route == "scored":
             return self._load_scored(tensors, dtype)
         up = torch.cat([tensors[f"e{e}.up"] for e in range(self.experts)], dim=0)
         if self.gated:
             gate = torch.cat([tensors[f"e{e}.gate"] for e in range(self.experts)], dim=0)
-            self.w_gate_up, self.fused = stack_gate_up(gate, up, dtype)
+            self.w_gate_up, self.fused = stack_gate_up(gate, up, dtype, self.gate_activation)
         else:
             self.w_gate_up, self.fused = prepare_weight(up.contiguous(), dtype), False
         self.w_down = prepare_weight(torch.cat([tensors[f"e{e}.down"] for e in range(self.experts)], dim=1).contiguous(), dtype)
@@ -197,7 +220,7 @@ class ExpertMixture(FeedForward):
         if self.top < self.experts:
             for e in range(self.experts):
                 if self.gated:
-                    gate_up, fused = stack_gate_up(tensors[f"e{e}.gate"], tensors[f"e{e}.up"], dtype)
+                    gate_up, fused = stack_gate_up(tensors[f"e{e}.gate"], tensors[f"e{e}.up"], dtype, self.gate_activation)
                 else:
                     gate_up, fused = prepare_weight(tensors[f"e{e}.up"], dtype), False
                 self.per_expert.append((gate_up, fused, prepare_weight(tensors[f"e{e}.down"], dtype)))
@@ -267,7 +290,7 @@ class ExpertMixture(FeedForward):
     def _activation(self, ctx, x, w_first, fused, dense=None):
         """An expert's (or all experts') hidden activation, times the dense weights if given."""
         if self.gated:
-            act = gated_activation(ctx, x, w_first, fused)
+            act = gated_activation(ctx, x, w_first, fused, self.gate_activation, self.glu)
             return act if dense is None else ops.moe_scale(act, dense, self.inter)
         return ops.moe_scale(ops.materialize(linear(ctx, x, w_first)), dense, self.inter, gelu=True)
 
@@ -283,10 +306,25 @@ class ExpertMixture(FeedForward):
                 y[lo:hi].copy_(linear(ctx, act, down, out_dtype=torch.float32))
         return ops.moe_combine(y, where, weights)
 
+    def _forward_table(self, ctx, x):
+        ids = ctx.extras.get("token_ids")
+        if ids is None:
+            raise ConfigError("moe: route 'table' needs the step's token ids, which the model's embedding does not publish")
+        if (self.per_expert and x.shape[0] >= self.GROUPED_FROM and not getattr(ctx, "all_decode", True)
+                and not torch.cuda.is_current_stream_capturing()):
+            chosen, weights, _ = ops.moe_table(ids, self.table, self.experts)
+            y = self._grouped(ctx, x, chosen, weights)
+        else:
+            act = ops.moe_scale_table(self._activation(ctx, x, self.w_gate_up, self.fused), ids, self.table, self.inter)
+            y = linear(ctx, act, self.w_down, out_dtype=torch.float32, allow_partial=self.partial_out)
+        return y if self.float32_out else ops.stream_sum(None, ops.materialize(y), out_dtype=x.dtype)
+
     def forward(self, ctx, x):
         x = ops.materialize(x)
         if self.route == "scored":
             return self._forward_scored(ctx, x)
+        if self.route == "table":
+            return self._forward_table(ctx, x)
         chosen, weights, dense = ops.moe_router(x, self.router, self.top, over_all=self.route == "softmax_renorm", scale=self.scale)
         if (self.per_expert and x.shape[0] >= self.GROUPED_FROM and not getattr(ctx, "all_decode", True)
                 and not torch.cuda.is_current_stream_capturing()):

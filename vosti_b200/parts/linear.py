@@ -34,10 +34,11 @@ def prepare_weight(w: torch.Tensor, serving_dtype: torch.dtype):
 
 def linear(ctx, x: torch.Tensor, w: torch.Tensor, *, out_dtype: Optional[torch.dtype] = None,
            row_index: Optional[torch.Tensor] = None, allow_partial: bool = False,
-           bias: Optional[torch.Tensor] = None):
+           bias: Optional[torch.Tensor] = None, scratch: str = "split_k"):
     """y = x @ w.T (+ bias). With `allow_partial` the result may come back as an `ops.PartialSum`
     (the K splits not yet summed) for a consumer that adds them itself; the caller must hand it
-    to such a consumer, or to `ops.materialize`, before any other product runs. With a `bias`
+    to such a consumer, or to `ops.materialize`, before any other product into the same `scratch`
+    buffer runs. With a `bias`
     (a vector of w's row count, float32 or bfloat16) the product is taken in float32, the bias
     is added there and the sum is rounded once; such a result is never partial."""
     x = ops.materialize(x)
@@ -51,5 +52,5 @@ def linear(ctx, x: torch.Tensor, w: torch.Tensor, *, out_dtype: Optional[torch.d
     if uses_tensor_cores(x.dtype, w):
         if row_index is not None:
             x = ops.gather_rows(x, row_index, ctx.status)
-        return ops.gemm_tc(x, w, ctx.status, out_dtype=out_dtype, allow_partial=allow_partial)
+        return ops.gemm_tc(x, w, ctx.status, out_dtype=out_dtype, allow_partial=allow_partial, scratch=scratch)
     return ops.gemm_simt(x, w, ctx.status, out_dtype=out_dtype, row_index=row_index)

@@ -89,8 +89,9 @@ class StreamRMSNorm(Norm):
     x / sqrt(mean(x^2) + eps) * (offset + weight), in float32, rounded to the serving type.
     Parameters: `eps`; `unit_offset` (default false): the weight is stored around zero and one is
     added to it. `forward_add` takes the stream and what is still to be added to it (a tensor or
-    an `ops.DeferredSum`), adds in float32, stores the sum as the new stream and norms it.
-    `out_dtype` "float32" keeps the normed rows unrounded (for a sublayer's output that is itself
+    an `ops.DeferredSum`, or an `ops.DeferredGated`: an output that joins through a gate), adds in
+    float32, stores the sum as the new stream and norms it. `scalar` (default false): the weight is one
+    number for all elements. `out_dtype` "float32" keeps the normed rows unrounded (for a sublayer's output that is itself
     added to the stream)."""
 
     def __init__(self, spec: PartSpec, width: int):
@@ -98,22 +99,38 @@ class StreamRMSNorm(Norm):
         self.eps = float(spec["eps"])
         self.offset = 1.0 if bool(spec.get("unit_offset", False)) else 0.0
         self.float32_out = spec.get("out_dtype") == "float32"
+        self.scalar = bool(spec.get("scalar", False))
         self.width = width
-        self.weight = None
+        self.weight, self.gain = None, 1.0
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        return {"weight": WeightSpec((self.width,), init="linear" if self.offset else "norm", std=0.1)}
+        return {"weight": WeightSpec(() if self.scalar else (self.width,), init="linear" if self.offset else "norm", std=0.1)}
 
     def load(self, tensors, dtype):
         self.weight = tensors["weight"]
+        if self.scalar:
+            self.gain, self.weight = self.offset + float(self.weight.float().item()), None
 
     def _out(self, ctx):
         return torch.float32 if self.float32_out else ctx.dtype
 
+    def forward_gated(self, ctx, x, stream, *, rows=None, conv=None):
+        """`ops.gated_rms_stream` with this norm: x an `ops.DeferredGated` still to be added, or None."""
+        return ops.gated_rms_stream(stream, x, self.eps, self._out(ctx), weight=self.weight, offset=self.offset, gain=self.gain,
+                                    rows=rows, conv=conv, ctx=ctx, status=ctx.status)
+
     def forward(self, ctx, x):
+        if self.scalar:
+            x = ops.materialize(x)
+            return self.forward_gated(ctx, None, x if x.dtype == torch.float32 else ops.stream_sum(None, x))
         return ops.rms_stream(x, self.weight, self.eps, self._out(ctx), offset=self.offset)
 
     def forward_add(self, ctx, x, residual):
+        if isinstance(x, ops.DeferredGated):
+            return self.forward_gated(ctx, x, residual), residual
+        if self.scalar:
+            residual = ops.stream_sum(residual, x)
+            return self.forward_gated(ctx, None, residual), residual
         if residual is None:
             first = ops.materialize(x.terms[0] if isinstance(x, ops.DeferredSum) else x)
             residual = torch.empty(first.shape, dtype=torch.float32, device=first.device)

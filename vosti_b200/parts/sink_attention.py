@@ -14,6 +14,7 @@ of them optional and a parameter of the spec:
   by distance n = i - j: row n below rows // 2, then logarithmic steps,
   min(rows - 1, half + floor(ln(n / half) / ln(far / half) * (rows - half))), which reach the
   last row at distance `far`. The scale does not multiply the bias;
+* `softcap` c > 0: the scaled score becomes c tanh(score / c), before the bias;
 * `sink`: a learned logit per head joins the softmax denominator once, with no key or value;
 * `value_mix`: "source" publishes this layer's values of the step's tokens for later layers;
   "mix" replaces its own values by (1 - l) v + l v_source before they are cached, with the learned
@@ -92,6 +93,9 @@ class SinkAttention(Mixer):
         self.has_sink = bool(spec.get("sink", False))
         self.sink_value = spec.get("sink_value")
         self.chunk = int(spec.get("chunk", 0) or 0)
+        self.softcap = float(spec.get("softcap", 0.0) or 0.0)
+        if self.softcap < 0:
+            raise ConfigError("sink_attention: softcap must be >= 0")
         self.value_mix = spec.get("value_mix")
         if self.value_mix not in (None, "source", "mix"):
             raise ConfigError("sink_attention: value_mix is 'source' or 'mix'")
@@ -159,6 +163,7 @@ class SinkAttention(Mixer):
         wide = max(self.dk, self.dv)
         self.expanded = wide if (self.maps > 1 and ops.attention_heads_supported(dtype, wide, self.nq // self.nkv)
                                  and not self.has_sink and self.sink_value is None and not self.bias_rows) else 0
+        # (a soft cap goes with maps of their own too: every map is capped by itself)
         q_rows, q_bias = tensors["q"], tensors.get("q.b")
         if self.expanded:
             # query heads in the order (kv head, map, head within the kv head's group)
@@ -229,7 +234,7 @@ class SinkAttention(Mixer):
         if self.expanded:
             D, m = self.expanded, self.maps
             each = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq * m, nkv=self.nkv * m, dk=D, dv=D,
-                                      scale=self.scale, window=self.window, bias=None, sink=None, chunk=self.chunk)
+                                      scale=self.scale, window=self.window, bias=None, sink=None, chunk=self.chunk, softcap=self.softcap)
             finish = ops.HeadFinish(lam=self.lam, unit_norm=True, eps=self.out_norm_eps, out_scale=1.0 - self.diff, gate=gate)
             attn = ops.head_finish(each, finish, nq=self.nq, maps=m, dv=self.dv, in_width=D, pair_group=self.nq // self.nkv)
             return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out)
@@ -238,7 +243,7 @@ class SinkAttention(Mixer):
             finish = ops.HeadFinish(lam=self.lam, unit_norm=self.maps == 2, eps=self.out_norm_eps, out_scale=1.0 - self.diff,
                                     gate=gate)
         attn = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq, nkv=self.nkv, dk=self.dk, dv=self.dv,
-                                  scale=self.scale, window=self.window, bias=self.bias_table, sink=self.sink, chunk=self.chunk,
+                                  scale=self.scale, window=self.window, bias=self.bias_table, sink=self.sink, chunk=self.chunk, softcap=self.softcap,
                                   maps=self.maps, finish=finish)
         return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out)
 
@@ -259,8 +264,9 @@ class SinkAttention(Mixer):
                           slot_mapping=group.slot_mapping, temp_coef=self.temp_coef, temp_every=self.temp_every,
                           status=ctx.status, freq=self.freq, magnitude=self.magnitude, v_first=v_source, v_mix=self.mix)
         attn = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq, nkv=self.nkv, dk=self.dk, dv=self.dv,
-                                  scale=self.scale, window=self.window, bias=self.bias_table, sink=self.sink, chunk=self.chunk)
-        return linear(ctx, attn, self.w_o, out_dtype=torch.float32)
+                                  scale=self.scale, window=self.window, bias=self.bias_table, sink=self.sink, chunk=self.chunk,
+                                  softcap=self.softcap)
+        return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out)
 
 
 register_part("mixer", "sink_attention", SinkAttention, replace=True)

@@ -62,6 +62,7 @@ class WeightSpec:
     std: float = 0.02
     integer: bool = False
     optional: bool = False
+    distinct_below: int = 0          # integer tables: a random row holds distinct values below this (0: zeros)
 
 
 def _resident_dtype(stored: torch.dtype, mode: torch.dtype, integer: bool) -> torch.dtype:

@@ -31,7 +31,12 @@ def draw_tensor(name: str, spec: WeightSpec, seed: int, *, device: torch.device 
     """Draw one tensor in float32 and round it once to `dtype`."""
     device = torch.device(device)
     if spec.integer:
-        return torch.zeros(spec.shape, dtype=torch.int32, device=device)
+        if spec.distinct_below <= 0:
+            return torch.zeros(spec.shape, dtype=torch.int32, device=device)
+        # a random permutation per row, cut to the row's length
+        picks = torch.Generator().manual_seed(_stream_seed(seed, name))
+        order = torch.rand((*spec.shape[:-1], spec.distinct_below), generator=picks).argsort(dim=-1)
+        return order[..., : spec.shape[-1]].to(torch.int32).contiguous().to(device)
     generator = torch.Generator(device=device)
     generator.manual_seed(_stream_seed(seed, name))
     if spec.init == "zeros":
