@@ -5,6 +5,9 @@
 //   h  = x / sqrt(mean(x^2) + eps) * (offset + w)     w a vector, or one number `gain`
 //   u  = h + conv(h)                                  (optional) the next mixer's causal convolution
 //
+// y may also be spread over several rows: token t's output is share * the sum of the rows where[t, 0 ..
+// picks - 1] of y (experts' outputs sorted by expert), picks in order, each with its splits.
+//
 // x goes back to the stream in float32, h (rounded to the serving type) is what the next gate and
 // feed-forward read, u what the next mixer reads. y and z may be a product's unsummed K splits
 // (float32 [splits, rows, width]), added in split order. With `rows` the kernel works on the rows
@@ -65,12 +68,16 @@ struct GatedBoundary {
   const float* stream;         // [source rows, width]
   const void* y;               // null: nothing to add
   int y_f32, y_splits;
+  const int* where;            // [source rows, picks]: y's rows of every row; null: row by row
+  int picks;
+  float share;
+  int64_t y_plane;             // one split of y
   const float* z;              // null: no gate
   int z_splits;
   const void* zb;              // the gate's bias, or null
   int zb_f32;
   float mult;
-  int64_t plane;               // source rows * width: one split of y or z
+  int64_t plane;               // source rows * width: one split of z
   const int* rows;             // the rows to make, or null: all
   int source_rows;
   float* stream_out;           // may be the stream; null: not wanted
@@ -107,8 +114,20 @@ gated_rms_stream_kernel(const GatedBoundary a, TO* __restrict__ out, TO* __restr
   auto sum4 = [&](int i) {
     float4 x = *reinterpret_cast<const float4*>(a.stream + from + i);
     if (a.y == nullptr) return x;
-    float4 y = a.y_splits > 1 ? sum_splits4(reinterpret_cast<const float*>(a.y) + from + i, a.y_splits, a.plane)
-                              : load_flex4(a.y, a.y_f32, from + i);
+    auto row4 = [&](int64_t base) {
+      return a.y_splits > 1 ? sum_splits4(reinterpret_cast<const float*>(a.y) + base + i, a.y_splits, a.y_plane)
+                            : load_flex4(a.y, a.y_f32, base + i);
+    };
+    float4 y;
+    if (a.where == nullptr) {
+      y = row4(from);
+    } else {
+      y = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int k = 0; k < a.picks; ++k) {
+        const float4 v = row4((int64_t)a.where[(int64_t)source * a.picks + k] * width);
+        y.x = fmaf(a.share, v.x, y.x); y.y = fmaf(a.share, v.y, y.y); y.z = fmaf(a.share, v.z, y.z); y.w = fmaf(a.share, v.w, y.w);
+      }
+    }
     if (a.z != nullptr) {
       float4 g = sum_splits4(a.z + from + i, a.z_splits, a.plane);
       if (a.zb != nullptr) {
@@ -123,8 +142,15 @@ gated_rms_stream_kernel(const GatedBoundary a, TO* __restrict__ out, TO* __restr
   auto sum1 = [&](int i) {
     float x = a.stream[from + i];
     if (a.y == nullptr) return x;
-    float y = load_flex(a.y, a.y_f32, from + i);
-    for (int s = 1; s < a.y_splits; ++s) y += reinterpret_cast<const float*>(a.y)[s * a.plane + from + i];
+    auto row1 = [&](int64_t base) {
+      float v = load_flex(a.y, a.y_f32, base + i);
+      for (int s = 1; s < a.y_splits; ++s) v += reinterpret_cast<const float*>(a.y)[s * a.y_plane + base + i];
+      return v;
+    };
+    float y = 0.f;
+    if (a.where == nullptr) y = row1(from);
+    else
+      for (int k = 0; k < a.picks; ++k) y = fmaf(a.share, row1((int64_t)a.where[(int64_t)source * a.picks + k] * width), y);
     if (a.z != nullptr) {
       float g = a.z[from + i];
       for (int s = 1; s < a.z_splits; ++s) g += a.z[s * a.plane + from + i];
@@ -212,11 +238,13 @@ gated_rms_stream_kernel(const GatedBoundary a, TO* __restrict__ out, TO* __restr
 }  // namespace
 
 // stream float32 [source_rows, width]; y (or null) float32 or bfloat16 [source_rows, width], or with y_splits
-// > 1 float32 [y_splits, source_rows, width]; z (or null) float32 likewise; zb [width] (or null); `rows`
+// > 1 float32 [y_splits, source_rows, width]; with `where` (int32 [source_rows, picks], every entry a row of y)
+// y has y_rows rows and a row's output is share * the sum of those; z (or null) float32 likewise; zb [width] (or null); `rows`
 // int32 [count] (or null: count = source_rows); stream_out float32 [count, width] (or null; not with
 // `rows`); out, conv_out [count, width] in the output type (conv_out null: no convolution; it needs
 // count = the step's requests, one row each). Without `weight` every element is multiplied by `gain`.
-VOSTI_API int vosti_gated_rms_stream(const float* stream, const void* y, int y_f32, int y_splits, const float* z, int z_splits,
+VOSTI_API int vosti_gated_rms_stream(const float* stream, const void* y, int y_f32, int y_splits, const int* where, int picks,
+                                     float share, int y_rows, const float* z, int z_splits,
                                      const void* zb, int zb_f32, float mult, const int* rows, int count, int source_rows,
                                      float* stream_out, const void* weight, int w_f32, float offset, float gain, float eps,
                                      const float* conv_w, int taps, float* state, int64_t state_stride, int64_t tail_offset,
@@ -225,6 +253,7 @@ VOSTI_API int vosti_gated_rms_stream(const float* stream, const void* y, int y_f
   VOSTI_REQUIRE(count >= 0 && source_rows >= 0 && width > 0, "gated_rms_stream: bad sizes rows=%d width=%d", count, width);
   VOSTI_REQUIRE(stream != nullptr && (out != nullptr || stream_out != nullptr), "gated_rms_stream: a stream and somewhere to write are needed");
   VOSTI_REQUIRE(y_splits >= 1 && (y_splits == 1 || y_f32) && z_splits >= 1, "gated_rms_stream: unsummed splits are float32");
+  VOSTI_REQUIRE(where == nullptr || (y != nullptr && picks >= 1 && y_rows >= 1), "gated_rms_stream: picked rows need their number");
   VOSTI_REQUIRE(z == nullptr || y != nullptr, "gated_rms_stream: a gate without something to gate");
   VOSTI_REQUIRE(rows == nullptr ? count == source_rows : stream_out == nullptr, "gated_rms_stream: the stream is stored for all rows or for none");
   VOSTI_REQUIRE(conv_out == nullptr || (out != nullptr && conv_w != nullptr && taps >= 1 &&
@@ -232,7 +261,8 @@ VOSTI_API int vosti_gated_rms_stream(const float* stream, const void* y, int y_f
                 "gated_rms_stream: the convolution needs its taps and, for more than one, the state slots");
   if (count == 0) return VOSTI_OK;
   GatedBoundary a = {};
-  a.stream = stream; a.y = y; a.y_f32 = y_f32; a.y_splits = y_splits; a.z = z; a.z_splits = z_splits; a.zb = zb; a.zb_f32 = zb_f32;
+  a.stream = stream; a.y = y; a.y_f32 = y_f32; a.y_splits = y_splits; a.where = where; a.picks = picks; a.share = share;
+  a.y_plane = (int64_t)(where != nullptr ? y_rows : source_rows) * width; a.z = z; a.z_splits = z_splits; a.zb = zb; a.zb_f32 = zb_f32;
   a.mult = mult; a.plane = (int64_t)source_rows * width; a.rows = rows; a.source_rows = source_rows; a.stream_out = stream_out;
   a.weight = weight; a.w_f32 = w_f32; a.offset = offset; a.gain = gain; a.eps = eps; a.conv_w = conv_w; a.taps = taps; a.state = state;
   a.state_stride = state_stride; a.tail_offset = tail_offset; a.state_slots = state_slots; a.num_slots = num_slots; a.width = width;

@@ -424,6 +424,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 }
 
 #include "gemm_tc_pair.cuh"
+#include "gemm_tc_grouped.cuh"
 
 // Sum the K splits in split order and apply the epilogue.
 __global__ void splitk_reduce_kernel(const float* __restrict__ partial, void* __restrict__ out, int splits,
@@ -514,10 +515,122 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int tokens, 
   return 0;
 }
 
+int device_sms() {
+  static int sms = 0;
+  if (sms == 0) {
+    int device = 0;
+    cudaGetDevice(&device);
+    if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess || sms <= 0) sms = 148;
+  }
+  return sms;
+}
+
+template <int BN, int STAGES>
+int launch_grouped_few(const CUtensorMap& mw, const CUtensorMap& mx, void* out, const int* offsets, int experts, int busy, int rows,
+                       int features, int tiles_per_expert, int k_blocks, int ld_out, int epilogue, int splits, int w_tiles, int x_rows,
+                       const GluConstants& glu, unsigned* status, cudaStream_t stream) {
+  constexpr size_t smem = (size_t)STAGES * (A_BYTES + BN * BK * 2) + 1024;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_grouped_few_kernel<BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) {
+      vosti_set_error("gemm_tc_grouped: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+      return (int)e;
+    }
+    configured = true;
+  }
+  vosti_launch(gemm_tc_grouped_few_kernel<BN, STAGES>, dim3(tiles_per_expert, busy, splits), dim3(THREADS), smem, stream, mw, mx, out,
+               offsets, experts, rows, features, tiles_per_expert, k_blocks, ld_out, epilogue, w_tiles, x_rows, glu, status);
+  return 0;
+}
+
 }  // namespace
 
 // Whether the tensor-core product takes a [features, k] bfloat16 weight at all.
 VOSTI_API int vosti_gemm_tc_supported(int features, int k) { return features >= 1 && k >= BK && k % 8 == 0; }
+
+// How many K splits a grouped product uses: a function of the sizes only (tokens of the step, (token, pick)
+// rows, experts).
+VOSTI_API int vosti_gemm_tc_grouped_splits(int tokens, int rows, int experts, int features, int k) {
+  if (tokens > 128 || g_vosti_fixed_order) return 1;
+  const int k_blocks = (k + BK - 1) / BK;
+  const int busy = rows < experts ? rows : experts;
+  const int tiles = ((features + BM - 1) / BM) * busy;
+  int splits = ((tokens <= 64 ? 2 : 1) * 148) / tiles;
+  if (splits > k_blocks / 4) splits = k_blocks / 4;         // at least 4 k-blocks (256 elements) per split
+  if (splits > 16) splits = 16;
+  return splits < 1 ? 1 : splits;
+}
+
+// Products of experts with their own rows (gemm_tc_grouped.cuh): x bf16 [rows, k] sorted by expert, offsets int32
+// [experts + 1] on the device; w packed: every expert's [features, k] padded to whole tiles of 128 features, one
+// expert after the other in one packed weight. `tokens`: how many tokens the step has, which no expert's
+// row count exceeds. Outputs as vosti_gemm_tc ([rows, features], or [rows, features / 2] for gated
+// epilogues); with more than one split and `defer_reduce` the sums stay in the workspace
+// [splits, rows, features].
+VOSTI_API int vosti_gemm_tc_grouped(const void* x, const void* w, void* y, const int* offsets, int tokens, int rows, int experts,
+                                    int features, int k, int epilogue, float* workspace, int64_t workspace_elems, int defer_reduce,
+                                    float glu_limit, float glu_sigmoid_scale, unsigned* status, cudaStream_t stream) {
+  VOSTI_REQUIRE(rows >= 0 && tokens >= 0 && experts > 0 && vosti_gemm_tc_supported(features, k), "gemm_tc_grouped: unsupported sizes F=%d K=%d", features, k);
+  VOSTI_REQUIRE((epilogue >= EPI_BF16 && epilogue <= EPI_SWIGLU) || is_gated(epilogue), "gemm_tc_grouped: unknown epilogue %d", epilogue);
+  VOSTI_REQUIRE(!is_gated(epilogue) || features % 32 == 0, "gemm_tc_grouped: a fused act(gate)*up needs features %% 32 == 0");
+  VOSTI_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0), "gemm_tc_grouped: operands must be 16-byte aligned");
+  VOSTI_REQUIRE(offsets != nullptr, "gemm_tc_grouped: the experts' row ranges are missing");
+  if (rows == 0) return VOSTI_OK;
+  const GluConstants glu = {glu_limit, glu_sigmoid_scale};
+  const int ld_out = is_gated(epilogue) ? features / 2 : features;
+  const int k_blocks = (k + BK - 1) / BK;
+  const int tiles_per_expert = (features + BM - 1) / BM;
+  const int64_t w_rows64 = (int64_t)k_blocks * experts * tiles_per_expert * BM;
+  VOSTI_REQUIRE(w_rows64 < (int64_t)1 << 31, "gemm_tc_grouped: the stacked experts are too large");
+  const int w_tiles = experts * tiles_per_expert, w_rows = (int)w_rows64;
+  CUtensorMap mw, mx;
+  if (tokens > 128) {
+    VOSTI_REQUIRE(weight_map(w, w_rows, BK, WIDE_BN, &mw) && make_map(&mx, x, rows, k, BM), "gemm_tc_grouped: cuTensorMapEncodeTiled failed");
+    constexpr size_t smem = (size_t)WIDE_STAGES * WIDE_STAGE_BYTES + 1024;
+    static bool configured = false;
+    if (!configured) {
+      cudaError_t e = cudaFuncSetAttribute(gemm_tc_grouped_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) {
+        vosti_set_error("gemm_tc_grouped: cannot configure the persistent kernel: %s", cudaGetErrorString(e));
+        return (int)e;
+      }
+      configured = true;
+    }
+    // no more CTAs than there can be tiles
+    const int64_t most = ((int64_t)rows / BM + (rows < experts ? rows : experts)) * ((features + WIDE_BN - 1) / WIDE_BN);
+    const int sms = device_sms();
+    vosti_launch(gemm_tc_grouped_wide_kernel, dim3((unsigned)(most < sms ? most : sms)), dim3(THREADS), smem, stream, mx, mw, y, offsets,
+                 experts, rows, features, tiles_per_expert, k_blocks, ld_out, epilogue, w_tiles, glu, status);
+    VOSTI_LAUNCH_CHECK();
+  }
+  const int splits = vosti_gemm_tc_grouped_splits(tokens, rows, experts, features, k);
+  VOSTI_REQUIRE(splits == 1 || (workspace != nullptr && workspace_elems >= (int64_t)splits * rows * features),
+                "gemm_tc_grouped: workspace too small for %d splits", splits);
+  const int bn = token_tile(tokens);
+  const int x_rows = (tokens + 7) / 8 * 8 < bn ? (tokens + 7) / 8 * 8 : bn;
+  VOSTI_REQUIRE(weight_map(w, w_rows, BK, BM, &mw) && make_map(&mx, x, rows, k, x_rows), "gemm_tc_grouped: cuTensorMapEncodeTiled failed");
+  void* dst = splits > 1 ? (void*)workspace : y;
+  const int epi = splits > 1 ? EPI_PARTIAL : epilogue;
+  const int ld = splits > 1 ? features : ld_out;
+  const int busy = rows < experts ? rows : experts;
+#define VOSTI_GROUPED_ARGS mw, mx, dst, offsets, experts, busy, rows, features, tiles_per_expert, k_blocks, ld, epi, splits, w_tiles, x_rows, glu, status, stream
+  int rc;
+  switch (bn) {
+    case 32: rc = launch_grouped_few<32, 5>(VOSTI_GROUPED_ARGS); break;
+    case 64: rc = launch_grouped_few<64, 4>(VOSTI_GROUPED_ARGS); break;
+    default: rc = launch_grouped_few<128, 6>(VOSTI_GROUPED_ARGS); break;
+  }
+#undef VOSTI_GROUPED_ARGS
+  if (rc != 0) return rc;
+  if (splits > 1 && !defer_reduce) {
+    const int64_t n = (int64_t)rows * features;
+    const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
+    vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)workspace, y, splits, rows, features, ld_out,
+                 epilogue, glu);
+  }
+  VOSTI_LAUNCH_CHECK();
+}
 
 // How many K splits a product of these sizes uses (a function of the sizes only; the
 // sum over splits is taken in split order). With one order of arithmetic asked for

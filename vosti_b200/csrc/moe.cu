@@ -404,6 +404,46 @@ moe_group_kernel(const int* __restrict__ chosen, int pairs, int top, int experts
   }
 }
 
+// Sort and gather in one kernel, for experts by token id: block i takes the (token, pick) pair i, finds its
+// place among the pairs sorted by expert (pairs of lower experts, then earlier pairs of its own: every
+// block counts by itself, so pairs * pairs table reads in all) and copies its token's row there;
+// blocks up to `experts` also count where an expert's rows start.
+template <int BYTES>
+__global__ void __launch_bounds__(256)
+moe_dispatch_kernel(const TokenTable by, int pairs, int experts, const char* __restrict__ x, int64_t row_bytes, char* __restrict__ sorted,
+                    int* __restrict__ offsets, int* __restrict__ where) {
+  __shared__ int counts[2][8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int i = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int mine = i < pairs ? table_row(by, i / by.top)[i % by.top] : -1;
+  int before = 0, start = 0;
+  for (int j = threadIdx.x; j < pairs; j += blockDim.x) {
+    const int e = table_row(by, j / by.top)[j % by.top];
+    before += (e < mine || (e == mine && j < i)) ? 1 : 0;
+    start += e < i ? 1 : 0;
+  }
+  for (int o = 16; o > 0; o >>= 1) {
+    before += __shfl_xor_sync(0xffffffffu, before, o);
+    start += __shfl_xor_sync(0xffffffffu, start, o);
+  }
+  if (lane == 0) { counts[0][warp] = before; counts[1][warp] = start; }
+  __syncthreads();
+  before = start = 0;
+  for (int w = 0; w < 8; ++w) { before += counts[0][w]; start += counts[1][w]; }
+  if (threadIdx.x == 0 && i <= experts) offsets[i] = start;
+  if (i >= pairs) return;
+  if (threadIdx.x == 0) where[i] = before;
+  const char* src = x + (int64_t)(i / by.top) * row_bytes;
+  char* dst = sorted + (int64_t)before * row_bytes;
+  if (BYTES == 16) {
+    for (int64_t c = threadIdx.x; c < row_bytes / 16; c += blockDim.x) reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+  } else {
+    for (int64_t c = threadIdx.x; c < row_bytes / 2; c += blockDim.x)
+      reinterpret_cast<unsigned short*>(dst)[c] = reinterpret_cast<const unsigned short*>(src)[c];
+  }
+}
+
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ where, const float* __restrict__ weights,
                    float* __restrict__ out, int top, int width) {
@@ -426,6 +466,24 @@ VOSTI_API int vosti_moe_group(const int* chosen, int tokens, int top, int expert
   VOSTI_REQUIRE((int64_t)tokens * top < (int64_t)1 << 30, "moe_group: too many pairs");
   vosti_launch(moe_group_kernel, dim3(1), dim3(1024), (size_t)(experts + 1) * sizeof(int), stream, chosen, tokens * top, top,
                experts, offsets, rows, where);
+  VOSTI_LAUNCH_CHECK();
+}
+
+// x: `tokens` rows of row_bytes (a multiple of 2); sorted: [tokens * top] rows; offsets int32 [experts + 1]; where int32
+// [tokens * top], the sorted place of every (token, pick) pair.
+VOSTI_API int vosti_moe_dispatch(const int* ids, const int* table, int vocab, int top, float share, int tokens, int experts, const void* x,
+                                 int64_t row_bytes, void* sorted, int* offsets, int* where, cudaStream_t stream) {
+  VOSTI_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && top <= experts && vocab > 0 && row_bytes > 0 && row_bytes % 2 == 0, "moe_dispatch: bad sizes");
+  VOSTI_REQUIRE((int64_t)tokens * top < (int64_t)1 << 24, "moe_dispatch: too many pairs");
+  VOSTI_REQUIRE(ids != nullptr && table != nullptr, "moe_dispatch: missing arrays");
+  if (tokens == 0) return VOSTI_OK;
+  const int pairs = tokens * top, blocks = pairs > experts + 1 ? pairs : experts + 1;
+  const bool words = row_bytes % 16 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(sorted) & 15) == 0;
+  const TokenTable by = {ids, table, top, vocab, share};
+  if (words)
+    vosti_launch(moe_dispatch_kernel<16>, dim3(blocks), dim3(256), 0, stream, by, pairs, experts, (const char*)x, row_bytes, (char*)sorted, offsets, where);
+  else
+    vosti_launch(moe_dispatch_kernel<2>, dim3(blocks), dim3(256), 0, stream, by, pairs, experts, (const char*)x, row_bytes, (char*)sorted, offsets, where);
   VOSTI_LAUNCH_CHECK();
 }
 

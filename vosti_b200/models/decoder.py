@@ -177,6 +177,8 @@ class DecoderModel:
                     # parts inside a part (the branches of a mixer) and lists of tensors
                     for item in value:
                         for inner in (item if isinstance(item, tuple) else (item,)):
+                            if isinstance(inner, ops.ExpertWeights):
+                                inner = inner.data
                             if isinstance(inner, Part):
                                 visit(inner)
                             elif isinstance(inner, torch.Tensor) and inner.is_cuda:

@@ -375,7 +375,7 @@ class PartialSum:
 
 
 def materialize(x):
-    return x.materialize() if isinstance(x, (PartialSum, StreamPair)) else x
+    return x.materialize() if isinstance(x, (PartialSum, StreamPair, PickedSum)) else x
 
 
 class PackedWeight:
@@ -408,6 +408,51 @@ class PackedWeight:
 
     def element_size(self) -> int:
         return self.data.element_size()
+
+
+class ExpertWeights(PackedWeight):
+    """The [features, k] bfloat16 weights of several experts as one packed weight, every expert's features
+    padded to whole tiles, for products in which every expert has rows of its own (`gemm_tc_grouped`)."""
+
+    def __init__(self, weights):
+        features, k = weights[0].shape
+        pad = -features % self.TILE_F
+        parts = []
+        for w in weights:
+            if tuple(w.shape) != (features, k):
+                raise KernelError("ExpertWeights: the experts' weights share a shape")
+            parts += [w] + ([w.new_zeros((pad, k))] if pad else [])
+        super().__init__(torch.cat(parts, dim=0))
+        self.experts, self.features, self.k = len(weights), features, k
+
+
+def gemm_tc_grouped(x: torch.Tensor, w: ExpertWeights, offsets: torch.Tensor, tokens: int, status: torch.Tensor, *,
+                    out_dtype: torch.dtype = torch.bfloat16, activation: Optional[str] = None, glu=(0.0, 0.0),
+                    allow_partial: bool = False, scratch: str = "split_k"):
+    """y[r] = x[r] @ w[expert of r].T for rows sorted by expert: expert e owns rows offsets[e] .. offsets[e + 1] - 1
+    (int32 [experts + 1], on the device; no expert has more than `tokens` of them). `activation`: the
+    gated epilogue of `gemm_tc` (bfloat16 out, half as many columns). csrc/gemm_tc_grouped.cuh."""
+    _contig(x, w.data, offsets)
+    if x.dtype != torch.bfloat16 or x.shape[1] != w.k or offsets.dtype != torch.int32 or offsets.shape[0] != w.experts + 1:
+        raise KernelError("gemm_tc_grouped: x is bfloat16 [rows, k], offsets int32 [experts + 1]")
+    rows, features = x.shape[0], w.features
+    epilogue, width = (EPI_F32 if out_dtype == torch.float32 else EPI_BF16), features
+    if activation is not None:
+        if out_dtype != torch.bfloat16:
+            raise KernelError("gemm_tc_grouped: the gated epilogues write bfloat16")
+        epilogue, width = FUSED_GLU_ACTIVATIONS[activation], features // 2
+    lib = library()
+    splits = lib.vosti_gemm_tc_grouped_splits(tokens, rows, w.experts, features, w.k)
+    ws = _workspace(x.device, splits * rows * features, scratch) if splits > 1 else None
+    defer = bool(allow_partial and splits > 1 and activation is None)
+    out = None if defer else torch.empty((rows, width), dtype=out_dtype, device=x.device)
+    if splits > 1:
+        _SPLIT_GENERATION[scratch] = _SPLIT_GENERATION.get(scratch, 0) + 1
+    _check(lib.vosti_gemm_tc_grouped(_p(x), _p(w.data), _p(out), _p(offsets), tokens, rows, w.experts, features, w.k, epilogue, _p(ws),
+                                     ctypes.c_int64(ws.numel() if ws is not None else 0), int(defer), ctypes.c_float(glu[0]),
+                                     ctypes.c_float(glu[1]), _p(status), _stream()), "gemm_tc_grouped",
+           kernels=2 if splits > 1 and not defer else 1)
+    return PartialSum(ws, splits, rows, features, out_dtype, status, scratch) if defer else out
 
 
 def gemm_tc(x: torch.Tensor, w, status: torch.Tensor, *, out_dtype: Optional[torch.dtype] = None,
@@ -797,17 +842,33 @@ def rms_stream(x, weight: Optional[torch.Tensor], eps: float, out_dtype: Optiona
     return out
 
 
+class PickedSum:
+    """share * the sum over picks of the rows where[t, pick] of y ([pairs, width] float32, or unsummed K splits
+    of them): experts' outputs sorted by expert that a later kernel (`gated_rms_stream`) adds up per token.
+    `materialize` gives the sums [tokens, width] in float32."""
+
+    def __init__(self, y, where: torch.Tensor, share: float):
+        self.y, self.where, self.share = y, where, float(share)
+        self.shape = (where.shape[0], y.shape[1])
+        self.dtype = torch.float32
+
+    def materialize(self) -> torch.Tensor:
+        weights = torch.full(tuple(self.where.shape), self.share, dtype=torch.float32, device=self.where.device)
+        return moe_combine(materialize(self.y), self.where, weights)
+
+
 class DeferredGated:
     """A sublayer's output y [rows, width] on its way into the float32 stream through a gate: what joins is
     scale * sigmoid(z + bias) * y, z a float32 product of the sublayer's input. The kernel that next reads
     the stream (`gated_rms_stream`) does it; y and z may be unsummed K splits (`PartialSum`, each in a
-    scratch of its own)."""
+    scratch of its own), y also a `PickedSum`."""
 
     def __init__(self, y, z, bias: Optional[torch.Tensor], scale: float):
-        for t in (y, z):
+        inner = y.y if isinstance(y, PickedSum) else y
+        for t in (inner, z):
             if isinstance(t, PartialSum) and t.dtype != torch.float32:
                 raise KernelError("deferred gate: unsummed products are float32")
-        if isinstance(y, PartialSum) and isinstance(z, PartialSum) and y.scratch == z.scratch:
+        if isinstance(inner, PartialSum) and isinstance(z, PartialSum) and inner.scratch == z.scratch:
             raise KernelError("deferred gate: two unsummed products need a scratch each")
         self.y, self.z, self.bias, self.scale = y, z, bias, float(scale)
         self.shape = tuple(y.shape)
@@ -851,7 +912,11 @@ def gated_rms_stream(stream: torch.Tensor, x: Optional[DeferredGated], eps: floa
     source, width = stream.shape
     if x is not None and tuple(x.shape) != (source, width):
         raise KernelError("gated_rms_stream: the sublayer's output does not match the stream")
-    yp, y_f32, y_splits = _splits_of(x.y if x is not None else None)
+    y, where, share = x.y if x is not None else None, None, 1.0
+    if isinstance(y, PickedSum):
+        y, where, share = y.y, y.where, y.share
+        _contig(where)
+    yp, y_f32, y_splits = _splits_of(y)
     zp, z_f32, z_splits = _splits_of(x.z if x is not None else None)
     bias = x.bias if x is not None else None
     _contig(bias)
@@ -872,7 +937,8 @@ def gated_rms_stream(stream: torch.Tensor, x: Optional[DeferredGated], eps: floa
         if stride < (taps - 1) * width:
             raise KernelError("gated_rms_stream: the state slots are too small for the convolution's tail")
     _check(library().vosti_gated_rms_stream(
-        _p(stream), yp, y_f32, y_splits, zp, z_splits, _p(bias), 0 if bias is None else _is_f32(bias),
+        _p(stream), yp, y_f32, y_splits, _p(where), 0 if where is None else where.shape[1], ctypes.c_float(share),
+        0 if where is None else y.shape[0], zp, z_splits, _p(bias), 0 if bias is None else _is_f32(bias),
         ctypes.c_float(x.scale if x is not None else 1.0), _p(rows), count, source, _p(stream) if store else None, _p(weight),
         0 if weight is None else _is_f32(weight), ctypes.c_float(offset), ctypes.c_float(gain), ctypes.c_float(eps), _p(cw),
         taps, _p(cs), ctypes.c_int64(stride), ctypes.c_int64(0), _p(slots), num_slots, _p(out), _p(u), _is_f32(out), width,
@@ -1572,6 +1638,27 @@ def moe_table(ids: torch.Tensor, table: torch.Tensor, experts: int, want_dense: 
     dense = torch.empty((tokens, experts), dtype=torch.float32, device=ids.device) if want_dense else None
     _check(library().vosti_moe_table(*args, tokens, experts, _p(chosen), _p(weights), _p(dense), _stream()), "moe_table")
     return chosen, weights, dense
+
+
+MOE_DISPATCH_PAIRS = 8192        # (token, pick) pairs up to which one kernel sorts and gathers (its counting is quadratic)
+
+
+def moe_dispatch(ids: torch.Tensor, table: torch.Tensor, experts: int, x: torch.Tensor, status: torch.Tensor):
+    """Every token's row once per expert its id is assigned to, sorted by expert: (rows [tokens * top, width], offsets
+    int32 [experts + 1] of the experts' runs, where int32 [tokens, top] the sorted place of every pair)."""
+    args = _table_args(ids, table)
+    _contig(x)
+    tokens, top = ids.shape[0], table.shape[1]
+    if tokens * top > MOE_DISPATCH_PAIRS:
+        chosen, _, _ = moe_table(ids, table, experts)
+        offsets, rows, where = moe_group(chosen, experts)
+        return gather_rows(x, rows, status), offsets, where
+    gathered = torch.empty((tokens * top, x.shape[1]), dtype=x.dtype, device=x.device)
+    offsets = torch.empty((experts + 1,), dtype=torch.int32, device=x.device)
+    where = torch.empty((tokens, top), dtype=torch.int32, device=x.device)
+    _check(library().vosti_moe_dispatch(*args, tokens, experts, _p(x), ctypes.c_int64(x.shape[1] * x.element_size()), _p(gathered),
+                                        _p(offsets), _p(where), _stream()), "moe_dispatch")
+    return gathered, offsets, where
 
 
 def moe_scale_table(act: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, ff: int) -> torch.Tensor:

@@ -43,9 +43,13 @@ def stack_gate_up(gate: torch.Tensor, up: torch.Tensor, dtype: torch.dtype, acti
              and activation in ops.FUSED_GLU_ACTIVATIONS)
     if not fused:
         return stacked.contiguous(), False
-    h = stacked.shape[1]
-    blocks = torch.stack([stacked[:inter].view(-1, 16, h), stacked[inter:].view(-1, 16, h)], dim=1)
-    return prepare_weight(blocks.reshape(2 * inter, h).contiguous(), dtype), True
+    return prepare_weight(interleave_gate_up(stacked[:inter], stacked[inter:]), dtype), True
+
+
+def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """Blocks of 16 gate rows followed by their 16 up rows."""
+    inter, h = gate.shape
+    return torch.stack([gate.view(-1, 16, h), up.view(-1, 16, h)], dim=1).reshape(2 * inter, h).contiguous()
 
 
 def gated_activation(ctx, x, w_gate_up, fused: bool, activation: str = "silu", glu=(0.0, 0.0)):
@@ -117,7 +121,12 @@ class ExpertMixture(FeedForward):
 
     With `route` "table" there is no router: `table` [vocab, top] (integers, the entries of a row differ)
     names the experts of every token id, each with weight 1 / top; the step's ids come from the
-    model's embedding part (`ctx.extras["token_ids"]`; `vocab`). Experts with a gate may be "clamped"
+    model's embedding part (`ctx.extras["token_ids"]`; `vocab`). In bfloat16 serving every step takes a sorted way
+    of its own: one kernel sorts the (token, pick) pairs by expert and gathers their rows, two grouped
+    products (`ops.gemm_tc_grouped`) run every expert over its own rows, on the device's word alone (no host
+    decision, so that decode steps may be recorded; experts without a token are not read), and a token's
+    picks are added by whatever kernel reads the result next. Sizes the grouped product does not take and
+    float32 serving run the ways described above. Experts with a gate may be "clamped"
     (`activation`): g sigmoid(`sigmoid_scale` g) (u + 1) of g = min(gate x, `limit`) and u = up x clamped to
     [-limit, limit].
 
@@ -180,8 +189,8 @@ class ExpertMixture(FeedForward):
                 raise ConfigError("moe: groups must divide experts + identity, and keep lie between 1 and groups")
             if self.top > routed // self.groups * self.keep:
                 raise ConfigError("moe: top exceeds the experts of the kept groups")
-        self.router = self.w_gate_up = self.w_down = None
-        self.fused = False
+        self.router = self.w_gate_up = self.w_down = self.grouped = None
+        self.fused, self.per_expert = False, []
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         h, i = self.hidden_size, self.inter
@@ -209,6 +218,12 @@ class ExpertMixture(FeedForward):
             self.router = tensors["router"].float().contiguous()        # 32-bit logits from exact 32-bit products
         if self.route == "scored":
             return self._load_scored(tensors, dtype)
+        if self.route == "table":
+            rows = self.table.sort(dim=1).values
+            if self.top > 1 and bool((rows[:, 1:] == rows[:, :-1]).any()):
+                raise ConfigError("moe: a row of the table names an expert twice")
+            if self.top < self.experts and self._load_grouped(tensors, dtype):
+                return
         up = torch.cat([tensors[f"e{e}.up"] for e in range(self.experts)], dim=0)
         if self.gated:
             gate = torch.cat([tensors[f"e{e}.gate"] for e in range(self.experts)], dim=0)
@@ -224,6 +239,16 @@ class ExpertMixture(FeedForward):
                 else:
                     gate_up, fused = prepare_weight(tensors[f"e{e}.up"], dtype), False
                 self.per_expert.append((gate_up, fused, prepare_weight(tensors[f"e{e}.down"], dtype)))
+
+    def _load_grouped(self, tensors, dtype) -> bool:
+        """The experts one after the other for the grouped products, if those take their sizes."""
+        downs = [tensors[f"e{e}.down"] for e in range(self.experts)]
+        pairs = [(tensors[f"e{e}.gate"], tensors[f"e{e}.up"]) for e in range(self.experts)]
+        if (dtype != torch.bfloat16 or self.inter % 16 or self.gate_activation not in ops.FUSED_GLU_ACTIVATIONS
+                or not all(uses_tensor_cores(dtype, w) for w in downs + [w for pair in pairs for w in pair])):
+            return False
+        self.grouped = (ops.ExpertWeights([interleave_gate_up(g, u) for g, u in pairs]), ops.ExpertWeights(downs))
+        return True
 
     def _load_scored(self, tensors, dtype):
         ups = [tensors[f"e{e}.up"] for e in range(self.experts)]
@@ -310,7 +335,15 @@ class ExpertMixture(FeedForward):
         ids = ctx.extras.get("token_ids")
         if ids is None:
             raise ConfigError("moe: route 'table' needs the step's token ids, which the model's embedding does not publish")
-        if (self.per_expert and x.shape[0] >= self.GROUPED_FROM and not getattr(ctx, "all_decode", True)
+        if self.grouped is not None:
+            gathered, offsets, where = ops.moe_dispatch(ids, self.table, self.experts, x, ctx.status)
+            act = ops.gemm_tc_grouped(gathered, self.grouped[0], offsets, x.shape[0], ctx.status, activation=self.gate_activation,
+                                      glu=self.glu)
+            y = ops.gemm_tc_grouped(act, self.grouped[1], offsets, x.shape[0], ctx.status, out_dtype=torch.float32,
+                                    allow_partial=self.partial_out)
+            y = ops.PickedSum(y, where, 1.0 / self.top)
+            y = y if self.partial_out else y.materialize()
+        elif (self.per_expert and x.shape[0] >= self.GROUPED_FROM and not getattr(ctx, "all_decode", True)
                 and not torch.cuda.is_current_stream_capturing()):
             chosen, weights, _ = ops.moe_table(ids, self.table, self.experts)
             y = self._grouped(ctx, x, chosen, weights)
