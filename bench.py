@@ -42,6 +42,12 @@ same sizes (`--design-sizes s,m`).
 gated attention and differential attention in turn, dense feed-forwards or, with size moe,
 experts chosen by corrected scores with identity experts and a shared expert) beside Qwen3
 (beside Mugizen where there are experts).
+
+`--design pubulix` does the same for the Pubulix design (gated pre-norm layers over a float32 stream
+with an input convolution: windowed latent attention, capped windowed attention, latent attention
+over the first layer's latents, and capped attention again, clamped experts by token table in every
+layer) beside Beralix, whose attention is closest (at sizes s and m, whose dense feed-forward does the
+work of the two experts a token has), and beside Mugizen's experts (size moe).
 """
 from __future__ import annotations
 
@@ -491,6 +497,47 @@ def nefipel_flops(size, tokens):
     return 2.0 * tokens * per_token + 2.0 * V * W + scores
 
 
+def pubulix_experts(size):
+    """The size's experts, or eight of half the dense feed-forward's width of which a token has two."""
+    return size["moe"] or dict(experts=8, top=2, ff=size["ff"] // 2)
+
+
+def pubulix_config(size):
+    """A Pubulix config.json of these sizes: latent attention (a latent of 512, 64 rotated and 128
+    unrotated elements a head) that keeps its own latents, capped grouped-query attention, latent
+    attention over the first layer's latents, capped attention; windows of 1,024; four taps."""
+    H, G, W, m = size["heads"], size["kv"], size["width"], pubulix_experts(size)
+    mlp = dict(kind="moe", expert=dict(ff=m["ff"], limit=7.0), router=dict(experts=m["experts"], top=m["top"]))
+    latent = dict(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, mask=dict(size=1024),
+                  rot=dict(base=10000.0, dims=64))
+    capped = dict(type="attention", mlp=mlp, mixer=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, softcap=50.0,
+                                                        mask=dict(size=1024), rot=dict(base=10000.0, dims=128)))
+    order = [dict(type="latent_attention", mlp=mlp, mixer=latent), capped,
+             dict(type="latent_attention", mlp=mlp, mixer=dict(latent, kv_from=0)), capped]
+    return dict(architecture="Pubulix", vocab=size["vocab"], width=W, norm=dict(eps=1e-5), canon=dict(taps=4), residual_mult=0.5,
+                embedding=dict(scale=W ** 0.5), logit_softcap=30.0, layers=[order[i % 4] for i in range(size["layers"])])
+
+
+def pubulix_flops(size, tokens):
+    """Multiply-add work of one prompt, times two, for `pubulix_config(size)`, the latent attention as the
+    engine computes it (scores and sums over the cached latents)."""
+    W, H, G, L, V, d = size["width"], size["heads"], size["kv"], size["layers"], size["vocab"], 128
+    m, rank, rot, taps = pubulix_experts(size), 512, 64, 4
+    query = W * H * (d + rot) + W * H * d + 2 * H * d * rank + H * d * W              # q, gate, into and out of the latent space, o
+    kinds = [query + W * (rank + rot), W * (H + 2 * G) * d + H * d * W, query, W * (H + 2 * G) * d + H * d * W]
+    per_token = sum(kinds[i % 4] + 2 * W * W + taps * W + 3 * W * m["ff"] * m["top"] for i in range(L))
+    pairs = sum(min(t + 1, 1024) for t in range(tokens))
+    scores = sum((H * (2 * rank + rot) * 2.0 if i % 2 == 0 else H * d * 4.0) * pairs for i in range(L))
+    return 2.0 * tokens * per_token + 2.0 * V * W + scores
+
+
+def unread_bytes(size, batch):
+    """Weight bytes of experts that a Pubulix decode step of `batch` requests of random tokens does not read."""
+    m = pubulix_experts(size)
+    idle = (1.0 - m["top"] / m["experts"]) ** batch * m["experts"]
+    return size["layers"] * idle * 3 * size["width"] * m["ff"] * 2.0
+
+
 def design_flops(size, tokens, design):
     """Multiply-add work of one prompt of `tokens` tokens, times two: the products and the attention."""
     if design == "vivesun":
@@ -499,6 +546,8 @@ def design_flops(size, tokens, design):
         return beralix_flops(size, tokens)
     if design == "nefipel":
         return nefipel_flops(size, tokens)
+    if design == "pubulix":
+        return pubulix_flops(size, tokens)
     W, H, G, F, L, V = size["width"], size["heads"], size["kv"], size["ff"], size["layers"], size["vocab"]
     d = 128
     attention = W * (H + 2 * G) * d + H * d * W
@@ -530,6 +579,8 @@ def design_engine(kind, size, max_batch):
         spec = model_spec_from_config(beralix_config(size))
     elif kind == "nefipel":
         spec = model_spec_from_config(nefipel_config(size))
+    elif kind == "pubulix":
+        spec = model_spec_from_config(pubulix_config(size))
     else:
         spec = model_spec_from_config(qwen3(size["layers"], size["width"], size["heads"], size["kv"], size["ff"],
                                             context=CONTEXT + 2048) | {"vocab_size": size["vocab"]})
@@ -566,7 +617,10 @@ def design_one(args, name, kind) -> dict:
     for batch in (8, 1):
         print(f"[bench] {name}: {kind}: decode at batch {batch}", file=sys.stderr, flush=True)
         run = decode_run(engine, batch, args.steps, args.warmup, seed=21 + batch, least_repeats=3)
-        step_bytes = weight_bytes + batch * (run["context"] * kv_bytes + 2 * state_bytes)
+        kv_read = run["context"] * kv_bytes
+        if kind == "pubulix":                   # windows of 1,024; the first layer's latents are read by two layers
+            kv_read = min(run["context"], 1024) * (kv_bytes + 576 * 2 * ((size["layers"] + 1) // 4))
+        step_bytes = weight_bytes + batch * (kv_read + 2 * state_bytes) - (unread_bytes(size, batch) if kind == "pubulix" else 0)
         entry[f"decode_b{batch}"] = {
             "tok_s": round(batch * 1e3 / run["device_ms"], 1), "ms_per_step": round(run["device_ms"], 4),
             "e2e_tok_s": round(batch * 1e3 / run["wall_ms"], 1), "launches_per_step": run["launches"] / args.steps,
@@ -574,12 +628,12 @@ def design_one(args, name, kind) -> dict:
     return entry
 
 
-BESIDE = {"mugizen": "qwen3", "vivesun": "mugizen", "beralix": "mugizen", "nefipel": "qwen3"}      # the engine's closest other model
+BESIDE = {"mugizen": "qwen3", "vivesun": "mugizen", "beralix": "mugizen", "nefipel": "qwen3", "pubulix": "beralix"}      # the engine's closest other model
 
 
 def design_main(args) -> int:
     """Prefill and decode of a design beside the engine's closest other model (Mugizen beside Qwen3,
-    Vivesun and Beralix beside Mugizen) at equal sizes; one JSON line. Every
+    Vivesun and Beralix beside Mugizen, Pubulix beside Beralix) at equal sizes; one JSON line. Every
     model is measured in a process of its own (this program started again with --design-one), so
     that no model's scratch buffers, graphs or allocator state reach the next one's timings."""
     if args.design_one:
@@ -598,6 +652,8 @@ def design_main(args) -> int:
                 if args.design != "nefipel":
                     continue                  # the engine has no other model with experts to stand beside
                 kind = "mugizen"              # Nefipel's experts stand beside Mugizen's
+            if kind == "beralix" and args.design == "pubulix" and size["moe"]:
+                kind = "mugizen"              # and so do Pubulix's
             child = subprocess.run([sys.executable, os.path.abspath(__file__), "--design", args.design, "--design-one",
                                     f"{name}:{kind}", "--steps", str(args.steps), "--warmup", str(args.warmup),
                                     "--context", str(CONTEXT), "--page", str(PAGE)],
@@ -635,7 +691,7 @@ def main() -> int:
                         help="read every step's tokens before the next step is planned (default: the engine's async scheduling)")
     parser.add_argument("--batch-invariant", default="off", choices=["off", "decode", "full"],
                         help="measure with the engine's bitwise-invariance modes (the default run has them off)")
-    parser.add_argument("--design", default="", choices=["", "mugizen", "vivesun", "beralix", "nefipel"],
+    parser.add_argument("--design", default="", choices=["", "mugizen", "vivesun", "beralix", "nefipel", "pubulix"],
                         help="measure this design beside the engine's closest other model at equal layer sizes instead of the headline")
     parser.add_argument("--design-sizes", default="s,m,moe", help="which of the sizes s, m, moe (comma-separated)")
     parser.add_argument("--design-one", default="", help=argparse.SUPPRESS)      # size:design, one model in this process

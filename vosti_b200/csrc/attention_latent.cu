@@ -410,7 +410,7 @@ VOSTI_API int vosti_head_project(const void* x, int x_f32, int64_t x_row, int64_
   const dim3 grid((out + HP_OUT - 1) / HP_OUT, heads, token_tiles), block(HP_OUT);
 #define VOSTI_HP(TX, TM, TY)                                                                                          \
   vosti_launch(head_project_kernel<TX, TM, TY>, grid, block, 0, stream, (const TX*)x, x_row, x_head, (const TM*)m, m_head, \
-               m_in, m_out, HeadGate{gate, element_gate, element_gate_f32, element_gate_row}, (TY*)y, y_row, y_head, tokens, heads, in, out)
+               m_in, m_out, HeadGate{gate, element_gate, element_gate_f32, element_gate_row, 0}, (TY*)y, y_row, y_head, tokens, heads, in, out)
   if (x_f32 && m_f32 && y_f32) VOSTI_HP(float, float, float);
   else if (x_f32 && !m_f32 && y_f32) VOSTI_HP(float, bf16, float);
   else if (x_f32 && !m_f32 && !y_f32) VOSTI_HP(float, bf16, bf16);

@@ -451,7 +451,8 @@ head_project_mma_kernel(const void* __restrict__ x_, int64_t x_row, int64_t x_he
     for (int nt = 0; nt < NT; ++nt) {
       const int o = o0 + n_warp + nt * 8 + (lane & 3) * 2;
       if (o >= out) continue;
-      store_pair(dst + o, acc[nt][2 * r] * gate.at(t, h, o, heads, out), acc[nt][2 * r + 1] * gate.at(t, h, o + 1, heads, out));
+      const float2 g = gate.at_pair(t, h, o, heads, out);
+      store_pair(dst + o, acc[nt][2 * r] * g.x, acc[nt][2 * r + 1] * g.y);
     }
   }
 }
@@ -533,7 +534,8 @@ VOSTI_API int vosti_head_project_mma(const void* x, int x_f32, int64_t x_row, in
                 reinterpret_cast<uintptr_t>(y) % 8 == 0, "head_project_mma: operands are not aligned");
   VOSTI_REQUIRE(element_gate == nullptr || (gate == nullptr && element_gate_row >= (int64_t)heads * out), "head_project_mma: one gate, with whole rows");
   if (tokens == 0) return VOSTI_OK;
-  const HeadGate head_gate = {gate, element_gate, element_gate_f32, element_gate_row};
+  const int pairs = !element_gate_f32 && element_gate_row % 2 == 0 && out % 2 == 0 && reinterpret_cast<uintptr_t>(element_gate) % 4 == 0;
+  const HeadGate head_gate = {gate, element_gate, element_gate_f32, element_gate_row, pairs};
   const bool kmajor = m_in == 1;
   const int64_t m_stride = kmajor ? m_out : m_in;
   const bool few = tokens <= 16;

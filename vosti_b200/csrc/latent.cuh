@@ -18,6 +18,14 @@ struct HeadGate {
   const void* per_element;     // [tokens, heads * out] before the sigmoid, rows `row` elements apart, or null
   int element_f32;
   int64_t row;
+  int pairs;                   // two neighbouring elements of per_element (bfloat16) are one aligned word
+  __device__ __forceinline__ float2 at_pair(int t, int h, int o, int heads, int out) const {
+    if (per_element == nullptr || !pairs) return make_float2(at(t, h, o, heads, out), at(t, h, o + 1, heads, out));
+    const __nv_bfloat162 raw = *reinterpret_cast<const __nv_bfloat162*>(reinterpret_cast<const bf16*>(per_element) +
+                                                                        (int64_t)t * row + (int64_t)h * out + o);
+    const float2 z = __bfloat1622float2(raw);
+    return make_float2(1.f / (1.f + expf(-z.x)), 1.f / (1.f + expf(-z.y)));
+  }
   __device__ __forceinline__ float at(int t, int h, int o, int heads, int out) const {
     if (per_head != nullptr) return per_head[(int64_t)t * heads + h];
     if (per_element != nullptr) return 1.f / (1.f + expf(-load_flex(per_element, element_f32, (int64_t)t * row + (int64_t)h * out + o)));

@@ -404,43 +404,72 @@ moe_group_kernel(const int* __restrict__ chosen, int pairs, int top, int experts
   }
 }
 
-// Sort and gather in one kernel, for experts by token id: block i takes the (token, pick) pair i, finds its
-// place among the pairs sorted by expert (pairs of lower experts, then earlier pairs of its own: every
-// block counts by itself, so pairs * pairs table reads in all) and copies its token's row there;
-// blocks up to `experts` also count where an expert's rows start.
-template <int BYTES>
+// Sort and gather in one kernel, for experts by token id. A block takes `chunk` neighbouring (token, pick)
+// pairs. It counts the pairs of every expert, all of them and those before its own (every block counts by
+// itself: the table's rows are few and cached), and so knows the place of each of its pairs among the
+// pairs sorted by expert (in their order inside an expert); then it copies its pairs' rows there. Block 0
+// also writes where the experts' rows start.
+constexpr int DISPATCH_CHUNK = 32;      // pairs of a block at most
+
 __global__ void __launch_bounds__(256)
-moe_dispatch_kernel(const TokenTable by, int pairs, int experts, const char* __restrict__ x, int64_t row_bytes, char* __restrict__ sorted,
-                    int* __restrict__ offsets, int* __restrict__ where) {
-  __shared__ int counts[2][8];
+moe_dispatch_kernel(const TokenTable by, int pairs, int experts, int chunk, int words, const char* __restrict__ x, int64_t row_bytes,
+                    char* __restrict__ sorted, int* __restrict__ offsets, int* __restrict__ where) {
+  extern __shared__ int counts[];                      // [experts] all pairs, then their exclusive sums; [experts] pairs before this block's
+  __shared__ int place[DISPATCH_CHUNK];
   pdl_wait();
   pdl_launch_dependents();
-  const int i = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int mine = i < pairs ? table_row(by, i / by.top)[i % by.top] : -1;
-  int before = 0, start = 0;
-  for (int j = threadIdx.x; j < pairs; j += blockDim.x) {
-    const int e = table_row(by, j / by.top)[j % by.top];
-    before += (e < mine || (e == mine && j < i)) ? 1 : 0;
-    start += e < i ? 1 : 0;
-  }
-  for (int o = 16; o > 0; o >>= 1) {
-    before += __shfl_xor_sync(0xffffffffu, before, o);
-    start += __shfl_xor_sync(0xffffffffu, start, o);
-  }
-  if (lane == 0) { counts[0][warp] = before; counts[1][warp] = start; }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  int* all = counts;
+  int* before = counts + experts;
+  const int first = blockIdx.x * chunk, mine = min(chunk, pairs - first);
+  for (int e = threadIdx.x; e < 2 * experts; e += blockDim.x) counts[e] = 0;
   __syncthreads();
-  before = start = 0;
-  for (int w = 0; w < 8; ++w) { before += counts[0][w]; start += counts[1][w]; }
-  if (threadIdx.x == 0 && i <= experts) offsets[i] = start;
-  if (i >= pairs) return;
-  if (threadIdx.x == 0) where[i] = before;
-  const char* src = x + (int64_t)(i / by.top) * row_bytes;
-  char* dst = sorted + (int64_t)before * row_bytes;
-  if (BYTES == 16) {
-    for (int64_t c = threadIdx.x; c < row_bytes / 16; c += blockDim.x) reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
-  } else {
-    for (int64_t c = threadIdx.x; c < row_bytes / 2; c += blockDim.x)
-      reinterpret_cast<unsigned short*>(dst)[c] = reinterpret_cast<const unsigned short*>(src)[c];
+  for (int j0 = warp * 32; j0 < pairs; j0 += blockDim.x) {
+    const int j = j0 + lane;
+    const bool live = j < pairs, early = live && j < first;
+    const int e = live ? table_row(by, j / by.top)[j % by.top] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e), ahead = __ballot_sync(0xffffffffu, early) & same;
+    if (live && lane == __ffs(same) - 1) {
+      atomicAdd(&all[e], __popc(same));
+      if (ahead) atomicAdd(&before[e], __popc(ahead));
+    }
+  }
+  __syncthreads();
+  if (warp == 0) {
+    int start = 0;                                     // exclusive sums over the experts, 32 at a time
+    for (int e0 = 0; e0 < experts; e0 += 32) {
+      const int n = e0 + lane < experts ? all[e0 + lane] : 0;
+      int sum = n;
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += v;
+      }
+      if (e0 + lane < experts) {
+        all[e0 + lane] = start + sum - n;
+        if (blockIdx.x == 0) offsets[e0 + lane] = start + sum - n;
+      }
+      start += __shfl_sync(0xffffffffu, sum, 31);
+    }
+    if (blockIdx.x == 0 && lane == 0) offsets[experts] = start;
+    __syncwarp();
+    const int e = lane < mine ? table_row(by, (first + lane) / by.top)[(first + lane) % by.top] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    if (lane < mine) {
+      place[lane] = all[e] + before[e] + __popc(same & ((1u << lane) - 1u));
+      where[first + lane] = place[lane];
+    }
+  }
+  __syncthreads();
+  for (int i = warp; i < mine; i += blockDim.x >> 5) { // a warp a row
+    const char* src = x + (int64_t)((first + i) / by.top) * row_bytes;
+    char* dst = sorted + (int64_t)place[i] * row_bytes;
+    if (words) {
+#pragma unroll 4
+      for (int64_t c = lane; c < row_bytes / 16; c += 32) reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+    } else {
+      for (int64_t c = lane; c < row_bytes / 2; c += 32)
+        reinterpret_cast<unsigned short*>(dst)[c] = reinterpret_cast<const unsigned short*>(src)[c];
+    }
   }
 }
 
@@ -477,13 +506,12 @@ VOSTI_API int vosti_moe_dispatch(const int* ids, const int* table, int vocab, in
   VOSTI_REQUIRE((int64_t)tokens * top < (int64_t)1 << 24, "moe_dispatch: too many pairs");
   VOSTI_REQUIRE(ids != nullptr && table != nullptr, "moe_dispatch: missing arrays");
   if (tokens == 0) return VOSTI_OK;
-  const int pairs = tokens * top, blocks = pairs > experts + 1 ? pairs : experts + 1;
+  VOSTI_REQUIRE(experts <= 4096, "moe_dispatch: %d experts (at most 4096 are taken)", experts);
+  // a warp of rows a block; few pairs: a row a block
+  const int pairs = tokens * top, chunk = pairs <= 148 ? 1 : pairs <= 148 * 8 ? 8 : DISPATCH_CHUNK;
   const bool words = row_bytes % 16 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(sorted) & 15) == 0;
-  const TokenTable by = {ids, table, top, vocab, share};
-  if (words)
-    vosti_launch(moe_dispatch_kernel<16>, dim3(blocks), dim3(256), 0, stream, by, pairs, experts, (const char*)x, row_bytes, (char*)sorted, offsets, where);
-  else
-    vosti_launch(moe_dispatch_kernel<2>, dim3(blocks), dim3(256), 0, stream, by, pairs, experts, (const char*)x, row_bytes, (char*)sorted, offsets, where);
+  vosti_launch(moe_dispatch_kernel, dim3((pairs + chunk - 1) / chunk), dim3(256), (size_t)2 * experts * sizeof(int), stream,
+               TokenTable{ids, table, top, vocab, share}, pairs, experts, chunk, (int)words, (const char*)x, row_bytes, (char*)sorted, offsets, where);
   VOSTI_LAUNCH_CHECK();
 }
 

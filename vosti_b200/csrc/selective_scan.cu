@@ -105,6 +105,91 @@ scan_conv_kernel(const T* __restrict__ xz, int64_t xz_stride, const void* __rest
   }
 }
 
+// The same for rows in whole words of four channels (up to CONV_WINDOW taps): a thread takes four neighbouring
+// channels, and the inputs of CONV_AHEAD tokens are in flight together. The arithmetic of a channel is
+// that of the kernel above, operation by operation.
+constexpr int CONV_AHEAD = 4;
+
+__device__ __forceinline__ float4 conv_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 conv_load4(const bf16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void conv_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void conv_store4(bf16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<const unsigned*>(&lo);
+  raw.y = *reinterpret_cast<const unsigned*>(&hi);
+  *reinterpret_cast<uint2*>(p) = raw;
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+scan_conv4_kernel(const T* __restrict__ xz, int64_t xz_stride, const void* __restrict__ conv_w, const void* __restrict__ conv_b,
+                  int w_f32, const float* state, int64_t state_stride, int64_t tail_offset, const int* __restrict__ request_of,
+                  const int* __restrict__ cu_q, const int* __restrict__ state_slots, int num_slots, int inner, int tokens,
+                  int per_block, int plain, T* __restrict__ out, unsigned* status) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  const int t_begin = blockIdx.y * per_block, t_end = min(tokens, t_begin + per_block);
+  if (c >= inner) return;
+  float w[TAPS][4], win[TAPS][4], bias[4];             // index TAPS - 1 is the current token
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    bias[u] = conv_b != nullptr ? load_flex(conv_b, w_f32, c + u) : 0.f;
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) { w[k][u] = load_flex(conv_w, w_f32, (int64_t)(c + u) * TAPS + k); win[k][u] = 0.f; }
+  }
+  int b = -1, next_first = 0;
+  bool usable = false;
+  for (int t0 = t_begin; t0 < t_end; t0 += CONV_AHEAD) {
+    float4 x[CONV_AHEAD];
+#pragma unroll
+    for (int a = 0; a < CONV_AHEAD; ++a)
+      if (t0 + a < t_end) x[a] = conv_load4(xz + (int64_t)(t0 + a) * xz_stride + c);
+#pragma unroll
+    for (int a = 0; a < CONV_AHEAD; ++a) {
+      const int t = t0 + a;
+      if (t >= t_end) break;
+      if (b < 0 || t >= next_first) {                  // a new request (or the block's first token): fill the window anew
+        b = request_of[t];
+        const int first = cu_q[b], slot = state_slots[b];
+        next_first = cu_q[b + 1];
+        usable = slot >= 0 && slot < num_slots;
+        if (!usable && threadIdx.x == 0) raise_fault(status, VOSTI_FAULT_SLOT_RANGE);
+        const float* tail = state + (int64_t)(usable ? slot : 0) * state_stride + tail_offset;
+#pragma unroll
+        for (int k = 1; k < TAPS; ++k) {               // the input k tokens back: of this portion, or from the tail
+          const int back = t - first;
+          const float4 v = k <= back ? conv_load4(xz + (int64_t)(t - k) * xz_stride + c)
+                                     : conv_load4(tail + (int64_t)(TAPS - 1 - (k - back)) * inner + c);
+          win[TAPS - 1 - k][0] = v.x; win[TAPS - 1 - k][1] = v.y; win[TAPS - 1 - k][2] = v.z; win[TAPS - 1 - k][3] = v.w;
+        }
+      } else {
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+          for (int u = 0; u < 4; ++u) win[k][u] = win[k + 1][u];
+      }
+      win[TAPS - 1][0] = x[a].x; win[TAPS - 1][1] = x[a].y; win[TAPS - 1][2] = x[a].z; win[TAPS - 1][3] = x[a].w;
+      if (!usable) continue;
+      float y[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        float acc = bias[u];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) acc = fmaf(w[k][u], win[k][u], acc);
+        y[u] = plain ? win[TAPS - 1][u] + acc : silu_f(acc);
+      }
+      conv_store4(out + (int64_t)t * inner + c, make_float4(y[0], y[1], y[2], y[3]));
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 scan_tail_kernel(const T* __restrict__ xz, int64_t xz_stride, float* state, int64_t state_stride, int64_t tail_offset,
@@ -269,6 +354,23 @@ scan_carry_kernel(const void* __restrict__ a_log, int w_f32, const float* state,
 
 }  // namespace
 
+// The tail's kernel, after the convolution's (nothing to keep with one tap).
+static int scan_tail(const void* xz, int64_t xz_stride, float* state, int64_t state_stride, int64_t tail_offset, const int* cu_q,
+                     const int* state_slots, int num_slots, int requests, int inner, int taps, int is_f32, cudaStream_t stream) {
+  if (taps > 1) {
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) { vosti_set_error("%s", cudaGetErrorString(e)); return (int)e; }
+    const int across = (inner + 255) / 256 < 64 ? (inner + 255) / 256 : 64;
+    if (is_f32)
+      vosti_launch(scan_tail_kernel<float>, dim3(across, requests), dim3(256), 0, stream, (const float*)xz, xz_stride, state,
+                   state_stride, tail_offset, cu_q, state_slots, num_slots, inner, taps);
+    else
+      vosti_launch(scan_tail_kernel<bf16>, dim3(across, requests), dim3(256), 0, stream, (const bf16*)xz, xz_stride, state,
+                   state_stride, tail_offset, cu_q, state_slots, num_slots, inner, taps);
+  }
+  VOSTI_LAUNCH_CHECK();
+}
+
 // xz [tokens, xz_stride] holds the convolution's inputs in its first `inner` columns; out [tokens, inner].
 // The state slot's tail [taps - 1, inner] starts tail_offset floats into the slot. Two launches
 // when taps > 1. `plain`: out = input + convolution, no SiLU (conv_b must be null).
@@ -279,6 +381,23 @@ VOSTI_API int vosti_scan_conv(const void* xz, int64_t xz_stride, const void* con
   VOSTI_REQUIRE(tokens >= 0 && requests >= 0 && inner > 0 && taps >= 1 && taps <= 64, "scan_conv: bad sizes");
   VOSTI_REQUIRE(!plain || conv_b == nullptr, "scan_conv: the plain form has no bias");
   if (tokens == 0) return VOSTI_OK;
+  // whole words of four channels, and taps the word kernel is built for
+  const uintptr_t mis = reinterpret_cast<uintptr_t>(xz) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(state);
+  if (taps >= 2 && taps <= 4 && inner % 4 == 0 && xz_stride % 4 == 0 && state_stride % 4 == 0 && tail_offset % 4 == 0 && (mis & 15) == 0) {
+    const int across4 = (inner / 4 + 127) / 128;
+    int per4 = 1;
+    while (per4 < 16 && (int64_t)across4 * ((tokens + per4 - 1) / per4) > 148 * 8) per4 *= 2;
+    VOSTI_REQUIRE((tokens + per4 - 1) / per4 <= 65535, "scan_conv: too many tokens for one launch");
+    const dim3 grid4(across4, (tokens + per4 - 1) / per4);
+#define VOSTI_CONV4(T, TAPS)                                                                                                   \
+  vosti_launch(scan_conv4_kernel<T, TAPS>, grid4, dim3(128), 0, stream, (const T*)xz, xz_stride, conv_w, conv_b, w_f32,        \
+               (const float*)state, state_stride, tail_offset, request_of, cu_q, state_slots, num_slots, inner, tokens, per4,  \
+               plain, (T*)out, status)
+    if (is_f32) { if (taps == 2) VOSTI_CONV4(float, 2); else if (taps == 3) VOSTI_CONV4(float, 3); else VOSTI_CONV4(float, 4); }
+    else { if (taps == 2) VOSTI_CONV4(bf16, 2); else if (taps == 3) VOSTI_CONV4(bf16, 3); else VOSTI_CONV4(bf16, 4); }
+#undef VOSTI_CONV4
+    return scan_tail(xz, xz_stride, state, state_stride, tail_offset, cu_q, state_slots, num_slots, requests, inner, taps, is_f32, stream);
+  }
   const int across_c = (inner + 255) / 256;
   int per_block = 1;                      // tokens a block takes: more once the grid fills the GPU several times over
   while (per_block < 16 && (int64_t)across_c * ((tokens + per_block - 1) / per_block) > 148 * 16) per_block *= 2;
@@ -293,18 +412,7 @@ VOSTI_API int vosti_scan_conv(const void* xz, int64_t xz_stride, const void* con
     vosti_launch(scan_conv_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)xz, xz_stride, conv_w, conv_b, w_f32,
                  (const float*)state, state_stride, tail_offset, request_of, cu_q, state_slots, num_slots, inner, taps,
                  tokens, per_block, plain, (bf16*)out, status);
-  if (taps > 1) {
-    cudaError_t e = cudaGetLastError();
-    if (e != cudaSuccess) { vosti_set_error("%s", cudaGetErrorString(e)); return (int)e; }
-    const int across = (inner + 255) / 256 < 64 ? (inner + 255) / 256 : 64;
-    if (is_f32)
-      vosti_launch(scan_tail_kernel<float>, dim3(across, requests), dim3(256), 0, stream, (const float*)xz, xz_stride, state,
-                   state_stride, tail_offset, cu_q, state_slots, num_slots, inner, taps);
-    else
-      vosti_launch(scan_tail_kernel<bf16>, dim3(across, requests), dim3(256), 0, stream, (const bf16*)xz, xz_stride, state,
-                   state_stride, tail_offset, cu_q, state_slots, num_slots, inner, taps);
-  }
-  VOSTI_LAUNCH_CHECK();
+  return scan_tail(xz, xz_stride, state, state_stride, tail_offset, cu_q, state_slots, num_slots, requests, inner, taps, is_f32, stream);
 }
 
 // Tokens a block of scan_run takes (a portion longer than this is run as chunks side by side):

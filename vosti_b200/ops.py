@@ -1640,7 +1640,7 @@ def moe_table(ids: torch.Tensor, table: torch.Tensor, experts: int, want_dense: 
     return chosen, weights, dense
 
 
-MOE_DISPATCH_PAIRS = 8192        # (token, pick) pairs up to which one kernel sorts and gathers (its counting is quadratic)
+MOE_DISPATCH_PAIRS = 16384       # (token, pick) pairs up to which one kernel sorts and gathers (beyond, three kernels)
 
 
 def moe_dispatch(ids: torch.Tensor, table: torch.Tensor, experts: int, x: torch.Tensor, status: torch.Tensor):

@@ -210,6 +210,7 @@ class ExpertMixture(FeedForward):
         return specs
 
     def load(self, tensors, dtype):
+        self.grouped, self.per_expert = None, []
         if self.route == "table":
             self.table = tensors["table"].to(torch.int32).contiguous()
             if self.table.numel() and (int(self.table.min()) < 0 or int(self.table.max()) >= self.experts):
