@@ -447,12 +447,17 @@ head_project_mma_kernel(const void* __restrict__ x_, int64_t x_row, int64_t x_he
     const int t = t0 + wm * 16 + (lane >> 2) + 8 * r;
     if (t >= tokens) continue;
     TY* dst = y + (int64_t)t * y_row + (int64_t)h * y_head;
+    float2 g[NT];                              // the gates first: a load does not wait for the stores before it
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const int o = o0 + n_warp + nt * 8 + (lane & 3) * 2;
+      g[nt] = o < out ? gate.at_pair(t, h, o, heads, out) : make_float2(0.f, 0.f);
+    }
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       const int o = o0 + n_warp + nt * 8 + (lane & 3) * 2;
       if (o >= out) continue;
-      const float2 g = gate.at_pair(t, h, o, heads, out);
-      store_pair(dst + o, acc[nt][2 * r] * g.x, acc[nt][2 * r + 1] * g.y);
+      store_pair(dst + o, acc[nt][2 * r] * g[nt].x, acc[nt][2 * r + 1] * g[nt].y);
     }
   }
 }

@@ -24,7 +24,7 @@ struct HeadGate {
     const __nv_bfloat162 raw = *reinterpret_cast<const __nv_bfloat162*>(reinterpret_cast<const bf16*>(per_element) +
                                                                         (int64_t)t * row + (int64_t)h * out + o);
     const float2 z = __bfloat1622float2(raw);
-    return make_float2(1.f / (1.f + expf(-z.x)), 1.f / (1.f + expf(-z.y)));
+    return make_float2(__fdividef(1.f, 1.f + __expf(-z.x)), __fdividef(1.f, 1.f + __expf(-z.y)));
   }
   __device__ __forceinline__ float at(int t, int h, int o, int heads, int out) const {
     if (per_head != nullptr) return per_head[(int64_t)t * heads + h];

@@ -424,14 +424,22 @@ moe_dispatch_kernel(const TokenTable by, int pairs, int experts, int chunk, int 
   const int first = blockIdx.x * chunk, mine = min(chunk, pairs - first);
   for (int e = threadIdx.x; e < 2 * experts; e += blockDim.x) counts[e] = 0;
   __syncthreads();
-  for (int j0 = warp * 32; j0 < pairs; j0 += blockDim.x) {
-    const int j = j0 + lane;
-    const bool live = j < pairs, early = live && j < first;
-    const int e = live ? table_row(by, j / by.top)[j % by.top] : -1;
-    const unsigned same = __match_any_sync(0xffffffffu, e), ahead = __ballot_sync(0xffffffffu, early) & same;
-    if (live && lane == __ffs(same) - 1) {
-      atomicAdd(&all[e], __popc(same));
-      if (ahead) atomicAdd(&before[e], __popc(ahead));
+  constexpr int AHEAD = 4;                             // table look-ups in flight together
+  for (int j0 = warp * 32; j0 < pairs; j0 += AHEAD * blockDim.x) {
+    int e[AHEAD];
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) {
+      const int j = j0 + a * (int)blockDim.x + lane;
+      e[a] = j < pairs ? table_row(by, j / by.top)[j % by.top] : -1;
+    }
+#pragma unroll
+    for (int a = 0; a < AHEAD; ++a) {
+      const int j = j0 + a * (int)blockDim.x + lane;
+      const unsigned same = __match_any_sync(0xffffffffu, e[a]), ahead = __ballot_sync(0xffffffffu, j < first) & same;
+      if (e[a] >= 0 && lane == __ffs(same) - 1) {
+        atomicAdd(&all[e[a]], __popc(same));
+        if (ahead) atomicAdd(&before[e[a]], __popc(ahead));
+      }
     }
   }
   __syncthreads();
@@ -473,6 +481,30 @@ moe_dispatch_kernel(const TokenTable by, int pairs, int experts, int chunk, int 
   }
 }
 
+// The same for at most 256 pairs, a pair a block and a thread a pair: two counts over the block place a row.
+__global__ void __launch_bounds__(256)
+moe_dispatch_few_kernel(const TokenTable by, int pairs, int experts, int words, const char* __restrict__ x, int64_t row_bytes,
+                        char* __restrict__ sorted, int* __restrict__ offsets, int* __restrict__ where) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int i = blockIdx.x, j = threadIdx.x;
+  const int mine = i < pairs ? table_row(by, i / by.top)[i % by.top] : -1;
+  const int e = j < pairs ? table_row(by, j / by.top)[j % by.top] : 0x7fffffff;
+  const int start = __syncthreads_count(e < i);                                   // rows of the experts before number i
+  const int place = __syncthreads_count(e < mine || (e == mine && j < i));
+  if (j == 0 && i <= experts) offsets[i] = start;
+  if (i >= pairs) return;
+  if (j == 0) where[i] = place;
+  const char* src = x + (int64_t)(i / by.top) * row_bytes;
+  char* dst = sorted + (int64_t)place * row_bytes;
+  if (words) {
+    for (int64_t c = j; c < row_bytes / 16; c += blockDim.x) reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
+  } else {
+    for (int64_t c = j; c < row_bytes / 2; c += blockDim.x)
+      reinterpret_cast<unsigned short*>(dst)[c] = reinterpret_cast<const unsigned short*>(src)[c];
+  }
+}
+
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ where, const float* __restrict__ weights,
                    float* __restrict__ out, int top, int width) {
@@ -507,9 +539,13 @@ VOSTI_API int vosti_moe_dispatch(const int* ids, const int* table, int vocab, in
   VOSTI_REQUIRE(ids != nullptr && table != nullptr, "moe_dispatch: missing arrays");
   if (tokens == 0) return VOSTI_OK;
   VOSTI_REQUIRE(experts <= 4096, "moe_dispatch: %d experts (at most 4096 are taken)", experts);
-  // a warp of rows a block; few pairs: a row a block
-  const int pairs = tokens * top, chunk = pairs <= 148 ? 1 : pairs <= 148 * 8 ? 8 : DISPATCH_CHUNK;
+  const int pairs = tokens * top, chunk = pairs <= 8192 ? 8 : DISPATCH_CHUNK;         // rows a block: a warp each, or four
   const bool words = row_bytes % 16 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(sorted) & 15) == 0;
+  if (pairs <= 256) {
+    vosti_launch(moe_dispatch_few_kernel, dim3(pairs > experts + 1 ? pairs : experts + 1), dim3(256), 0, stream,
+                 TokenTable{ids, table, top, vocab, share}, pairs, experts, (int)words, (const char*)x, row_bytes, (char*)sorted, offsets, where);
+    VOSTI_LAUNCH_CHECK();
+  }
   vosti_launch(moe_dispatch_kernel, dim3((pairs + chunk - 1) / chunk), dim3(256), (size_t)2 * experts * sizeof(int), stream,
                TokenTable{ids, table, top, vocab, share}, pairs, experts, chunk, (int)words, (const char*)x, row_bytes, (char*)sorted, offsets, where);
   VOSTI_LAUNCH_CHECK();
