@@ -47,8 +47,9 @@ struct ItemMeta {
 };
 
 // DMAX bounds the head size; with EXACT the head size is DMAX itself. FUSED: the query rows and
-// the token's own key and value are made here from the projection's partial sums (`fused`).
-template <int DMAX, bool EXACT, bool FUSED>
+// the token's own key and value are made here from the projection's partial sums (`fused`). CAPPED: the
+// scores pass a soft cap (fused.softcap).
+template <int DMAX, bool EXACT, bool FUSED, bool CAPPED>
 __global__ void __launch_bounds__(THREADS, DMAX <= 128 ? 2 : 1)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const bf16* __restrict__ q, float* __restrict__ partial, bf16* __restrict__ out,
@@ -434,7 +435,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         __syncwarp();
       }
 
-      attend_tile<DMAX, Q_IN_REGISTERS>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
+      attend_tile<DMAX, Q_IN_REGISTERS, CAPPED>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
                                         v_lane, v_xor, m_row, l_row, o,
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min(lane >> 2, group - 1)) * (fused.score_bias_last + 1),
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min((lane >> 2) + 8, group - 1)) * (fused.score_bias_last + 1),
@@ -772,23 +773,24 @@ int launch_decode(const void* q, const void* k_cache, const void* v_cache, void*
   VOSTI_REQUIRE(items < ((int64_t)1 << 30), "attention_decode: %lld work items are too many for one launch", (long long)items);
   const int64_t ctas = (int64_t)sm_count() * ctas_per_sm(d, group);
   dim3 grid((unsigned)(items < ctas ? items : ctas));
-#define LAUNCH_DECODE_AS(DMAX, EXACT, FUSED)                                                                        \
+#define LAUNCH_DECODE_AS(DMAX, EXACT, FUSED, CAPPED)                                                                \
   do {                                                                                                              \
     static bool configured = false;                                                                                 \
     if (!configured) {                                                                                              \
-      cudaFuncSetAttribute(attention_decode_kernel<DMAX, EXACT, FUSED>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+      cudaFuncSetAttribute(attention_decode_kernel<DMAX, EXACT, FUSED, CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                            (int)decode_smem_bytes(DMAX, 16));                                                       \
       configured = true;                                                                                            \
     }                                                                                                               \
-    vosti_launch(attention_decode_kernel<DMAX, EXACT, FUSED>, grid, dim3(THREADS), smem, stream, map_k, map_v,      \
+    vosti_launch(attention_decode_kernel<DMAX, EXACT, FUSED, CAPPED>, grid, dim3(THREADS), smem, stream, map_k, map_v, \
         (const bf16*)q, scratch, (bf16*)out, arrivals, token_list, positions, request_of,                          \
         block_table, max_pages, page_size, page_shift, num_pages, whole_pages, whole_rows, count, nq, nkv, d, segment_keys,     \
         segments, scale * LOG2E, window, status, fused);                                                            \
   } while (0)
 #define LAUNCH_DECODE(DMAX, EXACT)                                                                                  \
   do {                                                                                                              \
-    if (fused.partial != nullptr) LAUNCH_DECODE_AS(DMAX, EXACT, true);                                              \
-    else LAUNCH_DECODE_AS(DMAX, EXACT, false);                                                                      \
+    if (fused.partial != nullptr) LAUNCH_DECODE_AS(DMAX, EXACT, true, false);                                       \
+    else if (fused.softcap > 0.f) LAUNCH_DECODE_AS(DMAX, EXACT, false, true);                                       \
+    else LAUNCH_DECODE_AS(DMAX, EXACT, false, false);                                                               \
   } while (0)
   if (d == 64) LAUNCH_DECODE(64, true);
   else if (d == 128) LAUNCH_DECODE(128, true);

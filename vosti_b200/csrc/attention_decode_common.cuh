@@ -128,7 +128,7 @@ __device__ __forceinline__ void merge_segments(const float* __restrict__ base, b
 // One tile of 16 keys for one warp: S = Q K^T on the tensor cores, the online softmax of the
 // warp's 16 rows (base 2, float32; masked keys count as -inf), O = O * alpha + P V with P rounded
 // to bfloat16. ks / vs: shared-memory addresses of the tile's K and V blocks (128-byte swizzle).
-template <int DMAX, bool Q_IN_REGISTERS>
+template <int DMAX, bool Q_IN_REGISTERS, bool CAPPED = false>
 __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint32_t (&qa)[Q_IN_REGISTERS ? DMAX / 16 : 1][4],
                                             const uint8_t* q_s, int q_pitch, int d, int key0, int kstart, int pos,
                                             float scale_log2, bool upper_rows_live, uint32_t k_lane, uint32_t k_xor,
@@ -136,7 +136,7 @@ __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint
                                             float (&o)[DMAX / 8][4], const float* __restrict__ bias0 = nullptr,
                                             const float* __restrict__ bias1 = nullptr, int bias_last = 0,
                                             float softcap = 0.f) {
-  // softcap (base-2 units; 0: none) caps the scaled score; bias0 / bias1 (or null): the rows of a distance-bias table (base-2 units) of this lane's two
+  // softcap (base-2 units, CAPPED only) caps the scaled score; bias0 / bias1 (or null): the rows of a distance-bias table (base-2 units) of this lane's two
   // query heads, indexed by min(pos - key, bias_last) and added to the scaled score
   const int lane = threadIdx.x & 31;
   // ---- S = Q K^T for 16 keys: two 8-key column tiles
@@ -165,7 +165,7 @@ __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint
     for (int e = 0; e < 4; ++e) {
       const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
       const bool visible = key >= kstart && key <= pos;
-      if (softcap > 0.f) {
+      if (CAPPED) {
         s[nt][e] = soft_capped(s[nt][e] * scale_log2, softcap, 2.f * LOG2E / softcap);
         if (bias0 != nullptr) s[nt][e] += ((e >> 1) ? bias1 : bias0)[min(max(pos - key, 0), bias_last)];
         if (!visible) s[nt][e] = -INFINITY;
@@ -235,8 +235,9 @@ struct FusedProjection {
   // additions to the scores, for mixers that have them (all null / 0 otherwise; they do not need `partial`)
   const float* score_bias;     // [nq][score_bias_last + 1] float32, base-2 units, by min(distance, last)
   int score_bias_last;
+  float softcap;               // base-2 units: the scaled scores' soft cap (here it fills the padding: a launch with more
+                               // bytes of parameters was measured 1 us slower)
   const float* sink;           // [nq] float32, natural units: a logit in the denominator without key or value
-  float softcap;               // base-2 units: the scaled scores' soft cap
 };
 
 constexpr int ONCE_MAX_SEGMENTS = 16;     // CTAs per cluster of that kernel (above 8 it opts in to non-portable sizes)

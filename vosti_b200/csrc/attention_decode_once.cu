@@ -85,7 +85,7 @@ __device__ __forceinline__ int load_now(const int* p) {
 }
 
 
-template <int DMAX, bool EXACT, bool FUSED>
+template <int DMAX, bool EXACT, bool FUSED, bool CAPPED>
 __global__ void __launch_bounds__(THREADS, DMAX <= 128 ? 2 : 1)
 attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                              const bf16* __restrict__ q, bf16* __restrict__ out, const int* __restrict__ token_list,
@@ -323,7 +323,7 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
         }
         __syncwarp();
       }
-      attend_tile<DMAX, Q_IN_REGISTERS>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
+      attend_tile<DMAX, Q_IN_REGISTERS, CAPPED>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
                                         v_lane, v_xor, m_row, l_row, o,
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min(lane >> 2, group - 1)) * (fused.score_bias_last + 1),
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min((lane >> 2) + 8, group - 1)) * (fused.score_bias_last + 1),
@@ -429,9 +429,9 @@ int clusters_that_fit(Kernel kernel, int cluster, size_t smem) {
   return clusters;
 }
 
-template <int DMAX, bool EXACT, bool FUSED>
+template <int DMAX, bool EXACT, bool FUSED, bool CAPPED>
 int launch_as(const OnceLaunch& a, size_t smem) {
-  auto kernel = attention_decode_once_kernel<DMAX, EXACT, FUSED>;
+  auto kernel = attention_decode_once_kernel<DMAX, EXACT, FUSED, CAPPED>;
   static bool configured = false;
   if (!configured) {
     cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ONCE_SMEM_CAP);
@@ -462,7 +462,8 @@ int launch_as(const OnceLaunch& a, size_t smem) {
 
 template <int DMAX, bool EXACT>
 int launch_form(const OnceLaunch& a, size_t smem) {
-  return a.fused.partial != nullptr ? launch_as<DMAX, EXACT, true>(a, smem) : launch_as<DMAX, EXACT, false>(a, smem);
+  if (a.fused.partial != nullptr) return launch_as<DMAX, EXACT, true, false>(a, smem);
+  return a.fused.softcap > 0.f ? launch_as<DMAX, EXACT, false, true>(a, smem) : launch_as<DMAX, EXACT, false, false>(a, smem);
 }
 
 }  // namespace

@@ -56,10 +56,10 @@ __device__ __forceinline__ uint32_t swizzled(int row, int chunk) { return row * 
 
 // BIASED: the scaled score also gets bias[head][min(distance, bias_last)] (base-2 units; the
 // table's last column serves every larger distance, so a tile that lies wholly beyond it adds a
-// constant), and exp(sink[head]) joins the denominator once at the end (either may be null); softcap
-// (base-2 units) > 0 caps the scaled score before the bias.
+// constant), and exp(sink[head]) joins the denominator once at the end (either may be null). CAPPED
+// (with BIASED): the scaled score passes a soft cap (`softcap`, base-2 units) before the bias.
 // Without BIASED the arithmetic is what it was before the flag existed, bit for bit.
-template <int D, bool BIASED>
+template <int D, bool BIASED, bool CAPPED>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
@@ -172,15 +172,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&s_empty[wg]));       // the scores are in registers
-      if (BIASED && valid && softcap > 0.f) {
+      if (CAPPED && valid) {
         // the capped score; a bias, if there is one, is added to it below with a factor of one
         const float rate = 2.f * LOG2E / softcap;
 #pragma unroll
         for (int i = 0; i < KT; ++i)
           raw[i >> 5][i & 31] = __float_as_uint(soft_capped(__uint_as_float(raw[i >> 5][i & 31]) * scale_log2_in, softcap, rate));
       }
-      const float scale_here = BIASED && softcap > 0.f ? 1.f : scale_log2_in;
-      if (BIASED && valid && (softcap <= 0.f || bias_h != nullptr)) {
+      const float scale_here = CAPPED ? 1.f : scale_log2_in;
+      if (BIASED && valid && (!CAPPED || bias_h != nullptr)) {
         const int d0 = pos - key0;                               // key i of the tile is d0 - i positions back
         if (bias_h == nullptr || d0 - (KT - 1) >= bias_last) {
           const float far = bias_h != nullptr ? bias_h[bias_last] : 0.f;
@@ -479,24 +479,27 @@ int launch_prefill_tc(const void* q, const void* k_cache, const void* v_cache, v
   int page_shift = -1;
   if ((page_size & (page_size - 1)) == 0)
     for (page_shift = 0; (1 << page_shift) < page_size; ++page_shift) {}
-#define LAUNCH_PREFILL_TC(D, B)                                                                                      \
+#define LAUNCH_PREFILL_TC(D, B, C)                                                                                   \
   do {                                                                                                               \
     static bool configured = false;                                                                                  \
     if (!configured) {                                                                                               \
-      cudaFuncSetAttribute(attention_prefill_tc_kernel<D, B>, cudaFuncAttributeMaxDynamicSharedMemorySize,          \
+      cudaFuncSetAttribute(attention_prefill_tc_kernel<D, B, C>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
                            (int)prefill_tc_smem_bytes<D>());                                                         \
       configured = true;                                                                                             \
     }                                                                                                                \
-    vosti_launch(attention_prefill_tc_kernel<D, B>, grid, dim3(THREADS), prefill_tc_smem_bytes<D>(), stream, map_q,  \
+    vosti_launch(attention_prefill_tc_kernel<D, B, C>, grid, dim3(THREADS), prefill_tc_smem_bytes<D>(), stream, map_q,  \
         map_k, map_v, (bf16*)out, row_list, cu_q, kv_len, block_table, max_pages, page_size, page_shift, num_pages,   \
         nq, nkv, scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, status);                                               \
   } while (0)
-  if (biased) {
-    if (d == 64) LAUNCH_PREFILL_TC(64, true);
-    else LAUNCH_PREFILL_TC(128, true);
+  if (biased && softcap > 0.f) {
+    if (d == 64) LAUNCH_PREFILL_TC(64, true, true);
+    else LAUNCH_PREFILL_TC(128, true, true);
+  } else if (biased) {
+    if (d == 64) LAUNCH_PREFILL_TC(64, true, false);
+    else LAUNCH_PREFILL_TC(128, true, false);
   } else {
-    if (d == 64) LAUNCH_PREFILL_TC(64, false);
-    else LAUNCH_PREFILL_TC(128, false);
+    if (d == 64) LAUNCH_PREFILL_TC(64, false, false);
+    else LAUNCH_PREFILL_TC(128, false, false);
   }
 #undef LAUNCH_PREFILL_TC
   VOSTI_LAUNCH_CHECK();

@@ -32,11 +32,9 @@ constexpr int UMMA_K = 16;
 constexpr int A_BYTES = BM * BK * 2;
 constexpr int THREADS = 192;
 
-enum Epilogue : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3, EPI_REGLU = 4, EPI_RE2GLU = 5, EPI_CLAMPGLU = 6 };
-// Gated epilogues: act(gate) * up with act = SiLU, relu, or the square of relu; or, with a limit L and a
-// constant c, g sigmoid(c g) (u + 1) of g = min(gate, L) and u = up clamped to [-L, L].
-__host__ __device__ constexpr bool is_gated(int epilogue) { return epilogue == EPI_SWIGLU || (epilogue >= EPI_REGLU && epilogue <= EPI_CLAMPGLU); }
-struct GluConstants { float limit, sigmoid_scale; };      // of EPI_CLAMPGLU
+enum Epilogue : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_PARTIAL = 3, EPI_REGLU = 4, EPI_RE2GLU = 5 };
+// Gated epilogues: act(gate) * up with act = SiLU, relu, or the square of relu.
+__host__ __device__ constexpr bool is_gated(int epilogue) { return epilogue == EPI_SWIGLU || epilogue == EPI_REGLU || epilogue == EPI_RE2GLU; }
 
 // Instruction descriptor: D float32, A and B bfloat16, both K-major, M = 128, N = bn.
 __host__ __device__ constexpr uint32_t instr_desc(int bn) {
@@ -49,21 +47,13 @@ __device__ __forceinline__ float gate_act(int epilogue, float g) {
   const float r = fmaxf(g, 0.f);
   return epilogue == EPI_RE2GLU ? r * r : r;
 }
-__device__ __forceinline__ float gated(int epilogue, float g, float u, const GluConstants& glu) {
-  if (epilogue == EPI_CLAMPGLU) {
-    g = fminf(g, glu.limit);
-    u = fminf(fmaxf(u, -glu.limit), glu.limit);
-    return g / (1.f + __expf(-glu.sigmoid_scale * g)) * (u + 1.f);
-  }
-  return gate_act(epilogue, g) * u;
-}
 
 // ------------------------------------------------------------------ the kernel
 template <int BN, int STAGES, int KPS>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                void* __restrict__ out, int tokens, int features, int k_blocks, int ld_out, int epilogue,
-               int w_tiles, int x_rows, const GluConstants glu, unsigned* status) {
+               int w_tiles, int x_rows, unsigned* status) {
   // x_rows: rows of the token box map_x brings per k-block (the tokens rounded up to 8, at most BN):
   // with few tokens the rest of the tile is never fetched; what those rows of shared memory
   // hold only reaches output columns that are not stored.
@@ -197,7 +187,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const float other = __shfl_xor_sync(0xffffffffu, mine, 16);
             const int t = n0 + c0 + j;
             if (lane < 16 && t < tokens && out_feature < ld_out)
-              y[(int64_t)t * ld_out + out_feature] = __float2bfloat16_rn(gated(epilogue, mine, other, glu));
+              y[(int64_t)t * ld_out + out_feature] = __float2bfloat16_rn(gate_act(epilogue, mine) * other);
           }
         } else if (feature < features) {
           if (epilogue == EPI_BF16) {
@@ -236,15 +226,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 // One token's 32 consecutive accumulator columns (features f0 .. f0 + 31) through the epilogue
 // into the output: bf16, float32, or SiLU(gate) * up of 16 gate and 16 up columns.
 __device__ __forceinline__ void store_token_columns(const uint32_t (&r)[32], void* __restrict__ out, int token, int f0,
-                                                    int features, int ld_out, int epilogue, const GluConstants& glu) {
+                                                    int features, int ld_out, int epilogue) {
   if (is_gated(epilogue)) {
     // columns f0..f0+15 are gate rows, f0+16..f0+31 their up rows (features % 32 == 0)
     bf16* y = reinterpret_cast<bf16*>(out) + (int64_t)token * ld_out + f0 / 2;
     uint32_t packed[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const float a = gated(epilogue, __uint_as_float(r[2 * j]), __uint_as_float(r[16 + 2 * j]), glu);
-      const float b = gated(epilogue, __uint_as_float(r[2 * j + 1]), __uint_as_float(r[17 + 2 * j]), glu);
+      const float a = gate_act(epilogue, __uint_as_float(r[2 * j])) * __uint_as_float(r[16 + 2 * j]);
+      const float b = gate_act(epilogue, __uint_as_float(r[2 * j + 1])) * __uint_as_float(r[17 + 2 * j]);
       __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
       packed[j] = *reinterpret_cast<uint32_t*>(&v);
     }
@@ -302,7 +292,7 @@ constexpr int WIDE_STAGE_BYTES = A_BYTES + WIDE_B_BYTES;
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                     void* __restrict__ out, int tokens, int features, int k_blocks, int ld_out, int epilogue,
-                    int w_tiles, const GluConstants glu, unsigned* status) {
+                    int w_tiles, unsigned* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   __shared__ __align__(8) uint64_t full_bar[WIDE_STAGES];
@@ -403,7 +393,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
         uint32_t r[32];
         tmem_load32(tmem_base + as * WIDE_BN + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0, r);
         if (!row_ok) continue;
-        store_token_columns(r, out, token, f0, features, ld_out, epilogue, glu);
+        store_token_columns(r, out, token, f0, features, ld_out, epilogue);
       }
       // this warp is done reading the accumulator: hand it back to the MMA warp
       tc_fence_before();
@@ -428,7 +418,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 
 // Sum the K splits in split order and apply the epilogue.
 __global__ void splitk_reduce_kernel(const float* __restrict__ partial, void* __restrict__ out, int splits,
-                                     int tokens, int features, int ld_out, int epilogue, const GluConstants glu) {
+                                     int tokens, int features, int ld_out, int epilogue) {
   pdl_wait();
   pdl_launch_dependents();
   const int64_t plane = (int64_t)tokens * features;
@@ -443,7 +433,7 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ partial, void* __
         g += partial[s * plane + t * features + row_g];
         u += partial[s * plane + t * features + row_u];
       }
-      reinterpret_cast<bf16*>(out)[t * ld_out + f] = __float2bfloat16_rn(gated(epilogue, g, u, glu));
+      reinterpret_cast<bf16*>(out)[t * ld_out + f] = __float2bfloat16_rn(gate_act(epilogue, g) * u);
     }
     return;
   }
@@ -497,7 +487,7 @@ int token_tile(int tokens) { return tokens <= 32 ? 32 : tokens <= 64 ? 64 : toke
 
 template <int BN, int STAGES, int KPS = 1>
 int launch(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int tokens, int features, int k_blocks, int ld_out,
-           int epilogue, int splits, int w_tiles, int x_rows, const GluConstants& glu, unsigned* status, cudaStream_t stream) {
+           int epilogue, int splits, int w_tiles, int x_rows, unsigned* status, cudaStream_t stream) {
   constexpr size_t smem = (size_t)STAGES * KPS * (A_BYTES + BN * BK * 2) + 1024;
   static_assert(smem <= 232448, "the ring does not fit an SM's shared memory");
   static bool configured = false;
@@ -511,7 +501,7 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int tokens, 
   }
   dim3 grid((features + BM - 1) / BM, (tokens + BN - 1) / BN, splits);
   vosti_launch(gemm_tc_kernel<BN, STAGES, KPS>, grid, dim3(THREADS), smem, stream, mw, mx, out, tokens, features, k_blocks, ld_out,
-               epilogue, w_tiles, x_rows, glu, status);
+               epilogue, w_tiles, x_rows, status);
   return 0;
 }
 
@@ -572,13 +562,13 @@ VOSTI_API int vosti_gemm_tc_grouped(const void* x, const void* w, void* y, const
                                     int features, int k, int epilogue, float* workspace, int64_t workspace_elems, int defer_reduce,
                                     float glu_limit, float glu_sigmoid_scale, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(rows >= 0 && tokens >= 0 && experts > 0 && vosti_gemm_tc_supported(features, k), "gemm_tc_grouped: unsupported sizes F=%d K=%d", features, k);
-  VOSTI_REQUIRE((epilogue >= EPI_BF16 && epilogue <= EPI_SWIGLU) || is_gated(epilogue), "gemm_tc_grouped: unknown epilogue %d", epilogue);
-  VOSTI_REQUIRE(!is_gated(epilogue) || features % 32 == 0, "gemm_tc_grouped: a fused act(gate)*up needs features %% 32 == 0");
+  VOSTI_REQUIRE(epilogue == EPI_BF16 || epilogue == EPI_F32 || grouped_is_gated(epilogue), "gemm_tc_grouped: unknown epilogue %d", epilogue);
+  VOSTI_REQUIRE(!grouped_is_gated(epilogue) || features % 32 == 0, "gemm_tc_grouped: a fused act(gate)*up needs features %% 32 == 0");
   VOSTI_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0), "gemm_tc_grouped: operands must be 16-byte aligned");
   VOSTI_REQUIRE(offsets != nullptr, "gemm_tc_grouped: the experts' row ranges are missing");
   if (rows == 0) return VOSTI_OK;
   const GluConstants glu = {glu_limit, glu_sigmoid_scale};
-  const int ld_out = is_gated(epilogue) ? features / 2 : features;
+  const int ld_out = grouped_is_gated(epilogue) ? features / 2 : features;
   const int k_blocks = (k + BK - 1) / BK;
   const int tiles_per_expert = (features + BM - 1) / BM;
   const int64_t w_rows64 = (int64_t)k_blocks * experts * tiles_per_expert * BM;
@@ -626,8 +616,12 @@ VOSTI_API int vosti_gemm_tc_grouped(const void* x, const void* w, void* y, const
   if (splits > 1 && !defer_reduce) {
     const int64_t n = (int64_t)rows * features;
     const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
-    vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)workspace, y, splits, rows, features, ld_out,
-                 epilogue, glu);
+    if (epilogue == EPI_CLAMPGLU)
+      vosti_launch(grouped_clamped_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)workspace, (bf16*)y, splits, rows,
+                   features, glu);
+    else
+      vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)workspace, y, splits, rows, features, ld_out,
+                   epilogue);
   }
   VOSTI_LAUNCH_CHECK();
 }
@@ -657,14 +651,12 @@ VOSTI_API int vosti_gemm_tc_splits(int tokens, int features, int k) {
 
 // x: [tokens, k] bf16; w: [features, k] bf16; epilogue 0: y bf16 [tokens, features];
 // 1: y float32 [tokens, features]; 2: y bf16 [tokens, features / 2] = silu(gate) * up with
-// the weight rows interleaved in blocks of 16 gate rows and their 16 up rows (4, 5: relu and squared relu; 6: the
-// clamped form with glu_limit and glu_sigmoid_scale).
+// the weight rows interleaved in blocks of 16 gate rows and their 16 up rows.
 // With `defer_reduce` and more than one split the partial sums stay in the workspace
 // ([splits, tokens, features] float32) for a consumer that sums them itself; y is not written.
 VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, int features, int k, int epilogue,
-                            float* workspace, int64_t workspace_elems, int defer_reduce, int w_packed, float glu_limit,
-                            float glu_sigmoid_scale, unsigned* status, cudaStream_t stream) {
-  const GluConstants glu = {glu_limit, glu_sigmoid_scale};
+                            float* workspace, int64_t workspace_elems, int defer_reduce, int w_packed, unsigned* status,
+                            cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && vosti_gemm_tc_supported(features, k), "gemm_tc: unsupported sizes F=%d K=%d", features, k);
   VOSTI_REQUIRE((epilogue >= EPI_BF16 && epilogue <= EPI_SWIGLU) || is_gated(epilogue), "gemm_tc: unknown epilogue %d", epilogue);
   VOSTI_REQUIRE(!is_gated(epilogue) || features % 32 == 0, "gemm_tc: a fused act(gate)*up needs features %% 32 == 0");
@@ -706,7 +698,7 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
     const int tiles = ((tokens + 2 * BM - 1) / (2 * BM)) * ((features + PAIR_BN - 1) / PAIR_BN);
     const int pairs = tiles < pair_sms / 2 ? tiles : pair_sms / 2;
     vosti_launch_clusters(gemm_tc_pair_kernel, dim3(2 * pairs), dim3(PAIR_THREADS), 2, smem, stream, mx, *mw, y, tokens,
-                          features, k_blocks, ld_out, epilogue, w_tiles, glu, status);
+                          features, k_blocks, ld_out, epilogue, w_tiles, status);
     VOSTI_LAUNCH_CHECK();
   }
   if (tokens > 128) {
@@ -728,7 +720,7 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
     }
     const int tiles = ((tokens + BM - 1) / BM) * ((features + WIDE_BN - 1) / WIDE_BN);
     vosti_launch(gemm_tc_wide_kernel, dim3(tiles < sms ? tiles : sms), dim3(THREADS), smem, stream, mx, *mw, y, tokens,
-                 features, k_blocks, ld_out, epilogue, w_tiles, glu, status);
+                 features, k_blocks, ld_out, epilogue, w_tiles, status);
     VOSTI_LAUNCH_CHECK();
   }
   const int bn = token_tile(tokens);
@@ -741,7 +733,7 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
   // no more CTAs than SMs: each has an SM's shared memory to itself and takes two k-blocks per stage
   const int64_t ctas = (int64_t)((features + BM - 1) / BM) * ((tokens + bn - 1) / bn) * splits;
   const bool lone = ctas <= 148;
-#define VOSTI_GEMM_ARGS *mw, mx, dst, tokens, features, k_blocks, ld, epi, splits, w_tiles, x_rows, glu, status, stream
+#define VOSTI_GEMM_ARGS *mw, mx, dst, tokens, features, k_blocks, ld, epi, splits, w_tiles, x_rows, status, stream
   int rc;
   switch (bn) {
     case 32: rc = lone ? launch<32, 5, 2>(VOSTI_GEMM_ARGS) : launch<32, 5>(VOSTI_GEMM_ARGS); break;
@@ -755,7 +747,7 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
     const int64_t n = (int64_t)tokens * features;
     const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
     vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)workspace, y, splits, tokens,
-                 features, ld_out, epilogue, glu);
+                 features, ld_out, epilogue);
   }
   VOSTI_LAUNCH_CHECK();
 }
@@ -769,7 +761,7 @@ VOSTI_API int vosti_splitk_reduce(const float* partial, void* y, int splits, int
   const int64_t n = (int64_t)tokens * features;
   const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
   vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, partial, y, splits, tokens, features, features,
-               (int)(y_is_f32 ? EPI_F32 : EPI_BF16), GluConstants{});
+               (int)(y_is_f32 ? EPI_F32 : EPI_BF16));
   VOSTI_LAUNCH_CHECK();
 }
 
@@ -830,16 +822,16 @@ VOSTI_API int vosti_gemm_tc_split_static(const void* x, const void* w, void* y, 
   const int epi = splits > 1 ? EPI_PARTIAL : epilogue;
   int rc;
   switch (bn) {
-    case 32: rc = launch<32, 5>(mw, mx, dst, tokens, features, k_blocks, features, epi, splits, 0, bn, GluConstants{}, status, stream); break;
-    case 64: rc = launch<64, 4>(mw, mx, dst, tokens, features, k_blocks, features, epi, splits, 0, bn, GluConstants{}, status, stream); break;
-    default: rc = launch<128, 6>(mw, mx, dst, tokens, features, k_blocks, features, epi, splits, 0, bn, GluConstants{}, status, stream); break;
+    case 32: rc = launch<32, 5>(mw, mx, dst, tokens, features, k_blocks, features, epi, splits, 0, bn, status, stream); break;
+    case 64: rc = launch<64, 4>(mw, mx, dst, tokens, features, k_blocks, features, epi, splits, 0, bn, status, stream); break;
+    default: rc = launch<128, 6>(mw, mx, dst, tokens, features, k_blocks, features, epi, splits, 0, bn, status, stream); break;
   }
   if (rc != 0) return rc;
   if (splits > 1) {
     const int64_t n = (int64_t)tokens * features;
     const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
     vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)scratch, y, splits, tokens,
-                 features, features, epilogue, GluConstants{});
+                 features, features, epilogue);
   }
   VOSTI_LAUNCH_CHECK();
 }

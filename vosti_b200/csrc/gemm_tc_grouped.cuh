@@ -12,6 +12,23 @@
 // grouped_wide (more): rows on the M side as in gemm_tc_wide_kernel, persistent over the tiles
 // (expert, 128 rows, 256 features); a tile's rows beyond its expert's are computed and not stored.
 
+// Epilogues: bfloat16, float32, unsummed K splits, or a gated form (the features then are blocks of 16 gate
+// features and their 16 up features): those of gemm_tc.cu, and EPI_CLAMPGLU with a limit L and a constant c,
+// g sigmoid(c g) (u + 1) of g = min(gate, L) and u = up clamped to [-L, L]. (It is not one of gemm_tc_kernel's:
+// one more branch in that kernel's unrolled epilogue cost the other models' decode steps 2 %.)
+constexpr int EPI_CLAMPGLU = 6;
+struct GluConstants { float limit, sigmoid_scale; };
+
+__host__ __device__ constexpr bool grouped_is_gated(int epilogue) { return is_gated(epilogue) || epilogue == EPI_CLAMPGLU; }
+__device__ __forceinline__ float grouped_gate(int epilogue, float g, float u, const GluConstants& glu) {
+  if (epilogue == EPI_CLAMPGLU) {
+    g = fminf(g, glu.limit);
+    u = fminf(fmaxf(u, -glu.limit), glu.limit);
+    return g / (1.f + __expf(-glu.sigmoid_scale * g)) * (u + 1.f);
+  }
+  return gate_act(epilogue, g) * u;
+}
+
 // The n-th expert that has rows, and its rows [lo, hi); -1 if there are fewer. Every warp of the block alike.
 __device__ __forceinline__ int nth_busy_expert(const int* __restrict__ offsets, int experts, int n, int& lo, int& hi) {
   const int lane = threadIdx.x & 31;
@@ -123,7 +140,7 @@ gemm_tc_grouped_few_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = 0u;
         }
-        if (is_gated(epilogue)) {
+        if (grouped_is_gated(epilogue)) {
           bf16* y = reinterpret_cast<bf16*>(out);
           const int out_feature = (m0 + quarter * 32) / 2 + (lane & 15);
 #pragma unroll
@@ -131,7 +148,7 @@ gemm_tc_grouped_few_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
             const float mine = __uint_as_float(r[j]);
             const float other = __shfl_xor_sync(0xffffffffu, mine, 16);
             if (lane < 16 && c0 + j < n && out_feature < ld_out)
-              y[(int64_t)(row_lo + c0 + j) * ld_out + out_feature] = __float2bfloat16_rn(gated(epilogue, mine, other, glu));
+              y[(int64_t)(row_lo + c0 + j) * ld_out + out_feature] = __float2bfloat16_rn(grouped_gate(epilogue, mine, other, glu));
           }
         } else if (feature < features) {
           float* y = reinterpret_cast<float*>(out) + (epilogue == EPI_PARTIAL ? (int64_t)split * rows * ld_out : 0);
@@ -286,7 +303,27 @@ gemm_tc_grouped_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __g
         uint32_t r[32];
         tmem_load32(tmem_base + as * WIDE_BN + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0, r);
         if (!row_ok) continue;
-        store_token_columns(r, out, row, f0, features, ld_out, epilogue, glu);
+        if (epilogue == EPI_CLAMPGLU) {
+          // columns f0 .. f0 + 15 are gate features, f0 + 16 .. f0 + 31 their up features
+          uint32_t packed[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const __nv_bfloat162 v = __floats2bfloat162_rn(
+                grouped_gate(EPI_CLAMPGLU, __uint_as_float(r[2 * j]), __uint_as_float(r[16 + 2 * j]), glu),
+                grouped_gate(EPI_CLAMPGLU, __uint_as_float(r[2 * j + 1]), __uint_as_float(r[17 + 2 * j]), glu));
+            packed[j] = *reinterpret_cast<const uint32_t*>(&v);
+          }
+          bf16* y = reinterpret_cast<bf16*>(out) + (int64_t)row * ld_out + f0 / 2;
+          if ((ld_out & 7) == 0) {
+            reinterpret_cast<uint4*>(y)[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+            reinterpret_cast<uint4*>(y)[1] = make_uint4(packed[4], packed[5], packed[6], packed[7]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) reinterpret_cast<uint32_t*>(y)[j] = packed[j];   // ld_out is even
+          }
+          continue;
+        }
+        store_token_columns(r, out, row, f0, features, ld_out, epilogue);
       }
       tc_fence_before();
       __syncwarp();
@@ -302,5 +339,24 @@ gemm_tc_grouped_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __g
   if (warp == 1) {
     tc_fence_after();
     tmem_dealloc(tmem_base, 2 * WIDE_BN);
+  }
+}
+
+// The K splits of a clamped gated product, summed in split order, through the activation.
+__global__ void grouped_clamped_reduce_kernel(const float* __restrict__ partial, bf16* __restrict__ out, int splits, int rows,
+                                              int features, const GluConstants glu) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t plane = (int64_t)rows * features, n = plane / 2;
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t row = i / (features / 2);
+    const int f = (int)(i % (features / 2));
+    const float* p = partial + row * features + (f / 16) * 32 + f % 16;
+    float g = 0.f, u = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      g += p[s * plane];
+      u += p[s * plane + 16];
+    }
+    out[i] = __float2bfloat16_rn(grouped_gate(EPI_CLAMPGLU, g, u, glu));
   }
 }

@@ -78,7 +78,7 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
 __global__ void __launch_bounds__(pair_kernel::PAIR_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                     void* __restrict__ out, int tokens, int features, int k_blocks, int ld_out, int epilogue,
-                    int w_tiles, const GluConstants glu, unsigned* status) {
+                    int w_tiles, unsigned* status) {
   using namespace pair_kernel;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -194,7 +194,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
         uint32_t r[32];
         tmem_load32(tmem_base + as * PAIR_BN + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0, r);
         if (!row_ok) continue;
-        store_token_columns(r, out, token, f0, features, ld_out, epilogue, glu);
+        store_token_columns(r, out, token, f0, features, ld_out, epilogue);
       }
       tc_fence_before();
       __syncwarp();

@@ -175,7 +175,8 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
 
 
 GLU_ACTIVATIONS = {"silu": 0, "relu": 1, "relu2": 2, "clamped": 3}
-FUSED_GLU_ACTIVATIONS = {"silu": 2, "relu": 4, "relu2": 5, "clamped": 6}         # the tensor-core product's gated epilogues
+FUSED_GLU_ACTIVATIONS = {"silu": 2, "relu": 4, "relu2": 5}         # the tensor-core product's gated epilogues
+GROUPED_GLU_ACTIVATIONS = {**FUSED_GLU_ACTIVATIONS, "clamped": 6}                  # those of the grouped products
 
 
 def glu_mul(gate_up: torch.Tensor, activation: str, limit: float = 0.0, sigmoid_scale: float = 0.0) -> torch.Tensor:
@@ -430,8 +431,9 @@ def gemm_tc_grouped(x: torch.Tensor, w: ExpertWeights, offsets: torch.Tensor, to
                     out_dtype: torch.dtype = torch.bfloat16, activation: Optional[str] = None, glu=(0.0, 0.0),
                     allow_partial: bool = False, scratch: str = "split_k"):
     """y[r] = x[r] @ w[expert of r].T for rows sorted by expert: expert e owns rows offsets[e] .. offsets[e + 1] - 1
-    (int32 [experts + 1], on the device; no expert has more than `tokens` of them). `activation`: the
-    gated epilogue of `gemm_tc` (bfloat16 out, half as many columns). csrc/gemm_tc_grouped.cuh."""
+    (int32 [experts + 1], on the device; no expert has more than `tokens` of them). `activation`: a
+    gated epilogue (bfloat16 out, half as many columns), one of `gemm_tc`'s or "clamped" (see glu_mul; `glu` =
+    (limit, sigmoid_scale)). csrc/gemm_tc_grouped.cuh."""
     _contig(x, w.data, offsets)
     if x.dtype != torch.bfloat16 or x.shape[1] != w.k or offsets.dtype != torch.int32 or offsets.shape[0] != w.experts + 1:
         raise KernelError("gemm_tc_grouped: x is bfloat16 [rows, k], offsets int32 [experts + 1]")
@@ -440,7 +442,7 @@ def gemm_tc_grouped(x: torch.Tensor, w: ExpertWeights, offsets: torch.Tensor, to
     if activation is not None:
         if out_dtype != torch.bfloat16:
             raise KernelError("gemm_tc_grouped: the gated epilogues write bfloat16")
-        epilogue, width = FUSED_GLU_ACTIVATIONS[activation], features // 2
+        epilogue, width = GROUPED_GLU_ACTIVATIONS[activation], features // 2
     lib = library()
     splits = lib.vosti_gemm_tc_grouped_splits(tokens, rows, w.experts, features, w.k)
     ws = _workspace(x.device, splits * rows * features, scratch) if splits > 1 else None
@@ -456,14 +458,12 @@ def gemm_tc_grouped(x: torch.Tensor, w: ExpertWeights, offsets: torch.Tensor, to
 
 
 def gemm_tc(x: torch.Tensor, w, status: torch.Tensor, *, out_dtype: Optional[torch.dtype] = None,
-            swiglu: bool = False, allow_partial: bool = False, activation: str = "silu", glu=(0.0, 0.0),
-            scratch: str = "split_k"):
+            swiglu: bool = False, allow_partial: bool = False, activation: str = "silu", scratch: str = "split_k"):
     """y = x @ w.T on the tensor cores (bfloat16 operands, float32 accumulation); w is a
     [features, k] tensor or a `PackedWeight`. With `swiglu` the rows of w are blocks of 16 gate
     rows followed by their 16 up rows and y = act(gate) * up has half as many columns, act being
-    `activation`: "silu", "relu" or "relu2" (the square of relu), or the pair goes through the "clamped"
-    form (see glu_mul; `glu` = (limit, sigmoid_scale)). `scratch` names the buffer of the K splits: two
-    results that stay unsummed at the same time need buffers of their own."""
+    `activation`: "silu", "relu" or "relu2" (the square of relu). `scratch` names the buffer of the K splits:
+    two results that stay unsummed at the same time need buffers of their own."""
     packed = isinstance(w, PackedWeight)
     w_data = w.data if packed else w
     _contig(x, w_data)
@@ -491,8 +491,8 @@ def gemm_tc(x: torch.Tensor, w, status: torch.Tensor, *, out_dtype: Optional[tor
     if splits > 1:
         _SPLIT_GENERATION[scratch] = _SPLIT_GENERATION.get(scratch, 0) + 1
     _check(lib.vosti_gemm_tc(_p(x), _p(w_data), _p(out), tokens, features, k, epilogue, _p(ws),
-                             ctypes.c_int64(ws.numel() if ws is not None else 0), int(defer), int(packed), ctypes.c_float(glu[0]),
-                             ctypes.c_float(glu[1]), _p(status), _stream()),
+                             ctypes.c_int64(ws.numel() if ws is not None else 0), int(defer), int(packed), _p(status),
+                             _stream()),
            "gemm_tc", kernels=2 if splits > 1 and not defer else 1)
     if defer:
         return PartialSum(ws, splits, tokens, features, out_dtype, status, scratch)

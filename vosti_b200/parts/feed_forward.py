@@ -54,7 +54,7 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 def gated_activation(ctx, x, w_gate_up, fused: bool, activation: str = "silu", glu=(0.0, 0.0)):
     if fused:
-        return ops.gemm_tc(ops.materialize(x), w_gate_up, ctx.status, swiglu=True, activation=activation, glu=glu)
+        return ops.gemm_tc(ops.materialize(x), w_gate_up, ctx.status, swiglu=True, activation=activation)
     return ops.glu_mul(ops.materialize(linear(ctx, x, w_gate_up)), activation, *glu)
 
 
@@ -245,7 +245,7 @@ class ExpertMixture(FeedForward):
         """The experts one after the other for the grouped products, if those take their sizes."""
         downs = [tensors[f"e{e}.down"] for e in range(self.experts)]
         pairs = [(tensors[f"e{e}.gate"], tensors[f"e{e}.up"]) for e in range(self.experts)]
-        if (dtype != torch.bfloat16 or self.inter % 16 or self.gate_activation not in ops.FUSED_GLU_ACTIVATIONS
+        if (dtype != torch.bfloat16 or self.inter % 16 or self.gate_activation not in ops.GROUPED_GLU_ACTIVATIONS
                 or not all(uses_tensor_cores(dtype, w) for w in downs + [w for pair in pairs for w in pair])):
             return False
         self.grouped = (ops.ExpertWeights([interleave_gate_up(g, u) for g, u in pairs]), ops.ExpertWeights(downs))
