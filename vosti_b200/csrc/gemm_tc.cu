@@ -515,23 +515,30 @@ int device_sms() {
   return sms;
 }
 
-template <int BN, int STAGES>
-int launch_grouped_few(const CUtensorMap& mw, const CUtensorMap& mx, void* out, const int* offsets, int experts, int busy, int rows,
+template <int BN, int STAGES, int KIND>
+int launch_grouped_kind(const CUtensorMap& mw, const CUtensorMap& mx, void* out, const int* offsets, int experts, int busy, int rows,
                        int features, int tiles_per_expert, int k_blocks, int ld_out, int epilogue, int splits, int w_tiles, int x_rows,
                        const GluConstants& glu, unsigned* status, cudaStream_t stream) {
   constexpr size_t smem = (size_t)STAGES * (A_BYTES + BN * BK * 2) + 1024;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_tc_grouped_few_kernel<BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_grouped_few_kernel<BN, STAGES, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) {
       vosti_set_error("gemm_tc_grouped: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
       return (int)e;
     }
     configured = true;
   }
-  vosti_launch(gemm_tc_grouped_few_kernel<BN, STAGES>, dim3(tiles_per_expert, busy, splits), dim3(THREADS), smem, stream, mw, mx, out,
+  vosti_launch(gemm_tc_grouped_few_kernel<BN, STAGES, KIND>, dim3(tiles_per_expert, busy, splits), dim3(THREADS), smem, stream, mw, mx, out,
                offsets, experts, rows, features, tiles_per_expert, k_blocks, ld_out, epilogue, w_tiles, x_rows, glu, status);
   return 0;
+}
+
+template <int BN, int STAGES, typename... Args>
+int launch_grouped_few(int kind, const Args&... args) {
+  if (kind == 0) return launch_grouped_kind<BN, STAGES, 0>(args...);
+  if (kind == 1) return launch_grouped_kind<BN, STAGES, 1>(args...);
+  return kind == 2 ? launch_grouped_kind<BN, STAGES, 2>(args...) : launch_grouped_kind<BN, STAGES, 3>(args...);
 }
 
 }  // namespace
@@ -604,7 +611,7 @@ VOSTI_API int vosti_gemm_tc_grouped(const void* x, const void* w, void* y, const
   const int epi = splits > 1 ? EPI_PARTIAL : epilogue;
   const int ld = splits > 1 ? features : ld_out;
   const int busy = rows < experts ? rows : experts;
-#define VOSTI_GROUPED_ARGS mw, mx, dst, offsets, experts, busy, rows, features, tiles_per_expert, k_blocks, ld, epi, splits, w_tiles, x_rows, glu, status, stream
+#define VOSTI_GROUPED_ARGS grouped_kind(epi), mw, mx, dst, offsets, experts, busy, rows, features, tiles_per_expert, k_blocks, ld, epi, splits, w_tiles, x_rows, glu, status, stream
   int rc;
   switch (bn) {
     case 32: rc = launch_grouped_few<32, 5>(VOSTI_GROUPED_ARGS); break;

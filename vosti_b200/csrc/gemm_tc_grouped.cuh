@@ -49,7 +49,13 @@ __device__ __forceinline__ int nth_busy_expert(const int* __restrict__ offsets, 
   return -1;
 }
 
-template <int BN, int STAGES>
+// KIND of epilogue, known where the code is laid out so that a kernel's unrolled epilogue holds one form:
+// 0 bfloat16; 1 float32 or unsummed splits; 2 a gated form of gemm_tc.cu; 3 the clamped form.
+__host__ __device__ constexpr int grouped_kind(int epilogue) {
+  return epilogue == EPI_BF16 ? 0 : epilogue == EPI_CLAMPGLU ? 3 : is_gated(epilogue) ? 2 : 1;
+}
+
+template <int BN, int STAGES, int KIND>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_grouped_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                            void* __restrict__ out, const int* __restrict__ offsets, int experts, int rows, int features,
@@ -140,7 +146,7 @@ gemm_tc_grouped_few_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = 0u;
         }
-        if (grouped_is_gated(epilogue)) {
+        if (KIND >= 2) {
           bf16* y = reinterpret_cast<bf16*>(out);
           const int out_feature = (m0 + quarter * 32) / 2 + (lane & 15);
 #pragma unroll
@@ -148,15 +154,15 @@ gemm_tc_grouped_few_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
             const float mine = __uint_as_float(r[j]);
             const float other = __shfl_xor_sync(0xffffffffu, mine, 16);
             if (lane < 16 && c0 + j < n && out_feature < ld_out)
-              y[(int64_t)(row_lo + c0 + j) * ld_out + out_feature] = __float2bfloat16_rn(grouped_gate(epilogue, mine, other, glu));
+              y[(int64_t)(row_lo + c0 + j) * ld_out + out_feature] = __float2bfloat16_rn(grouped_gate(KIND == 3 ? EPI_CLAMPGLU : epilogue, mine, other, glu));
           }
         } else if (feature < features) {
-          float* y = reinterpret_cast<float*>(out) + (epilogue == EPI_PARTIAL ? (int64_t)split * rows * ld_out : 0);
+          float* y = reinterpret_cast<float*>(out) + (KIND == 1 && epilogue == EPI_PARTIAL ? (int64_t)split * rows * ld_out : 0);
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             if (c0 + j >= n) continue;
             const int64_t at = (int64_t)(row_lo + c0 + j) * ld_out + feature;
-            if (epilogue == EPI_BF16) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(__uint_as_float(r[j]));
+            if (KIND == 0) reinterpret_cast<bf16*>(out)[at] = __float2bfloat16_rn(__uint_as_float(r[j]));
             else y[at] = __uint_as_float(r[j]);
           }
         }
