@@ -4,8 +4,8 @@ of fixed size.
 
 Layers whose mixers keep everything share one group (one id space, one block table,
 as the reference's layers do: python/vosti_kernels/physical.py:124-147, 329-339);
-layers that only ever read a window of the past form a group of their own, whose pages
-are given back as soon as the window has passed them. A slot is ``page * page_size +
+layers that only ever read a window of the past (and perhaps a request's first tokens) form a group
+of their own, whose pages are given back as soon as the window has passed them. A slot is ``page * page_size +
 offset`` (kernels/triton_kernels/store_kv_cache.py:21-25); a layer's storage is
 ``[num_pages, heads, page_size, width]``, so the tokens one head holds in a page are
 contiguous (the reference keeps ``[pages, page_size, heads, width]``).
@@ -54,6 +54,7 @@ class CacheGroup:
     window: int
     layers: List[int]
     pool: PagePool
+    keep_first: int = 0          # tokens at a request's start whose pages a window never passes
 
 
 @dataclass
@@ -114,16 +115,19 @@ class CacheManager:
         self.page_size, self.num_pages, self.max_requests = page_size, num_pages, max_requests
         self.layer_caches: List[LayerCache] = []
         windows: List[int] = []
+        keeps: List[int] = []
         layers_of: List[List[int]] = []
-        by_window: Dict[int, int] = {}
+        by_window: Dict[Tuple[int, int], int] = {}
         for layer, spec in enumerate(cache_specs):
             cache = LayerCache(page_size=page_size)
             if spec is not None:
-                if spec.window not in by_window:
-                    by_window[spec.window] = len(windows)
-                    windows.append(spec.window)
+                reach = (spec.window, spec.keep_first if spec.window else 0)
+                if reach not in by_window:
+                    by_window[reach] = len(windows)
+                    windows.append(reach[0])
+                    keeps.append(reach[1])
                     layers_of.append([])
-                cache.group = by_window[spec.window]
+                cache.group = by_window[reach]
                 layers_of[cache.group].append(layer)
                 if device is not None:
                     # zeros, not empty: the decode kernel reads whole boxes of 16 keys and masks
@@ -147,7 +151,7 @@ class CacheManager:
         # with a windowed group or per-request state a prefix would need more than pages to
         # be reused, so the core switches reuse off then.
         self._lib = host.library()
-        self._ptr = self._lib.vh_create(len(windows), host.ints(windows), num_pages, page_size, max_requests,
+        self._ptr = self._lib.vh_create(len(windows), host.ints(windows), host.ints(keeps), num_pages, page_size, max_requests,
                                         int(prefix_reuse), int(self.has_state), max_requests, 4096, 0, 0, 0)
         if not self._ptr:
             raise ValueError("the host core refused the cache geometry")
@@ -155,8 +159,8 @@ class CacheManager:
         self.prefix_reuse = bool(self._lib.vh_prefix_reuse(self._h))
         self.has_windows = any(w > 0 for w in windows)
         self.groups: List[CacheGroup] = [
-            CacheGroup(window, layers, PagePool(borrowed=self._lib.vh_group_pool(self._h, g)))
-            for g, (window, layers) in enumerate(zip(windows, layers_of))]
+            CacheGroup(window, layers, PagePool(borrowed=self._lib.vh_group_pool(self._h, g)), keep)
+            for g, (window, keep, layers) in enumerate(zip(windows, keeps, layers_of))]
         self._handles: Dict[object, int] = {}
         self._names: Dict[int, object] = {}
         self._next_handle = 1
@@ -267,7 +271,8 @@ class CacheManager:
 
     def trim(self, request_id) -> int:
         """Give back the pages a window has passed: every query from now on sits at a
-        position >= length and reads keys > position - window only."""
+        position >= length and reads keys > position - window (and the request's first ones, if the
+        group keeps them) only."""
         return host.check(self._lib.vh_trim(self._h, self._rid(request_id)))
 
     def publish(self, request_id, tokens: Sequence[int]) -> int:

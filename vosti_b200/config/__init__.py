@@ -8,6 +8,7 @@ from . import vivesun as _vivesun
 from . import beralix as _beralix
 from . import nefipel as _nefipel
 from . import pubulix as _pubulix
+from . import difavik as _difavik
 
 register_architecture(_qwen3.ARCHITECTURE, _qwen3.spec_from_config, replace=True)
 register_architecture(_mugizen.ARCHITECTURE, _mugizen.spec_from_config, replace=True)
@@ -15,6 +16,7 @@ register_architecture(_vivesun.ARCHITECTURE, _vivesun.spec_from_config, replace=
 register_architecture(_beralix.ARCHITECTURE, _beralix.spec_from_config, replace=True)
 register_architecture(_nefipel.ARCHITECTURE, _nefipel.spec_from_config, replace=True)
 register_architecture(_pubulix.ARCHITECTURE, _pubulix.spec_from_config, replace=True)
+register_architecture(_difavik.ARCHITECTURE, _difavik.spec_from_config, replace=True)
 
 __all__ = [
     "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "Qwen3Config",

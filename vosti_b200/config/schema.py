@@ -64,6 +64,7 @@ class LayerSpec:
     out_norm: Optional[PartSpec] = None         # a norm on every sublayer's output before it joins the stream (arrangements that take one)
     layer_scale: bool = False                   # a learned vector per sublayer multiplies what joins the stream
     residual_scale: float = 1.0                 # a constant on what joins the stream (arrangements that take one)
+    number: Optional[int] = None                # the number its tensors carry in the checkpoint, where that is not its place in the list
     input_conv: int = 0                         # taps of a causal convolution on what the mixer reads (arrangements that take one)
 
     def name_of(self, role: str) -> str:

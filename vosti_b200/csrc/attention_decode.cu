@@ -43,13 +43,14 @@ namespace {
 using namespace decode_attention;
 
 struct ItemMeta {
-  int t, pos, item, g, seg, kstart, request, fresh;  // t < 0: no more items; fresh: the token's own key and value come with it
+  int t, pos, item, g, seg, kstart, request, fresh;  // t < 0: no more items; fresh: the token's own key and value come with it;
+                                                     // sloped: kstart is the window's first key, the keys are counted (KeyCount)
 };
 
 // DMAX bounds the head size; with EXACT the head size is DMAX itself. FUSED: the query rows and
 // the token's own key and value are made here from the projection's partial sums (`fused`). CAPPED: the
 // scores pass a soft cap (fused.softcap).
-template <int DMAX, bool EXACT, bool FUSED, bool CAPPED>
+template <int DMAX, bool EXACT, bool FUSED, bool CAPPED, bool SLOPED>
 __global__ void __launch_bounds__(THREADS, DMAX <= 128 ? 2 : 1)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const bf16* __restrict__ q, float* __restrict__ partial, bf16* __restrict__ out,
@@ -110,6 +111,10 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
   const int pairs = count * nkv;                      // the launcher keeps pairs * max_segments below 2^31
   const int total_items = pairs * max_segments;
   const int quarter = segment_keys / CONSUMERS;
+  const int keep = SLOPED ? fused.score_bias_last : 0;
+  // the sloped form counts the keys that may be visible: how, the count's place of the position and of the first key
+  auto counted = [&](int pos) { return SLOPED ? key_count(pos, window, keep) : KeyCount{0, 0}; };
+  auto first_counted = [&](int kstart, const KeyCount& c) { return SLOPED && (keep > 0 || c.gap > 0) ? 0 : kstart; };
 
   if (warp == 0) {
     // ------------------------------------------------------------ producer
@@ -146,7 +151,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
           next_pages[k] = (index >= lo && index <= hi && index < max_pages) ? table[index] : -1;
         }
       };
-      if (whole_pages) fetch_pages(0);
+      if (whole_pages && !SLOPED) fetch_pages(0);
       for (int j = 0; j < n; ++j) {
         const int t = __shfl_sync(0xffffffffu, t_l, j), pos = __shfl_sync(0xffffffffu, pos_l, j);
         const int req = __shfl_sync(0xffffffffu, req_l, j);
@@ -155,24 +160,28 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         const int g = (idx % pairs) % nkv;
         const int item = (idx % pairs) / nkv;
         const int kstart = first_visible_key(pos, window);
-        const int seg_begin = seg * segment_keys, seg_end = min(seg_begin + segment_keys, pos + 1);
-        if (whole_pages) {
+        const KeyCount kc = counted(pos);
+        const int vpos = pos - kc.gap, vstart = first_counted(kstart, kc);
+        const int seg_begin = seg * segment_keys, seg_end = min(seg_begin + segment_keys, vpos + 1);
+        if (whole_pages && !SLOPED) {
           __syncwarp();
 #pragma unroll
           for (int k = 0; k < MAX_SEGMENT_PAGES / 32; ++k) segment_pages[lane + 32 * k] = next_pages[k];
           __syncwarp();
           if (j + 1 < n) fetch_pages(j + 1);         // in flight while this item is described
         }
-        if (seg_begin > pos || seg_end <= kstart) continue;          // nothing visible in this segment
+        if (seg_begin > vpos || seg_end <= vstart) continue;         // nothing visible in this segment
         const uint32_t qb = q_issued % Q_BUFFERS;
         if (q_issued >= Q_BUFFERS)
           wait_or_abandon(smem_addr(&q_empty[qb]), ((q_issued / Q_BUFFERS) - 1) & 1, status, &abandoned);
         if (whole_pages) {
           const int first_index = seg_begin / page_size;
           for (int i = lane; i < segment_keys / TILE; i += 32) {
-            const int key0 = seg_begin + i * TILE;
+            const int key0 = SLOPED ? kc.key(seg_begin + i * TILE) : seg_begin + i * TILE;
             const int index = page_shift >= 0 ? key0 >> page_shift : key0 / page_size;
-            const int page = segment_pages[min(index - first_index, MAX_SEGMENT_PAGES - 1)];
+            int page;
+            if (SLOPED) page = (key0 <= pos && index < max_pages) ? block_table[(int64_t)req * max_pages + index] : -1;
+            else page = segment_pages[min(index - first_index, MAX_SEGMENT_PAGES - 1)];
             tile_rows[qb][i] = (page < 0 || page >= num_pages) ? -1 : (page * nkv + g) * page_size + (key0 - index * page_size);
           }
           __syncwarp();
@@ -268,10 +277,11 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 
   // This warp's tiles of an item: first key of its first tile, and their number.
   auto my_tiles = [&](const ItemMeta& m, int& first_tile, int& tiles) {
-    const int seg_begin = m.seg * segment_keys, seg_end = min(seg_begin + segment_keys, m.pos + 1);
+    const KeyCount kc = counted(m.pos);
+    const int seg_begin = m.seg * segment_keys, seg_end = min(seg_begin + segment_keys, m.pos - kc.gap + 1);
     const int my_begin = seg_begin + cw * quarter;
     const int my_end = min(my_begin + quarter, seg_end);
-    first_tile = max(my_begin, (m.kstart / TILE) * TILE);             // tiles stay aligned to the key index
+    first_tile = max(my_begin, (first_counted(m.kstart, kc) / TILE) * TILE);             // tiles stay aligned to the key index
     tiles = my_end > first_tile ? (my_end - first_tile + TILE - 1) / TILE : 0;
   };
   // Request the 16 keys from key0 of the item described in buffer `qslot` into the next ring slot.
@@ -301,9 +311,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       }
     } else {
       // any page size: one box of one row per key; lanes 0-15 fetch K rows, 16-31 V rows
-      const int key = key0 + (lane & 15);
+      const int key = (SLOPED ? counted(m.pos).key(key0) : key0) + (lane & 15);      // (key0: in the sloped form a place in the count)
       int row = -1;
-      if (key >= m.kstart && key <= m.pos) {
+      if ((key >= m.kstart || (SLOPED && key < keep)) && key <= m.pos) {
         const int index = page_shift >= 0 ? key >> page_shift : key / page_size;
         const int page = index < max_pages ? block_table[(int64_t)m.request * max_pages + index] : -1;
         if (page < 0 || page >= num_pages) raise_fault(status, VOSTI_FAULT_PAGE_RANGE);
@@ -338,7 +348,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       for (int row = cw; row < group; row += CONSUMERS) {
         const int h = p_g * group + row;
         merge_segments<true>(partial + ((int64_t)p_item * nq + h) * max_segments * record_floats(d), out + ((int64_t)p_t * nq + h) * d,
-                       p_first, p_last, d, fused.sink == nullptr ? -INFINITY : fused.sink[h] * LOG2E);
+                       p_first, p_last, d, fused.sink == nullptr ? -INFINITY : fused.sink[h] * LOG2E,
+                       SLOPED && fused.head_gate != nullptr ? 1.f / (1.f + expf(-fused.head_gate[(int64_t)p_t * nq + h])) : 1.f);
       }
     }
   };
@@ -354,6 +365,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     if (meta.t < 0) break;
     wait_or_abandon(smem_addr(&meta_bar[qb]), (q_seen / Q_BUFFERS) & 1, status, &abandoned);
     const int pos = meta.pos, kstart = meta.kstart, seg = meta.seg, g = meta.g;
+    const KeyCount kc = counted(pos);
     int first_tile, tiles;
     my_tiles(meta, first_tile, tiles);
     // tiles of this item requested so far: those the previous item's tail asked for, then up to a full ring
@@ -407,7 +419,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       wait_or_abandon(smem_addr(&full_bar[cw][slot]), (seen / RING) & 1, status, &abandoned);
       const uint32_t ks = smem_addr(ring_base + (cw * RING + slot) * slot_bytes);
       const uint32_t vs = ks + nb * BLOCK_BYTES;
-      const int key0 = first_tile + tile * TILE;
+      const int key0 = SLOPED ? kc.key(first_tile + tile * TILE) : first_tile + tile * TILE;
       bool edge = false;
       if (FUSED && meta.fresh && pos >= key0 && pos < key0 + TILE) {
         // the token's own key and value, made by the producer: over the row the box brought
@@ -430,12 +442,17 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         uint8_t* vrows = ring_base + (cw * RING + slot) * slot_bytes + nb * BLOCK_BYTES;
         for (int i = lane; i < nb * TILE * 8; i += 32) {
           const int r = (i >> 3) % TILE;
-          if (key0 + r < kstart || key0 + r > pos) reinterpret_cast<uint4*>(vrows)[i] = make_uint4(0, 0, 0, 0);
+          if ((key0 + r < kstart && (!SLOPED || key0 + r >= keep)) || key0 + r > pos) reinterpret_cast<uint4*>(vrows)[i] = make_uint4(0, 0, 0, 0);
         }
         __syncwarp();
       }
 
-      attend_tile<DMAX, Q_IN_REGISTERS, CAPPED>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
+      if (SLOPED)
+        attend_tile<DMAX, Q_IN_REGISTERS, false, true>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
+                                        v_lane, v_xor, m_row, l_row, o, fused.score_bias + g * group + min(lane >> 2, group - 1),
+                                        fused.score_bias + g * group + min((lane >> 2) + 8, group - 1), keep);
+      else
+        attend_tile<DMAX, Q_IN_REGISTERS, CAPPED>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
                                         v_lane, v_xor, m_row, l_row, o,
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min(lane >> 2, group - 1)) * (fused.score_bias_last + 1),
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min((lane >> 2) + 8, group - 1)) * (fused.score_bias_last + 1),
@@ -514,7 +531,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     if (pending) merge_if_last();
     pending = true;
     p_item = meta.item; p_g = g; p_t = meta.t;
-    p_first = kstart / segment_keys; p_last = pos / segment_keys;
+    p_first = first_counted(kstart, kc) / segment_keys; p_last = (pos - kc.gap) / segment_keys;
   }
   if (!waited) pdl_wait();                           // (a CTA without items: the chain of completed kernels stays unbroken)
   if (pending) {
@@ -701,13 +718,14 @@ int launch_decode(const void* q, const void* k_cache, const void* v_cache, void*
                   int64_t scratch_elems, int* arrivals, const int* token_list, int count, int tokens_total,
                   const int* positions, const int* request_of, const int* block_table, int max_pages,
                   int page_size, int num_pages, int nq, int nkv, int d, int max_kv_len, float scale,
-                  int window, unsigned* status, cudaStream_t stream, const FusedProjection& fused) {
+                  int window, unsigned* status, cudaStream_t stream, const FusedProjection& fused, bool sloped = false) {
   VOSTI_REQUIRE(count >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "attention_decode: bad head counts nq=%d nkv=%d", nq, nkv);
   VOSTI_REQUIRE(nq / nkv <= 16, "attention_decode: at most 16 query heads per kv head, got %d", nq / nkv);
   VOSTI_REQUIRE(d > 0 && d % 16 == 0 && d <= 256, "attention_decode: head_dim %d must be a multiple of 16 and <= 256", d);
   VOSTI_REQUIRE(page_size > 0 && max_pages > 0 && num_pages > 0, "attention_decode: bad cache geometry");
   VOSTI_REQUIRE(max_kv_len > 0, "attention_decode: max_kv_len %d must be positive", max_kv_len);
   if (count == 0) return VOSTI_OK;
+  if (sloped) max_kv_len = longest_count(max_kv_len, window, fused.score_bias_last);
   const int group = nq / nkv;
   const int64_t cache_rows = (int64_t)num_pages * nkv * page_size;
   VOSTI_REQUIRE(cache_rows < (int64_t)1 << 31, "attention_decode: cache of %lld rows is too large", (long long)cache_rows);
@@ -750,6 +768,7 @@ int launch_decode(const void* q, const void* k_cache, const void* v_cache, void*
       launch.segment_keys = once_keys;
       launch.scale_log2 = scale * LOG2E;
       launch.window = window;
+      launch.sloped = sloped ? 1 : 0;
       launch.status = status;
       launch.fused = fused;
       launch.stream = stream;
@@ -773,24 +792,25 @@ int launch_decode(const void* q, const void* k_cache, const void* v_cache, void*
   VOSTI_REQUIRE(items < ((int64_t)1 << 30), "attention_decode: %lld work items are too many for one launch", (long long)items);
   const int64_t ctas = (int64_t)sm_count() * ctas_per_sm(d, group);
   dim3 grid((unsigned)(items < ctas ? items : ctas));
-#define LAUNCH_DECODE_AS(DMAX, EXACT, FUSED, CAPPED)                                                                \
+#define LAUNCH_DECODE_AS(DMAX, EXACT, FUSED, CAPPED, SLOPED)                                                        \
   do {                                                                                                              \
     static bool configured = false;                                                                                 \
     if (!configured) {                                                                                              \
-      cudaFuncSetAttribute(attention_decode_kernel<DMAX, EXACT, FUSED, CAPPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+      cudaFuncSetAttribute(attention_decode_kernel<DMAX, EXACT, FUSED, CAPPED, SLOPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                            (int)decode_smem_bytes(DMAX, 16));                                                       \
       configured = true;                                                                                            \
     }                                                                                                               \
-    vosti_launch(attention_decode_kernel<DMAX, EXACT, FUSED, CAPPED>, grid, dim3(THREADS), smem, stream, map_k, map_v, \
+    vosti_launch(attention_decode_kernel<DMAX, EXACT, FUSED, CAPPED, SLOPED>, grid, dim3(THREADS), smem, stream, map_k, map_v, \
         (const bf16*)q, scratch, (bf16*)out, arrivals, token_list, positions, request_of,                          \
         block_table, max_pages, page_size, page_shift, num_pages, whole_pages, whole_rows, count, nq, nkv, d, segment_keys,     \
         segments, scale * LOG2E, window, status, fused);                                                            \
   } while (0)
 #define LAUNCH_DECODE(DMAX, EXACT)                                                                                  \
   do {                                                                                                              \
-    if (fused.partial != nullptr) LAUNCH_DECODE_AS(DMAX, EXACT, true, false);                                       \
-    else if (fused.softcap > 0.f) LAUNCH_DECODE_AS(DMAX, EXACT, false, true);                                       \
-    else LAUNCH_DECODE_AS(DMAX, EXACT, false, false);                                                               \
+    if (fused.partial != nullptr) LAUNCH_DECODE_AS(DMAX, EXACT, true, false, false);                                \
+    else if (sloped) LAUNCH_DECODE_AS(DMAX, EXACT, false, false, true);                                             \
+    else if (fused.softcap > 0.f) LAUNCH_DECODE_AS(DMAX, EXACT, false, true, false);                                \
+    else LAUNCH_DECODE_AS(DMAX, EXACT, false, false, false);                                                        \
   } while (0)
   if (d == 64) LAUNCH_DECODE(64, true);
   else if (d == 128) LAUNCH_DECODE(128, true);
@@ -834,6 +854,30 @@ VOSTI_API int vosti_attention_decode_biased(const void* q, const void* k_cache, 
   return launch_decode(q, k_cache, v_cache, out, scratch, scratch_elems, arrivals, token_list, count, tokens_total, positions,
                        request_of, block_table, max_pages, page_size, num_pages, nq, nkv, d, max_kv_len, scale, window,
                        status, stream, extras);
+}
+
+// The sloped form: `slopes` (float32 [nq], base-2 units) times the distance is taken off the scaled scores, keys before
+// `keep` are visible whatever the window, a sink as above, and every head's row is multiplied by the sigmoid
+// of head_gate (float32 [tokens_total, nq], or null). The segments then cut the keys that may be
+// visible, so the scratch is that of a context of vosti_attention_decode_sloped_keys keys.
+VOSTI_API int vosti_attention_decode_sloped_keys(int max_kv_len, int window, int keep) { return longest_count(max_kv_len, window, keep); }
+
+VOSTI_API int vosti_attention_decode_sloped(const void* q, const void* k_cache, const void* v_cache, void* out, float* scratch,
+                                            int64_t scratch_elems, int* arrivals, const int* token_list, int count,
+                                            int tokens_total, const int* positions, const int* request_of,
+                                            const int* block_table, int max_pages, int page_size, int num_pages, int nq,
+                                            int nkv, int d, int max_kv_len, float scale, int window, const float* slopes,
+                                            int keep, const float* sink, const float* head_gate, unsigned* status, cudaStream_t stream) {
+  VOSTI_REQUIRE(slopes != nullptr, "attention_decode: the slopes are missing");
+  VOSTI_REQUIRE(window >= 0 && keep >= 0 && (keep == 0 || window > 0), "attention_decode: kept first keys go with a window");
+  FusedProjection extras = {};
+  extras.score_bias = slopes;
+  extras.score_bias_last = keep;
+  extras.sink = sink;
+  extras.head_gate = head_gate;
+  return launch_decode(q, k_cache, v_cache, out, scratch, scratch_elems, arrivals, token_list, count, tokens_total, positions,
+                       request_of, block_table, max_pages, page_size, num_pages, nq, nkv, d, max_kv_len, scale, window,
+                       status, stream, extras, true);
 }
 
 // The fused form: `partial` holds the QKV projection's K-split partial sums of the step's tokens

@@ -52,10 +52,10 @@ __host__ __device__ inline int record_floats(int d) { return d + 4; }
 // GLOBAL: the records were written by other CTAs to global memory (read past L1); else they lie in
 // this CTA's shared memory.
 // `sink_l2` (base-2 units; -inf: none) is a logit without key or value that joins the denominator
-// once: it may raise the reference maximum and adds exp2(sink - max) to the sum.
+// once: it may raise the reference maximum and adds exp2(sink - max) to the sum. The row is multiplied by `factor`.
 template <bool GLOBAL>
 __device__ __forceinline__ void merge_segments(const float* __restrict__ base, bf16* __restrict__ dst, int first,
-                                               int last, int d, float sink_l2 = -INFINITY) {
+                                               int last, int d, float sink_l2 = -INFINITY, float factor = 1.f) {
   auto load2 = [](const float* p) { return GLOBAL ? __ldcg(reinterpret_cast<const float2*>(p)) : *reinterpret_cast<const float2*>(p); };
   auto load4 = [](const float* p) { return GLOBAL ? __ldcg(reinterpret_cast<const float4*>(p)) : *reinterpret_cast<const float4*>(p); };
   const int lane = threadIdx.x & 31;
@@ -118,7 +118,7 @@ __device__ __forceinline__ void merge_segments(const float* __restrict__ base, b
       }
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? factor / l : 0.f;
   if (owner)
     *reinterpret_cast<uint2*>(dst + 4 * lane) = make_uint2(pack_bf16(acc[0].x * inv, acc[0].y * inv), pack_bf16(acc[0].z * inv, acc[0].w * inv));
   if (second)
@@ -128,7 +128,7 @@ __device__ __forceinline__ void merge_segments(const float* __restrict__ base, b
 // One tile of 16 keys for one warp: S = Q K^T on the tensor cores, the online softmax of the
 // warp's 16 rows (base 2, float32; masked keys count as -inf), O = O * alpha + P V with P rounded
 // to bfloat16. ks / vs: shared-memory addresses of the tile's K and V blocks (128-byte swizzle).
-template <int DMAX, bool Q_IN_REGISTERS, bool CAPPED = false>
+template <int DMAX, bool Q_IN_REGISTERS, bool CAPPED = false, bool SLOPED = false>
 __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint32_t (&qa)[Q_IN_REGISTERS ? DMAX / 16 : 1][4],
                                             const uint8_t* q_s, int q_pitch, int d, int key0, int kstart, int pos,
                                             float scale_log2, bool upper_rows_live, uint32_t k_lane, uint32_t k_xor,
@@ -137,7 +137,9 @@ __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint
                                             const float* __restrict__ bias1 = nullptr, int bias_last = 0,
                                             float softcap = 0.f) {
   // softcap (base-2 units, CAPPED only) caps the scaled score; bias0 / bias1 (or null): the rows of a distance-bias table (base-2 units) of this lane's two
-  // query heads, indexed by min(pos - key, bias_last) and added to the scaled score
+  // query heads, indexed by min(pos - key, bias_last) and added to the scaled score. SLOPED: bias0 / bias1 point at
+  // the two heads' slopes (base-2 units), slope * (pos - key) is taken off the scaled score, and keys before
+  // `bias_last` are visible although they lie before kstart
   const int lane = threadIdx.x & 31;
   // ---- S = Q K^T for 16 keys: two 8-key column tiles
   float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
@@ -159,13 +161,16 @@ __device__ __forceinline__ void attend_tile(uint32_t ks, uint32_t vs, const uint
   }
   // ---- online softmax (rows lane/4 and lane/4 + 8)
   float tile_max[2] = {-INFINITY, -INFINITY};
+  const float slope[2] = {SLOPED ? *bias0 : 0.f, SLOPED ? *bias1 : 0.f};
 #pragma unroll
   for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int key = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
-      const bool visible = key >= kstart && key <= pos;
-      if (CAPPED) {
+      const bool visible = (key >= kstart || (SLOPED && key < bias_last)) && key <= pos;
+      if (SLOPED) {
+        s[nt][e] = visible ? fmaf(s[nt][e], scale_log2, -slope[e >> 1] * (float)(pos - key)) : -INFINITY;
+      } else if (CAPPED) {
         s[nt][e] = soft_capped(s[nt][e] * scale_log2, softcap, 2.f * LOG2E / softcap);
         if (bias0 != nullptr) s[nt][e] += ((e >> 1) ? bias1 : bias0)[min(max(pos - key, 0), bias_last)];
         if (!visible) s[nt][e] = -INFINITY;
@@ -221,7 +226,10 @@ struct FusedProjection {
   const float* partial;        // [splits][tokens][(nq + 2 nkv) d] float32
   int splits;
   long long plane;             // tokens * (nq + 2 nkv) * d
-  const void* q_norm_w;        // [d] or null: no head norm
+  union {                      // forms that exclude one another share their place (see softcap below)
+    const void* q_norm_w;      // fused: [d] or null: no head norm
+    const float* head_gate;    // sloped: float32 [tokens, nq], the head's row is multiplied by its sigmoid; or null
+  };
   const void* k_norm_w;
   int norm_w_is_f32;
   float eps;
@@ -233,12 +241,30 @@ struct FusedProjection {
   bf16* k_cache;
   bf16* v_cache;
   // additions to the scores, for mixers that have them (all null / 0 otherwise; they do not need `partial`)
-  const float* score_bias;     // [nq][score_bias_last + 1] float32, base-2 units, by min(distance, last)
-  int score_bias_last;
+  const float* score_bias;     // [nq][score_bias_last + 1] float32, base-2 units, by min(distance, last);
+                               // sloped: [nq] slopes, base-2 units, slope * distance is taken off the score
+  int score_bias_last;         // sloped: keys before this one are visible whatever the window
   float softcap;               // base-2 units: the scaled scores' soft cap (here it fills the padding: a launch with more
                                // bytes of parameters was measured 1 us slower)
   const float* sink;           // [nq] float32, natural units: a logit in the denominator without key or value
 };
+
+// The sloped form counts an item's keys without the gap between the kept first keys and the window: key v of
+// the count is key v of the request while v < head, and key v + gap from there on. Both are multiples of a
+// tile, so that tiles stay aligned to the key index. Without a window nothing is skipped.
+struct KeyCount {
+  int head, gap;
+  __host__ __device__ __forceinline__ int key(int v) const { return v < head ? v : v + gap; }
+};
+__host__ __device__ __forceinline__ KeyCount key_count(int pos, int window, int keep) {
+  const int head = (keep + TILE - 1) / TILE * TILE, from = first_visible_key(pos, window) / TILE * TILE;
+  return KeyCount{head, window > 0 && from > head ? from - head : 0};
+}
+// Longest such count of a context of max_kv_len keys.
+inline int longest_count(int max_kv_len, int window, int keep) {
+  const long long most = (long long)(keep + TILE - 1) / TILE * TILE + window + TILE - 1;
+  return window > 0 && most < max_kv_len ? (int)most : max_kv_len;
+}
 
 constexpr int ONCE_MAX_SEGMENTS = 16;     // CTAs per cluster of that kernel (above 8 it opts in to non-portable sizes)
 
@@ -255,6 +281,7 @@ struct OnceLaunch {
   int segments, segment_keys;          // CTAs per cluster and keys per segment
   float scale_log2;
   int window;
+  int sloped;                          // the sloped form (FusedProjection)
   unsigned* status;
   FusedProjection fused;               // partial == null: not fused
   cudaStream_t stream;

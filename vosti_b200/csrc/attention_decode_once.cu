@@ -85,7 +85,7 @@ __device__ __forceinline__ int load_now(const int* p) {
 }
 
 
-template <int DMAX, bool EXACT, bool FUSED, bool CAPPED>
+template <int DMAX, bool EXACT, bool FUSED, bool CAPPED, bool SLOPED>
 __global__ void __launch_bounds__(THREADS, DMAX <= 128 ? 2 : 1)
 attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                              const bf16* __restrict__ q, bf16* __restrict__ out, const int* __restrict__ token_list,
@@ -157,10 +157,13 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
   cluster_arrive_all();
   pdl_launch_dependents();
 
-  const int kstart = first_visible_key(pos, window);
-  const int seg_begin = seg * segment_keys, seg_end = min(seg_begin + segment_keys, pos + 1);
-  const bool visible = !(seg_begin > pos || seg_end <= kstart);
-  const int p_first = kstart / segment_keys, p_last = min(pos / segment_keys, segments - 1);   // the segments that hold visible keys
+  const int kstart = first_visible_key(pos, window), keep = SLOPED ? fused.score_bias_last : 0;
+  // segments cut the request's keys, or in the sloped form the count of those that may be visible
+  const KeyCount counted = SLOPED ? key_count(pos, window, keep) : KeyCount{0, 0};
+  const int vstart = SLOPED && (keep > 0 || counted.gap > 0) ? 0 : kstart, vpos = pos - counted.gap;
+  const int seg_begin = seg * segment_keys, seg_end = min(seg_begin + segment_keys, vpos + 1);
+  const bool visible = !(seg_begin > vpos || seg_end <= vstart);
+  const int p_first = vstart / segment_keys, p_last = min(vpos / segment_keys, segments - 1);   // the segments that hold visible keys
   const uint32_t leader_bar = map_to_rank(smem_addr(&records_bar), 0);
 
   if (!visible && seg != 0) {
@@ -227,7 +230,7 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
   if (visible) {
     // this warp's tiles: a quarter of the segment, aligned to the key index
     const int my_end = min(my_begin + quarter, seg_end);
-    const int first_tile = max(my_begin, (kstart / TILE) * TILE);
+    const int first_tile = max(my_begin, (vstart / TILE) * TILE);
     const int tiles = my_end > first_tile ? (my_end - first_tile + TILE - 1) / TILE : 0;      // <= 64
     // cache row of each tile's first key: lane i holds tiles i and i + 32
     int rows[2] = {-1, -1};
@@ -235,7 +238,7 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
     for (int k = 0; k < 2; ++k) {
       const int i = lane + 32 * k;
       if (i < tiles) {
-        const int key0 = first_tile + i * TILE;
+        const int key0 = SLOPED ? counted.key(first_tile + i * TILE) : first_tile + i * TILE;
         const int index = page_shift >= 0 ? key0 >> page_shift : key0 / page_size;
         int page = guessed_page[k];                    // (first_tile == my_begin when the guess was made)
         if (!guessed || req != t) page = index < max_pages ? block_table[(int64_t)req * max_pages + index] : -1;
@@ -297,7 +300,7 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
       wait_or_abandon(smem_addr(&full_bar[cw][ring_slot]), (uint32_t)(tile / RING) & 1, status, &abandoned);
       uint8_t* tile_s = ring_base + (cw * RING + ring_slot) * slot_bytes;
       const uint32_t ks = smem_addr(tile_s), vs = ks + nb * BLOCK_BYTES;
-      const int key0 = first_tile + tile * TILE;
+      const int key0 = SLOPED ? counted.key(first_tile + tile * TILE) : first_tile + tile * TILE;
       bool edge = false;
       if (FUSED && slot >= 0 && pos >= key0 && pos < key0 + TILE) {
         // the token's own key and value, made by the helper warp: over the row the box brought
@@ -319,11 +322,16 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
         uint8_t* vrows = tile_s + nb * BLOCK_BYTES;
         for (int i = lane; i < nb * TILE * 8; i += 32) {
           const int r = (i >> 3) % TILE;
-          if (key0 + r < kstart || key0 + r > pos) reinterpret_cast<uint4*>(vrows)[i] = make_uint4(0, 0, 0, 0);
+          if ((key0 + r < kstart && (!SLOPED || key0 + r >= keep)) || key0 + r > pos) reinterpret_cast<uint4*>(vrows)[i] = make_uint4(0, 0, 0, 0);
         }
         __syncwarp();
       }
-      attend_tile<DMAX, Q_IN_REGISTERS, CAPPED>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
+      if (SLOPED)
+        attend_tile<DMAX, Q_IN_REGISTERS, false, true>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
+                                        v_lane, v_xor, m_row, l_row, o, fused.score_bias + g * group + min(lane >> 2, group - 1),
+                                        fused.score_bias + g * group + min((lane >> 2) + 8, group - 1), keep);
+      else
+        attend_tile<DMAX, Q_IN_REGISTERS, CAPPED>(ks, vs, qa, q_s, q_pitch, d, key0, kstart, pos, scale_log2, upper_rows_live, k_lane, k_xor,
                                         v_lane, v_xor, m_row, l_row, o,
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min(lane >> 2, group - 1)) * (fused.score_bias_last + 1),
                                         fused.score_bias == nullptr ? nullptr : fused.score_bias + (int64_t)(g * group + min((lane >> 2) + 8, group - 1)) * (fused.score_bias_last + 1),
@@ -397,7 +405,8 @@ attention_decode_once_kernel(const __grid_constant__ CUtensorMap map_k, const __
   if (!mb_wait_cluster(smem_addr(&records_bar), 0, status)) return;
   for (int row = cw; row < group; row += CONSUMERS)
     merge_segments<false>(records + (int64_t)row * segments * grec, out + ((int64_t)t * nq + g * group + row) * d, p_first, p_last, d,
-                          fused.sink == nullptr ? -INFINITY : fused.sink[g * group + row] * LOG2E);
+                          fused.sink == nullptr ? -INFINITY : fused.sink[g * group + row] * LOG2E,
+                          SLOPED && fused.head_gate != nullptr ? 1.f / (1.f + expf(-fused.head_gate[(int64_t)t * nq + g * group + row])) : 1.f);
 }
 
 // How many clusters of `cluster` CTAs with `smem` bytes each the GPU can run at once (0: none, or
@@ -429,9 +438,9 @@ int clusters_that_fit(Kernel kernel, int cluster, size_t smem) {
   return clusters;
 }
 
-template <int DMAX, bool EXACT, bool FUSED, bool CAPPED>
+template <int DMAX, bool EXACT, bool FUSED, bool CAPPED, bool SLOPED = false>
 int launch_as(const OnceLaunch& a, size_t smem) {
-  auto kernel = attention_decode_once_kernel<DMAX, EXACT, FUSED, CAPPED>;
+  auto kernel = attention_decode_once_kernel<DMAX, EXACT, FUSED, CAPPED, SLOPED>;
   static bool configured = false;
   if (!configured) {
     cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ONCE_SMEM_CAP);
@@ -463,6 +472,7 @@ int launch_as(const OnceLaunch& a, size_t smem) {
 template <int DMAX, bool EXACT>
 int launch_form(const OnceLaunch& a, size_t smem) {
   if (a.fused.partial != nullptr) return launch_as<DMAX, EXACT, true, false>(a, smem);
+  if (a.sloped) return launch_as<DMAX, EXACT, false, false, true>(a, smem);
   return a.fused.softcap > 0.f ? launch_as<DMAX, EXACT, false, true>(a, smem) : launch_as<DMAX, EXACT, false, false>(a, smem);
 }
 

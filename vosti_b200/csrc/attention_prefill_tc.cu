@@ -58,8 +58,11 @@ __device__ __forceinline__ uint32_t swizzled(int row, int chunk) { return row * 
 // table's last column serves every larger distance, so a tile that lies wholly beyond it adds a
 // constant), and exp(sink[head]) joins the denominator once at the end (either may be null). CAPPED
 // (with BIASED): the scaled score passes a soft cap (`softcap`, base-2 units) before the bias.
+// SLOPED (with BIASED): `bias` holds one slope a head (base-2 units), slope * distance is taken off the scaled
+// score; keys before `bias_last` are visible whatever the window (tiles of them come first, in ascending key
+// order like all tiles); and every head's row is multiplied by the sigmoid of head_gate[token, head] (or null).
 // Without BIASED the arithmetic is what it was before the flag existed, bit for bit.
-template <int D, bool BIASED, bool CAPPED>
+template <int D, bool BIASED, bool CAPPED, bool SLOPED>
 __global__ void __launch_bounds__(THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
@@ -67,7 +70,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ kv_len, const int* __restrict__ block_table, int max_pages,
                             int page_size, int page_shift, int num_pages, int nq, int nkv, float scale_log2_in,
                             int window, const float* __restrict__ bias, int bias_last,
-                            const float* __restrict__ sink, float softcap, unsigned* status) {
+                            const float* __restrict__ sink, float softcap, const float* __restrict__ head_gate, unsigned* status) {
   const float scale_log2 = BIASED ? 1.f : scale_log2_in;      // BIASED: scores are scaled where the bias is added
   constexpr int NB = D / 64;                          // 64-element blocks of the head size
   constexpr int STAGES = kv_stages<D>();
@@ -103,12 +106,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   // its own end
   const int first_key = first_visible_key(shift + token0, window);
   const int tile_begin = (first_key / KT) * KT;
+  const int keep = SLOPED ? bias_last : 0;
+  const int head_tiles = SLOPED ? min((keep + KT - 1) / KT, tile_begin / KT) : 0;        // tiles of kept keys before the window
+  auto tile_key = [&](int t) { return SLOPED && t < head_tiles ? t * KT : tile_begin + (t - head_tiles) * KT; };
   int tiles_of[ROW_TILES], key_end = 0;
 #pragma unroll
   for (int w = 0; w < ROW_TILES; ++w) {
     const int t0 = token0 + w * tokens_per_tile;
     const int end = t0 < q_len ? shift + min(q_len - 1, t0 + tokens_per_tile - 1) + 1 : 0;    // exclusive
-    tiles_of[w] = end > tile_begin ? (end - tile_begin + KT - 1) / KT : 0;
+    tiles_of[w] = end > tile_begin ? head_tiles + (end - tile_begin + KT - 1) / KT : 0;
     key_end = max(key_end, end);
   }
   const int tiles = max(tiles_of[0], tiles_of[1]);
@@ -157,10 +163,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     bool ok = true;
     const uint32_t o_tmem = lane_base + PV_COL + wg * D;
     const int head = g * group + r % group;
-    const float* bias_h = (BIASED && bias != nullptr) ? bias + (int64_t)head * (bias_last + 1) : nullptr;
+    const float* bias_h = (BIASED && !SLOPED && bias != nullptr) ? bias + (int64_t)head * (bias_last + 1) : nullptr;
+    const float slope = SLOPED ? bias[min(head, nq - 1)] : 0.f;
 
     for (int t = 0; t < my_tiles && ok; ++t) {
-      const int key0 = tile_begin + t * KT;
+      const int key0 = tile_key(t);
       const int buf = t & 1;
       ok = mbar_wait(smem_u32(&s_full[wg]), t & 1, &abort_flag, status);
       if (!ok) break;
@@ -180,7 +187,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           raw[i >> 5][i & 31] = __float_as_uint(soft_capped(__uint_as_float(raw[i >> 5][i & 31]) * scale_log2_in, softcap, rate));
       }
       const float scale_here = CAPPED ? 1.f : scale_log2_in;
-      if (BIASED && valid && (!CAPPED || bias_h != nullptr)) {
+      if (SLOPED) {
+        const float behind = (float)(key0 - pos);                // key i of the tile is -(behind + i) positions back
+#pragma unroll
+        for (int i = 0; i < KT; ++i)
+          raw[i >> 5][i & 31] = __float_as_uint(fmaf(__uint_as_float(raw[i >> 5][i & 31]), scale_log2_in, slope * (behind + (float)i)));
+      } else if (BIASED && valid && (!CAPPED || bias_h != nullptr)) {
         const int d0 = pos - key0;                               // key i of the tile is d0 - i positions back
         if (bias_h == nullptr || d0 - (KT - 1) >= bias_last) {
           const float far = bias_h != nullptr ? bias_h[bias_last] : 0.f;
@@ -195,7 +207,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           }
         }
       }
-      const bool masked = key0 + KT - 1 > pos || key0 < kstart;
+      const bool masked = key0 + KT - 1 > pos || (key0 < kstart && (!SLOPED || key0 + KT > keep));
       // the maximum is exact in any order: four independent chains, scaled once at the end
       // (scale_log2 > 0, so max(s * scale) = max(s) * scale bit for bit)
       // A row of the tile that holds no token (a lone decode token fills 1 to 16 of the 128 rows)
@@ -206,7 +218,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       } else if (masked) {
 #pragma unroll
         for (int i = 0; i < KT; ++i)
-          if (key0 + i <= pos && key0 + i >= kstart) part_max[i & 3] = fmaxf(part_max[i & 3], __uint_as_float(raw[i >> 5][i & 31]));
+          if (key0 + i <= pos && (key0 + i >= kstart || (SLOPED && key0 + i < keep))) part_max[i & 3] = fmaxf(part_max[i & 3], __uint_as_float(raw[i >> 5][i & 31]));
       } else {
 #pragma unroll
         for (int i = 0; i < KT; ++i) part_max[i & 3] = fmaxf(part_max[i & 3], __uint_as_float(raw[i >> 5][i & 31]));
@@ -252,7 +264,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           for (int e = 0; e < 8; ++e) {
             const int i = 8 * c + e;
             p[e] = fast_exp2(__uint_as_float(raw[i >> 5][i & 31]) * scale_log2 - safe);
-            if (!(key0 + i <= pos && key0 + i >= kstart)) p[e] = 0.f;
+            if (!(key0 + i <= pos && (key0 + i >= kstart || (SLOPED && key0 + i < keep)))) p[e] = 0.f;
             part_sum[e & 3] += p[e];
           }
           *reinterpret_cast<uint4*>(p_dst + swizzled(r, c)) =
@@ -283,7 +295,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     tc_fence_after();
     if (my_tiles > 0) {
       if (BIASED && sink != nullptr && valid && m_run > -INFINITY) l_run += fast_exp2(sink[head] * LOG2E - m_run);
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (SLOPED && valid && head_gate != nullptr) inv *= 1.f / (1.f + expf(-head_gate[(int64_t)(q_start + token) * nq + head]));
       bf16* dst = out + ((int64_t)(q_start + token) * nq + g * group + r % group) * D;
 #pragma unroll 1
       for (int c0 = 0; c0 < D; c0 += 32) {
@@ -322,10 +335,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       const int stage = j % STAGES;
       if (j >= STAGES) ok = mbar_wait(smem_u32(&kv_empty[stage]), ((j / STAGES) - 1) & 1, &abort_flag, status);
       if (!ok) break;
-      const int lo = tile_begin + j * KT + w * GROUP_KEYS;
+      const int lo = tile_key(j) + w * GROUP_KEYS;
       uint8_t* dst = kv_s + stage * STAGE_BYTES + w * GROUP_KEYS * 128;     // + block * (KT * 128); V: + K_BYTES
       int row = -1;
-      if (lo + GROUP_KEYS - 1 >= first_key && lo < key_end) {
+      if ((lo + GROUP_KEYS - 1 >= first_key || (SLOPED && lo < keep)) && lo < key_end) {
         const int index = page_shift >= 0 ? lo >> page_shift : lo / page_size;
         const int page = index < max_pages ? table[index] : -1;
         if (page < 0 || page >= num_pages) raise_fault(status, VOSTI_FAULT_PAGE_RANGE);
@@ -452,7 +465,7 @@ int launch_prefill_tc(const void* q, const void* k_cache, const void* v_cache, v
                                          const int* block_table, int max_pages, int page_size, int num_pages, int nq,
                                          int nkv, int d, int max_q_len, int tokens_total, float scale, int window,
                                          bool biased, const float* bias, int bias_last, const float* sink, float softcap,
-                                         unsigned* status, cudaStream_t stream) {
+                                         unsigned* status, cudaStream_t stream, bool sloped = false, const float* head_gate = nullptr) {
   VOSTI_REQUIRE(count >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "attention_prefill_tc: bad head counts nq=%d nkv=%d", nq, nkv);
   VOSTI_REQUIRE(nq / nkv <= 16, "attention_prefill_tc: at most 16 query heads per kv head, got %d", nq / nkv);
   VOSTI_REQUIRE(vosti_attention_prefill_tc_supported(d, page_size),
@@ -479,27 +492,30 @@ int launch_prefill_tc(const void* q, const void* k_cache, const void* v_cache, v
   int page_shift = -1;
   if ((page_size & (page_size - 1)) == 0)
     for (page_shift = 0; (1 << page_shift) < page_size; ++page_shift) {}
-#define LAUNCH_PREFILL_TC(D, B, C)                                                                                   \
+#define LAUNCH_PREFILL_TC(D, B, C, S)                                                                                \
   do {                                                                                                               \
     static bool configured = false;                                                                                  \
     if (!configured) {                                                                                               \
-      cudaFuncSetAttribute(attention_prefill_tc_kernel<D, B, C>, cudaFuncAttributeMaxDynamicSharedMemorySize,       \
+      cudaFuncSetAttribute(attention_prefill_tc_kernel<D, B, C, S>, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
                            (int)prefill_tc_smem_bytes<D>());                                                         \
       configured = true;                                                                                             \
     }                                                                                                                \
-    vosti_launch(attention_prefill_tc_kernel<D, B, C>, grid, dim3(THREADS), prefill_tc_smem_bytes<D>(), stream, map_q,  \
+    vosti_launch(attention_prefill_tc_kernel<D, B, C, S>, grid, dim3(THREADS), prefill_tc_smem_bytes<D>(), stream, map_q,  \
         map_k, map_v, (bf16*)out, row_list, cu_q, kv_len, block_table, max_pages, page_size, page_shift, num_pages,   \
-        nq, nkv, scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, status);                                               \
+        nq, nkv, scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, head_gate, status);                   \
   } while (0)
-  if (biased && softcap > 0.f) {
-    if (d == 64) LAUNCH_PREFILL_TC(64, true, true);
-    else LAUNCH_PREFILL_TC(128, true, true);
+  if (sloped) {
+    if (d == 64) LAUNCH_PREFILL_TC(64, true, false, true);
+    else LAUNCH_PREFILL_TC(128, true, false, true);
+  } else if (biased && softcap > 0.f) {
+    if (d == 64) LAUNCH_PREFILL_TC(64, true, true, false);
+    else LAUNCH_PREFILL_TC(128, true, true, false);
   } else if (biased) {
-    if (d == 64) LAUNCH_PREFILL_TC(64, true, false);
-    else LAUNCH_PREFILL_TC(128, true, false);
+    if (d == 64) LAUNCH_PREFILL_TC(64, true, false, false);
+    else LAUNCH_PREFILL_TC(128, true, false, false);
   } else {
-    if (d == 64) LAUNCH_PREFILL_TC(64, false, false);
-    else LAUNCH_PREFILL_TC(128, false, false);
+    if (d == 64) LAUNCH_PREFILL_TC(64, false, false, false);
+    else LAUNCH_PREFILL_TC(128, false, false, false);
   }
 #undef LAUNCH_PREFILL_TC
   VOSTI_LAUNCH_CHECK();
@@ -532,4 +548,20 @@ VOSTI_API int vosti_attention_prefill_tc_biased(const void* q, const void* k_cac
   return launch_prefill_tc(q, k_cache, v_cache, out, row_list, count, cu_q, kv_len, block_table, max_pages, page_size,
                            num_pages, nq, nkv, d, max_q_len, tokens_total, scale, window, true, bias, bias_last, sink, softcap,
                            status, stream);
+}
+
+// The sloped form: `slopes` (float32 [nq], base-2 units) times the distance is taken off the scaled scores, keys before
+// `keep` are visible whatever the window, a sink as above, and every head's row is multiplied by the sigmoid
+// of head_gate (float32 [tokens_total, nq], or null).
+VOSTI_API int vosti_attention_prefill_tc_sloped(const void* q, const void* k_cache, const void* v_cache, void* out,
+                                                const int* row_list, int count, const int* cu_q, const int* kv_len,
+                                                const int* block_table, int max_pages, int page_size, int num_pages,
+                                                int nq, int nkv, int d, int max_q_len, int tokens_total, float scale,
+                                                int window, const float* slopes, int keep, const float* sink,
+                                                const float* head_gate, unsigned* status, cudaStream_t stream) {
+  VOSTI_REQUIRE(slopes != nullptr, "attention_prefill_tc: the slopes are missing");
+  VOSTI_REQUIRE(window >= 0 && keep >= 0 && (keep == 0 || window > 0), "attention_prefill_tc: kept first keys go with a window");
+  return launch_prefill_tc(q, k_cache, v_cache, out, row_list, count, cu_q, kv_len, block_table, max_pages, page_size,
+                           num_pages, nq, nkv, d, max_q_len, tokens_total, scale, window, true, slopes, keep, sink, 0.f, status,
+                           stream, true, head_gate);
 }

@@ -10,9 +10,12 @@
 //     bias[head][min(distance, last)] (already in base-2 units): beyond `last` the bias no
 //     longer changes, so the table is as long as the distances that differ;
 //   * a soft cap c on the scaled score, c tanh(score / c), before the bias;
+//   * a penalty linear in the distance, slope[head] * (i - j), taken off the scaled score;
+//   * a window that keeps a sequence's first keys: a query also sees every key before `keep`;
 //   * a sink: one more term exp(sink[head]) in the softmax denominator, with no key or value;
 //   * two score maps a head over the same values (differential attention), combined after the
-//     softmax, and a finish of the head's output: unit root mean square, a sigmoid gate (HeadFinish);
+//     softmax, and a finish of the head's output: unit root mean square, a sigmoid gate for every
+//     element or one for the head (HeadFinish);
 //   * a projection post-pass by heads (qkv_heads): bias, per-head RMS norm with a shared weight,
 //     rotation in pairs (i, i + n / 2) or (2i, 2i + 1), from a float32 product or its unsummed K splits.
 //
@@ -209,7 +212,7 @@ __device__ __forceinline__ void store_four(bf16* p, float4 v) {
 //     maps' softmax-weighted sums of the same values;
 //   * `unit_norm`: o / sqrt(mean(o^2) + eps) over the head's values (no weight), times `out_scale`;
 //   * `gate`: o * sigmoid(gate[t, h * dv + i]), the gate a product of the same input (float32 or
-//     bfloat16 rows `gate_stride` elements apart).
+//     bfloat16 rows `gate_stride` elements apart); with `gate_by_head` one for the head, gate[t, h].
 struct HeadFinish {
   float lambda;
   float out_scale;
@@ -218,7 +221,11 @@ struct HeadFinish {
   const void* gate;
   int gate_f32;
   long long gate_stride;
+  int gate_by_head;
 };
+__device__ __forceinline__ float head_gate_of(const HeadFinish& f, int64_t t, int h) {
+  return 1.f / (1.f + expf(-load_flex(f.gate, f.gate_f32, t * f.gate_stride + h)));
+}
 
 // acc[m][i]: map m's unnormalised sum for value element lane + 32 i; inv[m] = 1 / its denominator. One warp.
 template <typename T, int MAPS>
@@ -235,12 +242,14 @@ __device__ __forceinline__ void finish_head(const float (&acc)[MAPS][MAX_W / 32]
   }
   float by = 1.f;
   if (f.unit_norm) by = f.out_scale / sqrtf(warp_sum(ss) / (float)dv + f.eps);
+  const float head_gate = f.gate_by_head ? head_gate_of(f, t, h) : 1.f;
 #pragma unroll
   for (int i = 0; i < MAX_W / 32; ++i) {
     const int idx = lane + 32 * i;
     if (idx < dv) {
       float y = f.unit_norm ? o[i] * by : o[i];
-      if (f.gate != nullptr) y *= 1.f / (1.f + expf(-load_flex(f.gate, f.gate_f32, (int64_t)t * f.gate_stride + (int64_t)h * dv + idx)));
+      if (f.gate_by_head) y *= head_gate;
+      else if (f.gate != nullptr) y *= 1.f / (1.f + expf(-load_flex(f.gate, f.gate_f32, (int64_t)t * f.gate_stride + (int64_t)h * dv + idx)));
       orow[idx] = from_f32<T>(y);
     }
   }
@@ -260,7 +269,7 @@ head_finish_kernel(const T* __restrict__ a, T* __restrict__ out, int tokens, int
   if (wid >= (int64_t)tokens * nq) return;
   const int t = (int)(wid / nq), h = (int)(wid % nq);
   if (dv % 4 == 0 && a_width % 4 == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
-      (f.gate == nullptr || (f.gate_f32 && f.gate_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(f.gate) & 15) == 0))) {
+      (f.gate == nullptr || f.gate_by_head || (f.gate_f32 && f.gate_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(f.gate) & 15) == 0))) {
     // a lane takes four neighbouring elements (of every 128): whole words in and out
     constexpr int C = MAX_W / 128;
     float4 o[C];
@@ -282,12 +291,15 @@ head_finish_kernel(const T* __restrict__ a, T* __restrict__ out, int tokens, int
     }
     float by = 1.f;
     if (f.unit_norm) by = f.out_scale / sqrtf(warp_sum(ss) / (float)dv + f.eps);
+    const float head_gate = f.gate_by_head ? head_gate_of(f, t, h) : 1.f;
 #pragma unroll
     for (int c = 0; c < C; ++c) {
       const int i0 = 4 * lane + 128 * c;
       if (i0 < dv) {
         float4 y = f.unit_norm ? make_float4(o[c].x * by, o[c].y * by, o[c].z * by, o[c].w * by) : o[c];
-        if (f.gate != nullptr) {
+        if (f.gate_by_head) {
+          y.x *= head_gate; y.y *= head_gate; y.z *= head_gate; y.w *= head_gate;
+        } else if (f.gate != nullptr) {
           const float4 g = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(f.gate) + (int64_t)t * f.gate_stride + (int64_t)h * dv + i0);
           y.x *= 1.f / (1.f + expf(-g.x)); y.y *= 1.f / (1.f + expf(-g.y)); y.z *= 1.f / (1.f + expf(-g.z)); y.w *= 1.f / (1.f + expf(-g.w));
         }
@@ -587,8 +599,8 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
                       const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
                       const int* __restrict__ token_list, int tokens,
                       int nq, int nkv, int dk, int dv, float scale_log2, int window, const float* __restrict__ bias,
-                      int bias_last, const float* __restrict__ sink, float softcap, float* __restrict__ partial, int segment,
-                      unsigned* status, HeadFinish finish) {
+                      int bias_last, const float* __restrict__ sink, float softcap, const float* __restrict__ slopes, int keep,
+                      float* __restrict__ partial, int segment, unsigned* status, HeadFinish finish) {
   // MAPS score maps a head: the query row holds MAPS queries, a key entry MAPS keys side by side,
   // every map has a softmax of its own over the same values (a value row is loaded once for all).
   extern __shared__ float q_smem[];
@@ -608,11 +620,22 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
   const int pos = positions[t];
   int kstart = first_visible_key(pos, window);
   int kend = pos;                                   // inclusive
+  // the kept keys that lie before the window: [kept_from, kept_to)
+  int kept_from = 0, kept_to = min(keep, kstart);
   if (partial != nullptr) {                         // this warp's segment of the keys (segment: a multiple of 32)
-    const int seg = (window > 0 ? kstart / segment : 0) + (int)blockIdx.y;
-    kstart = max(kstart, seg * segment);
-    kend = min(kend, (seg + 1) * segment - 1);
+    const int kept_segments = (keep + segment - 1) / segment, piece = (int)blockIdx.y - kept_segments;
+    if (piece < 0) {
+      kept_from = (int)blockIdx.y * segment;
+      kept_to = min(kept_to, kept_from + segment);
+      kend = -1;                                    // nothing of the window
+    } else {
+      kept_to = 0;
+      const int seg = (window > 0 ? kstart / segment : 0) + piece;
+      kstart = max(kstart, seg * segment);
+      kend = min(kend, (seg + 1) * segment - 1);
+    }
   }
+  const float slope = slopes != nullptr ? slopes[h] : 0.f;
   const int* table = block_table + (int64_t)b * max_pages;
   const float* bias_h = bias != nullptr ? bias + (int64_t)h * (bias_last + 1) : nullptr;
 
@@ -626,9 +649,14 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
     for (int i = 0; i < MAX_W / 32; ++i) acc[a][i] = 0.f;
   }
 
-  for (int j0 = (kstart / 32) * 32; j0 <= kend; j0 += 32) {
+  // tiles of the kept keys, then those of the window
+  const int kept_tiles = kept_to > kept_from ? (kept_to - kept_from + 31) / 32 : 0, first_tile = (kstart / 32) * 32;
+  for (int tile = 0; tile < kept_tiles || first_tile + (tile - kept_tiles) * 32 <= kend; ++tile) {
+    const bool kept = tile < kept_tiles;
+    const int j0 = kept ? kept_from + tile * 32 : first_tile + (tile - kept_tiles) * 32;
+    const int tile_last = kept ? kept_to - 1 : kend;
     const int j = j0 + lane;
-    bool valid = j >= kstart && j <= kend;
+    bool valid = (kept || j >= kstart) && j <= tile_last;
     int64_t slot = 0;
     float s[MAPS];
 #pragma unroll
@@ -646,6 +674,7 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
           s[a] = dot_key(qs + a * dk, k_cache + (slot * MAPS + a) * dk, dk) * scale_log2;
           if (softcap > 0.f) s[a] = softcap * tanhf(s[a] / softcap);       // softcap in base-2 units like the scores
           if (bias_h != nullptr) s[a] += bias_h[min(pos - j, bias_last)];
+          if (slopes != nullptr) s[a] -= slope * (float)(pos - j);
         }
       }
     }
@@ -666,7 +695,7 @@ attention_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
       m[a] = m_new;
     }
     if (!any) continue;
-    const int last = min(31, kend - j0);
+    const int last = min(31, tile_last - j0);
     // four keys at a time, so that their value rows are in flight together (keys past the
     // end have p = 0 and slot 0, a row that exists)
     for (int kk = 0; kk <= last; kk += 4) {
@@ -797,20 +826,20 @@ VOSTI_API int vosti_qkv_store(const void* qkv, void* q_out, void* k_cache, void*
   VOSTI_LAUNCH_CHECK();
 }
 
-static const HeadFinish NO_FINISH = {0.f, 1.f, 0.f, 0, nullptr, 0, 0};
+static const HeadFinish NO_FINISH = {0.f, 1.f, 0.f, 0, nullptr, 0, 0, 0};
 
 template <typename T, int MAPS>
 static cudaError_t attention_sink_launch(const void* q, const void* k_cache, const void* v_cache, void* out, const int* positions,
                                          const int* request_of, const int* block_table, int max_pages, int page_size, int num_pages,
                                          const int* token_list, int tokens, int nq, int nkv, int dk, int dv, float scale, int window,
-                                         const float* bias, int bias_last, const float* sink, float softcap, float* partial, int segment,
-                                         int segments, unsigned* status, const HeadFinish& finish, cudaStream_t stream) {
+                                         const float* bias, int bias_last, const float* sink, float softcap, const float* slopes, int keep,
+                                         float* partial, int segment, int segments, unsigned* status, const HeadFinish& finish, cudaStream_t stream) {
   const int64_t blocks = ((int64_t)tokens * nq + WARPS - 1) / WARPS;
   const size_t smem = (size_t)WARPS * MAPS * dk * sizeof(float);
   const dim3 grid((unsigned)blocks, segments > 1 ? segments : 1);
   vosti_launch(attention_sink_kernel<T, MAPS>, grid, dim3(WARPS * 32), smem, stream, (const T*)q, (const T*)k_cache, (const T*)v_cache,
                (T*)out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list, tokens, nq, nkv, dk, dv,
-               scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, partial, segment, status, finish);
+               scale * LOG2E, window, bias, bias_last, sink, softcap * LOG2E, slopes, keep, partial, segment, status, finish);
   if (segments > 1) {
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return e;
@@ -826,15 +855,18 @@ static cudaError_t attention_sink_launch(const void* q, const void* k_cache, con
 // null: all of them) names the `tokens` rows to compute. With `segments` > 1 the keys are cut
 // into pieces of `segment` keys (a multiple of 32) and `scratch` holds tokens * nq * segments * maps *
 // (dv + 2) floats; with a window a row's pieces are counted from the one that holds its first key, so
-// (window - 1) / segment + 2 of them reach every key. `softcap` (natural units) > 0 caps the scores. maps is 1 or 2 (see HeadFinish for what follows the softmax: lambda, the unit norm
+// (window - 1) / segment + 2 of them reach every key. `keep` > 0 (with a window): keys before `keep` are seen by every
+// query; their pieces, keep / segment rounded up, come before the window's. `slopes` (float32 [nq], natural-log units times
+// log2(e), or null): slope[head] * distance is taken off the scores. `softcap` (natural units) > 0 caps the scores. maps is 1 or 2 (see HeadFinish for what follows the softmax: lambda, the unit norm
 // with eps and out_scale, the gate).
 VOSTI_API int vosti_attention_maps(const void* q, const void* k_cache, const void* v_cache, void* out, const int* positions,
                                    const int* request_of, const int* block_table, int max_pages, int page_size,
                                    int num_pages, const int* token_list, int tokens, int nq, int nkv, int maps, int dk, int dv,
                                    float scale, int window, const float* bias, int bias_last, const float* sink, float softcap,
-                                   float* scratch, int segment, int segments, float lambda, int unit_norm, float eps,
-                                   float out_scale, const void* gate, int gate_f32, long long gate_stride, int is_f32,
-                                   unsigned* status, cudaStream_t stream) {
+                                   const float* slopes, int keep, float* scratch, int segment, int segments, float lambda,
+                                   int unit_norm, float eps, float out_scale, const void* gate, int gate_f32, long long gate_stride,
+                                   int gate_by_head, int is_f32, unsigned* status, cudaStream_t stream) {
+  VOSTI_REQUIRE(keep >= 0 && (keep == 0 || window > 0), "attention: kept first keys go with a window");
   VOSTI_REQUIRE(tokens >= 0 && nq > 0 && nkv > 0 && nq % nkv == 0, "attention: bad head counts nq=%d nkv=%d", nq, nkv);
   VOSTI_REQUIRE(maps == 1 || maps == 2, "attention: one or two score maps a head, not %d", maps);
   VOSTI_REQUIRE(dk > 0 && dv > 0 && dk <= MAX_W && dv <= MAX_W, "attention: head widths %d / %d must be at most %d", dk, dv, MAX_W);
@@ -843,14 +875,15 @@ VOSTI_API int vosti_attention_maps(const void* q, const void* k_cache, const voi
   VOSTI_REQUIRE(softcap >= 0.f, "attention: the soft cap is positive, or 0 for none");
   VOSTI_REQUIRE(segments >= 1 && segments <= 65535 && (segments == 1 || (scratch != nullptr && segment > 0 && segment % 32 == 0)),
                 "attention: key segments need scratch and a length that is a multiple of 32");
-  VOSTI_REQUIRE(gate == nullptr || gate_stride >= (long long)nq * dv, "attention: the gate's rows are narrower than the heads");
+  VOSTI_REQUIRE(!gate_by_head || gate != nullptr, "attention: the heads' gates are missing");
+  VOSTI_REQUIRE(gate == nullptr || gate_stride >= (gate_by_head ? nq : (long long)nq * dv), "attention: the gate's rows are narrower than the heads");
   if (tokens == 0) return VOSTI_OK;
   VOSTI_REQUIRE(((int64_t)tokens * nq + WARPS - 1) / WARPS <= 0x7fffffffLL, "attention: too many (token, head) pairs");
-  const HeadFinish finish = {lambda, out_scale, eps, unit_norm, gate, gate_f32, gate_stride};
+  const HeadFinish finish = {lambda, out_scale, eps, unit_norm, gate, gate_f32, gate_stride, gate_by_head};
   float* partial = segments > 1 ? scratch : nullptr;
   cudaError_t e;
 #define VOSTI_SINK_ARGS q, k_cache, v_cache, out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list, \
-                        tokens, nq, nkv, dk, dv, scale, window, bias, bias_last, sink, softcap, partial, segment, segments, status, finish, stream
+                        tokens, nq, nkv, dk, dv, scale, window, bias, bias_last, sink, softcap, slopes, keep, partial, segment, segments, status, finish, stream
   if (is_f32) e = maps == 2 ? attention_sink_launch<float, 2>(VOSTI_SINK_ARGS) : attention_sink_launch<float, 1>(VOSTI_SINK_ARGS);
   else e = maps == 2 ? attention_sink_launch<bf16, 2>(VOSTI_SINK_ARGS) : attention_sink_launch<bf16, 1>(VOSTI_SINK_ARGS);
 #undef VOSTI_SINK_ARGS
@@ -865,20 +898,21 @@ VOSTI_API int vosti_attention_sink(const void* q, const void* k_cache, const voi
                                    float* scratch, int segment, int segments, int is_f32, unsigned* status,
                                    cudaStream_t stream) {
   return vosti_attention_maps(q, k_cache, v_cache, out, positions, request_of, block_table, max_pages, page_size, num_pages, token_list,
-                              tokens, nq, nkv, 1, dk, dv, scale, window, bias, bias_last, sink, 0.f, scratch, segment, segments,
-                              NO_FINISH.lambda, 0, 0.f, 1.f, nullptr, 0, 0, is_f32, status, stream);
+                              tokens, nq, nkv, 1, dk, dv, scale, window, bias, bias_last, sink, 0.f, nullptr, 0, scratch, segment, segments,
+                              NO_FINISH.lambda, 0, 0.f, 1.f, nullptr, 0, 0, 0, is_f32, status, stream);
 }
 
 // a: [tokens, nq, maps, dv] attention outputs -> out [tokens, nq, dv] (see HeadFinish).
 VOSTI_API int vosti_head_finish(const void* a, void* out, int tokens, int nq, int maps, int dv, int a_width, int pair_group,
                                 float lambda, int unit_norm, float eps,
-                                float out_scale, const void* gate, int gate_f32, long long gate_stride, int is_f32,
+                                float out_scale, const void* gate, int gate_f32, long long gate_stride, int gate_by_head, int is_f32,
                                 cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && nq > 0 && dv > 0 && dv <= MAX_W && (maps == 1 || maps == 2), "head_finish: bad sizes");
   VOSTI_REQUIRE(a_width >= dv && pair_group >= 0 && (pair_group == 0 || nq % pair_group == 0), "head_finish: bad input layout");
-  VOSTI_REQUIRE(gate == nullptr || gate_stride >= (long long)nq * dv, "head_finish: the gate's rows are narrower than the heads");
+  VOSTI_REQUIRE(!gate_by_head || gate != nullptr, "head_finish: the heads' gates are missing");
+  VOSTI_REQUIRE(gate == nullptr || gate_stride >= (gate_by_head ? nq : (long long)nq * dv), "head_finish: the gate's rows are narrower than the heads");
   if (tokens == 0) return VOSTI_OK;
-  const HeadFinish f = {lambda, out_scale, eps, unit_norm, gate, gate_f32, gate_stride};
+  const HeadFinish f = {lambda, out_scale, eps, unit_norm, gate, gate_f32, gate_stride, gate_by_head};
   const unsigned blocks = (unsigned)(((int64_t)tokens * nq + WARPS - 1) / WARPS);
   if (is_f32) {
     if (maps == 2) vosti_launch(head_finish_kernel<float, 2>, dim3(blocks), dim3(WARPS * 32), 0, stream, (const float*)a, (float*)out, tokens, nq, dv, a_width, pair_group, f);

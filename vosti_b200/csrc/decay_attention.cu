@@ -1,0 +1,763 @@
+// Linear attention with one fixed decay per head: per request and head a float32 state S [dk, dv],
+//
+//   S_t = decay * S_(t-1) + k_t v_t^T,    o_t = S_t^T q_t
+//
+// q, k and v are columns of one projection (the serving type, or float32 unsummed K splits, added in
+// split order and rounded to the serving type); on the way in they may pass SiLU, or q and k a rotation
+// of the first 2 * rot_half elements of each head (element i with i + rot_half, by position * freq[i],
+// formed in float32); k is then multiplied by a constant. The state slot of a request holds S of all heads
+// ([heads, dk, dv]).
+//
+// decay_scan: token by token, for steps of few tokens a request and for float32 serving. A block takes a
+// piece of the value columns of one (request, head); a thread keeps a few rows of S in registers, the
+// state is read and written once.
+//
+// Long portions in bfloat16 run as chunks of 128 tokens, on the tensor cores (mma.sync):
+//   decay_chunk_state  U_c = sum over the chunk's tokens of decay^(tokens after it) k v^T, all chunks side by side;
+//   decay_chunk_scan   S before every chunk, S_(c+1) = decay^(n_c) S_c + U_c, written over U; the last one to the slot;
+//   decay_chunk_out    o_t = decay^(t+1) q_t S_c + sum over j <= t of decay^(t-j) (q_t . k_j) v_j, all chunks side by side.
+// What is float32 in the recurrence (decayed keys, rotated queries and keys, S, the weights of the second
+// product) enters a product as two bfloat16 terms; the product of the two remainders is left out. SiLU'd
+// queries, keys and values are activations of a projection and are rounded to bfloat16.
+//
+// decay_out: the read-outs normed (each head by its own root mean square, or all heads together with a
+// weight) and gated (SiLU or sigmoid of further columns of the projection), rounded for the output product.
+#include "common.cuh"
+#include "mma_util.cuh"
+
+namespace {
+
+constexpr int MAX_DK = 256;
+constexpr int CHUNK = 128;
+
+__device__ __forceinline__ float silu_of(float x) { return x / (1.f + expf(-x)); }
+template <typename T> __device__ __forceinline__ float rounded_to(float x) { return to_f32(from_f32<T>(x)); }
+
+struct Projection {
+  const void* data;            // T [tokens, stride], or float32 [splits, tokens, stride] with `plane` between splits
+  int splits;
+  int64_t stride, plane;
+  int off_q, off_k, off_v, off_g;
+};
+// Column `col` of token t, rounded to the serving type.
+template <typename T>
+__device__ __forceinline__ float column(const Projection& p, int64_t t, int col) {
+  const int64_t at = t * p.stride + col;
+  if (p.splits == 0) return to_f32(reinterpret_cast<const T*>(p.data)[at]);
+  const float* src = reinterpret_cast<const float*>(p.data) + at;
+  float x = src[0];
+  for (int s = 1; s < p.splits; ++s) x += src[s * p.plane];
+  return rounded_to<T>(x);
+}
+
+struct Recurrence {
+  int heads, dk, dv, silu;
+  const float* decay;          // [heads]
+  const float* log2_decay;     // [heads]
+  float key_scale;
+  const float* freq;           // [rot_half]
+  int rot_half;
+  const int* positions;
+  float* state;
+  int64_t state_stride;
+  const int* cu_q;
+  const int* state_slots;
+  int num_slots;
+};
+
+// ------------------------------------------------------------------ token by token
+constexpr int SCAN_THREADS = 256;
+constexpr int SCAN_LANES = 8;                        // threads side by side along the value columns
+constexpr int SCAN_ROWS = SCAN_THREADS / SCAN_LANES; // row groups: a thread keeps rows rg, rg + 32, ...
+constexpr int SCAN_TOKENS = 8;                       // tokens staged together
+
+template <typename T, int V, int R>
+__global__ void __launch_bounds__(SCAN_THREADS)
+decay_scan_kernel(const Projection p, const Recurrence c, float* __restrict__ out, int max_len) {
+  constexpr int COLS = SCAN_LANES * V;
+  __shared__ float qs[SCAN_TOKENS][32 * R], ks[SCAN_TOKENS][32 * R], vs[SCAN_TOKENS][COLS];
+  __shared__ float red[SCAN_TOKENS][SCAN_THREADS / 32][COLS];
+  extern __shared__ float turns[];                   // [SCAN_TOKENS][rot_half] cosines, then sines
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * COLS;
+  const int slot = c.state_slots[b];
+  const int start = c.cu_q[b], n = c.cu_q[b + 1] - start;
+  if (slot < 0 || slot >= c.num_slots || n <= 0 || (max_len > 0 && n > max_len)) return;
+  const int lane8 = threadIdx.x % SCAN_LANES, rg = threadIdx.x / SCAN_LANES;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int dk = c.dk, dv = c.dv;
+  const int col = col0 + lane8 * V;
+  const bool live = col < dv;                        // (V = 4 only where dv is a multiple of 4)
+  float* S = c.state + (int64_t)slot * c.state_stride + (int64_t)h * dk * dv + col;
+  float s[R][V];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = rg + SCAN_ROWS * i;
+    if (V == 4) {
+      const float4 x = (live && r < dk) ? *reinterpret_cast<const float4*>(S + (int64_t)r * dv) : make_float4(0.f, 0.f, 0.f, 0.f);
+      s[i][0] = x.x; s[i][V > 1 ? 1 : 0] = x.y; s[i][V > 2 ? 2 : 0] = x.z; s[i][V > 3 ? 3 : 0] = x.w;
+    } else {
+      s[i][0] = (live && r < dk) ? S[(int64_t)r * dv] : 0.f;
+    }
+  }
+  const float decay = c.decay[h];
+  float* cosines = turns;
+  float* sines = turns + SCAN_TOKENS * c.rot_half;
+  for (int t0 = 0; t0 < n; t0 += SCAN_TOKENS) {
+    const int count = min(SCAN_TOKENS, n - t0);
+    if (c.rot_half > 0) {
+      for (int i = threadIdx.x; i < count * c.rot_half; i += SCAN_THREADS) {
+        const int tt = i / c.rot_half, f = i - tt * c.rot_half;
+        const float angle = (float)c.positions[start + t0 + tt] * c.freq[f];
+        cosines[tt * c.rot_half + f] = cosf(angle);
+        sines[tt * c.rot_half + f] = sinf(angle);
+      }
+      __syncthreads();
+    }
+    for (int i = threadIdx.x; i < count * dk; i += SCAN_THREADS) {
+      const int tt = i / dk, e = i - tt * dk;
+      const int64_t t = start + t0 + tt;
+      const int cq = p.off_q + h * dk, ck = p.off_k + h * dk;
+      float q = column<T>(p, t, cq + e), k = column<T>(p, t, ck + e);
+      if (c.silu) { q = silu_of(q); k = silu_of(k); }
+      if (e < 2 * c.rot_half) {
+        const bool low = e < c.rot_half;
+        const int other = low ? e + c.rot_half : e - c.rot_half, f = low ? e : other;
+        const float cs = cosines[tt * c.rot_half + f], sn = low ? -sines[tt * c.rot_half + f] : sines[tt * c.rot_half + f];
+        q = q * cs + column<T>(p, t, cq + other) * sn;
+        k = k * cs + column<T>(p, t, ck + other) * sn;
+      }
+      qs[tt][e] = q;
+      ks[tt][e] = k * c.key_scale;
+    }
+    for (int i = threadIdx.x; i < count * COLS; i += SCAN_THREADS) {
+      const int tt = i / COLS, e = i - tt * COLS;
+      float v = col0 + e < dv ? column<T>(p, start + t0 + tt, p.off_v + h * dv + col0 + e) : 0.f;
+      vs[tt][e] = c.silu ? silu_of(v) : v;
+    }
+    __syncthreads();
+    for (int tt = 0; tt < count; ++tt) {
+      float o[V], v[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) { o[e] = 0.f; v[e] = vs[tt][lane8 * V + e]; }
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int r = rg + SCAN_ROWS * i;
+        if (r < dk) {
+          const float k = ks[tt][r], q = qs[tt][r];
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            s[i][e] = fmaf(k, v[e], s[i][e] * decay);
+            o[e] = fmaf(q, s[i][e], o[e]);
+          }
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        o[e] += __shfl_xor_sync(0xffffffffu, o[e], 8);
+        o[e] += __shfl_xor_sync(0xffffffffu, o[e], 16);
+        if (lane < SCAN_LANES) red[tt][warp][lane8 * V + e] = o[e];
+      }
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < count * COLS; i += SCAN_THREADS) {
+      const int tt = i / COLS, e = i - tt * COLS;
+      if (col0 + e < dv) {
+        float sum = 0.f;
+#pragma unroll
+        for (int w = 0; w < SCAN_THREADS / 32; ++w) sum += red[tt][w][e];
+        out[(int64_t)(start + t0 + tt) * c.heads * dv + h * dv + col0 + e] = sum;
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int r = rg + SCAN_ROWS * i;
+    if (!live || r >= dk) continue;
+    if (V == 4) *reinterpret_cast<float4*>(S + (int64_t)r * dv) = make_float4(s[i][0], s[i][V > 1 ? 1 : 0], s[i][V > 2 ? 2 : 0], s[i][V > 3 ? 3 : 0]);
+    else S[(int64_t)r * dv] = s[i][0];
+  }
+}
+
+// ------------------------------------------------------------------ chunks on the tensor cores
+constexpr int CHUNK_THREADS = 256;
+constexpr int VT = 64;                  // value columns of a block
+constexpr int V_PITCH = VT + 8;         // elements: rows 16 bytes apart modulo 128, conflict-free ldmatrix
+constexpr int CHUNK_MAX_DK = 128;
+
+struct Chunks {
+  const int* request;                   // [chunks] the request a chunk belongs to
+  const int* first;                     // [chunks] its first token, counted in the request's portion
+  const float2* turns;                  // [tokens][rot_half] (cosine, sine), or null
+  float* states;                        // [chunks][heads][dk][dv]
+};
+
+__global__ void __launch_bounds__(256)
+rotation_table_kernel(const float* __restrict__ freq, int half, const int* __restrict__ positions, int64_t n, float2* __restrict__ out) {
+  pdl_wait();
+  pdl_launch_dependents();
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / half;
+    const float angle = (float)positions[t] * freq[i - t * half];
+    out[i] = make_float2(cosf(angle), sinf(angle));
+  }
+}
+
+__device__ __forceinline__ void two_terms(float x, bf16& hi, bf16& lo) {
+  hi = __float2bfloat16_rn(x);
+  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
+}
+__device__ __forceinline__ uint32_t pair_of(bf16 a, bf16 b) {
+  const __nv_bfloat162 v(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+__device__ __forceinline__ void unpack8(uint4 raw, float (&x)[8]) {
+  const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 f = __bfloat1622float2(p[e]);
+    x[2 * e] = f.x;
+    x[2 * e + 1] = f.y;
+  }
+}
+
+// A chunk's rows of one head's queries or keys (columns col0 .. col0 + dk - 1 of the projection) as two bfloat16
+// terms in shared memory, [CHUNK][pitch] each, zeros beyond row n and column dk. weight: 0: times `scale`;
+// 1: times scale * decay^(n - 1 - row).
+template <bool WEIGHTED>
+__device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int dk, int dkp,
+                                           int pitch, int silu, const float2* __restrict__ turns, int rot_half, float scale,
+                                           float log2_decay, bf16* hi, bf16* lo, bool want_lo) {
+  const int words = dkp / 8;
+  const bool wide = dk % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0 && rot_half % 8 == 0;
+  for (int i = threadIdx.x; i < CHUNK * words; i += CHUNK_THREADS) {
+    const int r = i / words, e0 = (i - r * words) * 8;
+    float x[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = 0.f;
+    if (r < n && e0 < dk) {
+      const bf16* src = proj + (start + r) * stride + col0;
+      if (wide) {
+        unpack8(*reinterpret_cast<const uint4*>(src + e0), x);
+        if (silu) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) x[e] = rounded_to<bf16>(silu_of(x[e]));
+        }
+        if (e0 < 2 * rot_half) {
+          const bool low = e0 < rot_half;
+          float y[8];
+          unpack8(*reinterpret_cast<const uint4*>(src + (low ? e0 + rot_half : e0 - rot_half)), y);
+          const float4* cs = reinterpret_cast<const float4*>(turns + (start + r) * rot_half + (low ? e0 : e0 - rot_half));
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float4 a = cs[e];
+            x[2 * e] = x[2 * e] * a.x + y[2 * e] * (low ? -a.y : a.y);
+            x[2 * e + 1] = x[2 * e + 1] * a.z + y[2 * e + 1] * (low ? -a.w : a.w);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const int j = e0 + e;
+          if (j >= dk) continue;
+          float v = to_f32(src[j]);
+          if (silu) v = rounded_to<bf16>(silu_of(v));
+          if (j < 2 * rot_half) {
+            const bool low = j < rot_half;
+            const float2 a = turns[(start + r) * rot_half + (low ? j : j - rot_half)];
+            v = v * a.x + to_f32(src[low ? j + rot_half : j - rot_half]) * (low ? -a.y : a.y);
+          }
+          x[e] = v;
+        }
+      }
+      const float by = WEIGHTED ? scale * exp2f(log2_decay * (float)(n - 1 - r)) : scale;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] *= by;
+    }
+    uint32_t h[4], l[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      bf16 h0, l0, h1, l1;
+      two_terms(x[2 * e], h0, l0);
+      two_terms(x[2 * e + 1], h1, l1);
+      h[e] = pair_of(h0, h1);
+      l[e] = pair_of(l0, l1);
+    }
+    *reinterpret_cast<uint4*>(hi + r * pitch + e0) = make_uint4(h[0], h[1], h[2], h[3]);
+    if (want_lo) *reinterpret_cast<uint4*>(lo + r * pitch + e0) = make_uint4(l[0], l[1], l[2], l[3]);
+  }
+}
+
+// A chunk's values, columns v0 .. v0 + VT - 1 of one head, [CHUNK][V_PITCH], zeros beyond row n and column dv.
+__device__ __forceinline__ void stage_values(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int v0, int dv,
+                                             int silu, bf16* vs) {
+  const bool wide = dv % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0;
+  for (int i = threadIdx.x; i < CHUNK * (VT / 8); i += CHUNK_THREADS) {
+    const int r = i / (VT / 8), e0 = (i % (VT / 8)) * 8;
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    if (r < n && v0 + e0 < dv) {
+      const bf16* src = proj + (start + r) * stride + col0 + v0 + e0;
+      bf16* x = reinterpret_cast<bf16*>(&raw);
+      if (wide) {
+        raw = *reinterpret_cast<const uint4*>(src);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e)
+          if (v0 + e0 + e < dv) x[e] = src[e];
+      }
+      if (silu) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = __float2bfloat16_rn(silu_of(__bfloat162float(x[e])));
+      }
+    }
+    *reinterpret_cast<uint4*>(vs + r * V_PITCH + e0) = raw;
+  }
+}
+
+__device__ __forceinline__ int chunk_rows(const Recurrence& c, const Chunks& k, int chunk, int64_t& start) {
+  const int b = k.request[chunk];
+  start = c.cu_q[b] + k.first[chunk];
+  return min(CHUNK, (int)(c.cu_q[b + 1] - start));
+}
+
+__global__ void __launch_bounds__(CHUNK_THREADS, 2)
+decay_chunk_state_kernel(const Projection p, const Recurrence c, const Chunks k) {
+  extern __shared__ __align__(16) uint8_t chunk_smem[];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT;
+  const int dk = c.dk, dv = c.dv, dkp = (dk + 15) & ~15, pitch = dkp + 8;
+  bf16* kh = reinterpret_cast<bf16*>(chunk_smem);
+  bf16* kl = kh + CHUNK * pitch;
+  bf16* vs = kl + CHUNK * pitch;
+  int64_t start;
+  const int n = chunk_rows(c, k, chunk, start);
+  if (n <= 0) return;
+  const bf16* proj = reinterpret_cast<const bf16*>(p.data);
+  stage_rows<true>(proj, p.stride, start, n, p.off_k + h * dk, dk, dkp, pitch, c.silu, k.turns, c.rot_half, c.key_scale, c.log2_decay[h],
+                   kh, kl, true);
+  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, c.silu, vs);
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int steps = (n + 15) / 16;                                      // tokens in steps of 16
+  float* U = k.states + ((int64_t)chunk * c.heads + h) * dk * dv;
+  // units of 16 key channels x 32 value columns
+  const uint32_t a_off = (uint32_t)((((lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 8) * 2);
+  const uint32_t b_off = (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * V_PITCH + (lane >> 4) * 8) * 2);
+  for (int unit = warp; unit < dkp / 16 * 2; unit += CHUNK_THREADS / 32) {
+    const int m0 = (unit >> 1) * 16, n0 = (unit & 1) * 32;
+    float acc[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    for (int s = 0; s < steps; ++s) {
+      uint32_t ah[4], al[4], b0[4], b1[4];
+      ldmatrix_x4_trans(ah, smem_addr(kh) + a_off + (uint32_t)((s * 16 * pitch + m0) * 2));
+      ldmatrix_x4_trans(al, smem_addr(kl) + a_off + (uint32_t)((s * 16 * pitch + m0) * 2));
+      ldmatrix_x4_trans(b0, smem_addr(vs) + b_off + (uint32_t)((s * 16 * V_PITCH + n0) * 2));
+      ldmatrix_x4_trans(b1, smem_addr(vs) + b_off + (uint32_t)((s * 16 * V_PITCH + n0 + 16) * 2));
+      mma_bf16(acc[0], ah, b0[0], b0[1]); mma_bf16(acc[1], ah, b0[2], b0[3]);
+      mma_bf16(acc[2], ah, b1[0], b1[1]); mma_bf16(acc[3], ah, b1[2], b1[3]);
+      mma_bf16(acc[0], al, b0[0], b0[1]); mma_bf16(acc[1], al, b0[2], b0[3]);
+      mma_bf16(acc[2], al, b1[0], b1[1]); mma_bf16(acc[3], al, b1[2], b1[3]);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int row = m0 + (lane >> 2) + 8 * r, col = v0 + n0 + 8 * j + (lane & 3) * 2;
+        if (row >= dk) continue;
+        if (dv % 2 == 0) {
+          if (col < dv) *reinterpret_cast<float2*>(U + (int64_t)row * dv + col) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
+        } else {
+          if (col < dv) U[(int64_t)row * dv + col] = acc[j][2 * r];
+          if (col + 1 < dv) U[(int64_t)row * dv + col + 1] = acc[j][2 * r + 1];
+        }
+      }
+  }
+}
+
+// V floats a thread. long_requests: which requests; chunk0: a request's first chunk.
+template <int V>
+__global__ void __launch_bounds__(256)
+decay_chunk_scan_kernel(const Recurrence c, const int* __restrict__ long_requests, const int* __restrict__ chunk0, float* __restrict__ states) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = long_requests[blockIdx.z], h = blockIdx.y;
+  const int slot = c.state_slots[b], n = c.cu_q[b + 1] - c.cu_q[b];
+  const int64_t size = (int64_t)c.dk * c.dv, i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (i >= size || slot < 0 || slot >= c.num_slots) return;
+  const int chunks = (n + CHUNK - 1) / CHUNK;
+  const int64_t step = (int64_t)c.heads * size;
+  float* S = c.state + (int64_t)slot * c.state_stride + (int64_t)h * size + i;
+  float* at = states + ((int64_t)chunk0[blockIdx.z] * c.heads + h) * size + i;
+  const float whole = exp2f(c.log2_decay[h] * (float)CHUNK), last = exp2f(c.log2_decay[h] * (float)(n - (chunks - 1) * CHUNK));
+  float s[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) s[e] = S[e];
+  constexpr int AHEAD = 8;
+  for (int k0 = 0; k0 < chunks; k0 += AHEAD) {
+    float u[AHEAD][V];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+      if (k0 + k >= chunks) continue;
+      if (V == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(at + (k0 + k) * step);
+        u[k][0] = x.x; u[k][V > 1 ? 1 : 0] = x.y; u[k][V > 2 ? 2 : 0] = x.z; u[k][V > 3 ? 3 : 0] = x.w;
+      } else {
+        u[k][0] = at[(k0 + k) * step];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+      if (k0 + k >= chunks) continue;
+      if (V == 4) *reinterpret_cast<float4*>(at + (k0 + k) * step) = make_float4(s[0], s[V > 1 ? 1 : 0], s[V > 2 ? 2 : 0], s[V > 3 ? 3 : 0]);
+      else at[(k0 + k) * step] = s[0];
+      const float by = k0 + k + 1 < chunks ? whole : last;
+#pragma unroll
+      for (int e = 0; e < V; ++e) s[e] = fmaf(by, s[e], u[k][e]);
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < V; ++e) S[e] = s[e];
+}
+
+// LO: queries and keys have a second term (they are rotated); else they are bfloat16 (SiLU'd activations).
+template <bool LO>
+__global__ void __launch_bounds__(CHUNK_THREADS, 2)
+decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, float* __restrict__ out) {
+  extern __shared__ __align__(16) uint8_t chunk_smem[];
+  constexpr int KS = CHUNK_MAX_DK / 16;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT;
+  const int dk = c.dk, dv = c.dv, dkp = (dk + 15) & ~15, pitch = dkp + 8;
+  bf16* kh = reinterpret_cast<bf16*>(chunk_smem);      // queries, then the state (pitch V_PITCH), then keys
+  bf16* kl = kh + CHUNK * pitch;
+  bf16* vs = kl + CHUNK * pitch;
+  int64_t start;
+  const int n = chunk_rows(c, k, chunk, start);
+  if (n <= 0) return;
+  const bf16* proj = reinterpret_cast<const bf16*>(p.data);
+  const float l2d = c.log2_decay[h];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int row0 = warp * 16;                          // this warp's tokens of the chunk
+  stage_rows<false>(proj, p.stride, start, n, p.off_q + h * dk, dk, dkp, pitch, c.silu, k.turns, c.rot_half, 1.f, 0.f, kh, kl, LO);
+  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, c.silu, vs);
+  __syncthreads();
+  uint32_t qh[KS][4], ql[LO ? KS : 1][4];
+  {
+    const uint32_t off = (uint32_t)(((row0 + (lane & 15)) * pitch + (lane >> 4) * 8) * 2);
+#pragma unroll
+    for (int s = 0; s < KS; ++s)
+      if (s * 16 < dkp) {
+        ldmatrix_x4(qh[s], smem_addr(kh) + off + s * 32);
+        if (LO) ldmatrix_x4(ql[LO ? s : 0], smem_addr(kl) + off + s * 32);
+      }
+  }
+  __syncthreads();
+  // ---- the state before the chunk: [dkp][V_PITCH] in two terms, in the place of the queries
+  bf16* sh = kh;
+  bf16* sl = kh + (int64_t)dkp * V_PITCH;
+  {
+    const float* S = k.states + ((int64_t)chunk * c.heads + h) * dk * dv + v0;
+    const bool wide = dv % 4 == 0;
+    for (int i = threadIdx.x; i < dkp * (VT / 4); i += CHUNK_THREADS) {
+      const int r = i / (VT / 4), e0 = (i % (VT / 4)) * 4;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < dk) {
+        const float* src = S + (int64_t)r * dv + e0;
+        if (wide) {
+          if (v0 + e0 < dv) x = *reinterpret_cast<const float4*>(src);
+        } else {
+          if (v0 + e0 < dv) x.x = src[0];
+          if (v0 + e0 + 1 < dv) x.y = src[1];
+          if (v0 + e0 + 2 < dv) x.z = src[2];
+          if (v0 + e0 + 3 < dv) x.w = src[3];
+        }
+      }
+      bf16 a0, b0, a1, b1, a2, b2, a3, b3;
+      two_terms(x.x, a0, b0); two_terms(x.y, a1, b1); two_terms(x.z, a2, b2); two_terms(x.w, a3, b3);
+      *reinterpret_cast<uint2*>(sh + r * V_PITCH + e0) = make_uint2(pair_of(a0, a1), pair_of(a2, a3));
+      *reinterpret_cast<uint2*>(sl + r * V_PITCH + e0) = make_uint2(pair_of(b0, b1), pair_of(b2, b3));
+    }
+  }
+  __syncthreads();
+  float o[VT / 8][4];
+#pragma unroll
+  for (int j = 0; j < VT / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  const uint32_t b_off = (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * V_PITCH + (lane >> 4) * 8) * 2);
+  if (row0 < n) {
+#pragma unroll
+    for (int s = 0; s < KS; ++s)
+      if (s * 16 < dkp) {
+#pragma unroll
+        for (int j = 0; j < VT / 16; ++j) {
+          uint32_t b[4], bl[4];
+          ldmatrix_x4_trans(b, smem_addr(sh) + b_off + (uint32_t)((s * 16 * V_PITCH + j * 16) * 2));
+          ldmatrix_x4_trans(bl, smem_addr(sl) + b_off + (uint32_t)((s * 16 * V_PITCH + j * 16) * 2));
+          mma_bf16(o[2 * j], qh[s], b[0], b[1]); mma_bf16(o[2 * j + 1], qh[s], b[2], b[3]);
+          mma_bf16(o[2 * j], qh[s], bl[0], bl[1]); mma_bf16(o[2 * j + 1], qh[s], bl[2], bl[3]);
+          if (LO) { mma_bf16(o[2 * j], ql[LO ? s : 0], b[0], b[1]); mma_bf16(o[2 * j + 1], ql[LO ? s : 0], b[2], b[3]); }
+        }
+      }
+    const int r0 = row0 + (lane >> 2);
+    const float d0 = exp2f(l2d * (float)(r0 + 1)), d1 = exp2f(l2d * (float)(r0 + 9));
+#pragma unroll
+    for (int j = 0; j < VT / 8; ++j) { o[j][0] *= d0; o[j][1] *= d0; o[j][2] *= d1; o[j][3] *= d1; }
+  }
+  __syncthreads();
+  // ---- the chunk's own keys
+  stage_rows<false>(proj, p.stride, start, n, p.off_k + h * dk, dk, dkp, pitch, c.silu, k.turns, c.rot_half, c.key_scale, 0.f, kh, kl, true);
+  __syncthreads();
+  if (row0 >= n) return;
+  const uint32_t k_off = (uint32_t)((((lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 8) * 2);
+  for (int t = 0; t <= warp; ++t) {                    // tiles of 16 keys up to the warp's own rows
+    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+    for (int kk = 0; kk < KS; ++kk)
+      if (kk * 16 < dkp) {
+        uint32_t b[4], bl[4];
+        ldmatrix_x4(b, smem_addr(kh) + k_off + (uint32_t)((t * 16 * pitch + kk * 16) * 2));
+        mma_bf16(s[0], qh[kk], b[0], b[1]); mma_bf16(s[1], qh[kk], b[2], b[3]);
+        ldmatrix_x4(bl, smem_addr(kl) + k_off + (uint32_t)((t * 16 * pitch + kk * 16) * 2));
+        mma_bf16(s[0], qh[kk], bl[0], bl[1]); mma_bf16(s[1], qh[kk], bl[2], bl[3]);
+        if (LO) { mma_bf16(s[0], ql[LO ? kk : 0], b[0], b[1]); mma_bf16(s[1], ql[LO ? kk : 0], b[2], b[3]); }
+      }
+    uint32_t ph[4], pl[4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        bf16 h0, l0, h1, l1;
+        const int back = row0 + (lane >> 2) + 8 * r - (t * 16 + 8 * j + (lane & 3) * 2);
+        two_terms(back >= 0 ? s[j][2 * r] * exp2f(l2d * (float)back) : 0.f, h0, l0);
+        two_terms(back >= 1 ? s[j][2 * r + 1] * exp2f(l2d * (float)(back - 1)) : 0.f, h1, l1);
+        ph[2 * j + r] = pair_of(h0, h1);
+        pl[2 * j + r] = pair_of(l0, l1);
+      }
+#pragma unroll
+    for (int j = 0; j < VT / 16; ++j) {
+      uint32_t b[4];
+      ldmatrix_x4_trans(b, smem_addr(vs) + b_off + (uint32_t)((t * 16 * V_PITCH + j * 16) * 2));
+      mma_bf16(o[2 * j], ph, b[0], b[1]); mma_bf16(o[2 * j + 1], ph, b[2], b[3]);
+      mma_bf16(o[2 * j], pl, b[0], b[1]); mma_bf16(o[2 * j + 1], pl, b[2], b[3]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < VT / 8; ++j)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int row = row0 + (lane >> 2) + 8 * r, col = v0 + 8 * j + (lane & 3) * 2;
+      if (row >= n) continue;
+      float* dst = out + (start + row) * c.heads * dv + (int64_t)h * dv + col;
+      if (dv % 2 == 0) {
+        if (col < dv) *reinterpret_cast<float2*>(dst) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
+      } else {
+        if (col < dv) dst[0] = o[j][2 * r];
+        if (col + 1 < dv) dst[1] = o[j][2 * r + 1];
+      }
+    }
+}
+
+// ------------------------------------------------------------------ norm and gate
+// joint: one root mean square over the whole row, times a weight [width]; else one per head, no weight.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+decay_out_kernel(const float* __restrict__ o, const Projection p, int heads, int dv, int joint, const void* __restrict__ w, int w_f32,
+                 float eps, int gate_silu, T* __restrict__ y) {
+  __shared__ float scratch[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const int width = heads * dv;
+  const float* row = o + t * width;
+  auto gate_of = [&](float g) { return gate_silu ? silu_of(g) : 1.f / (1.f + expf(-g)); };
+  const bool vec = dv % 4 == 0 && p.stride % 4 == 0 && p.off_g % 4 == 0;
+  // four neighbouring gate columns
+  auto gates4 = [&](int i) {
+    const int64_t at = t * p.stride + p.off_g + i;
+    float4 g;
+    if (p.splits == 0) {
+      if (sizeof(T) == 4) {
+        g = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.data) + at);
+      } else {
+        const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p.data) + at);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        g = make_float4(a.x, a.y, b.x, b.y);
+      }
+    } else {
+      const float* src = reinterpret_cast<const float*>(p.data) + at;
+      g = *reinterpret_cast<const float4*>(src);
+      for (int s = 1; s < p.splits; ++s) {
+        const float4 u = *reinterpret_cast<const float4*>(src + s * p.plane);
+        g.x += u.x; g.y += u.y; g.z += u.z; g.w += u.w;
+      }
+      g = make_float4(rounded_to<T>(g.x), rounded_to<T>(g.y), rounded_to<T>(g.z), rounded_to<T>(g.w));
+    }
+    return make_float4(gate_of(g.x), gate_of(g.y), gate_of(g.z), gate_of(g.w));
+  };
+  auto put = [&](int i, float4 v) {
+    T* dst = y + t * width + i;
+    if (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(dst) = v;
+    } else {
+      const uint2 raw = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+      *reinterpret_cast<uint2*>(dst) = raw;
+    }
+  };
+  if (joint) {
+    float ss = 0.f;
+    if (vec) {
+      for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+        const float4 x = *reinterpret_cast<const float4*>(row + i);
+        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+      }
+    } else {
+      for (int i = threadIdx.x; i < width; i += blockDim.x) ss += row[i] * row[i];
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+    if (vec) {
+      for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
+        const float4 x = *reinterpret_cast<const float4*>(row + i), g = gates4(i);
+        put(i, make_float4(x.x * inv * load_flex(w, w_f32, i) * g.x, x.y * inv * load_flex(w, w_f32, i + 1) * g.y,
+                           x.z * inv * load_flex(w, w_f32, i + 2) * g.z, x.w * inv * load_flex(w, w_f32, i + 3) * g.w));
+      }
+    } else {
+      for (int i = threadIdx.x; i < width; i += blockDim.x)
+        y[t * width + i] = from_f32<T>(row[i] * inv * load_flex(w, w_f32, i) * gate_of(column<T>(p, t, p.off_g + i)));
+    }
+    return;
+  }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  for (int h = blockIdx.y * nwarps + warp; h < heads; h += gridDim.y * nwarps) {
+    float ss = 0.f;
+    if (vec) {
+      for (int i = lane * 4; i < dv; i += 128) {
+        const float4 x = *reinterpret_cast<const float4*>(row + h * dv + i);
+        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+      }
+    } else {
+      for (int i = lane; i < dv; i += 32) ss += row[h * dv + i] * row[h * dv + i];
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
+    if (vec) {
+      for (int i = lane * 4; i < dv; i += 128) {
+        const float4 x = *reinterpret_cast<const float4*>(row + h * dv + i), g = gates4(h * dv + i);
+        put(h * dv + i, make_float4(x.x * inv * g.x, x.y * inv * g.y, x.z * inv * g.z, x.w * inv * g.w));
+      }
+    } else {
+      for (int i = lane; i < dv; i += 32)
+        y[t * width + h * dv + i] = from_f32<T>(row[h * dv + i] * inv * gate_of(column<T>(p, t, p.off_g + h * dv + i)));
+    }
+  }
+}
+
+template <typename T, int V>
+void launch_scan(const Projection& p, const Recurrence& c, float* out, int requests, int max_len, cudaStream_t stream) {
+  const dim3 grid((c.dv + SCAN_LANES * V - 1) / (SCAN_LANES * V), c.heads, requests);
+  const size_t smem = (size_t)2 * SCAN_TOKENS * c.rot_half * sizeof(float);
+  if (c.dk <= 64) vosti_launch(decay_scan_kernel<T, V, 2>, grid, dim3(SCAN_THREADS), smem, stream, p, c, out, max_len);
+  else if (c.dk <= 128) vosti_launch(decay_scan_kernel<T, V, 4>, grid, dim3(SCAN_THREADS), smem, stream, p, c, out, max_len);
+  else vosti_launch(decay_scan_kernel<T, V, 8>, grid, dim3(SCAN_THREADS), smem, stream, p, c, out, max_len);
+}
+}  // namespace
+
+#define VOSTI_DECAY_CHECKS(name)                                                                                                       \
+  VOSTI_REQUIRE(heads > 0 && dk > 0 && dk <= MAX_DK && dv > 0 && requests >= 0 && splits >= 0, name ": bad sizes heads=%d dk=%d dv=%d", heads, dk, dv); \
+  VOSTI_REQUIRE(heads <= 65535 && requests <= 65535, name ": too many heads or requests for one launch");                              \
+  VOSTI_REQUIRE(state_stride >= (int64_t)heads * dk * dv && state_stride % 4 == 0, name ": the state slots are too small");            \
+  VOSTI_REQUIRE(rot_half >= 0 && 2 * rot_half <= dk && (rot_half == 0 || (freq != nullptr && positions != nullptr)), name ": the rotation takes at most the whole head"); \
+  VOSTI_REQUIRE(!(silu && rot_half > 0), name ": SiLU or a rotation, not both")
+
+// proj: the serving type [tokens, stride] (splits 0) or float32 [splits, tokens, stride]. Requests with more than max_len
+// tokens are left out (0: none is). out: float32 [tokens, heads * dv].
+VOSTI_API int vosti_decay_scan(const void* proj, int splits, int64_t stride, int tokens, int off_q, int off_k, int off_v, int heads, int dk,
+                               int dv, int silu, const float* decay, float key_scale, const float* freq, int rot_half,
+                               const int* positions, float* state, int64_t state_stride, const int* cu_q, const int* state_slots,
+                               int num_slots, int requests, int max_len, float* out, int is_f32, cudaStream_t stream) {
+  VOSTI_DECAY_CHECKS("decay_scan");
+  if (tokens == 0 || requests == 0) return VOSTI_OK;
+  const Projection p = {proj, splits, stride, (int64_t)tokens * stride, off_q, off_k, off_v, 0};
+  const Recurrence c = {heads, dk, dv, silu, decay, nullptr, key_scale, freq, rot_half, positions, state, state_stride, cu_q, state_slots, num_slots};
+  if (is_f32) {
+    if (dv % 4 == 0) launch_scan<float, 4>(p, c, out, requests, max_len, stream);
+    else launch_scan<float, 1>(p, c, out, requests, max_len, stream);
+  } else {
+    if (dv % 4 == 0) launch_scan<bf16, 4>(p, c, out, requests, max_len, stream);
+    else launch_scan<bf16, 1>(p, c, out, requests, max_len, stream);
+  }
+  VOSTI_LAUNCH_CHECK();
+}
+
+// Tokens of a chunk, and whether the chunk kernels take heads of this width.
+VOSTI_API int vosti_decay_chunk() { return CHUNK; }
+VOSTI_API int vosti_decay_chunk_fits(int dk) { return dk > 0 && dk <= CHUNK_MAX_DK; }
+
+// out float32 pairs [tokens, half]: cosine and sine of positions[t] * freq[i].
+VOSTI_API int vosti_rotation_table(const float* freq, int half, const int* positions, int tokens, void* out, cudaStream_t stream) {
+  VOSTI_REQUIRE(half > 0 && tokens >= 0 && freq != nullptr && positions != nullptr && out != nullptr, "rotation_table: bad arguments");
+  if (tokens == 0) return VOSTI_OK;
+  const int64_t n = (int64_t)tokens * half;
+  const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
+  vosti_launch(rotation_table_kernel, dim3(blocks), dim3(256), 0, stream, freq, half, positions, n, (float2*)out);
+  VOSTI_LAUNCH_CHECK();
+}
+
+// The long portions of a step: proj bfloat16 [tokens, stride]; chunk_request / chunk_first int32 [chunks] (see Chunks),
+// long_requests / long_chunk0 int32 [longs]; turns the rotation table of the step's tokens, or null;
+// states float32 scratch [chunks, heads, dk, dv].
+VOSTI_API int vosti_decay_chunks(const void* proj, int64_t stride, int tokens, int off_q, int off_k, int off_v, int heads, int dk, int dv,
+                                 int silu, const float* log2_decay, float key_scale, const float* freq, const void* turns, int rot_half,
+                                 const int* positions, float* state, int64_t state_stride, const int* cu_q, const int* state_slots,
+                                 int num_slots, const int* chunk_request, const int* chunk_first, int chunks, const int* long_requests,
+                                 const int* long_chunk0, int requests, float* states, float* out, cudaStream_t stream) {
+  const int splits = 0;
+  VOSTI_DECAY_CHECKS("decay_chunks");
+  VOSTI_REQUIRE(dk <= CHUNK_MAX_DK, "decay_chunks: heads of %d (at most %d)", dk, CHUNK_MAX_DK);
+  VOSTI_REQUIRE(rot_half == 0 || turns != nullptr, "decay_chunks: the rotation table is missing");
+  VOSTI_REQUIRE(((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(states) | reinterpret_cast<uintptr_t>(turns)) & 15) == 0,
+                "decay_chunks: operands must be 16-byte aligned");
+  if (tokens == 0 || chunks == 0) return VOSTI_OK;
+  const Projection p = {proj, 0, stride, 0, off_q, off_k, off_v, 0};
+  const Recurrence c = {heads, dk, dv, silu, nullptr, log2_decay, key_scale, freq, rot_half, positions, state, state_stride, cu_q, state_slots, num_slots};
+  const Chunks k = {chunk_request, chunk_first, (const float2*)turns, states};
+  const int dkp = (dk + 15) & ~15;
+  // (queries and keys take [CHUNK][dkp + 8] twice, the state [dkp][V_PITCH] twice in the same place, which is no larger)
+  static_assert(CHUNK_MAX_DK <= CHUNK && V_PITCH <= CHUNK, "the state must fit the keys' place");
+  const size_t smem = (size_t)2 * CHUNK * (dkp + 8) * 2 + (size_t)CHUNK * V_PITCH * 2;
+  constexpr int MOST = 2 * CHUNK * (CHUNK_MAX_DK + 8) * 2 + CHUNK * V_PITCH * 2;
+  static bool configured = false;
+  if (!configured) {
+    cudaFuncSetAttribute(decay_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST);
+    cudaFuncSetAttribute(decay_chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST);
+    cudaFuncSetAttribute(decay_chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST);
+    configured = true;
+  }
+  const dim3 grid(chunks, heads, (dv + VT - 1) / VT);
+  vosti_launch(decay_chunk_state_kernel, grid, dim3(CHUNK_THREADS), smem, stream, p, c, k);
+  const int64_t size = (int64_t)dk * dv;
+  if (size % 4 == 0)
+    vosti_launch(decay_chunk_scan_kernel<4>, dim3((unsigned)((size / 4 + 255) / 256), heads, requests), dim3(256), 0, stream, c, long_requests, long_chunk0, states);
+  else
+    vosti_launch(decay_chunk_scan_kernel<1>, dim3((unsigned)((size + 255) / 256), heads, requests), dim3(256), 0, stream, c, long_requests, long_chunk0, states);
+  if (rot_half > 0) vosti_launch(decay_chunk_out_kernel<true>, grid, dim3(CHUNK_THREADS), smem, stream, p, c, k, out);
+  else vosti_launch(decay_chunk_out_kernel<false>, grid, dim3(CHUNK_THREADS), smem, stream, p, c, k, out);
+  VOSTI_LAUNCH_CHECK();
+}
+
+// o float32 [tokens, heads * dv]; the gate: columns off_g .. off_g + heads * dv - 1 of proj. joint: w [heads * dv].
+VOSTI_API int vosti_decay_out(const float* o, const void* proj, int splits, int64_t stride, int off_g, int tokens, int heads, int dv,
+                              int joint, const void* w, int w_f32, float eps, int gate_silu, void* y, int is_f32, cudaStream_t stream) {
+  VOSTI_REQUIRE(tokens >= 0 && heads > 0 && dv > 0 && splits >= 0, "decay_out: bad sizes");
+  VOSTI_REQUIRE(!joint || w != nullptr, "decay_out: the joint norm's weight is missing");
+  if (tokens == 0) return VOSTI_OK;
+  const Projection p = {proj, splits, stride, (int64_t)tokens * stride, 0, 0, 0, off_g};
+  const int width = heads * dv;
+  int threads = 256;
+  if (joint && tokens <= 64) threads = width / 4 >= 1024 ? 1024 : ((width / 4 + 31) / 32 * 32 > 256 ? (width / 4 + 31) / 32 * 32 : 256);
+  const dim3 grid(tokens, joint ? 1 : (heads + 7) / 8);
+  if (is_f32) vosti_launch(decay_out_kernel<float>, grid, dim3(threads), 0, stream, o, p, heads, dv, joint, w, w_f32, eps, gate_silu, (float*)y);
+  else vosti_launch(decay_out_kernel<bf16>, grid, dim3(threads), 0, stream, o, p, heads, dv, joint, w, w_f32, eps, gate_silu, (bf16*)y);
+  VOSTI_LAUNCH_CHECK();
+}

@@ -48,6 +48,13 @@ __device__ __forceinline__ float gate_act(int epilogue, float g) {
   return epilogue == EPI_RE2GLU ? r * r : r;
 }
 
+// g sigmoid(scale g) (u + 1) of g = min(gate, limit) and u = up clamped to [-limit, limit].
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float scale) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + __expf(-scale * g)) * (u + 1.f);
+}
+
 // ------------------------------------------------------------------ the kernel
 template <int BN, int STAGES, int KPS>
 __global__ void __launch_bounds__(THREADS, 1)
@@ -695,7 +702,7 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
       int device = 0;
       cudaGetDevice(&device);
       cudaDeviceGetAttribute(&pair_sms, cudaDevAttrMultiProcessorCount, device);
-      cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel<PlainEpilogue>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess || pair_sms <= 1) {
         pair_sms = 0;
         vosti_set_error("gemm_tc: cannot configure the paired kernel: %s", cudaGetErrorString(e));
@@ -704,8 +711,8 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
     }
     const int tiles = ((tokens + 2 * BM - 1) / (2 * BM)) * ((features + PAIR_BN - 1) / PAIR_BN);
     const int pairs = tiles < pair_sms / 2 ? tiles : pair_sms / 2;
-    vosti_launch_clusters(gemm_tc_pair_kernel, dim3(2 * pairs), dim3(PAIR_THREADS), 2, smem, stream, mx, *mw, y, tokens,
-                          features, k_blocks, ld_out, epilogue, w_tiles, status);
+    vosti_launch_clusters(gemm_tc_pair_kernel<PlainEpilogue>, dim3(2 * pairs), dim3(PAIR_THREADS), 2, smem, stream, mx, *mw, y, tokens,
+                          features, k_blocks, ld_out, epilogue, w_tiles, PlainEpilogue{}, status);
     VOSTI_LAUNCH_CHECK();
   }
   if (tokens > 128) {
@@ -756,6 +763,35 @@ VOSTI_API int vosti_gemm_tc(const void* x, const void* w, void* y, int tokens, i
     vosti_launch(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, (const float*)workspace, y, splits, tokens,
                  features, ld_out, epilogue);
   }
+  VOSTI_LAUNCH_CHECK();
+}
+
+// A gate | up product of more than 128 tokens with biases and the clamped activation as its epilogue (two SMs per tile):
+// y bf16 [tokens, features / 2] = clamped_glu(gate + bias, up + bias), the packed weight's rows (and the float32 bias)
+// in blocks of 16 gate rows and their 16 up rows.
+VOSTI_API int vosti_gemm_tc_clamped(const void* x, const void* w, void* y, int tokens, int features, int k, const float* bias,
+                                    float limit, float sigmoid_scale, unsigned* status, cudaStream_t stream) {
+  using namespace pair_kernel;
+  VOSTI_REQUIRE(tokens > 128 && vosti_gemm_tc_supported(features, k) && features % 32 == 0, "gemm_tc_clamped: unsupported sizes T=%d F=%d K=%d", tokens, features, k);
+  VOSTI_REQUIRE(bias != nullptr && limit > 0.f, "gemm_tc_clamped: a bias and a positive limit are needed");
+  VOSTI_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0) && ((uintptr_t)bias % 16 == 0), "gemm_tc_clamped: operands must be 16-byte aligned");
+  const int k_blocks = (k + BK - 1) / BK, w_tiles = (features + BM - 1) / BM;
+  CUtensorMap mw, mx;
+  VOSTI_REQUIRE(weight_map(w, k_blocks * w_tiles * BM, BK, BM, &mw) && make_map(&mx, x, tokens, k, BM), "gemm_tc_clamped: cuTensorMapEncodeTiled failed");
+  constexpr size_t smem = (size_t)PAIR_STAGES * PAIR_STAGE_BYTES + 1024;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_pair_kernel<ClampedEpilogue>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) {
+      vosti_set_error("gemm_tc_clamped: cannot configure the paired kernel: %s", cudaGetErrorString(e));
+      return (int)e;
+    }
+    configured = true;
+  }
+  const int tiles = ((tokens + 2 * BM - 1) / (2 * BM)) * ((features + PAIR_BN - 1) / PAIR_BN);
+  const int pairs = tiles < device_sms() / 2 ? tiles : device_sms() / 2;
+  vosti_launch_clusters(gemm_tc_pair_kernel<ClampedEpilogue>, dim3(2 * pairs), dim3(PAIR_THREADS), 2, smem, stream, mx, mw, y, tokens,
+                        features, k_blocks, features / 2, (int)EPI_SWIGLU, w_tiles, ClampedEpilogue{bias, limit, sigmoid_scale}, status);
   VOSTI_LAUNCH_CHECK();
 }
 

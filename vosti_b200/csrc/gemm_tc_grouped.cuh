@@ -22,9 +22,7 @@ struct GluConstants { float limit, sigmoid_scale; };
 __host__ __device__ constexpr bool grouped_is_gated(int epilogue) { return is_gated(epilogue) || epilogue == EPI_CLAMPGLU; }
 __device__ __forceinline__ float grouped_gate(int epilogue, float g, float u, const GluConstants& glu) {
   if (epilogue == EPI_CLAMPGLU) {
-    g = fminf(g, glu.limit);
-    u = fminf(fmaxf(u, -glu.limit), glu.limit);
-    return g / (1.f + __expf(-glu.sigmoid_scale * g)) * (u + 1.f);
+    return clamped_glu(g, u, glu.limit, glu.sigmoid_scale);
   }
   return gate_act(epilogue, g) * u;
 }

@@ -73,12 +73,44 @@ __device__ __forceinline__ void umma_commit_pair(uint32_t bar) {
                ::"r"(bar), "h"((uint16_t)3)
                : "memory");
 }
+// What the epilogue needs beside its kind: nothing, or for the clamped gated form (a kernel of its own) the bias in the
+// features' order and the activation's constants.
+struct PlainEpilogue {};
+struct ClampedEpilogue {
+  const float* bias;
+  float limit, sigmoid_scale;
+};
+__device__ __forceinline__ void store_columns(const uint32_t (&r)[32], void* out, int token, int f0, int features, int ld_out,
+                                              int epilogue, const PlainEpilogue&) {
+  store_token_columns(r, out, token, f0, features, ld_out, epilogue);
+}
+__device__ __forceinline__ void store_columns(const uint32_t (&r)[32], void* out, int token, int f0, int, int ld_out, int,
+                                              const ClampedEpilogue& c) {
+  // columns f0..f0+15 are gate rows, f0+16..f0+31 their up rows
+  const float4* b4 = reinterpret_cast<const float4*>(c.bias + f0);
+  uint32_t packed[8];
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    const float4 bg = __ldg(b4 + q), bu = __ldg(b4 + 4 + q);
+    const float v0 = clamped_glu(__uint_as_float(r[4 * q]) + bg.x, __uint_as_float(r[16 + 4 * q]) + bu.x, c.limit, c.sigmoid_scale);
+    const float v1 = clamped_glu(__uint_as_float(r[4 * q + 1]) + bg.y, __uint_as_float(r[17 + 4 * q]) + bu.y, c.limit, c.sigmoid_scale);
+    const float v2 = clamped_glu(__uint_as_float(r[4 * q + 2]) + bg.z, __uint_as_float(r[18 + 4 * q]) + bu.z, c.limit, c.sigmoid_scale);
+    const float v3 = clamped_glu(__uint_as_float(r[4 * q + 3]) + bg.w, __uint_as_float(r[19 + 4 * q]) + bu.w, c.limit, c.sigmoid_scale);
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v0, v1), hi = __floats2bfloat162_rn(v2, v3);
+    packed[2 * q] = *reinterpret_cast<const uint32_t*>(&lo);
+    packed[2 * q + 1] = *reinterpret_cast<const uint32_t*>(&hi);
+  }
+  uint4* y = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(out) + (int64_t)token * ld_out + f0 / 2);    // ld_out is a multiple of 16
+  y[0] = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+  y[1] = make_uint4(packed[4], packed[5], packed[6], packed[7]);
+}
 }  // namespace pair_kernel
 
+template <typename EpilogueExtra>
 __global__ void __launch_bounds__(pair_kernel::PAIR_THREADS, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                     void* __restrict__ out, int tokens, int features, int k_blocks, int ld_out, int epilogue,
-                    int w_tiles, unsigned* status) {
+                    int w_tiles, const EpilogueExtra extra, unsigned* status) {
   using namespace pair_kernel;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -194,7 +226,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
         uint32_t r[32];
         tmem_load32(tmem_base + as * PAIR_BN + ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0, r);
         if (!row_ok) continue;
-        store_token_columns(r, out, token, f0, features, ld_out, epilogue);
+        store_columns(r, out, token, f0, features, ld_out, epilogue, extra);
       }
       tc_fence_before();
       __syncwarp();

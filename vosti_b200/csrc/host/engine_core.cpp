@@ -215,10 +215,11 @@ struct Residency {
 
 class CacheCore {
  public:
-  CacheCore(int groups, const int* group_windows, int pages, int page, int requests, bool reuse, bool has_state)
+  CacheCore(int groups, const int* group_windows, const int* group_keeps, int pages, int page, int requests, bool reuse, bool has_state)
       : page_size(page), num_pages(pages), max_requests(requests), has_state(has_state) {
     for (int g = 0; g < groups; ++g) {
       windows.push_back(group_windows[g]);
+      keeps.push_back(group_keeps[g] > 0 ? group_keeps[g] : 0);
       pools.emplace_back(new PagePool(pages));
     }
     prefix_reuse = reuse && groups == 1 && windows[0] == 0 && !has_state;
@@ -306,7 +307,7 @@ class CacheCore {
       const int first_needed = res.length - windows[g] + 1;
       if (first_needed <= 0) continue;
       const int upto = std::min(first_needed / page_size, (int)res.pages[g].size());
-      for (int index = 0; index < upto; ++index) {
+      for (int index = pages_for(keeps[g]); index < upto; ++index) {       // (the pages of a request's kept first tokens stay)
         if (res.pages[g][index] != RELEASED) {
           const int rc = pools[g]->release(res.pages[g][index]);
           if (rc != VH_OK) return rc;
@@ -378,6 +379,7 @@ class CacheCore {
   std::vector<int> fresh_slots;                           // handed out by begin() since they were last taken
   bool prefix_reuse = false;
   std::vector<int> windows;
+  std::vector<int> keeps;                                 // first tokens of a request a group's window never passes
   std::vector<std::unique_ptr<PagePool>> pools;
   std::map<int64_t, Residency> live;
   std::vector<int> free_slots;
@@ -714,12 +716,12 @@ VH_API int vh_pool_check(void* pool, const int32_t* pages, const int32_t* counts
 }
 
 // ---- cache manager and scheduler
-VH_API void* vh_create(int groups, const int32_t* windows, int num_pages, int page_size, int max_requests,
+VH_API void* vh_create(int groups, const int32_t* windows, const int32_t* keeps, int num_pages, int page_size, int max_requests,
                        int prefix_reuse, int has_state, int max_num_seqs, int max_batched_tokens, int chunk_size,
                        int vocab_size, int max_context) {
   if (groups < 0 || num_pages <= 0 || page_size <= 0 || max_requests <= 0) return nullptr;
   Host* h = new Host;
-  h->cache.reset(new CacheCore(groups, windows, num_pages, page_size, max_requests, prefix_reuse != 0, has_state != 0));
+  h->cache.reset(new CacheCore(groups, windows, keeps, num_pages, page_size, max_requests, prefix_reuse != 0, has_state != 0));
   h->scheduler.reset(new SchedulerCore(h->cache.get(), max_num_seqs, max_batched_tokens, chunk_size, vocab_size, max_context));
   return h;
 }

@@ -3,7 +3,7 @@
 // moe_route: per token, the `top` experts with the largest float32 router logits (the lowest
 // index wins a tie) and their weights: the softmax over the chosen logits only, or (`over_all`)
 // the softmax over all experts, of which the chosen ones' scores are divided by their sum (plus
-// 1e-20); either way times a constant `scale`. It writes the
+// 1e-20) or left as they are (`over_all` 2); each way times a constant `scale`. It writes the
 // choice twice: as lists (expert ids and weights, [tokens, top]) and as a dense float32 matrix
 // [tokens, experts] that is zero where an expert was not chosen.
 //
@@ -66,7 +66,7 @@ __device__ __forceinline__ void route_row(const float* row, int t, int experts, 
     float z = 0.f;
     for (int e = lane; e < experts; e += 32) z += expf(row[e] - first);
     z = warp_sum(z);
-    inv = (1.f / z) / (total / z + 1e-20f);
+    inv = over_all == 2 ? 1.f / z : (1.f / z) / (total / z + 1e-20f);
   }
   inv *= scale;
   if (lane == 0)
@@ -281,13 +281,13 @@ __device__ __forceinline__ float moe_activation(float x, int mode) {
 
 // Experts by token id: table [vocab, top] (entries of a row differ), every listed expert with weight `share`.
 struct TokenTable {
-  const int* ids;          // [tokens], or null: the weights are in `dense`
+  const int* ids;          // [tokens], or null: in moe_scale the weights are in `dense`, else token t's row is row t
   const int* table;
   int top, vocab;
   float share;
 };
 __device__ __forceinline__ const int* table_row(const TokenTable& by, int64_t t) {
-  const int id = by.ids[t];
+  const int id = by.ids != nullptr ? by.ids[t] : (int)t;
   return by.table + (int64_t)(id < 0 || id >= by.vocab ? 0 : id) * by.top;
 }
 __device__ __forceinline__ float table_weight(const TokenTable& by, int64_t t, int e) {
@@ -530,13 +530,13 @@ VOSTI_API int vosti_moe_group(const int* chosen, int tokens, int top, int expert
   VOSTI_LAUNCH_CHECK();
 }
 
-// x: `tokens` rows of row_bytes (a multiple of 2); sorted: [tokens * top] rows; offsets int32 [experts + 1]; where int32
+// ids null: the table has a row per token (a router's choice). x: `tokens` rows of row_bytes (a multiple of 2); sorted: [tokens * top] rows; offsets int32 [experts + 1]; where int32
 // [tokens * top], the sorted place of every (token, pick) pair.
 VOSTI_API int vosti_moe_dispatch(const int* ids, const int* table, int vocab, int top, float share, int tokens, int experts, const void* x,
                                  int64_t row_bytes, void* sorted, int* offsets, int* where, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && top <= experts && vocab > 0 && row_bytes > 0 && row_bytes % 2 == 0, "moe_dispatch: bad sizes");
   VOSTI_REQUIRE((int64_t)tokens * top < (int64_t)1 << 24, "moe_dispatch: too many pairs");
-  VOSTI_REQUIRE(ids != nullptr && table != nullptr, "moe_dispatch: missing arrays");
+  VOSTI_REQUIRE(table != nullptr && (ids != nullptr || vocab >= tokens), "moe_dispatch: missing arrays");
   if (tokens == 0) return VOSTI_OK;
   VOSTI_REQUIRE(experts <= 4096, "moe_dispatch: %d experts (at most 4096 are taken)", experts);
   const int pairs = tokens * top, chunk = pairs <= 8192 ? 8 : DISPATCH_CHUNK;         // rows a block: a warp each, or four

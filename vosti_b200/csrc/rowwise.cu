@@ -396,6 +396,84 @@ VOSTI_API int vosti_glu_mul(const void* gate_up, void* out, int rows, int inter,
   VOSTI_LAUNCH_CHECK();
 }
 
+// The clamped activation of a gate | up projection with biases, g sigmoid(sigmoid_scale g) (u + 1) of g = min(gate + bg,
+// limit) and u = up + bu clamped to [-limit, limit], from a product of the serving type or from its float32
+// unsummed K splits, added in split order. `block` 0: the gate columns come first; > 0: blocks of `block` gate
+// columns followed by their up columns. The bias is float32 in the projection's column order.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+glu_bias_kernel(const void* __restrict__ gate_up, int in_f32, int splits, const float* __restrict__ bias, T* __restrict__ out,
+                int64_t rows, int inter, int block, float limit, float sigmoid_scale) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t words = rows * inter / V, width = 2 * (int64_t)inter, plane = rows * width;
+  for (int64_t w = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; w < words; w += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t r = w * V / inter;
+    const int c = (int)(w * V - r * inter);
+    const int gc = block > 0 ? c / block * 2 * block + c % block : c, uc = gc + (block > 0 ? block : inter);
+    float g[V], u[V];
+    auto load = [&](int64_t at, float (&x)[V]) {
+      if (V == 4 && in_f32) {
+        const float4 f = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(gate_up) + at);
+        x[0] = f.x; x[V > 1 ? 1 : 0] = f.y; x[V > 2 ? 2 : 0] = f.z; x[V > 3 ? 3 : 0] = f.w;
+      } else if (V == 4) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(gate_up) + at);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        x[0] = a.x; x[V > 1 ? 1 : 0] = a.y; x[V > 2 ? 2 : 0] = b.x; x[V > 3 ? 3 : 0] = b.y;
+      } else {
+        x[0] = load_flex(gate_up, in_f32, at);
+      }
+    };
+    load(r * width + gc, g);
+    load(r * width + uc, u);
+#pragma unroll 2
+    for (int s = 1; s < splits; ++s) {
+      float a[V], b[V];
+      load(s * plane + r * width + gc, a);
+      load(s * plane + r * width + uc, b);
+#pragma unroll
+      for (int e = 0; e < V; ++e) { g[e] += a[e]; u[e] += b[e]; }
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      const float a = fminf(g[e] + bias[gc + e], limit), b = fminf(fmaxf(u[e] + bias[uc + e], -limit), limit);
+      g[e] = a * (1.f / (1.f + expf(-sigmoid_scale * a))) * (b + 1.f);
+    }
+    T* dst = out + w * V;
+    if (V == 4 && sizeof(T) == 2) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(g[0], g[V > 1 ? 1 : 0]), hi = __floats2bfloat162_rn(g[V > 2 ? 2 : 0], g[V > 3 ? 3 : 0]);
+      uint2 raw;
+      raw.x = *reinterpret_cast<const unsigned*>(&lo);
+      raw.y = *reinterpret_cast<const unsigned*>(&hi);
+      *reinterpret_cast<uint2*>(dst) = raw;
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) dst[e] = from_f32<T>(g[e]);
+    }
+  }
+}
+
+VOSTI_API int vosti_glu_bias(const void* gate_up, int in_f32, int splits, const float* bias, void* out, int rows, int inter, int block,
+                             float limit, float sigmoid_scale, int out_f32, cudaStream_t stream) {
+  VOSTI_REQUIRE(rows >= 0 && inter > 0 && splits >= 1 && (splits == 1 || in_f32), "glu_bias: bad sizes rows=%d inter=%d splits=%d", rows, inter, splits);
+  VOSTI_REQUIRE(block == 0 || (block > 0 && inter % block == 0), "glu_bias: blocks of %d do not divide %d columns", block, inter);
+  VOSTI_REQUIRE(bias != nullptr && limit > 0.f, "glu_bias: a bias and a positive limit are needed");
+  if (rows == 0) return VOSTI_OK;
+  const bool words = inter % 4 == 0 && block % 4 == 0 && ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const int64_t n = (int64_t)rows * inter / (words ? 4 : 1);
+  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+#define VOSTI_GLU_ARGS(T) gate_up, in_f32, splits, bias, (T*)out, (int64_t)rows, inter, block, limit, sigmoid_scale
+  if (out_f32) {
+    if (words) vosti_launch(glu_bias_kernel<float, 4>, dim3(blocks), dim3(256), 0, stream, VOSTI_GLU_ARGS(float));
+    else vosti_launch(glu_bias_kernel<float, 1>, dim3(blocks), dim3(256), 0, stream, VOSTI_GLU_ARGS(float));
+  } else {
+    if (words) vosti_launch(glu_bias_kernel<bf16, 4>, dim3(blocks), dim3(256), 0, stream, VOSTI_GLU_ARGS(bf16));
+    else vosti_launch(glu_bias_kernel<bf16, 1>, dim3(blocks), dim3(256), 0, stream, VOSTI_GLU_ARGS(bf16));
+  }
+#undef VOSTI_GLU_ARGS
+  VOSTI_LAUNCH_CHECK();
+}
+
 VOSTI_API int vosti_silu_mul(const void* gate_up, void* out, int rows, int inter, int is_f32,
                              cudaStream_t stream) {
   VOSTI_REQUIRE(rows >= 0 && inter > 0, "silu_mul: bad sizes rows=%d inter=%d", rows, inter);

@@ -2,7 +2,8 @@
 //
 // pair_embedding: x[t] = table[id] + pairs[row] in float32, where row hashes the token with the
 // one before it in its sequence, (prev * mul_prev + id * mul_cur) mod buckets, and a sequence's
-// first token (position 0) takes the row after the hashed ones (row `buckets`). The token before
+// first token (position 0) takes the row after the hashed ones (row `buckets`); the rows' rounding may be
+// written beside them. The token before
 // the first one of a step's portion is the last token of the request's step before: it lives in
 // the request's state slot (one int32), which pair_state rewrites after every token of the step
 // has been read. Token ids a sampler left on the device (`source`, `values`: see the embedding
@@ -23,7 +24,7 @@ __global__ void __launch_bounds__(128)
 pair_embedding_kernel(const int* __restrict__ ids, const int* __restrict__ source, const int* __restrict__ values,
                       const int* __restrict__ positions, const int* __restrict__ request_of, const int* __restrict__ cu_q,
                       const int* __restrict__ state_slots, const int* __restrict__ last_token, int num_slots,
-                      const T* __restrict__ table, const T* __restrict__ pairs, float* __restrict__ out,
+                      const T* __restrict__ table, const T* __restrict__ pairs, float* __restrict__ out, bf16* __restrict__ low,
                       int* __restrict__ resolved, int hidden, int vocab, long long buckets, long long mul_prev,
                       long long mul_cur, unsigned* status) {
   pdl_wait();
@@ -71,10 +72,21 @@ pair_embedding_kernel(const int* __restrict__ ids, const int* __restrict__ sourc
       }
       reinterpret_cast<float4*>(dst)[2 * i] = make_float4(r[0], r[1], r[2], r[3]);
       reinterpret_cast<float4*>(dst)[2 * i + 1] = make_float4(r[4], r[5], r[6], r[7]);
+      if (low != nullptr) {
+        uint4 raw;
+        __nv_bfloat162* z = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) z[e] = __floats2bfloat162_rn(r[2 * e], r[2 * e + 1]);
+        reinterpret_cast<uint4*>(low + (int64_t)t * hidden)[i] = raw;
+      }
     }
     return;
   }
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = bad ? 0.f : to_f32(a[i]) + to_f32(p[i]);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    const float x = bad ? 0.f : to_f32(a[i]) + to_f32(p[i]);
+    dst[i] = x;
+    if (low != nullptr) low[(int64_t)t * hidden + i] = __float2bfloat16_rn(x);
+  }
 }
 
 // One thread per request: the last token of its portion becomes the slot's last token.
@@ -114,11 +126,11 @@ token_gate_kernel(const T* __restrict__ z, const int* __restrict__ ids, const TS
 }  // namespace
 
 // table [vocab, hidden] and pairs [buckets + 1, hidden] share a type; out float32 [tokens, hidden];
-// resolved int32 [tokens]; last_token int32 [num_slots] (a view with stride 1).
+// low: the rows' rounding to bfloat16 [tokens, hidden], or null; resolved int32 [tokens]; last_token int32 [num_slots] (a view with stride 1).
 VOSTI_API int vosti_pair_embedding(const int* ids, const int* source, const int* values, const int* positions,
                                    const int* request_of, const int* cu_q, const int* state_slots, int* last_token,
                                    int num_slots, int requests, const void* table, const void* pairs, int is_f32,
-                                   float* out, int* resolved, int tokens, int hidden, int vocab, long long buckets,
+                                   float* out, void* low, int* resolved, int tokens, int hidden, int vocab, long long buckets,
                                    long long mul_prev, long long mul_cur, unsigned* status, cudaStream_t stream) {
   VOSTI_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0 && buckets > 0 && requests >= 0,
                 "pair_embedding: bad sizes T=%d H=%d V=%d buckets=%lld", tokens, hidden, vocab, buckets);
@@ -127,11 +139,11 @@ VOSTI_API int vosti_pair_embedding(const int* ids, const int* source, const int*
   if (tokens == 0) return VOSTI_OK;
   if (is_f32)
     vosti_launch(pair_embedding_kernel<float>, dim3(tokens), dim3(128), 0, stream, ids, source, values, positions, request_of,
-                 cu_q, state_slots, (const int*)last_token, num_slots, (const float*)table, (const float*)pairs, out, resolved,
+                 cu_q, state_slots, (const int*)last_token, num_slots, (const float*)table, (const float*)pairs, out, (bf16*)low, resolved,
                  hidden, vocab, buckets, mul_prev, mul_cur, status);
   else
     vosti_launch(pair_embedding_kernel<bf16>, dim3(tokens), dim3(128), 0, stream, ids, source, values, positions, request_of,
-                 cu_q, state_slots, (const int*)last_token, num_slots, (const bf16*)table, (const bf16*)pairs, out, resolved,
+                 cu_q, state_slots, (const int*)last_token, num_slots, (const bf16*)table, (const bf16*)pairs, out, (bf16*)low, resolved,
                  hidden, vocab, buckets, mul_prev, mul_cur, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) { vosti_set_error("%s", cudaGetErrorString(e)); return (int)e; }

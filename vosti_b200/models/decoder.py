@@ -74,7 +74,7 @@ class DecoderModel:
             for spec in (self.blocks[i].mixer.cache_spec() for i in layers):
                 if pages[index] is not None and spec is not None and pages[index].window:
                     wider = max(pages[index].window, spec.window) if spec.window else 0
-                    pages[index] = dataclasses.replace(pages[index], window=wider)
+                    pages[index] = dataclasses.replace(pages[index], window=wider, keep_first=max(pages[index].keep_first, spec.keep_first))
         pages = [spec if i in owned else None for i, spec in enumerate(pages)]
         return (pages + ([None] if own else []),
                 [self.blocks[i].state_spec() for i in self.cache_layers] + ([self.embedding.state_spec()] if own else []))
@@ -112,12 +112,16 @@ class DecoderModel:
         return {key: tensors[cls._part_tensor_name(name, part, key)] for key in part.weight_specs()
                 if cls._part_tensor_name(name, part, key) in tensors}
 
+    def _layer_prefix(self, i: int) -> str:
+        number = self.spec.layers[i].number
+        return self.spec.layer_prefix.format(i=i if number is None else number)
+
     def expected_weights(self) -> Dict[str, WeightSpec]:
         spec = self.spec
         out = {self._part_tensor_name(spec.embed_name, self.embedding, key): w
                for key, w in self.embedding.weight_specs().items()}
         for i, block in enumerate(self.blocks):
-            prefix = spec.layer_prefix.format(i=i)
+            prefix = self._layer_prefix(i)
             for key, w in block.weight_specs().items():
                 out[prefix + key] = w
         for key, w in self.final_norm.weight_specs().items():
@@ -144,7 +148,7 @@ class DecoderModel:
         under = lambda prefix: {k[len(prefix):]: v for k, v in tensors.items() if k.startswith(prefix)}
         self.embedding.load(self._own(tensors, spec.embed_name, self.embedding), dtype)
         for i, block in enumerate(self.blocks):
-            block.load(under(spec.layer_prefix.format(i=i)), dtype)
+            block.load(under(self._layer_prefix(i)), dtype)
         self.final_norm.load(self._own(tensors, spec.final_norm_name, self.final_norm), dtype)
         self.head.load(self._own(tensors, spec.lm_head_name, self.head), dtype,
                        tied=self.embedding.table() if spec.tie_word_embeddings else None)

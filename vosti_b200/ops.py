@@ -193,6 +193,38 @@ def glu_mul(gate_up: torch.Tensor, activation: str, limit: float = 0.0, sigmoid_
     return out
 
 
+def glu_bias(gate_up, bias: torch.Tensor, out_dtype: torch.dtype, *, block: int, limit: float, sigmoid_scale: float) -> torch.Tensor:
+    """The clamped activation (see `glu_mul`) of a gate | up projection plus its float32 bias; `gate_up` is a tensor or a
+    float32 product's unsummed K splits (`PartialSum`). `block` 0: the gate columns come first; > 0: blocks of `block` gate
+    columns followed by their up columns (the bias in the same order)."""
+    p, in_f32, splits = _splits_of(gate_up)
+    rows, width = gate_up.shape
+    if bias.dtype != torch.float32 or bias.shape[0] != width:
+        raise KernelError("glu_bias: the bias is float32 over the projection's columns")
+    out = torch.empty((rows, width // 2), dtype=out_dtype, device=bias.device)
+    _check(library().vosti_glu_bias(p, in_f32, splits, _p(bias), _p(out), rows, width // 2, block, ctypes.c_float(limit),
+                                    ctypes.c_float(sigmoid_scale), _is_f32(out), _stream()), "glu_bias")
+    return out
+
+
+CLAMPED_EPILOGUE_FROM = 128      # more tokens than this: the product applies bias and activation itself
+
+
+def gemm_tc_clamped(x: torch.Tensor, w: "PackedWeight", bias: torch.Tensor, status: torch.Tensor, *, limit: float,
+                    sigmoid_scale: float) -> torch.Tensor:
+    """`glu_bias` of x @ w.T as the product's epilogue, for more than 128 tokens; w's rows and the bias are blocks of 16
+    gate rows followed by their 16 up rows."""
+    _contig(x, w.data, bias)
+    tokens, k = x.shape
+    features = w.shape[0]
+    if x.dtype != torch.bfloat16 or w.shape[1] != k or bias.dtype != torch.float32 or bias.shape[0] != features:
+        raise KernelError("gemm_tc_clamped: x is bfloat16 [tokens, k], the bias float32 over the weight's rows")
+    out = torch.empty((tokens, features // 2), dtype=torch.bfloat16, device=x.device)
+    _check(library().vosti_gemm_tc_clamped(_p(x), _p(w.data), _p(out), tokens, features, k, _p(bias), ctypes.c_float(limit),
+                                           ctypes.c_float(sigmoid_scale), _p(status), _stream()), "gemm_tc_clamped")
+    return out
+
+
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, status: torch.Tensor, *,
               out_dtype: Optional[torch.dtype] = None,
               row_index: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -376,7 +408,7 @@ class PartialSum:
 
 
 def materialize(x):
-    return x.materialize() if isinstance(x, (PartialSum, StreamPair, PickedSum)) else x
+    return x.materialize() if isinstance(x, (PartialSum, StreamPair, PickedSum, BranchMean)) else x
 
 
 class PackedWeight:
@@ -844,16 +876,19 @@ def rms_stream(x, weight: Optional[torch.Tensor], eps: float, out_dtype: Optiona
 
 class PickedSum:
     """share * the sum over picks of the rows where[t, pick] of y ([pairs, width] float32, or unsummed K splits
-    of them): experts' outputs sorted by expert that a later kernel (`gated_rms_stream`) adds up per token.
-    `materialize` gives the sums [tokens, width] in float32."""
+    of them): experts' outputs sorted by expert that a later kernel (`gated_rms_stream`, `out_norm_stream`) adds up
+    per token. With `weights` (float32 [tokens, picks], `out_norm_stream` only) every pick has a weight of its own
+    instead of the share. `materialize` gives the sums [tokens, width] in float32."""
 
-    def __init__(self, y, where: torch.Tensor, share: float):
-        self.y, self.where, self.share = y, where, float(share)
+    def __init__(self, y, where: torch.Tensor, share: float, weights: Optional[torch.Tensor] = None):
+        self.y, self.where, self.share, self.weights = y, where, float(share), weights
         self.shape = (where.shape[0], y.shape[1])
         self.dtype = torch.float32
 
     def materialize(self) -> torch.Tensor:
-        weights = torch.full(tuple(self.where.shape), self.share, dtype=torch.float32, device=self.where.device)
+        weights = self.weights
+        if weights is None:
+            weights = torch.full(tuple(self.where.shape), self.share, dtype=torch.float32, device=self.where.device)
         return moe_combine(materialize(self.y), self.where, weights)
 
 
@@ -864,6 +899,8 @@ class DeferredGated:
     scratch of its own), y also a `PickedSum`."""
 
     def __init__(self, y, z, bias: Optional[torch.Tensor], scale: float):
+        if isinstance(y, PickedSum) and y.weights is not None:
+            y = y.materialize()
         inner = y.y if isinstance(y, PickedSum) else y
         for t in (inner, z):
             if isinstance(t, PartialSum) and t.dtype != torch.float32:
@@ -946,6 +983,61 @@ def gated_rms_stream(stream: torch.Tensor, x: Optional[DeferredGated], eps: floa
     return out if conv is None else (out, u)
 
 
+class BranchMean:
+    """The mean of two side-by-side branches' outputs, each first divided by its root mean square and multiplied by
+    a weight, still to be formed: tensors or float32 unsummed K splits (`PartialSum`, each in a scratch of its own).
+    `out_norm_stream` forms it on the way; `materialize` gives it as a tensor (`branch_merge`)."""
+
+    def __init__(self, xs, weights, eps: float):
+        if len(xs) != 2:
+            raise KernelError("branch mean: two branches")
+        scratches = [x.scratch for x in xs if isinstance(x, PartialSum)]
+        if len(set(scratches)) != len(scratches):
+            raise KernelError("branch mean: unsummed products need a scratch each")
+        self.xs, self.weights, self.eps = tuple(xs), tuple(weights), float(eps)
+        self.shape, self.dtype = tuple(xs[0].shape), torch.float32
+
+    def materialize(self) -> torch.Tensor:
+        return branch_merge(self.xs, self.weights, self.eps)
+
+
+def out_norm_stream(pair: "StreamPair", y, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, status: torch.Tensor, *,
+                    offset: float = 0.0, scale: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> "StreamPair":
+    """The boundary between sublayers that are normed on their way into the stream (csrc/out_norm.cu):
+    x + scale * z / sqrt(mean(z^2) + eps) * (offset + weight) with z = y + bias, written over the float32 stream x
+    together with its rounding to `out_dtype`. y: a tensor, float32 unsummed K splits, a `PickedSum` or a `BranchMean`."""
+    stream = pair.stream
+    _contig(stream, weight, scale, bias)
+    rows, width = stream.shape
+    lib = library()
+    if isinstance(y, BranchMean) and width > lib.vosti_out_norm_max_width(2):
+        y = y.materialize()
+    if tuple(y.shape) != (rows, width) or stream.dtype != torch.float32:
+        raise KernelError("out_norm_stream: the stream is float32 and the output has its shape")
+    where = picks = branch_w = None
+    branch_eps, branch_f32, share = 0.0, 0, 1.0
+    terms = [y]
+    if isinstance(y, BranchMean):
+        terms, branch_eps, branch_f32 = list(y.xs), y.eps, _is_f32(y.weights[0])
+        if _is_f32(y.weights[1]) != branch_f32:
+            raise KernelError("out_norm_stream: the branches' weights must share a dtype")
+        _contig(*y.weights)
+        branch_w = (ctypes.c_void_p * 2)(*[w.data_ptr() for w in y.weights])
+    elif isinstance(y, PickedSum):
+        terms, where, picks, share = [y.y], y.where, y.weights, y.share
+        _contig(where, picks)
+    flat = [_splits_of(t) for t in terms]
+    n = len(flat)
+    out = None if out_dtype == torch.float32 else torch.empty((rows, width), dtype=out_dtype, device=stream.device)
+    _check(lib.vosti_out_norm_stream(
+        (ctypes.c_void_p * n)(*[p for p, _, _ in flat]), (ctypes.c_int * n)(*[f for _, f, _ in flat]),
+        (ctypes.c_int * n)(*[s for _, _, s in flat]), n, _p(bias), 0 if bias is None else _is_f32(bias), _p(where), _p(picks),
+        0 if where is None else where.shape[1], 0 if where is None else terms[0].shape[0], ctypes.c_float(share), branch_w, branch_f32,
+        ctypes.c_float(branch_eps), _p(stream), _p(stream), _p(weight), _is_f32(weight), ctypes.c_float(offset), ctypes.c_float(eps),
+        _p(scale), 0 if scale is None else _is_f32(scale), _p(out), rows, width, _p(status), _stream()), "out_norm_stream")
+    return StreamPair(stream if out is None else out, stream)
+
+
 # ---------------------------------------------------------------- token inputs
 class StreamPair:
     """A float32 residual stream [rows, width] together with its rounding to the serving type: what a
@@ -986,12 +1078,13 @@ def post_norm_stream(stream: torch.Tensor, x, weight: torch.Tensor, alpha: float
 
 
 def pair_embedding(ids: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, last_token: torch.Tensor, ctx, *,
-                   buckets: int, mul_prev: int, mul_cur: int, feedback: Optional[tuple] = None):
+                   buckets: int, mul_prev: int, mul_cur: int, feedback: Optional[tuple] = None, rounded: bool = False):
     """table[id] + pairs[(prev * mul_prev + id * mul_cur) % buckets] in float32, row `buckets` of
     `pairs` for tokens at position 0; `prev` is the token before in the step, or, for the first
     token of a request's portion, what `last_token` (int32 [slots]) holds for its slot, which is
     then set to the portion's last token. Returns (rows float32 [tokens, hidden], the token ids
-    int32 [tokens] with those a sampler left on the device filled in)."""
+    int32 [tokens] with those a sampler left on the device filled in); with `rounded` the rows come as a
+    `StreamPair` with their rounding to bfloat16, written by the same kernel."""
     _contig(ids, table, pairs, last_token)
     source, values = feedback if feedback is not None else (None, None)
     if source is not None:
@@ -1000,13 +1093,14 @@ def pair_embedding(ids: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, 
         raise KernelError("pair_embedding: the tables must share a type, the pair table has buckets + 1 rows")
     tokens = ids.shape[0]
     out = torch.empty((tokens, table.shape[1]), dtype=torch.float32, device=table.device)
+    low = torch.empty((tokens, table.shape[1]), dtype=torch.bfloat16, device=table.device) if rounded else None
     resolved = torch.empty((tokens,), dtype=torch.int32, device=table.device)
     _check(library().vosti_pair_embedding(
         _p(ids), _p(source), _p(values), _p(ctx.positions), _p(ctx.request_of), _p(ctx.cu_q), _p(ctx.state_slots),
-        _p(last_token), last_token.shape[0], ctx.num_requests, _p(table), _p(pairs), _is_f32(table), _p(out), _p(resolved),
+        _p(last_token), last_token.shape[0], ctx.num_requests, _p(table), _p(pairs), _is_f32(table), _p(out), _p(low), _p(resolved),
         tokens, table.shape[1], table.shape[0], ctypes.c_longlong(buckets), ctypes.c_longlong(mul_prev),
         ctypes.c_longlong(mul_cur), _p(ctx.status), _stream()), "pair_embedding", kernels=2)
-    return out, resolved
+    return (StreamPair(low, out) if rounded else out), resolved
 
 
 def token_gate(z: torch.Tensor, ids: torch.Tensor, side: torch.Tensor, offset: int) -> torch.Tensor:
@@ -1072,10 +1166,12 @@ class HeadFinish:
     """What follows a head's softmax-weighted sum before the output projection, in float32 (the
     kernels' HeadFinish): with two score maps a head o = a1 - `lam` * a2; with `unit_norm`
     o / sqrt(mean(o^2) + eps) * out_scale over the head's values; with `gate` ([tokens, >= nq * dv],
-    float32 or bfloat16, rows may be strided: a view of a wider product) o * sigmoid(gate)."""
+    float32 or bfloat16, rows may be strided: a view of a wider product) o * sigmoid(gate); `by_head`: the
+    gate is [tokens, >= nq], one number a head."""
 
     def __init__(self, *, lam: float = 0.0, unit_norm: bool = False, eps: float = 0.0, out_scale: float = 1.0,
-                 gate: Optional[torch.Tensor] = None):
+                 gate: Optional[torch.Tensor] = None, by_head: bool = False):
+        self.by_head = bool(by_head)
         self.lam, self.unit_norm, self.eps, self.out_scale, self.gate = float(lam), bool(unit_norm), float(eps), float(out_scale), gate
         if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1):
             raise KernelError("head finish: the gate is [tokens, heads * width] with contiguous rows")
@@ -1083,7 +1179,7 @@ class HeadFinish:
     def args(self):
         g = self.gate
         return (ctypes.c_float(self.lam), int(self.unit_norm), ctypes.c_float(self.eps), ctypes.c_float(self.out_scale), _p(g),
-                0 if g is None else _is_f32(g), ctypes.c_longlong(0 if g is None else g.stride(0)))
+                0 if g is None else _is_f32(g), ctypes.c_longlong(0 if g is None else g.stride(0)), int(self.by_head))
 
 
 _NO_FINISH = HeadFinish()
@@ -1166,20 +1262,50 @@ def qkv_heads(proj: torch.Tensor, k_cache: Optional[torch.Tensor], v_cache: Opti
     return q if splits == 1 else (q, extra)
 
 
+def qk_joint(proj, k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], *, nq: int, nkv: int, dk: int, page_size: int,
+             slot_mapping: Optional[torch.Tensor], out_dtype: torch.dtype, status: torch.Tensor, q_norm: torch.Tensor,
+             k_norm: torch.Tensor, eps: float, bias: Optional[torch.Tensor] = None, extra_width: int = 0):
+    """After a q | k | further projection whose values are its keys (csrc/qk_joint.cu): the bias (float32 over q | k) is
+    added, the keys go to the value slots as they are, and queries and keys are divided by the root mean square
+    of their whole projection (all heads at once) and multiplied by `q_norm` [nq * dk] / `k_norm` [nkv * dk]; float32,
+    rounded once. `proj` may be float32 unsummed K splits. Returns (queries [tokens, nq * dk], the `extra_width`
+    columns after k in float32 or None)."""
+    p, proj_f32, splits = _splits_of(proj)
+    tokens, stride = proj.shape
+    _contig(k_cache, v_cache, slot_mapping, bias, q_norm, k_norm)
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape[0] != (nq + nkv) * dk):
+        raise KernelError("qk_joint: the bias is float32 over the q | k columns")
+    if _is_f32(q_norm) != _is_f32(k_norm) or q_norm.shape[0] != nq * dk or k_norm.shape[0] != nkv * dk:
+        raise KernelError("qk_joint: the norms' weights cover their whole projections and share a dtype")
+    if any(cache is not None and cache.dtype != out_dtype for cache in (k_cache, v_cache)):
+        raise KernelError("qk_joint: the caches hold the output type")
+    device = q_norm.device
+    q = torch.empty((tokens, nq * dk), dtype=out_dtype, device=device)
+    extra = torch.empty((tokens, extra_width), dtype=torch.float32, device=device) if extra_width else None
+    num_slots = 0 if k_cache is None else k_cache.numel() // (nkv * dk)
+    _check(library().vosti_qk_joint(p, proj_f32, splits, ctypes.c_int64(stride), _p(bias), _p(q_norm), _p(k_norm), _is_f32(q_norm),
+                                    ctypes.c_float(eps), _p(q), _p(k_cache), _p(v_cache), _p(slot_mapping), ctypes.c_int64(num_slots),
+                                    page_size, tokens, nq, nkv, dk, _p(extra), extra_width, 1 if out_dtype == torch.float32 else 0,
+                                    _p(status), _stream()), "qk_joint")
+    return q, extra
+
+
 def _attention_sink_rows(ctx, q, k_cache, v_cache, out, group, *, token_list, count, nq, nkv, dk, dv, scale, window,
-                         bias, sink, softcap=0.0, maps=1, finish=None) -> None:
+                         bias, sink, softcap=0.0, maps=1, finish=None, slopes=None, keep=0) -> None:
     """The CUDA-core kernel over `count` rows of the step (all of them if `token_list` is None)."""
     flag = _same_dtype(q, k_cache, v_cache)
     num_pages = k_cache.numel() // (group.page_size * nkv * maps * dk)
     segments, scratch = 1, None
     if count * nq <= SINK_SPLIT_MAX_ROWS:
         segments = key_segments(ctx.max_kv_len, window, SINK_SEGMENT)
+        if keep and segments > 1:                       # the kept keys' pieces come before the window's
+            segments += -(-keep // SINK_SEGMENT)
     if segments > 1:
         scratch = _workspace(q.device, count * nq * segments * maps * (dv + 2))
     _check(library().vosti_attention_maps(
         _p(q), _p(k_cache), _p(v_cache), _p(out), _p(ctx.positions), _p(ctx.request_of), _p(group.block_table),
         group.block_table.shape[1], group.page_size, num_pages, _p(token_list), count, nq, nkv, maps, dk, dv,
-        ctypes.c_float(scale), window, _p(bias), 0 if bias is None else bias.shape[1] - 1, _p(sink), ctypes.c_float(softcap), _p(scratch),
+        ctypes.c_float(scale), window, _p(bias), 0 if bias is None else bias.shape[1] - 1, _p(sink), ctypes.c_float(softcap), _p(slopes), keep, _p(scratch),
         SINK_SEGMENT, segments, *(finish or _NO_FINISH).args(), flag, _p(ctx.status), _stream()), "attention_sink",
         kernels=2 if segments > 1 else 1)
 
@@ -1187,12 +1313,13 @@ def _attention_sink_rows(ctx, q, k_cache, v_cache, out, group, *, token_list, co
 def attention_sink(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, group, *, nq: int, nkv: int,
                    dk: int, dv: int, scale: float, window: int, bias: Optional[torch.Tensor],
                    sink: Optional[torch.Tensor], chunk: int = 0, softcap: float = 0.0, maps: int = 1,
-                   finish: Optional["HeadFinish"] = None) -> torch.Tensor:
+                   finish: Optional["HeadFinish"] = None, slopes: Optional[torch.Tensor] = None, keep: int = 0) -> torch.Tensor:
     """Causal attention of every query row over its request's cached keys (the last `window` of
     them, or with `chunk` those of the query's own chunk of positions), with an optional bias
     table float32 [nq, distances] (base-2 units, the last column serving every larger distance)
     and an optional sink logit per head (float32 [nq], natural units); `softcap` c > 0 makes the scaled
-    scores c tanh(score / c). Returns [tokens, nq * dv].
+    scores c tanh(score / c); `slopes` (float32 [nq], base-2 units) times the distance is taken off the scores; with
+    `keep` > 0 and a window every query also sees the keys before `keep`. Returns [tokens, nq * dv].
     With `maps` = 2 a head has two score maps (queries [tokens, nq, 2, dk], the key cache's entries
     2 * dk wide) over the same values; `finish` (a `HeadFinish`) says how they are combined and what
     else follows the softmax (unit norm, gate).
@@ -1202,23 +1329,50 @@ def attention_sink(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.T
     bias and the sink, and `finish` is a kernel of its own after them. Everything else runs on the
     CUDA-core kernel, with the keys cut into segments when the step has few rows, and `finish` is
     its last step."""
-    _contig(q, k_cache, v_cache, bias, sink)
+    _contig(q, k_cache, v_cache, bias, sink, slopes)
     tokens = q.shape[0]
     out = torch.empty((tokens, nq * dv), dtype=q.dtype, device=q.device)
     if chunk < 0 or window < 0 or (chunk and window):
         raise KernelError("attention_sink: a window or a chunk, not both, and neither negative")
+    if keep < 0 or (keep and not window):
+        raise KernelError("attention_sink: kept first keys go with a window")
     window = -chunk if chunk else window            # the kernels take a chunk as a negative window
     common = dict(nq=nq, nkv=nkv, dk=dk, dv=dv, scale=scale, window=window, bias=bias, sink=sink, softcap=softcap)
     lib = library()
+    sloped = slopes is not None or keep > 0
+    head_gate = finish.gate if finish is not None and finish.by_head else None
     tensor_memory = (q.dtype == torch.bfloat16 and dk == dv and nq // nkv <= 16 and maps == 1
+                     and (not sloped or (slopes is not None and chunk == 0 and bias is None and softcap == 0.0
+                                         and (finish is None or (head_gate is not None and not finish.unit_norm
+                                                                 and head_gate.dtype == torch.float32 and head_gate.is_contiguous()))))
                      and lib.vosti_attention_prefill_tc_supported(dk, group.page_size))
     if not tensor_memory or getattr(ctx, "layout", None) is None or "attention" not in ctx.layout:
-        _attention_sink_rows(ctx, q, k_cache, v_cache, out, group, token_list=None, count=tokens, maps=maps, finish=finish, **common)
+        _attention_sink_rows(ctx, q, k_cache, v_cache, out, group, token_list=None, count=tokens, maps=maps, finish=finish,
+                             slopes=slopes, keep=keep, **common)
         return out
     # as for `attention`: requests that bring a few tokens one query at a time with split keys,
     # longer portions tile by tile on the tensor-memory kernel (the step's work lists)
     lists = ctx.layout["attention"]
     num_pages = k_cache.numel() // (group.page_size * nkv * dk)
+    if sloped:
+        # the kernels' sloped form, the head gate as its last step
+        tail = (ctypes.c_float(scale), window, _p(slopes), keep, _p(sink), _p(head_gate), _p(ctx.status), _stream())
+        if lists["num_short_tokens"]:
+            count = lists["num_short_tokens"]
+            lib.vosti_attention_decode_scratch.restype = ctypes.c_int64
+            keys = lib.vosti_attention_decode_sloped_keys(ctx.max_kv_len, window, keep)
+            scratch = _workspace(q.device, lib.vosti_attention_decode_scratch(count, nq, nkv, dk, keys))
+            _check(lib.vosti_attention_decode_sloped(
+                _p(q), _p(k_cache), _p(v_cache), _p(out), _p(scratch), ctypes.c_int64(scratch.numel()),
+                _p(_counters(q.device, count * nkv)), _p(ctx.extras.get("attention.short_tokens")), count, tokens, _p(ctx.positions),
+                _p(ctx.request_of), _p(group.block_table), group.block_table.shape[1], group.page_size, num_pages, nq, nkv, dk,
+                ctx.max_kv_len, *tail), "attention_decode_sloped")
+        if lists["num_long_rows"]:
+            _check(lib.vosti_attention_prefill_tc_sloped(
+                _p(q), _p(k_cache), _p(v_cache), _p(out), _p(ctx.extras.get("attention.long_rows")), lists["num_long_rows"],
+                _p(ctx.cu_q), _p(ctx.kv_len), _p(group.block_table), group.block_table.shape[1], group.page_size, num_pages,
+                nq, nkv, dk, lists["max_long_q_len"], tokens, *tail), "attention_prefill_tc_sloped")
+        return out
     bias_last = 0 if bias is None else bias.shape[1] - 1
     if lists["num_short_tokens"]:
         count = lists["num_short_tokens"]
@@ -1553,12 +1707,97 @@ def general_delta_scan(r, k, v, decay, unit, removal, state: torch.Tensor, ctx, 
     return out
 
 
+# ---------------------------------------------------------------- linear attention with a fixed decay
+DECAY_CHUNK = 128    # tokens of a chunk (csrc/decay_attention.cu)
+DECAY_SHORT = 16     # requests that bring at most this many tokens are served token by token
+
+
+def decay_step_layout(q_lens):
+    """How the fixed-decay recurrence divides a step (registered with the step layout as "decay"): requests that bring
+    more than DECAY_SHORT tokens are cut into chunks that run side by side, the others go token by
+    token; with one order of arithmetic asked for (set_fixed_order) all of them do."""
+    chunk = DECAY_CHUNK
+    requests, firsts, longs, starts = [], [], [], []
+    if not FIXED_ORDER and max(q_lens, default=0) > DECAY_SHORT:
+        for i, n in enumerate(q_lens):
+            if n > DECAY_SHORT:
+                longs.append(i)
+                starts.append(len(requests))
+                requests.extend([i] * -(-n // chunk))
+                firsts.extend(range(0, n, chunk))
+    arrays = {"chunk_request": requests, "chunk_first": firsts, "long_requests": longs, "long_chunk0": starts} if longs else {}
+    return arrays, {"chunks": len(requests), "longs": len(longs), "shorts": len(q_lens) - len(longs)}
+
+
+def decay_attention(proj, offsets: dict, state: torch.Tensor, ctx, *, heads: int, dk: int, dv: int, decay: torch.Tensor,
+                    log2_decay: torch.Tensor, silu: bool, key_scale: float, freq: Optional[torch.Tensor]) -> torch.Tensor:
+    """S <- decay S + k v^T, o = S^T q per head over every request's tokens of this step, from and to its state slot
+    (csrc/decay_attention.cu); `proj` (a tensor of the serving type or unsummed K splits that are rounded to it) holds
+    the columns q | k | v at `offsets`, which pass SiLU (`silu`) or of which q and k are rotated (`freq`, float32 [n],
+    the first 2n elements of a head). `decay` and its base-2 logarithm: float32 [heads]. Returns float32 [tokens, heads * dv]."""
+    dtype = proj.dtype
+    layout = (getattr(ctx, "layout", None) or {}).get("decay")
+    lib = library()
+    chunked = dtype == torch.bfloat16 and layout is not None and layout["longs"] > 0 and lib.vosti_decay_chunk_fits(dk)
+    if chunked:
+        proj = materialize(proj)
+    p, _, splits = _splits_of(proj)
+    splits = splits if isinstance(proj, PartialSum) else 0
+    tokens, stride = proj.shape
+    _contig(state, decay, log2_decay, freq)
+    if state.dtype != torch.float32 or decay.dtype != torch.float32 or log2_decay.dtype != torch.float32:
+        raise KernelError("decay_attention: the state and the decays are float32")
+    out = torch.empty((tokens, heads * dv), dtype=torch.float32, device=state.device)
+    half = 0 if freq is None else freq.shape[0]
+    common = (offsets["q"], offsets["k"], offsets["v"], heads, dk, dv, int(silu))
+    slots = (_p(state), ctypes.c_int64(state.shape[1]), _p(ctx.cu_q), _p(ctx.state_slots), state.shape[0])
+    if chunked:
+        turns = None
+        if half:
+            # one table of angles a step and set of frequencies, shared by the layers that rotate alike
+            key = ("rotation_table", freq.data_ptr())
+            turns = ctx.extras.get(key)
+            if turns is None:
+                turns = torch.empty((tokens, half, 2), dtype=torch.float32, device=state.device)
+                _check(lib.vosti_rotation_table(_p(freq), half, _p(ctx.positions), tokens, _p(turns), _stream()), "rotation_table")
+                ctx.extras[key] = turns
+        states = torch.empty((layout["chunks"], heads, dk, dv), dtype=torch.float32, device=state.device)
+        arrays = ctx.extras
+        _check(lib.vosti_decay_chunks(
+            p, ctypes.c_int64(stride), tokens, *common, _p(log2_decay), ctypes.c_float(key_scale), _p(freq), _p(turns), half,
+            _p(ctx.positions), *slots, _p(arrays["decay.chunk_request"]), _p(arrays["decay.chunk_first"]), layout["chunks"],
+            _p(arrays["decay.long_requests"]), _p(arrays["decay.long_chunk0"]), layout["longs"], _p(states), _p(out), _stream()),
+            "decay_chunks", kernels=3)
+    if not chunked or layout["shorts"] > 0:
+        _check(lib.vosti_decay_scan(
+            p, splits, ctypes.c_int64(stride), tokens, *common, _p(decay), ctypes.c_float(key_scale), _p(freq), half,
+            _p(ctx.positions), *slots, ctx.num_requests, DECAY_SHORT if chunked else 0, _p(out), 1 if dtype == torch.float32 else 0,
+            _stream()), "decay_scan")
+    return out
+
+
+def decay_out(o: torch.Tensor, proj, offset: int, *, heads: int, dv: int, eps: float, weight: Optional[torch.Tensor], gate_silu: bool,
+              out_dtype: torch.dtype) -> torch.Tensor:
+    """o [tokens, heads * dv] float32 divided by its root mean square (every head by its own, or with `weight` [heads * dv]
+    all heads together, times the weight) and multiplied by SiLU or sigmoid of the columns from `offset` of `proj`."""
+    p, _, splits = _splits_of(proj)
+    _contig(o, weight)
+    tokens, stride = proj.shape
+    y = torch.empty(o.shape, dtype=out_dtype, device=o.device)
+    _check(library().vosti_decay_out(
+        _p(o), p, splits if isinstance(proj, PartialSum) else 0, ctypes.c_int64(stride), offset, tokens, heads, dv,
+        int(weight is not None), _p(weight), 0 if weight is None else _is_f32(weight), ctypes.c_float(eps), int(gate_silu), _p(y),
+        _is_f32(y), _stream()), "decay_out")
+    return y
+
+
 # ---------------------------------------------------------------- mixture of experts
-def moe_route(logits: torch.Tensor, top: int, *, over_all: bool = False, scale: float = 1.0):
+def moe_route(logits: torch.Tensor, top: int, *, over_all: int = 0, scale: float = 1.0):
     """The `top` largest of each row of float32 router logits: (expert ids int32 [tokens, top],
     their weights float32 [tokens, top], the same weights as a dense [tokens, experts]). The
     weights are the softmax over the chosen logits, or with `over_all` the chosen experts' shares
-    of a softmax over all experts divided by their sum (+ 1e-20); both times `scale`."""
+    of a softmax over all experts divided by their sum (+ 1e-20), or with `over_all` 2 not divided; each times
+    `scale`."""
     if logits.dtype != torch.float32:
         raise KernelError("moe_route: router logits are float32")
     _contig(logits)
@@ -1571,7 +1810,7 @@ def moe_route(logits: torch.Tensor, top: int, *, over_all: bool = False, scale: 
     return chosen, weights, dense
 
 
-def moe_router(x: torch.Tensor, router: torch.Tensor, top: int, *, over_all: bool = False, scale: float = 1.0,
+def moe_router(x: torch.Tensor, router: torch.Tensor, top: int, *, over_all: int = 0, scale: float = 1.0,
                want_logits: bool = False):
     """The router's product x @ router.T (float32 arithmetic, router float32 [experts, k]) and
     `moe_route` of it in one kernel: (chosen, weights, dense), and the logits too if asked for."""
@@ -1623,7 +1862,7 @@ def moe_router_scored(x: torch.Tensor, router: torch.Tensor, top: int, *, identi
 
 def _table_args(ids: torch.Tensor, table: torch.Tensor):
     _contig(ids, table)
-    if ids.dtype != torch.int32 or table.dtype != torch.int32 or table.dim() != 2:
+    if (ids is not None and ids.dtype != torch.int32) or table.dtype != torch.int32 or table.dim() != 2:
         raise KernelError("moe: token ids and the table [vocab, top] are int32")
     return _p(ids), _p(table), table.shape[0], table.shape[1], ctypes.c_float(1.0 / table.shape[1])
 
@@ -1643,14 +1882,14 @@ def moe_table(ids: torch.Tensor, table: torch.Tensor, experts: int, want_dense: 
 MOE_DISPATCH_PAIRS = 16384       # (token, pick) pairs up to which one kernel sorts and gathers (beyond, three kernels)
 
 
-def moe_dispatch(ids: torch.Tensor, table: torch.Tensor, experts: int, x: torch.Tensor, status: torch.Tensor):
-    """Every token's row once per expert its id is assigned to, sorted by expert: (rows [tokens * top, width], offsets
+def moe_dispatch(ids: Optional[torch.Tensor], table: torch.Tensor, experts: int, x: torch.Tensor, status: torch.Tensor):
+    """Every token's row once per expert its id is assigned to (ids None: `table` is a router's choice, a row per token), sorted by expert: (rows [tokens * top, width], offsets
     int32 [experts + 1] of the experts' runs, where int32 [tokens, top] the sorted place of every pair)."""
     args = _table_args(ids, table)
     _contig(x)
-    tokens, top = ids.shape[0], table.shape[1]
+    tokens, top = (table if ids is None else ids).shape[0], table.shape[1]
     if tokens * top > MOE_DISPATCH_PAIRS:
-        chosen, _, _ = moe_table(ids, table, experts)
+        chosen = table if ids is None else moe_table(ids, table, experts)[0]
         offsets, rows, where = moe_group(chosen, experts)
         return gather_rows(x, rows, status), offsets, where
     gathered = torch.empty((tokens * top, x.shape[1]), dtype=x.dtype, device=x.device)

@@ -9,12 +9,13 @@ from .feed_forward import ExpertMixture, SwiGLU
 from .sink_attention import SinkAttention
 from .gated_delta import GatedDeltaRule
 from .general_delta import GeneralDeltaRule
+from .decay_attention import DecayAttention
 from .latent_attention import LatentAttention
 from .selective_scan import SelectiveScan
 from .token_input import GatedTokenInput
 from .branches import BranchMixer
 from .reentry import ConcatReentry
-from .block import GatedStreamBlock, ParallelBlock, PostNormStreamBlock, PreNormBlock, SandwichStreamBlock, StreamPreNormBlock, build_block
+from .block import GatedStreamBlock, OutNormStreamBlock, ParallelBlock, PostNormStreamBlock, PreNormBlock, SandwichStreamBlock, StreamPreNormBlock, build_block
 from .embedding import PairHashEmbedding, TableEmbedding
 from .head import LinearHead
 
@@ -24,5 +25,5 @@ __all__ = [
     "register_part", "register_step_layout", "unregister_part", "linear", "RMSNorm", "RotaryEncoding", "Attention",
     "SwiGLU", "PreNormBlock", "build_block", "build_reentry", "DynamicTanh", "ExpertMixture", "SinkAttention",
     "GatedDeltaRule", "BranchMixer", "ConcatReentry", "ParallelBlock", "StreamRMSNorm", "GeneralDeltaRule",
-    "GatedTokenInput", "StreamPreNormBlock", "LayerNormStream", "LatentAttention", "SelectiveScan", "SandwichStreamBlock", "PostNormStreamBlock", "GatedStreamBlock", "PairHashEmbedding", "TokenInput", "build_token_input",
+    "GatedTokenInput", "StreamPreNormBlock", "LayerNormStream", "LatentAttention", "SelectiveScan", "SandwichStreamBlock", "PostNormStreamBlock", "GatedStreamBlock", "OutNormStreamBlock", "DecayAttention", "PairHashEmbedding", "TokenInput", "build_token_input",
 ]

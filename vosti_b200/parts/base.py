@@ -39,12 +39,14 @@ from ..weights.loader import WeightSpec
 class PagedCacheSpec:
     """Per-token cache of a mixer: `entries` tensors (keys and values: 2), each
     [tokens, heads, width] per token; `window` > 0 means only the last `window`
-    tokens are ever read again, so older pages may be given back."""
+    tokens, and a request's first `keep_first`, are ever read again, so the pages
+    between them may be given back."""
 
     entries: int
     heads: int
     width: int
     window: int = 0
+    keep_first: int = 0
     widths: Tuple[int, ...] = ()      # width of every entry where they differ (else `width` for all)
 
     def entry_widths(self) -> Tuple[int, ...]:

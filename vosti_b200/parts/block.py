@@ -306,6 +306,18 @@ class SandwichStreamBlock(StreamPreNormBlock):
 register_part("arrangement", "sandwich_stream", SandwichStreamBlock, replace=True)
 
 
+def stream_pair(ctx, hidden) -> "ops.StreamPair":
+    """The float32 stream and its rounding: what the block before handed on, or the embedding's rows, which start the
+    stream (float32 rows as they are, others widened)."""
+    if isinstance(hidden, ops.StreamPair):
+        return hidden
+    hidden = ops.materialize(hidden)
+    stream = hidden if hidden.dtype == torch.float32 else ops.stream_sum(None, hidden)
+    rounded = stream if ctx.dtype == torch.float32 else (
+        hidden if hidden.dtype == ctx.dtype else ops.stream_sum(stream, None, out_dtype=ctx.dtype))
+    return ops.StreamPair(rounded, stream)
+
+
 class PostNormStreamBlock(StreamPreNormBlock):
     """'post_norm_stream': the norm comes after the sum, over a float32 residual stream,
 
@@ -348,15 +360,7 @@ class PostNormStreamBlock(StreamPreNormBlock):
     def forward(self, ctx, hidden, residual, cache, writes_cache=True):
         if residual is not None:
             raise ConfigError("post_norm_stream block: the block before it left a residual; it follows blocks of its own kind")
-        if isinstance(hidden, ops.StreamPair):
-            pair = hidden
-        else:
-            # the embedding's rows start the stream: float32 rows as they are, others widened
-            hidden = ops.materialize(hidden)
-            stream = hidden if hidden.dtype == torch.float32 else ops.stream_sum(None, hidden)
-            rounded = stream if ctx.dtype == torch.float32 else (
-                hidden if hidden.dtype == ctx.dtype else ops.stream_sum(stream, None, out_dtype=ctx.dtype))
-            pair = ops.StreamPair(rounded, stream)
+        pair = stream_pair(ctx, hidden)
         pair = self._after(ctx, self.input_norm, pair, self.mixer.forward(ctx, pair.rounded, cache, writes_cache))
         if self.feed_forward is not None:
             pair = self._after(ctx, self.post_norm, pair, self.feed_forward.forward(ctx, pair.rounded))
@@ -464,3 +468,78 @@ class GatedStreamBlock(StreamPreNormBlock):
 
 
 register_part("arrangement", "gated_pre_norm_stream", GatedStreamBlock, replace=True)
+
+
+class OutNormStreamBlock(StreamPreNormBlock):
+    """'out_norm_stream': norms on the sublayers' outputs only, over a float32 residual stream, and an optional
+    learned scale on what joins the stream,
+
+        x <- x + s1 * norm1(mixer(x));   x <- x + s2 * norm2(ff(x))
+
+    The sublayers read x itself, rounded to the serving type. `LayerSpec.norm` is a root-mean-square norm over the
+    stream (`rms_stream`); with `LayerSpec.layer_scale` the vectors s1, s2 exist. One kernel per sublayer
+    boundary sums the sublayer's unsummed product (or its experts' rows, or the mean of its two branches), adds the
+    product's bias (the feed-forward's `out_bias`), norms, scales, adds, and writes the stream and its rounding
+    (`ops.out_norm_stream`); a block hands the next one both (`ops.StreamPair`) and no residual.
+
+    Checkpoint names: `LayerSpec.names` maps the roles "mixer_out_norm", "ff_out_norm", "mixer", "feed_forward",
+    "mixer_scale", "ff_scale" to name fragments; a norm's `weight` and a scale are called by the fragment itself,
+    every other tensor `<fragment>.<key>`. Of a layer without a feed-forward a checkpoint may carry its norm
+    and scale all the same."""
+
+    def __init__(self, spec: LayerSpec, hidden_size: int):
+        super().__init__(spec, hidden_size)
+        if spec.token_input is not None or spec.out_norm is not None or spec.input_conv:
+            raise ConfigError("out_norm_stream block: it takes no token input, second norm or input convolution")
+        self.width, self.scaled = hidden_size, bool(spec.layer_scale)
+        self.mixer_out_norm, self.ff_out_norm = self.input_norm, build_norm(spec.norm, hidden_size)
+        for norm in (self.mixer_out_norm, self.ff_out_norm):
+            if not hasattr(norm, "offset") or getattr(norm, "scalar", False):
+                raise ConfigError("out_norm_stream block: the norm must be a root-mean-square norm over the stream with a weight vector (rms_stream)")
+        self.mixer_scale = self.ff_scale = None
+
+    def _children(self):
+        n = self.spec.name_of
+        yield n("mixer"), self.mixer
+        yield n("mixer_out_norm"), self.mixer_out_norm
+        if self.feed_forward is not None:
+            yield n("feed_forward"), self.feed_forward
+            yield n("ff_out_norm"), self.ff_out_norm
+
+    def _scales(self):
+        n = self.spec.name_of
+        if self.scaled:
+            yield n("mixer_scale"), "mixer_scale", False
+            yield n("ff_scale"), "ff_scale", self.feed_forward is None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        specs = super().weight_specs()
+        for name, _, unused in self._scales():
+            specs[name] = WeightSpec((self.width,), init="norm", std=0.1, optional=unused)
+        if self.feed_forward is None:
+            n = self.spec.name_of("ff_out_norm")
+            for key, w in self.ff_out_norm.weight_specs().items():
+                specs[n if key == "weight" else f"{n}.{key}"] = dataclasses.replace(w, optional=True)
+        return specs
+
+    def load(self, tensors, dtype):
+        super().load(tensors, dtype)
+        for name, attribute, unused in self._scales():
+            setattr(self, attribute, None if unused else tensors[name])
+
+    def _join(self, ctx, pair, y, norm, scale, bias=None):
+        return ops.out_norm_stream(pair, y, norm.weight, norm.eps, ctx.dtype, ctx.status, offset=norm.offset, scale=scale, bias=bias)
+
+    def forward(self, ctx, hidden, residual, cache, writes_cache=True):
+        if residual is not None:
+            raise ConfigError("out_norm_stream block: the block before it left a residual; it follows blocks of its own kind")
+        pair = stream_pair(ctx, hidden)
+        pair = self._join(ctx, pair, self.mixer.forward(ctx, pair.rounded, cache, writes_cache), self.mixer_out_norm, self.mixer_scale)
+        if self.feed_forward is not None:
+            out = self.feed_forward.forward(ctx, pair.rounded)
+            bias = getattr(self.feed_forward, "out_bias", None) if getattr(self.feed_forward, "partial_out", False) else None
+            pair = self._join(ctx, pair, out, self.ff_out_norm, self.ff_scale, bias)
+        return pair, None
+
+
+register_part("arrangement", "out_norm_stream", OutNormStreamBlock, replace=True)

@@ -8,6 +8,9 @@ layer run has one paged cache and one state. The result is float32.
 
 `merge` = "sum" with `scales` (one constant per branch) gives sum_b scales[b] * branch_b instead:
 no norm, no weight vectors.
+
+`defer` (default false, two branches): the mean is left to the kernel that reads it next (`ops.BranchMean`),
+and the branches' output products may stay unsummed until then.
 """
 from __future__ import annotations
 
@@ -37,6 +40,12 @@ class BranchMixer(Mixer):
         if sum(b.cache_spec() is not None for _, b in self.branches) > 1 or \
                 sum(b.state_spec() is not None for _, b in self.branches) > 1:
             raise ConfigError("branches: at most one branch may keep pages and at most one a state slot")
+        self.defer = bool(spec.get("defer", False))
+        if self.defer:
+            if self.merge != "unit_rms_mean" or len(self.branches) != 2:
+                raise ConfigError("branches: the mean of two branches can be deferred, nothing else")
+            for i, (_, branch) in enumerate(self.branches):
+                branch.out_scratch = f"split_k_branch{i}"       # two products stay unsummed at the same time
         self.capture_safe = all(getattr(b, "capture_safe", True) for _, b in self.branches)
         self.out_weights = []
 
@@ -76,6 +85,8 @@ class BranchMixer(Mixer):
         outs = [branch.forward(ctx, x, cache, writes_cache) for _, branch in self.branches]
         if self.merge == "sum":
             return ops.branch_sum(outs, self.scales)
+        if self.defer:
+            return ops.BranchMean(outs, self.out_weights, self.eps)
         return ops.branch_merge(outs, self.out_weights, self.eps)
 
 

@@ -66,7 +66,9 @@ class PairHashEmbedding(Embedding):
     `side` [vocab, side_width] of per-token vectors for sublayers that read the token ids again
     (parts of role "token_input"), which this part publishes in `ctx.extras["token_table"]`
     beside the step's token ids in `ctx.extras["token_ids"]`; `names`: checkpoint names of the
-    tensors `pairs` and `side` where they are not `<embedding>.pairs` / `<embedding>.side`."""
+    tensors `pairs` and `side` where they are not `<embedding>.pairs` / `<embedding>.side`; `rounded` (default
+    false): in bfloat16 serving the same kernel writes the rows' rounding beside them and the part returns both,
+    an `ops.StreamPair`."""
 
     def __init__(self, spec: PartSpec, hidden_size: int, vocab_size: int):
         super().__init__(spec, hidden_size, vocab_size)
@@ -74,6 +76,7 @@ class PairHashEmbedding(Embedding):
         self.side_width = int(spec.get("side_width", 0) or 0)
         if self.buckets <= 0 or not 0 <= self.mul_prev < 1 << 31 or not 0 <= self.mul_cur < 1 << 31:
             raise ConfigError("pair_hash: buckets must be positive and the multipliers in [0, 2^31)")
+        self.rounded = bool(spec.get("rounded", False))
         self.weight = self.pairs = self.side = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -98,7 +101,8 @@ class PairHashEmbedding(Embedding):
         if cache is None or cache.state is None:
             raise ConfigError("pair_hash: the embedding needs its state slots (the token before a portion)")
         rows, ids = ops.pair_embedding(tokens, self.weight, self.pairs, cache.state.view(-1), ctx, buckets=self.buckets,
-                                       mul_prev=self.mul_prev, mul_cur=self.mul_cur, feedback=feedback)
+                                       mul_prev=self.mul_prev, mul_cur=self.mul_cur, feedback=feedback,
+                                       rounded=self.rounded and ctx.dtype == torch.bfloat16)
         ctx.extras["token_ids"] = ids
         if self.side is not None:
             ctx.extras["token_table"] = self.side

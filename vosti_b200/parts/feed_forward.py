@@ -8,7 +8,10 @@ gate * sigmoid(gate) * up in float32 (kernels/triton_kernels/silu_mul.py:66-87).
 Parameters besides `intermediate_size`: `tensor_names`, the checkpoint's names of the gate, up
 and down matrices (default: Qwen3's), `float32_out`, for models whose residual stream is
 float32: the down projection is then not rounded to the serving type, and `activation`: "silu"
-(the default), "relu" or "relu2" (the square of relu) on the gate.
+(the default), "relu" or "relu2" (the square of relu) on the gate, or with `bias` "clamped": g sigmoid(`sigmoid_scale` g)
+(u + 1) of g = min(gate x + bg, `limit`) and u = up x + bu clamped to [-limit, limit]. `bias`: all three projections have
+biases (the tensor's name with ".b"); the down projection's joins in the kernel that reads the product next
+(an arrangement that asks for `out_bias`), the others in the activation.
 
 `ExpertMixture` is the same feed-forward as `experts` small ones, of which each token uses
 the `top` with the largest router logits, weighted by the softmax over the chosen logits only.
@@ -68,25 +71,63 @@ class SwiGLU(FeedForward):
         self.float32_out = bool(spec.get("float32_out", False))
         self.activation = str(spec.get("activation", "silu") or "silu")
         self.partial_out = bool(spec.get("partial_out", False))   # with float32_out: the next kernel sums the down product's K splits
+        self.has_bias, self.limit, self.sigmoid_scale = bool(spec.get("bias", False)), 0.0, 0.0
+        self.bias_gate_up = self.out_bias = None
+        if self.has_bias != (self.activation == "clamped"):
+            raise ConfigError("swiglu: the clamped activation and biases go together")
+        if self.has_bias:
+            self.limit, self.sigmoid_scale = float(spec["limit"]), float(spec["sigmoid_scale"])
+            if not self.limit > 0:
+                raise ConfigError("swiglu: the clamped activation's limit must be positive")
         if self.activation not in ops.GLU_ACTIVATIONS:
             raise ConfigError(f"swiglu: activation is one of {sorted(ops.GLU_ACTIVATIONS)}")
         self.w_gate_up = self.w_down = None
-        self.fused = False
+        self.fused = self.fused_packed = False
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         h, i = self.hidden_size, self.inter
         gate, up, down = self.names
-        return {gate: WeightSpec((i, h)), up: WeightSpec((i, h)), down: WeightSpec((h, i))}
+        specs = {gate: WeightSpec((i, h)), up: WeightSpec((i, h)), down: WeightSpec((h, i))}
+        if self.has_bias:
+            specs.update({gate + ".b": WeightSpec((i,), std=0.1), up + ".b": WeightSpec((i,), std=0.1), down + ".b": WeightSpec((h,), std=0.1)})
+        return specs
 
     def load(self, tensors, dtype):
         gate, up, down = self.names
         self.w_down = prepare_weight(tensors[down], dtype)
+        if self.has_bias:
+            pair, biases = (tensors[gate], tensors[up]), (tensors[gate + ".b"].float(), tensors[up + ".b"].float())
+            # blocks of 16 gate and 16 up rows where the tensor-core product may apply the activation itself
+            self.fused = dtype == torch.bfloat16 and self.inter % 16 == 0 and all(uses_tensor_cores(dtype, w) for w in pair)
+            if self.fused:
+                self.w_gate_up = prepare_weight(interleave_gate_up(*pair), dtype)
+                self.bias_gate_up = interleave_gate_up(*(b.view(-1, 1) for b in biases)).view(-1).contiguous()
+                self.fused_packed = isinstance(self.w_gate_up, ops.PackedWeight)
+            else:
+                common = torch.float32 if torch.float32 in (pair[0].dtype, pair[1].dtype) else pair[0].dtype
+                self.w_gate_up = prepare_weight(torch.cat([w.to(common) for w in pair], dim=0).contiguous(), dtype)
+                self.bias_gate_up = torch.cat(biases).contiguous()
+            self.out_bias = tensors[down + ".b"].float().contiguous()
+            return
         self.w_gate_up, self.fused = stack_gate_up(tensors[gate], tensors[up], dtype, self.activation)
 
     def first_weight(self):
         return self.w_gate_up
 
+    def _biased_activation(self, ctx, x):
+        x = ops.materialize(x)
+        if self.fused and self.fused_packed and x.shape[0] > ops.CLAMPED_EPILOGUE_FROM:
+            return ops.gemm_tc_clamped(x, self.w_gate_up, self.bias_gate_up, ctx.status, limit=self.limit, sigmoid_scale=self.sigmoid_scale)
+        product = linear(ctx, x, self.w_gate_up, out_dtype=torch.float32, allow_partial=True)
+        return ops.glu_bias(product, self.bias_gate_up, x.dtype, block=16 if self.fused else 0, limit=self.limit,
+                            sigmoid_scale=self.sigmoid_scale)
+
     def forward(self, ctx, x):
+        if self.has_bias:
+            y = linear(ctx, self._biased_activation(ctx, x), self.w_down, out_dtype=torch.float32, allow_partial=self.partial_out)
+            # an arrangement that leaves the product unsummed adds `out_bias` itself
+            y = y if self.partial_out else ops.affine_rows(y, bias=self.out_bias)
+            return y if self.float32_out else ops.stream_sum(None, ops.materialize(y), out_dtype=x.dtype)
         mlp = gated_activation(ctx, x, self.w_gate_up, self.fused, self.activation)
         if self.float32_out:
             return linear(ctx, mlp, self.w_down, out_dtype=torch.float32, allow_partial=self.partial_out)
@@ -101,7 +142,8 @@ class ExpertMixture(FeedForward):
     `router` [experts, hidden] and `e<i>.gate`, `e<i>.up`, `e<i>.down`. Further parameters:
     `gated` (default true; false: experts are down(gelu(up(x))), no `gate` tensors), `route`
     ("top_softmax", the default: softmax over the chosen logits; "softmax_renorm": softmax over
-    all experts, the chosen scores divided by their sum + 1e-20) and `scale`, a constant on the
+    all experts, the chosen scores divided by their sum + 1e-20; "softmax": the same, not divided; in bfloat16
+    serving it takes the sorted way described for "table" below, the router's choice in the table's place) and `scale`, a constant on the
     weights (default 1).
 
     With `route` "scored" (experts without a gate only): the router has experts + `identity` rows;
@@ -174,8 +216,8 @@ class ExpertMixture(FeedForward):
         self.correction = None
         if self.experts <= 0 or not 0 < self.top <= self.experts + self.identity or self.inter <= 0:
             raise ConfigError("moe: experts, top (at most experts) and intermediate_size must be positive")
-        if self.route not in ("top_softmax", "softmax_renorm", "scored", "table") or self.scale != self.scale:
-            raise ConfigError("moe: route is 'top_softmax', 'softmax_renorm', 'scored' or 'table' and scale a number")
+        if self.route not in ("top_softmax", "softmax_renorm", "softmax", "scored", "table") or self.scale != self.scale:
+            raise ConfigError("moe: route is 'top_softmax', 'softmax_renorm', 'softmax', 'scored' or 'table' and scale a number")
         if self.route == "table" and (not self.gated or self.scale != 1.0 or self.vocab <= 0):
             raise ConfigError("moe: route 'table' takes gated experts, no scale, and the size of the vocabulary")
         if self.route != "scored" and (self.identity or self.has_correction or self.groups != 1 or self.shared
@@ -225,6 +267,8 @@ class ExpertMixture(FeedForward):
                 raise ConfigError("moe: a row of the table names an expert twice")
             if self.top < self.experts and self._load_grouped(tensors, dtype):
                 return
+        if self.route == "softmax" and self.gated and self.top < self.experts and self._load_grouped(tensors, dtype):
+            return
         up = torch.cat([tensors[f"e{e}.up"] for e in range(self.experts)], dim=0)
         if self.gated:
             gate = torch.cat([tensors[f"e{e}.gate"] for e in range(self.experts)], dim=0)
@@ -332,18 +376,22 @@ class ExpertMixture(FeedForward):
                 y[lo:hi].copy_(linear(ctx, act, down, out_dtype=torch.float32))
         return ops.moe_combine(y, where, weights)
 
+    def _sorted_products(self, ctx, x, ids, table, weights=None):
+        """The experts over their own rows: `table` by token id, or (ids None) a router's choice with its weights."""
+        gathered, offsets, where = ops.moe_dispatch(ids, table, self.experts, x, ctx.status)
+        act = ops.gemm_tc_grouped(gathered, self.grouped[0], offsets, x.shape[0], ctx.status, activation=self.gate_activation,
+                                  glu=self.glu)
+        y = ops.gemm_tc_grouped(act, self.grouped[1], offsets, x.shape[0], ctx.status, out_dtype=torch.float32,
+                                allow_partial=self.partial_out)
+        y = ops.PickedSum(y, where, 1.0 / self.top, weights)
+        return y if self.partial_out else y.materialize()
+
     def _forward_table(self, ctx, x):
         ids = ctx.extras.get("token_ids")
         if ids is None:
             raise ConfigError("moe: route 'table' needs the step's token ids, which the model's embedding does not publish")
         if self.grouped is not None:
-            gathered, offsets, where = ops.moe_dispatch(ids, self.table, self.experts, x, ctx.status)
-            act = ops.gemm_tc_grouped(gathered, self.grouped[0], offsets, x.shape[0], ctx.status, activation=self.gate_activation,
-                                      glu=self.glu)
-            y = ops.gemm_tc_grouped(act, self.grouped[1], offsets, x.shape[0], ctx.status, out_dtype=torch.float32,
-                                    allow_partial=self.partial_out)
-            y = ops.PickedSum(y, where, 1.0 / self.top)
-            y = y if self.partial_out else y.materialize()
+            y = self._sorted_products(ctx, x, ids, self.table)
         elif (self.per_expert and x.shape[0] >= self.GROUPED_FROM and not getattr(ctx, "all_decode", True)
                 and not torch.cuda.is_current_stream_capturing()):
             chosen, weights, _ = ops.moe_table(ids, self.table, self.experts)
@@ -359,7 +407,11 @@ class ExpertMixture(FeedForward):
             return self._forward_scored(ctx, x)
         if self.route == "table":
             return self._forward_table(ctx, x)
-        chosen, weights, dense = ops.moe_router(x, self.router, self.top, over_all=self.route == "softmax_renorm", scale=self.scale)
+        over_all = {"softmax_renorm": 1, "softmax": 2}.get(self.route, 0)
+        chosen, weights, dense = ops.moe_router(x, self.router, self.top, over_all=over_all, scale=self.scale)
+        if self.grouped is not None:
+            y = self._sorted_products(ctx, x, None, chosen, weights)
+            return y if self.float32_out else ops.stream_sum(None, ops.materialize(y), out_dtype=x.dtype)
         if (self.per_expert and x.shape[0] >= self.GROUPED_FROM and not getattr(ctx, "all_decode", True)
                 and not torch.cuda.is_current_stream_capturing()):
             out = self._grouped(ctx, x, chosen, weights)

@@ -37,7 +37,16 @@ of them optional and a parameter of the spec:
 * `partial_out`: the output projection may come back as unsummed K splits (`ops.PartialSum`) for an
   arrangement whose next kernel adds them (the norm after the sum);
 * `out_gate`: the concatenated heads are multiplied element by element by sigmoid(W_g x) (`g`), a
-  product of the mixer's own input, before the output projection.
+  product of the mixer's own input, before the output projection; `head_gate`: the same with one
+  number a head (`g` [heads, hidden]);
+* `slope_range` r > 0: a penalty linear in the distance, slope_h * (i - j) with
+  slope_h = 2^(-r (h + 1) / heads), is taken off the scaled scores;
+* `keep_first`, with a window: every query also sees the sequence's first `keep_first` tokens, at their
+  true positions;
+* `value_is_key`: the values are the projected keys (bias included) before any norm; no `v` tensors;
+* `joint_norm_eps`: queries and keys are divided by the root mean square of their whole projection, all heads
+  at once, and multiplied by weights of that size (`q.norm` [heads * head_dim], `k.norm`); goes with
+  `value_is_key` and without a rotation; `qk_bias`: `q.b` and `k.b` exist.
 
 In bfloat16 serving a layer with two maps whose wider head width (of key and value) is one the
 tensor-core attention kernels take runs every map as a head of its own on those kernels
@@ -46,9 +55,9 @@ the q projection's rows reordered so that the query heads of a key head stand to
 maps are combined by a kernel after them. Such a layer's cache holds 2 * maps * kv heads entries
 of that width a token.
 
-With any of these five the projection (q | k | v | g as one product) stays float32 and one kernel
+With the ones from `qkv_bias` to `out_gate` the projection (q | k | v | g as one product) stays float32 and one kernel
 (`ops.qkv_heads`) adds the bias, norms, rotates and stores, rounding once; what follows the softmax is
-the attention kernel's last step (`ops.HeadFinish`).
+the attention kernel's last step (`ops.HeadFinish`). With joint norms `ops.qk_joint` takes the other kernel's place.
 
 Other parameters: num_heads, num_kv_heads (query head h reads kv head h // (heads / kv_heads)),
 head_dim, v_head_dim, scale, window (0: every earlier key). Keys and values live in the paged
@@ -109,6 +118,25 @@ class SinkAttention(Mixer):
         self.out_gate = bool(spec.get("out_gate", False))
         self.lam = 0.0
         self.expanded = 0
+        self.out_scratch = "split_k"
+        self.keep_first = int(spec.get("keep_first", 0) or 0) if self.window else 0
+        self.slope_range = float(spec.get("slope_range", 0.0) or 0.0)
+        self.slopes = None
+        self.head_gate = bool(spec.get("head_gate", False))
+        self.value_is_key = bool(spec.get("value_is_key", False))
+        eps = spec.get("joint_norm_eps")
+        self.joint_norm_eps = None if eps is None else float(eps)
+        self.qk_bias = bool(spec.get("qk_bias", False))
+        if (self.joint_norm_eps is not None) != self.value_is_key or (self.value_is_key and self.dv != self.dk):
+            raise ConfigError("sink_attention: joint norms and values that are the keys go together, with one head width")
+        if (self.qk_bias or self.head_gate) and not self.value_is_key:
+            raise ConfigError("sink_attention: qk_bias and head_gate go with value_is_key")
+        if self.value_is_key and (self.qkv_bias or self.head_norm_eps is not None or self.maps > 1 or self.out_gate
+                                  or spec.get("position") is not None or self.temp_coef or self.value_mix is not None):
+            raise ConfigError("sink_attention: value_is_key takes no rotation, temperature, per-head norms, maps, value mixing or "
+                              "element gate")
+        if self.keep_first < 0 or self.slope_range < 0 or (self.slope_range and (self.bias_rows or self.softcap or self.maps > 1)):
+            raise ConfigError("sink_attention: keep_first and slope_range are not negative; slopes take no bias table, soft cap or maps")
         self.partial_out = bool(spec.get("partial_out", False))     # the block's next kernel sums the output product's K splits
         self.b_qkv = self.q_norm = self.k_norm = None
         if self.maps not in (1, 2):
@@ -139,6 +167,16 @@ class SinkAttention(Mixer):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         h, nq, nkv, dk, dv = self.hidden_size, self.nq, self.nkv, self.dk, self.dv
+        if self.value_is_key:
+            specs = {"q": WeightSpec((nq * dk, h)), "k": WeightSpec((nkv * dk, h)), "o": WeightSpec((h, nq * dv)),
+                     "q.norm": WeightSpec((nq * dk,), init="norm", std=0.1), "k.norm": WeightSpec((nkv * dk,), init="norm", std=0.1)}
+            if self.qk_bias:
+                specs.update({"q.b": WeightSpec((nq * dk,), std=0.1), "k.b": WeightSpec((nkv * dk,), std=0.1)})
+            if self.head_gate:
+                specs["g"] = WeightSpec((nq, h))
+            if self.has_sink:
+                specs["sink"] = WeightSpec((nq,), std=1.0)
+            return specs
         m = self.maps
         specs = {"q": WeightSpec((nq * m * dk, h)), "k": WeightSpec((nkv * m * dk, h)), "v": WeightSpec((nkv * dv, h)),
                  "o": WeightSpec((h, nq * dv))}
@@ -159,7 +197,19 @@ class SinkAttention(Mixer):
             specs["vmix"] = WeightSpec((), std=0.3, optional=self.value_mix == "source")
         return specs
 
+    def _load_joint(self, tensors, dtype):
+        parts = [tensors["q"], tensors["k"]] + ([tensors["g"]] if self.head_gate else [])
+        common = torch.float32 if any(p.dtype == torch.float32 for p in parts) else parts[0].dtype
+        self.w_qkv = prepare_weight(torch.cat([p.to(common) for p in parts], dim=0).contiguous(), dtype)
+        self.w_o = prepare_weight(tensors["o"], dtype)
+        self.q_norm, self.k_norm = tensors["q.norm"].float().contiguous(), tensors["k.norm"].float().contiguous()
+        if self.qk_bias:
+            self.b_qkv = torch.cat([tensors["q.b"].float(), tensors["k.b"].float()]).contiguous()
+        self.sink = tensors["sink"].float().contiguous() if self.has_sink else None
+
     def load(self, tensors, dtype):
+        if self.value_is_key:
+            return self._load_joint(tensors, dtype)
         wide = max(self.dk, self.dv)
         self.expanded = wide if (self.maps > 1 and ops.attention_heads_supported(dtype, wide, self.nq // self.nkv)
                                  and not self.has_sink and self.sink_value is None and not self.bias_rows) else 0
@@ -201,6 +251,9 @@ class SinkAttention(Mixer):
             self.bias_table = (rel[index].T * LOG2E).contiguous()
 
     def setup(self, device, dtype):
+        if self.slope_range:
+            slopes = [2.0 ** (-self.slope_range * (h + 1) / self.nq) * LOG2E for h in range(self.nq)]
+            self.slopes = torch.tensor(slopes, dtype=torch.float64).to(torch.float32).to(device)      # base-2 units, like the kernels' scores
         if self.rotation is not None:
             self.freq = self.rotation.frequencies().to(device=device, dtype=torch.float32).contiguous()
             self.magnitude = float(self.rotation.magnitude()) if hasattr(self.rotation, "magnitude") else 1.0
@@ -212,9 +265,9 @@ class SinkAttention(Mixer):
 
     def cache_spec(self) -> PagedCacheSpec:
         if getattr(self, "expanded", 0):
-            return PagedCacheSpec(entries=2, heads=self.nkv * self.maps, width=self.expanded, window=self.window)
+            return PagedCacheSpec(entries=2, heads=self.nkv * self.maps, width=self.expanded, window=self.window, keep_first=self.keep_first)
         # with maps, a kv head's entry holds its keys of all maps side by side
-        return PagedCacheSpec(entries=2, heads=self.nkv, width=self.maps * self.dk, window=self.window,
+        return PagedCacheSpec(entries=2, heads=self.nkv, width=self.maps * self.dk, window=self.window, keep_first=self.keep_first,
                               widths=(self.maps * self.dk, self.dv))
 
     def _forward_by_heads(self, ctx, x, cache, writes_cache, group):
@@ -234,21 +287,36 @@ class SinkAttention(Mixer):
         if self.expanded:
             D, m = self.expanded, self.maps
             each = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq * m, nkv=self.nkv * m, dk=D, dv=D,
-                                      scale=self.scale, window=self.window, bias=None, sink=None, chunk=self.chunk, softcap=self.softcap)
+                                      scale=self.scale, window=self.window, bias=None, sink=None, chunk=self.chunk, softcap=self.softcap,
+                                      keep=self.keep_first)
             finish = ops.HeadFinish(lam=self.lam, unit_norm=True, eps=self.out_norm_eps, out_scale=1.0 - self.diff, gate=gate)
             attn = ops.head_finish(each, finish, nq=self.nq, maps=m, dv=self.dv, in_width=D, pair_group=self.nq // self.nkv)
-            return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out)
+            return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out, scratch=self.out_scratch)
         finish = None
         if self.maps == 2 or self.out_gate:
             finish = ops.HeadFinish(lam=self.lam, unit_norm=self.maps == 2, eps=self.out_norm_eps, out_scale=1.0 - self.diff,
                                     gate=gate)
         attn = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq, nkv=self.nkv, dk=self.dk, dv=self.dv,
                                   scale=self.scale, window=self.window, bias=self.bias_table, sink=self.sink, chunk=self.chunk, softcap=self.softcap,
-                                  maps=self.maps, finish=finish)
-        return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out)
+                                  maps=self.maps, finish=finish, slopes=self.slopes, keep=self.keep_first)
+        return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out, scratch=self.out_scratch)
+
+    def _forward_joint(self, ctx, x, cache, writes_cache, group):
+        proj = linear(ctx, x, self.w_qkv, out_dtype=torch.float32, allow_partial=True)   # K splits are summed by qk_joint
+        q, gate = ops.qk_joint(proj, cache.k if writes_cache else None, cache.v if writes_cache else None, nq=self.nq, nkv=self.nkv,
+                               dk=self.dk, page_size=group.page_size, slot_mapping=group.slot_mapping, out_dtype=ctx.dtype,
+                               status=ctx.status, q_norm=self.q_norm, k_norm=self.k_norm, eps=self.joint_norm_eps, bias=self.b_qkv,
+                               extra_width=self.nq if self.head_gate else 0)
+        finish = ops.HeadFinish(gate=gate, by_head=True) if self.head_gate else None
+        attn = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq, nkv=self.nkv, dk=self.dk, dv=self.dv, scale=self.scale,
+                                  window=self.window, bias=None, sink=self.sink, chunk=self.chunk, softcap=self.softcap, finish=finish,
+                                  slopes=self.slopes, keep=self.keep_first)
+        return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out, scratch=self.out_scratch)
 
     def forward(self, ctx, x, cache, writes_cache: bool = True):
         group = ctx.group(cache.group)
+        if self.value_is_key:
+            return self._forward_joint(ctx, x, cache, writes_cache, group)
         if self.by_heads:
             return self._forward_by_heads(ctx, x, cache, writes_cache, group)
         qkv = ops.materialize(linear(ctx, x, self.w_qkv))
@@ -265,8 +333,8 @@ class SinkAttention(Mixer):
                           status=ctx.status, freq=self.freq, magnitude=self.magnitude, v_first=v_source, v_mix=self.mix)
         attn = ops.attention_sink(ctx, q, cache.k, cache.v, group, nq=self.nq, nkv=self.nkv, dk=self.dk, dv=self.dv,
                                   scale=self.scale, window=self.window, bias=self.bias_table, sink=self.sink, chunk=self.chunk,
-                                  softcap=self.softcap)
-        return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out)
+                                  softcap=self.softcap, slopes=self.slopes, keep=self.keep_first)
+        return linear(ctx, attn, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out, scratch=self.out_scratch)
 
 
 register_part("mixer", "sink_attention", SinkAttention, replace=True)
