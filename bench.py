@@ -48,6 +48,9 @@ with an input convolution: windowed latent attention, capped windowed attention,
 over the first layer's latents, and capped attention again, clamped experts by token table in every
 layer) beside Beralix, whose attention is closest (at sizes s and m, whose dense feed-forward does the
 work of the two experts a token has), and beside Mugizen's experts (size moe).
+`--design difavik` does the same for the Difavik design (output norms over a float32 stream, windowed attention
+with linear penalties and kept first tokens beside retention, lightning attention, clamped feed-forwards with
+biases or experts by a plain softmax) beside Mugizen at the same sizes (`--design-sizes s,m,moe`).
 """
 from __future__ import annotations
 
@@ -531,8 +534,37 @@ def pubulix_flops(size, tokens):
     return 2.0 * tokens * per_token + 2.0 * V * W + scores
 
 
+def difavik_config(size):
+    """A Difavik config.json of these sizes: parallel layers (windowed attention whose values are its keys, a window
+    of 1,024 and 64 kept tokens, beside retention) and lightning layers in turn, heads of 128 everywhere."""
+    H, G, W = size["heads"], size["kv"], size["width"]
+    if size["moe"]:
+        mlp = dict(kind="moe", expert=dict(ff=size["moe"]["ff"], limit=7.0), router=dict(experts=size["moe"]["experts"], top=size["moe"]["top"]))
+    else:
+        mlp = dict(kind="dense", ff=size["ff"], limit=7.0)
+    decay = [1.0 - 2.0 ** (-5.0 - 6.0 * h / H) for h in range(H)]
+    parallel = dict(type="parallel", mlp=mlp, mixer=dict(
+        left=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=64)),
+        right=dict(heads=H, dim=128, vdim=128, rot=dict(base=10000.0, dims=128), decay=decay)))
+    light = dict(type="lightning", mlp=mlp, mixer=dict(heads=H, dim=128, vdim=128, decay=decay))
+    return dict(architecture="Difavik", vocab=size["vocab"], width=W, norm=dict(eps=1e-5),
+                embedding=dict(bigram=dict(buckets=65521, mul_prev=1000003, mul_cur=31)),
+                layers=[parallel if i % 2 == 0 else light for i in range(size["layers"])])
+
+
+def difavik_flops(size, tokens):
+    """Multiply-add work of one prompt, times two, for `difavik_config(size)`."""
+    W, H, G, L, V, d = size["width"], size["heads"], size["kv"], size["layers"], size["vocab"], 128
+    feed = 3 * W * size["ff"] if not size["moe"] else 3 * W * size["moe"]["ff"] * size["moe"]["top"] + W * size["moe"]["experts"]
+    recurrent, attention = 5 * W * H * d, W * ((H + G) * d + H) + H * d * W
+    per_token = L * (recurrent + feed) + (L - L // 2) * attention
+    pairs = sum(min(t + 1, 1024 + min(max(t - 1023, 0), 64)) for t in range(tokens))
+    scores = (L - L // 2) * H * d * 4.0 * pairs + L * tokens * H * 4.0 * d * d       # attention; 2 passes over a 128 x 128 state
+    return 2.0 * tokens * per_token + 2.0 * V * W + scores
+
+
 def unread_bytes(size, batch):
-    """Weight bytes of experts that a Pubulix decode step of `batch` requests of random tokens does not read."""
+    """Weight bytes of experts that a Pubulix or Difavik decode step of `batch` requests of random tokens does not read."""
     m = pubulix_experts(size)
     idle = (1.0 - m["top"] / m["experts"]) ** batch * m["experts"]
     return size["layers"] * idle * 3 * size["width"] * m["ff"] * 2.0
@@ -546,6 +578,8 @@ def design_flops(size, tokens, design):
         return beralix_flops(size, tokens)
     if design == "nefipel":
         return nefipel_flops(size, tokens)
+    if design == "difavik":
+        return difavik_flops(size, tokens)
     if design == "pubulix":
         return pubulix_flops(size, tokens)
     W, H, G, F, L, V = size["width"], size["heads"], size["kv"], size["ff"], size["layers"], size["vocab"]
@@ -579,6 +613,8 @@ def design_engine(kind, size, max_batch):
         spec = model_spec_from_config(beralix_config(size))
     elif kind == "nefipel":
         spec = model_spec_from_config(nefipel_config(size))
+    elif kind == "difavik":
+        spec = model_spec_from_config(difavik_config(size))
     elif kind == "pubulix":
         spec = model_spec_from_config(pubulix_config(size))
     else:
@@ -620,7 +656,10 @@ def design_one(args, name, kind) -> dict:
         kv_read = run["context"] * kv_bytes
         if kind == "pubulix":                   # windows of 1,024; the first layer's latents are read by two layers
             kv_read = min(run["context"], 1024) * (kv_bytes + 576 * 2 * ((size["layers"] + 1) // 4))
-        step_bytes = weight_bytes + batch * (kv_read + 2 * state_bytes) - (unread_bytes(size, batch) if kind == "pubulix" else 0)
+        if kind == "difavik":                   # a window of 1,024 and 64 kept tokens
+            kv_read = min(run["context"], 1024 + 64) * kv_bytes
+        step_bytes = weight_bytes + batch * (kv_read + 2 * state_bytes) - (unread_bytes(size, batch) if kind == "pubulix" else
+                                                                                        unread_bytes(size, batch) if kind == "difavik" and size["moe"] else 0)
         entry[f"decode_b{batch}"] = {
             "tok_s": round(batch * 1e3 / run["device_ms"], 1), "ms_per_step": round(run["device_ms"], 4),
             "e2e_tok_s": round(batch * 1e3 / run["wall_ms"], 1), "launches_per_step": run["launches"] / args.steps,
@@ -628,12 +667,12 @@ def design_one(args, name, kind) -> dict:
     return entry
 
 
-BESIDE = {"mugizen": "qwen3", "vivesun": "mugizen", "beralix": "mugizen", "nefipel": "qwen3", "pubulix": "beralix"}      # the engine's closest other model
+BESIDE = {"mugizen": "qwen3", "vivesun": "mugizen", "beralix": "mugizen", "nefipel": "qwen3", "pubulix": "beralix", "difavik": "mugizen"}      # the engine's closest other model
 
 
 def design_main(args) -> int:
     """Prefill and decode of a design beside the engine's closest other model (Mugizen beside Qwen3,
-    Vivesun and Beralix beside Mugizen, Pubulix beside Beralix) at equal sizes; one JSON line. Every
+    Vivesun, Beralix and Difavik beside Mugizen, Pubulix beside Beralix) at equal sizes; one JSON line. Every
     model is measured in a process of its own (this program started again with --design-one), so
     that no model's scratch buffers, graphs or allocator state reach the next one's timings."""
     if args.design_one:
@@ -691,7 +730,7 @@ def main() -> int:
                         help="read every step's tokens before the next step is planned (default: the engine's async scheduling)")
     parser.add_argument("--batch-invariant", default="off", choices=["off", "decode", "full"],
                         help="measure with the engine's bitwise-invariance modes (the default run has them off)")
-    parser.add_argument("--design", default="", choices=["", "mugizen", "vivesun", "beralix", "nefipel", "pubulix"],
+    parser.add_argument("--design", default="", choices=["", "mugizen", "vivesun", "beralix", "nefipel", "pubulix", "difavik"],
                         help="measure this design beside the engine's closest other model at equal layer sizes instead of the headline")
     parser.add_argument("--design-sizes", default="s,m,moe", help="which of the sizes s, m, moe (comma-separated)")
     parser.add_argument("--design-one", default="", help=argparse.SUPPRESS)      # size:design, one model in this process

@@ -561,96 +561,121 @@ decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, f
 }
 
 // ------------------------------------------------------------------ norm and gate
-// joint: one root mean square over the whole row, times a weight [width]; else one per head, no weight.
-template <typename T>
+__device__ __forceinline__ float gate_value(float g, int silu) { return silu ? silu_of(g) : 1.f / (1.f + expf(-g)); }
+// V neighbouring gates of token t from column off_g + i on, summed and rounded like `column`.
+template <typename T, int V>
+__device__ __forceinline__ void load_gates(const Projection& p, int64_t t, int i, int silu, float (&g)[V]) {
+  const int64_t at = t * p.stride + p.off_g + i;
+  if (V == 1) {
+    g[0] = gate_value(column<T>(p, t, p.off_g + i), silu);
+    return;
+  }
+  float4 v;
+  if (p.splits == 0 && sizeof(T) == 2) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p.data) + at);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    v = make_float4(a.x, a.y, b.x, b.y);
+  } else {
+    const float* src = reinterpret_cast<const float*>(p.data) + at;
+    v = *reinterpret_cast<const float4*>(src);
+    for (int s = 1; s < p.splits; ++s) {
+      const float4 u = *reinterpret_cast<const float4*>(src + s * p.plane);
+      v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
+    }
+    v = make_float4(rounded_to<T>(v.x), rounded_to<T>(v.y), rounded_to<T>(v.z), rounded_to<T>(v.w));
+  }
+  g[0] = gate_value(v.x, silu);
+  g[V > 1 ? 1 : 0] = gate_value(v.y, silu);
+  g[V > 2 ? 2 : 0] = gate_value(v.z, silu);
+  g[V > 3 ? 3 : 0] = gate_value(v.w, silu);
+}
+template <int V>
+__device__ __forceinline__ void load_row(const float* p, float (&x)[V]) {
+  if (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    x[0] = v.x; x[V > 1 ? 1 : 0] = v.y; x[V > 2 ? 2 : 0] = v.z; x[V > 3 ? 3 : 0] = v.w;
+  } else {
+    x[0] = p[0];
+  }
+}
+template <int V> __device__ __forceinline__ void store_row(float* p, const float (&x)[V]) {
+  if (V == 4) *reinterpret_cast<float4*>(p) = make_float4(x[0], x[V > 1 ? 1 : 0], x[V > 2 ? 2 : 0], x[V > 3 ? 3 : 0]);
+  else p[0] = x[0];
+}
+template <int V> __device__ __forceinline__ void store_row(bf16* p, const float (&x)[V]) {
+  if (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x[0], x[V > 1 ? 1 : 0]), pack_bf16(x[V > 2 ? 2 : 0], x[V > 3 ? 3 : 0]));
+  else p[0] = __float2bfloat16_rn(x[0]);
+}
+
+// One root mean square over the whole row (all heads together), times a weight [width]. A block a token; V elements a
+// thread at a time.
+template <typename T, int V>
 __global__ void __launch_bounds__(1024)
-decay_out_kernel(const float* __restrict__ o, const Projection p, int heads, int dv, int joint, const void* __restrict__ w, int w_f32,
-                 float eps, int gate_silu, T* __restrict__ y) {
+decay_out_joint_kernel(const float* __restrict__ o, const Projection p, int width, const void* __restrict__ w, int w_f32, float eps,
+                       int gate_silu, T* __restrict__ y) {
   __shared__ float scratch[32];
   pdl_wait();
   pdl_launch_dependents();
   const int64_t t = blockIdx.x;
-  const int width = heads * dv;
+  const int words = width / V, step = blockDim.x;
   const float* row = o + t * width;
-  auto gate_of = [&](float g) { return gate_silu ? silu_of(g) : 1.f / (1.f + expf(-g)); };
-  const bool vec = dv % 4 == 0 && p.stride % 4 == 0 && p.off_g % 4 == 0;
-  // four neighbouring gate columns
-  auto gates4 = [&](int i) {
-    const int64_t at = t * p.stride + p.off_g + i;
-    float4 g;
-    if (p.splits == 0) {
-      if (sizeof(T) == 4) {
-        g = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.data) + at);
-      } else {
-        const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(p.data) + at);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-        g = make_float4(a.x, a.y, b.x, b.y);
-      }
-    } else {
-      const float* src = reinterpret_cast<const float*>(p.data) + at;
-      g = *reinterpret_cast<const float4*>(src);
-      for (int s = 1; s < p.splits; ++s) {
-        const float4 u = *reinterpret_cast<const float4*>(src + s * p.plane);
-        g.x += u.x; g.y += u.y; g.z += u.z; g.w += u.w;
-      }
-      g = make_float4(rounded_to<T>(g.x), rounded_to<T>(g.y), rounded_to<T>(g.z), rounded_to<T>(g.w));
-    }
-    return make_float4(gate_of(g.x), gate_of(g.y), gate_of(g.z), gate_of(g.w));
-  };
-  auto put = [&](int i, float4 v) {
-    T* dst = y + t * width + i;
-    if (sizeof(T) == 4) {
-      *reinterpret_cast<float4*>(dst) = v;
-    } else {
-      const uint2 raw = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
-      *reinterpret_cast<uint2*>(dst) = raw;
-    }
-  };
-  if (joint) {
-    float ss = 0.f;
-    if (vec) {
-      for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
-        const float4 x = *reinterpret_cast<const float4*>(row + i);
-        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
-      }
-    } else {
-      for (int i = threadIdx.x; i < width; i += blockDim.x) ss += row[i] * row[i];
-    }
-    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
-    if (vec) {
-      for (int i = threadIdx.x * 4; i < width; i += blockDim.x * 4) {
-        const float4 x = *reinterpret_cast<const float4*>(row + i), g = gates4(i);
-        put(i, make_float4(x.x * inv * load_flex(w, w_f32, i) * g.x, x.y * inv * load_flex(w, w_f32, i + 1) * g.y,
-                           x.z * inv * load_flex(w, w_f32, i + 2) * g.z, x.w * inv * load_flex(w, w_f32, i + 3) * g.w));
-      }
-    } else {
-      for (int i = threadIdx.x; i < width; i += blockDim.x)
-        y[t * width + i] = from_f32<T>(row[i] * inv * load_flex(w, w_f32, i) * gate_of(column<T>(p, t, p.off_g + i)));
-    }
+  float ss = 0.f;
+  for (int n = threadIdx.x; n < words; n += step) {
+    float x[V];
+    load_row<V>(row + n * V, x);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  for (int n = threadIdx.x; n < words; n += step) {
+    float x[V], g[V];
+    load_row<V>(row + n * V, x);
+    load_gates<T, V>(p, t, n * V, gate_silu, g);
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = x[e] * inv * load_flex(w, w_f32, n * V + e) * g[e];
+    store_row<V>(y + t * width + n * V, x);
+  }
+}
+
+// Every head by its own root mean square, no weight. A warp a head.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+decay_out_heads_kernel(const float* __restrict__ o, const Projection p, int heads, int dv, float eps, int gate_silu, T* __restrict__ y) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const int lane = threadIdx.x & 31, h = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (h >= heads) return;
+  const int words = dv / V;
+  const float* row = o + (t * heads + h) * dv;
+  float ss = 0.f;
+  for (int n = lane; n < words; n += 32) {
+    float x[V];
+    load_row<V>(row + n * V, x);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
+  for (int n = lane; n < words; n += 32) {
+    float x[V], g[V];
+    load_row<V>(row + n * V, x);
+    load_gates<T, V>(p, t, h * dv + n * V, gate_silu, g);
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = x[e] * inv * g[e];
+    store_row<V>(y + (t * heads + h) * dv + n * V, x);
+  }
+}
+
+template <typename T, int V>
+void launch_decay_out(const float* o, const Projection& p, int tokens, int heads, int dv, int joint, const void* w, int w_f32, float eps,
+                      int gate_silu, void* y, cudaStream_t stream) {
+  if (!joint) {
+    vosti_launch(decay_out_heads_kernel<T, V>, dim3(tokens, (heads + 7) / 8), dim3(256), 0, stream, o, p, heads, dv, eps, gate_silu, (T*)y);
     return;
   }
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-  for (int h = blockIdx.y * nwarps + warp; h < heads; h += gridDim.y * nwarps) {
-    float ss = 0.f;
-    if (vec) {
-      for (int i = lane * 4; i < dv; i += 128) {
-        const float4 x = *reinterpret_cast<const float4*>(row + h * dv + i);
-        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
-      }
-    } else {
-      for (int i = lane; i < dv; i += 32) ss += row[h * dv + i] * row[h * dv + i];
-    }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
-    if (vec) {
-      for (int i = lane * 4; i < dv; i += 128) {
-        const float4 x = *reinterpret_cast<const float4*>(row + h * dv + i), g = gates4(h * dv + i);
-        put(h * dv + i, make_float4(x.x * inv * g.x, x.y * inv * g.y, x.z * inv * g.z, x.w * inv * g.w));
-      }
-    } else {
-      for (int i = lane; i < dv; i += 32)
-        y[t * width + h * dv + i] = from_f32<T>(row[h * dv + i] * inv * gate_of(column<T>(p, t, p.off_g + h * dv + i)));
-    }
-  }
+  const int width = heads * dv, wanted = (width / V + 31) / 32 * 32;
+  const int threads = tokens > 64 || wanted < 256 ? 256 : wanted > 1024 ? 1024 : wanted;      // few rows: a thread a word
+  vosti_launch(decay_out_joint_kernel<T, V>, dim3(tokens), dim3(threads), 0, stream, o, p, width, w, w_f32, eps, gate_silu, (T*)y);
 }
 
 template <typename T, int V>
@@ -753,11 +778,16 @@ VOSTI_API int vosti_decay_out(const float* o, const void* proj, int splits, int6
   VOSTI_REQUIRE(!joint || w != nullptr, "decay_out: the joint norm's weight is missing");
   if (tokens == 0) return VOSTI_OK;
   const Projection p = {proj, splits, stride, (int64_t)tokens * stride, 0, 0, 0, off_g};
-  const int width = heads * dv;
-  int threads = 256;
-  if (joint && tokens <= 64) threads = width / 4 >= 1024 ? 1024 : ((width / 4 + 31) / 32 * 32 > 256 ? (width / 4 + 31) / 32 * 32 : 256);
-  const dim3 grid(tokens, joint ? 1 : (heads + 7) / 8);
-  if (is_f32) vosti_launch(decay_out_kernel<float>, grid, dim3(threads), 0, stream, o, p, heads, dv, joint, w, w_f32, eps, gate_silu, (float*)y);
-  else vosti_launch(decay_out_kernel<bf16>, grid, dim3(threads), 0, stream, o, p, heads, dv, joint, w, w_f32, eps, gate_silu, (bf16*)y);
+  const bool words = dv % 4 == 0 && stride % 4 == 0 && off_g % 4 == 0 &&
+                     ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
+#define VOSTI_OUT_ARGS o, p, tokens, heads, dv, joint, w, w_f32, eps, gate_silu, y, stream
+  if (is_f32) {
+    if (words) launch_decay_out<float, 4>(VOSTI_OUT_ARGS);
+    else launch_decay_out<float, 1>(VOSTI_OUT_ARGS);
+  } else {
+    if (words) launch_decay_out<bf16, 4>(VOSTI_OUT_ARGS);
+    else launch_decay_out<bf16, 1>(VOSTI_OUT_ARGS);
+  }
+#undef VOSTI_OUT_ARGS
   VOSTI_LAUNCH_CHECK();
 }
