@@ -12,7 +12,8 @@
 // piece of the value columns of one (request, head); a thread keeps a few rows of S in registers, the
 // state is read and written once.
 //
-// Long portions in bfloat16 run as chunks of 128 tokens, on the tensor cores (mma.sync):
+// Long portions in bfloat16 run as chunks of 128 tokens, on the 5th-generation tensor cores (tcgen05, accumulators in
+// tensor memory, operands made by the block's threads in the 128-byte-swizzled layout):
 //   decay_chunk_state  U_c = sum over the chunk's tokens of decay^(tokens after it) k v^T, all chunks side by side;
 //   decay_chunk_scan   S before every chunk, S_(c+1) = decay^(n_c) S_c + U_c, written over U; the last one to the slot;
 //   decay_chunk_out    o_t = decay^(t+1) q_t S_c + sum over j <= t of decay^(t-j) (q_t . k_j) v_j, all chunks side by side.
@@ -24,6 +25,7 @@
 // weight) and gated (SiLU or sigmoid of further columns of the projection), rounded for the output product.
 #include "common.cuh"
 #include "mma_util.cuh"
+#include "tcgen05.cuh"
 
 namespace {
 
@@ -181,10 +183,10 @@ decay_scan_kernel(const Projection p, const Recurrence c, float* __restrict__ ou
 }
 
 // ------------------------------------------------------------------ chunks on the tensor cores
-constexpr int CHUNK_THREADS = 256;
-constexpr int VT = 64;                  // value columns of a block
-constexpr int V_PITCH = VT + 8;         // elements: rows 16 bytes apart modulo 128, conflict-free ldmatrix
+constexpr int CHUNK_THREADS = 512;
 constexpr int CHUNK_MAX_DK = 128;
+constexpr int VT = 128;                 // value columns of a block
+constexpr int BLOCK_BYTES = CHUNK * 128;        // [128 rows][64 elements], 128-byte swizzle
 
 struct Chunks {
   const int* request;                   // [chunks] the request a chunk belongs to
@@ -204,6 +206,7 @@ rotation_table_kernel(const float* __restrict__ freq, int half, const int* __res
   }
 }
 
+__device__ __forceinline__ float gate_value(float g, int silu) { return silu ? silu_of(g) : 1.f / (1.f + expf(-g)); }
 __device__ __forceinline__ void two_terms(float x, bf16& hi, bf16& lo) {
   hi = __float2bfloat16_rn(x);
   lo = __float2bfloat16_rn(x - __bfloat162float(hi));
@@ -221,18 +224,37 @@ __device__ __forceinline__ void unpack8(uint4 raw, float (&x)[8]) {
     x[2 * e + 1] = f.y;
   }
 }
+// Byte offset of 16-byte word `word` (8 elements) of row `row` in the tensor cores' layout: blocks of 64 elements,
+// [rows][128 bytes] each with the 128-byte swizzle, `block_bytes` apart.
+__device__ __forceinline__ uint32_t operand_offset(int row, int word, int block_bytes) {
+  return (uint32_t)((word >> 3) * block_bytes + row * 128 + (((word & 7) ^ (row & 7)) << 4));
+}
+// Eight values as one or two bfloat16 terms, a 16-byte word each.
+__device__ __forceinline__ void put_terms(const float (&x)[8], uint8_t* hi, uint8_t* lo, uint32_t at) {
+  uint32_t h[4], l[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    bf16 h0, l0, h1, l1;
+    two_terms(x[2 * e], h0, l0);
+    two_terms(x[2 * e + 1], h1, l1);
+    h[e] = pair_of(h0, h1);
+    l[e] = pair_of(l0, l1);
+  }
+  *reinterpret_cast<uint4*>(hi + at) = make_uint4(h[0], h[1], h[2], h[3]);
+  if (lo != nullptr) *reinterpret_cast<uint4*>(lo + at) = make_uint4(l[0], l[1], l[2], l[3]);
+}
 
-// A chunk's rows of one head's queries or keys (columns col0 .. col0 + dk - 1 of the projection) as two bfloat16
-// terms in shared memory, [CHUNK][pitch] each, zeros beyond row n and column dk. weight: 0: times `scale`;
-// 1: times scale * decay^(n - 1 - row).
+// A chunk's rows of one head's queries or keys (columns col0 .. col0 + dk - 1 of the projection) as one or two (lo not
+// null) bfloat16 terms, zeros beyond row n and column dk up to `padded` elements. Times `scale`, and if WEIGHTED
+// times decay^(n - 1 - row).
 template <bool WEIGHTED>
-__device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int dk, int dkp,
-                                           int pitch, int silu, const float2* __restrict__ turns, int rot_half, float scale,
-                                           float log2_decay, bf16* hi, bf16* lo, bool want_lo) {
-  const int words = dkp / 8;
+__device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int dk, int padded,
+                                           int silu, const float2* __restrict__ turns, int rot_half, float scale, float log2_decay,
+                                           uint8_t* hi, uint8_t* lo) {
+  const int words = padded / 8;
   const bool wide = dk % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0 && rot_half % 8 == 0;
   for (int i = threadIdx.x; i < CHUNK * words; i += CHUNK_THREADS) {
-    const int r = i / words, e0 = (i - r * words) * 8;
+    const int r = i / words, word = i - r * words, e0 = word * 8;
     float x[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) x[e] = 0.f;
@@ -275,26 +297,17 @@ __device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int64_
 #pragma unroll
       for (int e = 0; e < 8; ++e) x[e] *= by;
     }
-    uint32_t h[4], l[4];
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      bf16 h0, l0, h1, l1;
-      two_terms(x[2 * e], h0, l0);
-      two_terms(x[2 * e + 1], h1, l1);
-      h[e] = pair_of(h0, h1);
-      l[e] = pair_of(l0, l1);
-    }
-    *reinterpret_cast<uint4*>(hi + r * pitch + e0) = make_uint4(h[0], h[1], h[2], h[3]);
-    if (want_lo) *reinterpret_cast<uint4*>(lo + r * pitch + e0) = make_uint4(l[0], l[1], l[2], l[3]);
+    put_terms(x, hi, lo, operand_offset(r, word, BLOCK_BYTES));
   }
 }
 
-// A chunk's values, columns v0 .. v0 + VT - 1 of one head, [CHUNK][V_PITCH], zeros beyond row n and column dv.
+// A chunk's values, columns v0 .. v0 + padded - 1 of one head, zeros beyond row n and column dv.
 __device__ __forceinline__ void stage_values(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int v0, int dv,
-                                             int silu, bf16* vs) {
+                                             int padded, int silu, uint8_t* vs) {
+  const int words = padded / 8;
   const bool wide = dv % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0;
-  for (int i = threadIdx.x; i < CHUNK * (VT / 8); i += CHUNK_THREADS) {
-    const int r = i / (VT / 8), e0 = (i % (VT / 8)) * 8;
+  for (int i = threadIdx.x; i < CHUNK * words; i += CHUNK_THREADS) {
+    const int r = i / words, word = i - r * words, e0 = word * 8;
     uint4 raw = make_uint4(0, 0, 0, 0);
     if (r < n && v0 + e0 < dv) {
       const bf16* src = proj + (start + r) * stride + col0 + v0 + e0;
@@ -311,7 +324,7 @@ __device__ __forceinline__ void stage_values(const bf16* __restrict__ proj, int6
         for (int e = 0; e < 8; ++e) x[e] = __float2bfloat16_rn(silu_of(__bfloat162float(x[e])));
       }
     }
-    *reinterpret_cast<uint4*>(vs + r * V_PITCH + e0) = raw;
+    *reinterpret_cast<uint4*>(vs + operand_offset(r, word, BLOCK_BYTES)) = raw;
   }
 }
 
@@ -320,61 +333,121 @@ __device__ __forceinline__ int chunk_rows(const Recurrence& c, const Chunks& k, 
   start = c.cu_q[b] + k.first[chunk];
   return min(CHUNK, (int)(c.cu_q[b + 1] - start));
 }
+__host__ __device__ __forceinline__ int blocks_of(int elements) { return (elements + 63) / 64; }       // blocks of 64 elements
 
+// Instruction descriptor for kind::f16 with A MN-major too (rows of A's tile are the K index).
+__host__ __device__ constexpr uint32_t instr_both_mn(int n) { return umma_instr_desc(CHUNK, n, true) | (1u << 15); }
+
+// An operand in shared memory: its descriptor, and how it moves on along K: `step` bytes for 16 elements, after
+// `per_block` steps to the next block, `block_bytes` further on.
+struct Operand {
+  uint64_t desc;
+  int step, per_block, block_bytes;
+  __device__ __forceinline__ uint64_t at(int k) const {
+    return desc + (uint64_t)(((k / per_block) * block_bytes + (k % per_block) * step) >> 4);
+  }
+};
+__device__ __forceinline__ Operand k_major(uint32_t addr) { return Operand{smem_desc_sw128(addr), 32, 4, BLOCK_BYTES}; }
+__device__ __forceinline__ Operand mn_major(uint32_t addr, int block_bytes) { return Operand{smem_desc_sw128_mn(addr, (uint32_t)block_bytes), 16 * 128, 1 << 20, 0}; }
+// D += A B over `steps` steps of 16 along K (the first MMA of a sum overwrites D). One thread.
+__device__ __forceinline__ void multiply(uint32_t tmem, const Operand& a, const Operand& b, uint32_t idesc, int steps, bool& started) {
+  for (int k = 0; k < steps; ++k) {
+    umma_bf16(tmem, a.at(k), b.at(k), idesc, started ? 1u : 0u);
+    started = true;
+  }
+}
+
+// What the two kernels have in common: barriers and tensor memory, operands, the way out.
+template <int BARS>
+__device__ __forceinline__ void tensor_setup(uint64_t (&bars)[BARS], uint32_t* holder, volatile int* abort_flag, uint32_t cols) {
+  if (threadIdx.x == 0) {
+    *abort_flag = 0;
+    for (int i = 0; i < BARS; ++i) mbar_init(smem_u32(&bars[i]), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (threadIdx.x < 32) tmem_alloc(smem_u32(holder), cols);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  pdl_launch_dependents();            // after the tensor memory is ours: a dependent must not take it first
+}
+// Every thread's writes to shared memory are seen by the tensor cores after this.
+__device__ __forceinline__ void operands_ready() {
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+}
+__device__ __forceinline__ void tensor_leave(uint32_t tmem, uint32_t cols, volatile int* abort_flag) {
+  tc_fence_before();
+  __syncthreads();
+  if (*abort_flag) {
+    for (int i = 0; i < 64; ++i) __nanosleep(1000);
+    __syncthreads();
+  }
+  if (threadIdx.x < 32) {
+    tc_fence_after();
+    tmem_dealloc(tmem, cols);
+  }
+}
+
+constexpr uint32_t STATE_TMEM = 128;
+
+// grid (chunks, heads, value tiles): U[dk, dv] = K^T V, the head's key channels on the MMA's M side (128, zeros beyond dk).
 __global__ void __launch_bounds__(CHUNK_THREADS, 2)
-decay_chunk_state_kernel(const Projection p, const Recurrence c, const Chunks k) {
-  extern __shared__ __align__(16) uint8_t chunk_smem[];
+decay_chunk_state_kernel(const Projection p, const Recurrence c, const Chunks k, unsigned* status) {
+  extern __shared__ uint8_t chunk_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(chunk_raw) + 1023) & ~(uintptr_t)1023);
+  __shared__ __align__(8) uint64_t done[1];
+  __shared__ uint32_t tmem_holder;
+  __shared__ volatile int abort_flag;
   pdl_wait();
-  pdl_launch_dependents();
   const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT;
-  const int dk = c.dk, dv = c.dv, dkp = (dk + 15) & ~15, pitch = dkp + 8;
-  bf16* kh = reinterpret_cast<bf16*>(chunk_smem);
-  bf16* kl = kh + CHUNK * pitch;
-  bf16* vs = kl + CHUNK * pitch;
+  const int dk = c.dk, dv = c.dv;
   int64_t start;
   const int n = chunk_rows(c, k, chunk, start);
-  if (n <= 0) return;
+  if (n <= 0) return;                                  // (the whole block: nothing is allocated yet)
+  const int vblocks = blocks_of(min(dv - v0, VT));
+  uint8_t* kh = smem;                                  // two blocks of 64 key channels
+  uint8_t* kl = kh + 2 * BLOCK_BYTES;
+  uint8_t* vs = kl + 2 * BLOCK_BYTES;                  // [vblocks]
+  tensor_setup(done, &tmem_holder, &abort_flag, STATE_TMEM);
+  const uint32_t tmem = tmem_holder;
   const bf16* proj = reinterpret_cast<const bf16*>(p.data);
-  stage_rows<true>(proj, p.stride, start, n, p.off_k + h * dk, dk, dkp, pitch, c.silu, k.turns, c.rot_half, c.key_scale, c.log2_decay[h],
-                   kh, kl, true);
-  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, c.silu, vs);
-  __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int steps = (n + 15) / 16;                                      // tokens in steps of 16
-  float* U = k.states + ((int64_t)chunk * c.heads + h) * dk * dv;
-  // units of 16 key channels x 32 value columns
-  const uint32_t a_off = (uint32_t)((((lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 8) * 2);
-  const uint32_t b_off = (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * V_PITCH + (lane >> 4) * 8) * 2);
-  for (int unit = warp; unit < dkp / 16 * 2; unit += CHUNK_THREADS / 32) {
-    const int m0 = (unit >> 1) * 16, n0 = (unit & 1) * 32;
-    float acc[4][4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-    for (int s = 0; s < steps; ++s) {
-      uint32_t ah[4], al[4], b0[4], b1[4];
-      ldmatrix_x4_trans(ah, smem_addr(kh) + a_off + (uint32_t)((s * 16 * pitch + m0) * 2));
-      ldmatrix_x4_trans(al, smem_addr(kl) + a_off + (uint32_t)((s * 16 * pitch + m0) * 2));
-      ldmatrix_x4_trans(b0, smem_addr(vs) + b_off + (uint32_t)((s * 16 * V_PITCH + n0) * 2));
-      ldmatrix_x4_trans(b1, smem_addr(vs) + b_off + (uint32_t)((s * 16 * V_PITCH + n0 + 16) * 2));
-      mma_bf16(acc[0], ah, b0[0], b0[1]); mma_bf16(acc[1], ah, b0[2], b0[3]);
-      mma_bf16(acc[2], ah, b1[0], b1[1]); mma_bf16(acc[3], ah, b1[2], b1[3]);
-      mma_bf16(acc[0], al, b0[0], b0[1]); mma_bf16(acc[1], al, b0[2], b0[3]);
-      mma_bf16(acc[2], al, b1[0], b1[1]); mma_bf16(acc[3], al, b1[2], b1[3]);
-    }
-#pragma unroll
-    for (int j = 0; j < 4; ++j)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int row = m0 + (lane >> 2) + 8 * r, col = v0 + n0 + 8 * j + (lane & 3) * 2;
-        if (row >= dk) continue;
-        if (dv % 2 == 0) {
-          if (col < dv) *reinterpret_cast<float2*>(U + (int64_t)row * dv + col) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
-        } else {
-          if (col < dv) U[(int64_t)row * dv + col] = acc[j][2 * r];
-          if (col + 1 < dv) U[(int64_t)row * dv + col + 1] = acc[j][2 * r + 1];
-        }
-      }
+  stage_rows<true>(proj, p.stride, start, n, p.off_k + h * dk, dk, 128, c.silu, k.turns, c.rot_half, c.key_scale, c.log2_decay[h], kh, kl);
+  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, 64 * vblocks, c.silu, vs);
+  operands_ready();
+  if (threadIdx.x == 0) {
+    const uint32_t idesc = instr_both_mn(64 * vblocks);
+    const Operand v = mn_major(smem_u32(vs), BLOCK_BYTES);
+    bool started = false;
+    multiply(tmem, mn_major(smem_u32(kh), BLOCK_BYTES), v, idesc, (n + 15) / 16, started);
+    multiply(tmem, mn_major(smem_u32(kl), BLOCK_BYTES), v, idesc, (n + 15) / 16, started);
+    umma_commit(smem_u32(&done[0]));
   }
+  __syncwarp();
+  const bool ok = mbar_wait_warp(smem_u32(&done[0]), 0, &abort_flag, status);
+  tc_fence_after();
+  // a thread a key channel and 32 value columns
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, row = (warp & 3) * 32 + lane, c0 = (warp >> 2) * 32;
+  if (ok && c0 < 64 * vblocks) {
+    uint32_t r[32];
+    tmem_load32(tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)c0, r);
+    if (row < dk) {
+      float* dst = k.states + (((int64_t)chunk * c.heads + h) * dk + row) * dv + v0 + c0;
+      if (dv % 4 == 0) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (v0 + c0 + 4 * j < dv)
+            reinterpret_cast<float4*>(dst)[j] = make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]), __uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3]));
+      } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+          if (v0 + c0 + j < dv) dst[j] = __uint_as_float(r[j]);
+      }
+    }
+  }
+  tensor_leave(tmem, STATE_TMEM, &abort_flag);
 }
 
 // V floats a thread. long_requests: which requests; chunk0: a request's first chunk.
@@ -422,146 +495,207 @@ decay_chunk_scan_kernel(const Recurrence c, const int* __restrict__ long_request
   for (int e = 0; e < V; ++e) S[e] = s[e];
 }
 
-// LO: queries and keys have a second term (they are rotated); else they are bfloat16 (SiLU'd activations).
+constexpr uint32_t OUT_TMEM = 512, SCORE_COL = 0, CARRIED_COL = 128, INNER_COL = 256;
+
+// What may follow a head's read-out at once where a block holds the whole head: unit root mean square and gate.
+struct HeadOut {
+  bf16* y;                              // [tokens, heads * dv], or null: the read-outs go out as they are
+  float eps;
+  int gate_silu;
+};
+
+// grid (chunks, heads, value tiles). LO: queries and keys have a second term (they are rotated); else they are bfloat16
+// (SiLU'd activations). Scores Q K^T, the carried part Q S and the inner part P V have tensor memory of their own;
+// P, the decayed scores in two terms, takes the place of the queries and keys.
 template <bool LO>
-__global__ void __launch_bounds__(CHUNK_THREADS, 2)
-decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, float* __restrict__ out) {
-  extern __shared__ __align__(16) uint8_t chunk_smem[];
-  constexpr int KS = CHUNK_MAX_DK / 16;
+__global__ void __launch_bounds__(CHUNK_THREADS, 1)
+decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, float* __restrict__ out, const HeadOut fin, unsigned* status) {
+  extern __shared__ uint8_t chunk_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(chunk_raw) + 1023) & ~(uintptr_t)1023);
+  __shared__ __align__(8) uint64_t done[3];
+  __shared__ uint32_t tmem_holder;
+  __shared__ volatile int abort_flag;
   pdl_wait();
-  pdl_launch_dependents();
   const int chunk = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT;
-  const int dk = c.dk, dv = c.dv, dkp = (dk + 15) & ~15, pitch = dkp + 8;
-  bf16* kh = reinterpret_cast<bf16*>(chunk_smem);      // queries, then the state (pitch V_PITCH), then keys
-  bf16* kl = kh + CHUNK * pitch;
-  bf16* vs = kl + CHUNK * pitch;
+  const int dk = c.dk, dv = c.dv;
   int64_t start;
   const int n = chunk_rows(c, k, chunk, start);
   if (n <= 0) return;
+  const int kblocks = blocks_of(dk), vblocks = blocks_of(min(dv - v0, VT));
+  const int q_bytes = kblocks * BLOCK_BYTES, s_block = 64 * kblocks * 128;
+  uint8_t* qh = smem;
+  uint8_t* ql = qh + (LO ? q_bytes : 0);
+  uint8_t* kh = ql + q_bytes;
+  uint8_t* kl = kh + (LO ? q_bytes : 0);
+  uint8_t* ph = smem;                                  // after the queries and keys have been read: two blocks of 64 keys a term
+  uint8_t* pl = ph + 2 * BLOCK_BYTES;
+  uint8_t* vs = smem + max((LO ? 4 : 2) * q_bytes, 4 * BLOCK_BYTES);
+  uint8_t* sh = vs + vblocks * BLOCK_BYTES;            // [vblocks][64 * kblocks rows][64 columns]
+  uint8_t* sl = sh + vblocks * s_block;
+  tensor_setup(done, &tmem_holder, &abort_flag, OUT_TMEM);
+  const uint32_t tmem = tmem_holder;
   const bf16* proj = reinterpret_cast<const bf16*>(p.data);
   const float l2d = c.log2_decay[h];
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int row0 = warp * 16;                          // this warp's tokens of the chunk
-  stage_rows<false>(proj, p.stride, start, n, p.off_q + h * dk, dk, dkp, pitch, c.silu, k.turns, c.rot_half, 1.f, 0.f, kh, kl, LO);
-  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, c.silu, vs);
-  __syncthreads();
-  uint32_t qh[KS][4], ql[LO ? KS : 1][4];
-  {
-    const uint32_t off = (uint32_t)(((row0 + (lane & 15)) * pitch + (lane >> 4) * 8) * 2);
-#pragma unroll
-    for (int s = 0; s < KS; ++s)
-      if (s * 16 < dkp) {
-        ldmatrix_x4(qh[s], smem_addr(kh) + off + s * 32);
-        if (LO) ldmatrix_x4(ql[LO ? s : 0], smem_addr(kl) + off + s * 32);
-      }
+  stage_rows<false>(proj, p.stride, start, n, p.off_q + h * dk, dk, 64 * kblocks, c.silu, k.turns, c.rot_half, 1.f, 0.f, qh, LO ? ql : nullptr);
+  stage_rows<false>(proj, p.stride, start, n, p.off_k + h * dk, dk, 64 * kblocks, c.silu, k.turns, c.rot_half, c.key_scale, 0.f, kh, LO ? kl : nullptr);
+  operands_ready();
+  if (threadIdx.x == 0) {
+    const uint32_t idesc = umma_instr_desc(CHUNK, CHUNK, false);
+    bool started = false;
+    multiply(tmem + SCORE_COL, k_major(smem_u32(qh)), k_major(smem_u32(kh)), idesc, 4 * kblocks, started);
+    if (LO) {
+      multiply(tmem + SCORE_COL, k_major(smem_u32(ql)), k_major(smem_u32(kh)), idesc, 4 * kblocks, started);
+      multiply(tmem + SCORE_COL, k_major(smem_u32(qh)), k_major(smem_u32(kl)), idesc, 4 * kblocks, started);
+    }
+    umma_commit(smem_u32(&done[0]));
   }
-  __syncthreads();
-  // ---- the state before the chunk: [dkp][V_PITCH] in two terms, in the place of the queries
-  bf16* sh = kh;
-  bf16* sl = kh + (int64_t)dkp * V_PITCH;
+  __syncwarp();
+  // the state before the chunk and the values, while the scores are made
   {
     const float* S = k.states + ((int64_t)chunk * c.heads + h) * dk * dv + v0;
+    const int words = 8 * vblocks, rows = 64 * kblocks;
     const bool wide = dv % 4 == 0;
-    for (int i = threadIdx.x; i < dkp * (VT / 4); i += CHUNK_THREADS) {
-      const int r = i / (VT / 4), e0 = (i % (VT / 4)) * 4;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = threadIdx.x; i < rows * words; i += CHUNK_THREADS) {
+      const int r = i / words, word = i - r * words, e0 = word * 8;
+      float x[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = 0.f;
       if (r < dk) {
         const float* src = S + (int64_t)r * dv + e0;
         if (wide) {
-          if (v0 + e0 < dv) x = *reinterpret_cast<const float4*>(src);
+          if (v0 + e0 < dv) {
+            const float4 a = *reinterpret_cast<const float4*>(src);
+            x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
+          }
+          if (v0 + e0 + 4 < dv) {
+            const float4 a = *reinterpret_cast<const float4*>(src + 4);
+            x[4] = a.x; x[5] = a.y; x[6] = a.z; x[7] = a.w;
+          }
         } else {
-          if (v0 + e0 < dv) x.x = src[0];
-          if (v0 + e0 + 1 < dv) x.y = src[1];
-          if (v0 + e0 + 2 < dv) x.z = src[2];
-          if (v0 + e0 + 3 < dv) x.w = src[3];
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            if (v0 + e0 + e < dv) x[e] = src[e];
         }
       }
-      bf16 a0, b0, a1, b1, a2, b2, a3, b3;
-      two_terms(x.x, a0, b0); two_terms(x.y, a1, b1); two_terms(x.z, a2, b2); two_terms(x.w, a3, b3);
-      *reinterpret_cast<uint2*>(sh + r * V_PITCH + e0) = make_uint2(pair_of(a0, a1), pair_of(a2, a3));
-      *reinterpret_cast<uint2*>(sl + r * V_PITCH + e0) = make_uint2(pair_of(b0, b1), pair_of(b2, b3));
+      put_terms(x, sh, sl, operand_offset(r, word, s_block));
     }
   }
-  __syncthreads();
-  float o[VT / 8][4];
+  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, 64 * vblocks, c.silu, vs);
+  operands_ready();
+  const uint32_t idesc_v = umma_instr_desc(CHUNK, 64 * vblocks, true);
+  if (threadIdx.x == 0) {
+    bool started = false;
+    multiply(tmem + CARRIED_COL, k_major(smem_u32(qh)), mn_major(smem_u32(sh), s_block), idesc_v, 4 * kblocks, started);
+    multiply(tmem + CARRIED_COL, k_major(smem_u32(qh)), mn_major(smem_u32(sl), s_block), idesc_v, 4 * kblocks, started);
+    if (LO) multiply(tmem + CARRIED_COL, k_major(smem_u32(ql)), mn_major(smem_u32(sh), s_block), idesc_v, 4 * kblocks, started);
+    umma_commit(smem_u32(&done[1]));
+  }
+  __syncwarp();
+  // ---- the decayed scores: a thread a token and 32 keys
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, row = (warp & 3) * 32 + lane, part = warp >> 2, c0 = part * 32;
+  const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
+  bool ok = mbar_wait_warp(smem_u32(&done[0]), 0, &abort_flag, status);
+  ok = ok && mbar_wait_warp(smem_u32(&done[1]), 0, &abort_flag, status);      // (the queries may be overwritten)
+  tc_fence_after();
+  if (ok) {
+    uint32_t r[32];
+    tmem_load32(lanes + SCORE_COL + c0, r);
 #pragma unroll
-  for (int j = 0; j < VT / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-  const uint32_t b_off = (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * V_PITCH + (lane >> 4) * 8) * 2);
-  if (row0 < n) {
+    for (int w = 0; w < 4; ++w) {
+      float x[8];
 #pragma unroll
-    for (int s = 0; s < KS; ++s)
-      if (s * 16 < dkp) {
+      for (int e = 0; e < 8; ++e) {
+        const int back = row - (c0 + 8 * w + e);
+        x[e] = back >= 0 ? __uint_as_float(r[8 * w + e]) * exp2f(l2d * (float)back) : 0.f;
+      }
+      put_terms(x, ph, pl, operand_offset(row, c0 / 8 + w, BLOCK_BYTES));
+    }
+  }
+  operands_ready();
+  if (threadIdx.x == 0 && ok) {
+    const Operand v = mn_major(smem_u32(vs), BLOCK_BYTES);
+    const int steps = (n + 15) / 16;
+    bool started = false;
+    multiply(tmem + INNER_COL, k_major(smem_u32(ph)), v, idesc_v, steps, started);
+    multiply(tmem + INNER_COL, k_major(smem_u32(pl)), v, idesc_v, steps, started);
+    umma_commit(smem_u32(&done[2]));
+  }
+  __syncwarp();
+  // ---- carried part times decay^(token + 1), plus the inner part: a thread a token and 32 value columns
+  const bool mine = c0 < 64 * vblocks;
+  float o[32];
+  {
+    uint32_t r[32];
+    const float by = exp2f(l2d * (float)(row + 1));
+    if (ok && mine) {
+      tmem_load32(lanes + CARRIED_COL + c0, r);
 #pragma unroll
-        for (int j = 0; j < VT / 16; ++j) {
-          uint32_t b[4], bl[4];
-          ldmatrix_x4_trans(b, smem_addr(sh) + b_off + (uint32_t)((s * 16 * V_PITCH + j * 16) * 2));
-          ldmatrix_x4_trans(bl, smem_addr(sl) + b_off + (uint32_t)((s * 16 * V_PITCH + j * 16) * 2));
-          mma_bf16(o[2 * j], qh[s], b[0], b[1]); mma_bf16(o[2 * j + 1], qh[s], b[2], b[3]);
-          mma_bf16(o[2 * j], qh[s], bl[0], bl[1]); mma_bf16(o[2 * j + 1], qh[s], bl[2], bl[3]);
-          if (LO) { mma_bf16(o[2 * j], ql[LO ? s : 0], b[0], b[1]); mma_bf16(o[2 * j + 1], ql[LO ? s : 0], b[2], b[3]); }
+      for (int j = 0; j < 32; ++j) o[j] = __uint_as_float(r[j]) * by;
+    }
+    ok = ok && mbar_wait_warp(smem_u32(&done[2]), 0, &abort_flag, status);
+    tc_fence_after();
+    if (ok && mine) {
+      tmem_load32(lanes + INNER_COL + c0, r);
+#pragma unroll
+      for (int j = 0; j < 32; ++j) o[j] += __uint_as_float(r[j]);
+    }
+  }
+  if (fin.y != nullptr) {
+    // (one value tile: the block holds the whole head, columns beyond dv are zero)
+    float* squares = reinterpret_cast<float*>(smem);     // [4][CHUNK], in the place of the decayed scores, which have been read
+    float ss = 0.f;
+    if (ok && mine) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) ss += o[j] * o[j];
+    }
+    squares[part * CHUNK + row] = ss;
+    __syncthreads();
+    const float inv = 1.f / sqrtf((squares[row] + squares[CHUNK + row] + squares[2 * CHUNK + row] + squares[3 * CHUNK + row]) / (float)dv + fin.eps);
+    if (ok && mine && row < n) {
+      const int64_t at = (start + row) * p.stride + p.off_g + (int64_t)h * dv + c0;
+      bf16* dst = fin.y + ((start + row) * c.heads + h) * dv + c0;
+      const bool words = dv % 8 == 0 && p.stride % 8 == 0 && p.off_g % 8 == 0;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        if (words) {
+          if (c0 + 8 * w < dv) {
+            float g[8];
+            unpack8(*reinterpret_cast<const uint4*>(proj + at + 8 * w), g);
+            uint32_t v[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              v[e] = pack_bf16(o[8 * w + 2 * e] * inv * gate_value(g[2 * e], fin.gate_silu), o[8 * w + 2 * e + 1] * inv * gate_value(g[2 * e + 1], fin.gate_silu));
+            *reinterpret_cast<uint4*>(dst + 8 * w) = make_uint4(v[0], v[1], v[2], v[3]);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            if (c0 + 8 * w + e < dv) dst[8 * w + e] = __float2bfloat16_rn(o[8 * w + e] * inv * gate_value(to_f32(proj[at + 8 * w + e]), fin.gate_silu));
         }
       }
-    const int r0 = row0 + (lane >> 2);
-    const float d0 = exp2f(l2d * (float)(r0 + 1)), d1 = exp2f(l2d * (float)(r0 + 9));
+    }
+  } else if (ok && mine && row < n) {
+    float* dst = out + (start + row) * c.heads * dv + (int64_t)h * dv + v0 + c0;
+    if (dv % 4 == 0) {
 #pragma unroll
-    for (int j = 0; j < VT / 8; ++j) { o[j][0] *= d0; o[j][1] *= d0; o[j][2] *= d1; o[j][3] *= d1; }
-  }
-  __syncthreads();
-  // ---- the chunk's own keys
-  stage_rows<false>(proj, p.stride, start, n, p.off_k + h * dk, dk, dkp, pitch, c.silu, k.turns, c.rot_half, c.key_scale, 0.f, kh, kl, true);
-  __syncthreads();
-  if (row0 >= n) return;
-  const uint32_t k_off = (uint32_t)((((lane & 7) + (lane >> 4) * 8) * pitch + ((lane >> 3) & 1) * 8) * 2);
-  for (int t = 0; t <= warp; ++t) {                    // tiles of 16 keys up to the warp's own rows
-    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+      for (int j = 0; j < 8; ++j)
+        if (v0 + c0 + 4 * j < dv) reinterpret_cast<float4*>(dst)[j] = make_float4(o[4 * j], o[4 * j + 1], o[4 * j + 2], o[4 * j + 3]);
+    } else {
 #pragma unroll
-    for (int kk = 0; kk < KS; ++kk)
-      if (kk * 16 < dkp) {
-        uint32_t b[4], bl[4];
-        ldmatrix_x4(b, smem_addr(kh) + k_off + (uint32_t)((t * 16 * pitch + kk * 16) * 2));
-        mma_bf16(s[0], qh[kk], b[0], b[1]); mma_bf16(s[1], qh[kk], b[2], b[3]);
-        ldmatrix_x4(bl, smem_addr(kl) + k_off + (uint32_t)((t * 16 * pitch + kk * 16) * 2));
-        mma_bf16(s[0], qh[kk], bl[0], bl[1]); mma_bf16(s[1], qh[kk], bl[2], bl[3]);
-        if (LO) { mma_bf16(s[0], ql[LO ? kk : 0], b[0], b[1]); mma_bf16(s[1], ql[LO ? kk : 0], b[2], b[3]); }
-      }
-    uint32_t ph[4], pl[4];
-#pragma unroll
-    for (int j = 0; j < 2; ++j)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        bf16 h0, l0, h1, l1;
-        const int back = row0 + (lane >> 2) + 8 * r - (t * 16 + 8 * j + (lane & 3) * 2);
-        two_terms(back >= 0 ? s[j][2 * r] * exp2f(l2d * (float)back) : 0.f, h0, l0);
-        two_terms(back >= 1 ? s[j][2 * r + 1] * exp2f(l2d * (float)(back - 1)) : 0.f, h1, l1);
-        ph[2 * j + r] = pair_of(h0, h1);
-        pl[2 * j + r] = pair_of(l0, l1);
-      }
-#pragma unroll
-    for (int j = 0; j < VT / 16; ++j) {
-      uint32_t b[4];
-      ldmatrix_x4_trans(b, smem_addr(vs) + b_off + (uint32_t)((t * 16 * V_PITCH + j * 16) * 2));
-      mma_bf16(o[2 * j], ph, b[0], b[1]); mma_bf16(o[2 * j + 1], ph, b[2], b[3]);
-      mma_bf16(o[2 * j], pl, b[0], b[1]); mma_bf16(o[2 * j + 1], pl, b[2], b[3]);
+      for (int j = 0; j < 32; ++j)
+        if (v0 + c0 + j < dv) dst[j] = o[j];
     }
   }
-#pragma unroll
-  for (int j = 0; j < VT / 8; ++j)
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int row = row0 + (lane >> 2) + 8 * r, col = v0 + 8 * j + (lane & 3) * 2;
-      if (row >= n) continue;
-      float* dst = out + (start + row) * c.heads * dv + (int64_t)h * dv + col;
-      if (dv % 2 == 0) {
-        if (col < dv) *reinterpret_cast<float2*>(dst) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
-      } else {
-        if (col < dv) dst[0] = o[j][2 * r];
-        if (col + 1 < dv) dst[1] = o[j][2 * r + 1];
-      }
-    }
+  tensor_leave(tmem, OUT_TMEM, &abort_flag);
+}
+
+size_t state_smem(int dv) { return 1024 + (size_t)(4 + blocks_of(dv < VT ? dv : VT)) * BLOCK_BYTES; }
+size_t out_smem(int dk, int dv, bool lo) {
+  const size_t kb = blocks_of(dk), vb = blocks_of(dv < VT ? dv : VT), rows = (lo ? 4 : 2) * kb;
+  return 1024 + ((rows > 4 ? rows : 4) + vb + vb * kb) * BLOCK_BYTES;      // (a term of the state: vb * kb blocks of 64 rows)
 }
 
 // ------------------------------------------------------------------ norm and gate
-__device__ __forceinline__ float gate_value(float g, int silu) { return silu ? silu_of(g) : 1.f / (1.f + expf(-g)); }
 // V neighbouring gates of token t from column off_g + i on, summed and rounded like `column`.
 template <typename T, int V>
 __device__ __forceinline__ void load_gates(const Projection& p, int64_t t, int i, int silu, float (&g)[V]) {
@@ -731,43 +865,43 @@ VOSTI_API int vosti_rotation_table(const float* freq, int half, const int* posit
 
 // The long portions of a step: proj bfloat16 [tokens, stride]; chunk_request / chunk_first int32 [chunks] (see Chunks),
 // long_requests / long_chunk0 int32 [longs]; turns the rotation table of the step's tokens, or null;
-// states float32 scratch [chunks, heads, dk, dv].
+// states float32 scratch [chunks, heads, dk, dv]. With y (bfloat16 [tokens, heads * dv]; dv <= 128) every head's read-out is
+// divided by its root mean square, gated by the columns from off_g on and written there; else out receives the read-outs.
 VOSTI_API int vosti_decay_chunks(const void* proj, int64_t stride, int tokens, int off_q, int off_k, int off_v, int heads, int dk, int dv,
                                  int silu, const float* log2_decay, float key_scale, const float* freq, const void* turns, int rot_half,
                                  const int* positions, float* state, int64_t state_stride, const int* cu_q, const int* state_slots,
                                  int num_slots, const int* chunk_request, const int* chunk_first, int chunks, const int* long_requests,
-                                 const int* long_chunk0, int requests, float* states, float* out, cudaStream_t stream) {
+                                 const int* long_chunk0, int requests, float* states, float* out, int off_g, float eps, int gate_silu,
+                                 void* y, unsigned* status, cudaStream_t stream) {
   const int splits = 0;
   VOSTI_DECAY_CHECKS("decay_chunks");
   VOSTI_REQUIRE(dk <= CHUNK_MAX_DK, "decay_chunks: heads of %d (at most %d)", dk, CHUNK_MAX_DK);
   VOSTI_REQUIRE(rot_half == 0 || turns != nullptr, "decay_chunks: the rotation table is missing");
-  VOSTI_REQUIRE(((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(states) | reinterpret_cast<uintptr_t>(turns)) & 15) == 0,
+  VOSTI_REQUIRE(y != nullptr ? dv <= VT : out != nullptr, "decay_chunks: nowhere to write, or a head too wide to be normed at once");
+  VOSTI_REQUIRE(((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(states) | reinterpret_cast<uintptr_t>(turns) |
+                  reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(y)) & 15) == 0,
                 "decay_chunks: operands must be 16-byte aligned");
   if (tokens == 0 || chunks == 0) return VOSTI_OK;
-  const Projection p = {proj, 0, stride, 0, off_q, off_k, off_v, 0};
+  const Projection p = {proj, 0, stride, 0, off_q, off_k, off_v, off_g};
   const Recurrence c = {heads, dk, dv, silu, nullptr, log2_decay, key_scale, freq, rot_half, positions, state, state_stride, cu_q, state_slots, num_slots};
   const Chunks k = {chunk_request, chunk_first, (const float2*)turns, states};
-  const int dkp = (dk + 15) & ~15;
-  // (queries and keys take [CHUNK][dkp + 8] twice, the state [dkp][V_PITCH] twice in the same place, which is no larger)
-  static_assert(CHUNK_MAX_DK <= CHUNK && V_PITCH <= CHUNK, "the state must fit the keys' place");
-  const size_t smem = (size_t)2 * CHUNK * (dkp + 8) * 2 + (size_t)CHUNK * V_PITCH * 2;
-  constexpr int MOST = 2 * CHUNK * (CHUNK_MAX_DK + 8) * 2 + CHUNK * V_PITCH * 2;
+  const HeadOut fin = {(bf16*)y, eps, gate_silu};
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(decay_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST);
-    cudaFuncSetAttribute(decay_chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST);
-    cudaFuncSetAttribute(decay_chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, MOST);
+    cudaFuncSetAttribute(decay_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)state_smem(VT));
+    cudaFuncSetAttribute(decay_chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem(CHUNK_MAX_DK, VT, true));
+    cudaFuncSetAttribute(decay_chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem(CHUNK_MAX_DK, VT, false));
     configured = true;
   }
   const dim3 grid(chunks, heads, (dv + VT - 1) / VT);
-  vosti_launch(decay_chunk_state_kernel, grid, dim3(CHUNK_THREADS), smem, stream, p, c, k);
+  vosti_launch(decay_chunk_state_kernel, grid, dim3(CHUNK_THREADS), state_smem(dv), stream, p, c, k, status);
   const int64_t size = (int64_t)dk * dv;
   if (size % 4 == 0)
     vosti_launch(decay_chunk_scan_kernel<4>, dim3((unsigned)((size / 4 + 255) / 256), heads, requests), dim3(256), 0, stream, c, long_requests, long_chunk0, states);
   else
     vosti_launch(decay_chunk_scan_kernel<1>, dim3((unsigned)((size + 255) / 256), heads, requests), dim3(256), 0, stream, c, long_requests, long_chunk0, states);
-  if (rot_half > 0) vosti_launch(decay_chunk_out_kernel<true>, grid, dim3(CHUNK_THREADS), smem, stream, p, c, k, out);
-  else vosti_launch(decay_chunk_out_kernel<false>, grid, dim3(CHUNK_THREADS), smem, stream, p, c, k, out);
+  if (rot_half > 0) vosti_launch(decay_chunk_out_kernel<true>, grid, dim3(CHUNK_THREADS), out_smem(dk, dv, true), stream, p, c, k, out, fin, status);
+  else vosti_launch(decay_chunk_out_kernel<false>, grid, dim3(CHUNK_THREADS), out_smem(dk, dv, false), stream, p, c, k, out, fin, status);
   VOSTI_LAUNCH_CHECK();
 }
 

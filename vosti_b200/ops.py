@@ -1729,12 +1729,23 @@ def decay_step_layout(q_lens):
     return arrays, {"chunks": len(requests), "longs": len(longs), "shorts": len(q_lens) - len(longs)}
 
 
+class DecayOut:
+    """What follows the fixed-decay recurrence (see `decay_out`): the gate's first column in the projection, the norm's
+    eps and weight (None: every head by its own root mean square), the gate's activation and the result's type."""
+
+    def __init__(self, offset: int, eps: float, weight: Optional[torch.Tensor], gate_silu: bool, out_dtype: torch.dtype):
+        self.offset, self.eps, self.weight, self.gate_silu, self.out_dtype = offset, float(eps), weight, bool(gate_silu), out_dtype
+
+
 def decay_attention(proj, offsets: dict, state: torch.Tensor, ctx, *, heads: int, dk: int, dv: int, decay: torch.Tensor,
-                    log2_decay: torch.Tensor, silu: bool, key_scale: float, freq: Optional[torch.Tensor]) -> torch.Tensor:
+                    log2_decay: torch.Tensor, silu: bool, key_scale: float, freq: Optional[torch.Tensor],
+                    finish: Optional[DecayOut] = None) -> torch.Tensor:
     """S <- decay S + k v^T, o = S^T q per head over every request's tokens of this step, from and to its state slot
     (csrc/decay_attention.cu); `proj` (a tensor of the serving type or unsummed K splits that are rounded to it) holds
     the columns q | k | v at `offsets`, which pass SiLU (`silu`) or of which q and k are rotated (`freq`, float32 [n],
-    the first 2n elements of a head). `decay` and its base-2 logarithm: float32 [heads]. Returns float32 [tokens, heads * dv]."""
+    the first 2n elements of a head). `decay` and its base-2 logarithm: float32 [heads]. Returns o, float32
+    [tokens, heads * dv], or with `finish` what `decay_out` makes of it (in one kernel with the recurrence where a step
+    brings long portions only and every head is normed by itself)."""
     dtype = proj.dtype
     layout = (getattr(ctx, "layout", None) or {}).get("decay")
     lib = library()
@@ -1747,7 +1758,10 @@ def decay_attention(proj, offsets: dict, state: torch.Tensor, ctx, *, heads: int
     _contig(state, decay, log2_decay, freq)
     if state.dtype != torch.float32 or decay.dtype != torch.float32 or log2_decay.dtype != torch.float32:
         raise KernelError("decay_attention: the state and the decays are float32")
-    out = torch.empty((tokens, heads * dv), dtype=torch.float32, device=state.device)
+    at_once = bool(chunked and finish is not None and finish.weight is None and finish.out_dtype == torch.bfloat16 and dv <= 128
+                   and layout["shorts"] == 0)
+    y = torch.empty((tokens, heads * dv), dtype=torch.bfloat16, device=state.device) if at_once else None
+    out = None if at_once else torch.empty((tokens, heads * dv), dtype=torch.float32, device=state.device)
     half = 0 if freq is None else freq.shape[0]
     common = (offsets["q"], offsets["k"], offsets["v"], heads, dk, dv, int(silu))
     slots = (_p(state), ctypes.c_int64(state.shape[1]), _p(ctx.cu_q), _p(ctx.state_slots), state.shape[0])
@@ -1763,17 +1777,23 @@ def decay_attention(proj, offsets: dict, state: torch.Tensor, ctx, *, heads: int
                 ctx.extras[key] = turns
         states = torch.empty((layout["chunks"], heads, dk, dv), dtype=torch.float32, device=state.device)
         arrays = ctx.extras
+        gate = (finish.offset, ctypes.c_float(finish.eps), int(finish.gate_silu)) if at_once else (0, ctypes.c_float(0.0), 0)
         _check(lib.vosti_decay_chunks(
             p, ctypes.c_int64(stride), tokens, *common, _p(log2_decay), ctypes.c_float(key_scale), _p(freq), _p(turns), half,
             _p(ctx.positions), *slots, _p(arrays["decay.chunk_request"]), _p(arrays["decay.chunk_first"]), layout["chunks"],
-            _p(arrays["decay.long_requests"]), _p(arrays["decay.long_chunk0"]), layout["longs"], _p(states), _p(out), _stream()),
-            "decay_chunks", kernels=3)
+            _p(arrays["decay.long_requests"]), _p(arrays["decay.long_chunk0"]), layout["longs"], _p(states), _p(out), *gate, _p(y),
+            _p(ctx.status), _stream()), "decay_chunks", kernels=3)
+    if at_once:
+        return y
     if not chunked or layout["shorts"] > 0:
         _check(lib.vosti_decay_scan(
             p, splits, ctypes.c_int64(stride), tokens, *common, _p(decay), ctypes.c_float(key_scale), _p(freq), half,
             _p(ctx.positions), *slots, ctx.num_requests, DECAY_SHORT if chunked else 0, _p(out), 1 if dtype == torch.float32 else 0,
             _stream()), "decay_scan")
-    return out
+    if finish is None:
+        return out
+    return decay_out(out, proj, finish.offset, heads=heads, dv=dv, eps=finish.eps, weight=finish.weight, gate_silu=finish.gate_silu,
+                     out_dtype=finish.out_dtype)
 
 
 def decay_out(o: torch.Tensor, proj, offset: int, *, heads: int, dv: int, eps: float, weight: Optional[torch.Tensor], gate_silu: bool,

@@ -92,10 +92,9 @@ class DecayAttention(Mixer):
         proj = linear(ctx, x, self.w_in, allow_partial=True)
         if isinstance(proj, ops.PartialSum) and proj.dtype == torch.float32:
             proj = proj.materialize()
-        o = ops.decay_attention(proj, self.offsets, cache.state, ctx, heads=self.heads, dk=self.dk, dv=self.dv, decay=self.decay,
-                                log2_decay=self.log2_decay, silu=self.silu, key_scale=self.key_scale, freq=self.freq)
-        y = ops.decay_out(o, proj, self.offsets["g"], heads=self.heads, dv=self.dv, eps=self.eps, weight=self.norm,
-                          gate_silu=self.gate_silu, out_dtype=ctx.dtype)
+        y = ops.decay_attention(proj, self.offsets, cache.state, ctx, heads=self.heads, dk=self.dk, dv=self.dv, decay=self.decay,
+                                log2_decay=self.log2_decay, silu=self.silu, key_scale=self.key_scale, freq=self.freq,
+                                finish=ops.DecayOut(self.offsets["g"], self.eps, self.norm, self.gate_silu, ctx.dtype))
         return linear(ctx, y, self.w_o, out_dtype=torch.float32, allow_partial=self.partial_out, scratch=self.out_scratch)
 
 
