@@ -207,13 +207,13 @@ rotation_table_kernel(const float* __restrict__ freq, int half, const int* __res
 }
 
 __device__ __forceinline__ float gate_value(float g, int silu) { return silu ? silu_of(g) : 1.f / (1.f + expf(-g)); }
-__device__ __forceinline__ void two_terms(float x, bf16& hi, bf16& lo) {
-  hi = __float2bfloat16_rn(x);
-  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
-}
-__device__ __forceinline__ uint32_t pair_of(bf16 a, bf16 b) {
-  const __nv_bfloat162 v(a, b);
-  return *reinterpret_cast<const uint32_t*>(&v);
+// SiLU and sigmoid gates on the special-function unit, for results that are rounded to bfloat16.
+__device__ __forceinline__ float quick_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+__device__ __forceinline__ float quick_gate(float g, int silu) { return silu ? quick_silu(g) : __fdividef(1.f, 1.f + __expf(-g)); }
+// Two values as two bfloat16 terms each: hi = round(x), lo = round(x - hi).
+__device__ __forceinline__ void two_terms(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(a, b);
+  lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 __device__ __forceinline__ void unpack8(uint4 raw, float (&x)[8]) {
   const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
@@ -233,98 +233,130 @@ __device__ __forceinline__ uint32_t operand_offset(int row, int word, int block_
 __device__ __forceinline__ void put_terms(const float (&x)[8], uint8_t* hi, uint8_t* lo, uint32_t at) {
   uint32_t h[4], l[4];
 #pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    bf16 h0, l0, h1, l1;
-    two_terms(x[2 * e], h0, l0);
-    two_terms(x[2 * e + 1], h1, l1);
-    h[e] = pair_of(h0, h1);
-    l[e] = pair_of(l0, l1);
-  }
+  for (int e = 0; e < 4; ++e) two_terms(x[2 * e], x[2 * e + 1], h[e], l[e]);
   *reinterpret_cast<uint4*>(hi + at) = make_uint4(h[0], h[1], h[2], h[3]);
   if (lo != nullptr) *reinterpret_cast<uint4*>(lo + at) = make_uint4(l[0], l[1], l[2], l[3]);
 }
 
 // A chunk's rows of one head's queries or keys (columns col0 .. col0 + dk - 1 of the projection) as one or two (lo not
-// null) bfloat16 terms, zeros beyond row n and column dk up to `padded` elements. Times `scale`, and if WEIGHTED
-// times decay^(n - 1 - row).
-template <bool WEIGHTED>
-__device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int dk, int padded,
+// null) bfloat16 terms in `blocks` blocks of 64 elements, zeros beyond row n and column dk. Times `scale`, and if
+// WEIGHTED times decay^(n - 1 - row). ROTATED: with a rotation (no activation), else perhaps with SiLU. The loads of
+// BATCH words of a thread are in flight together.
+template <bool WEIGHTED, bool ROTATED>
+__device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int dk, int blocks,
                                            int silu, const float2* __restrict__ turns, int rot_half, float scale, float log2_decay,
                                            uint8_t* hi, uint8_t* lo) {
-  const int words = padded / 8;
-  const bool wide = dk % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0 && rot_half % 8 == 0;
-  for (int i = threadIdx.x; i < CHUNK * words; i += CHUNK_THREADS) {
-    const int r = i / words, word = i - r * words, e0 = word * 8;
-    float x[8];
+  constexpr int BATCH = ROTATED ? 2 : 4;
+  const int shift = blocks == 1 ? 3 : 4, total = CHUNK << shift;        // words of a row: 8 or 16
+  const bool wide = dk % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0 && (!ROTATED || rot_half % 8 == 0);
+  for (int i0 = threadIdx.x; i0 < total; i0 += BATCH * CHUNK_THREADS) {
+    uint4 raw[BATCH], other[ROTATED ? BATCH : 1];
+    float4 cs[ROTATED ? BATCH : 1][4];
+    if (wide) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) x[e] = 0.f;
-    if (r < n && e0 < dk) {
-      const bf16* src = proj + (start + r) * stride + col0;
-      if (wide) {
-        unpack8(*reinterpret_cast<const uint4*>(src + e0), x);
-        if (silu) {
+      for (int b = 0; b < BATCH; ++b) {
+        const int i = i0 + b * CHUNK_THREADS, r = i >> shift, e0 = (i & ((1 << shift) - 1)) * 8;
+        raw[b] = make_uint4(0, 0, 0, 0);
+        if (r < n && e0 < dk) {                        // (n <= CHUNK: words beyond the total are left out too)
+          const bf16* src = proj + (start + r) * stride + col0;
+          raw[b] = *reinterpret_cast<const uint4*>(src + e0);
+          if (ROTATED && e0 < 2 * rot_half) {
+            const bool low = e0 < rot_half;
+            other[ROTATED ? b : 0] = *reinterpret_cast<const uint4*>(src + (low ? e0 + rot_half : e0 - rot_half));
+            const float4* t = reinterpret_cast<const float4*>(turns + (start + r) * rot_half + (low ? e0 : e0 - rot_half));
 #pragma unroll
-          for (int e = 0; e < 8; ++e) x[e] = rounded_to<bf16>(silu_of(x[e]));
-        }
-        if (e0 < 2 * rot_half) {
-          const bool low = e0 < rot_half;
-          float y[8];
-          unpack8(*reinterpret_cast<const uint4*>(src + (low ? e0 + rot_half : e0 - rot_half)), y);
-          const float4* cs = reinterpret_cast<const float4*>(turns + (start + r) * rot_half + (low ? e0 : e0 - rot_half));
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float4 a = cs[e];
-            x[2 * e] = x[2 * e] * a.x + y[2 * e] * (low ? -a.y : a.y);
-            x[2 * e + 1] = x[2 * e + 1] * a.z + y[2 * e + 1] * (low ? -a.w : a.w);
+            for (int e = 0; e < 4; ++e) cs[ROTATED ? b : 0][e] = t[e];
           }
-        }
-      } else {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const int j = e0 + e;
-          if (j >= dk) continue;
-          float v = to_f32(src[j]);
-          if (silu) v = rounded_to<bf16>(silu_of(v));
-          if (j < 2 * rot_half) {
-            const bool low = j < rot_half;
-            const float2 a = turns[(start + r) * rot_half + (low ? j : j - rot_half)];
-            v = v * a.x + to_f32(src[low ? j + rot_half : j - rot_half]) * (low ? -a.y : a.y);
-          }
-          x[e] = v;
         }
       }
-      const float by = WEIGHTED ? scale * exp2f(log2_decay * (float)(n - 1 - r)) : scale;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] *= by;
     }
-    put_terms(x, hi, lo, operand_offset(r, word, BLOCK_BYTES));
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b) {
+      const int i = i0 + b * CHUNK_THREADS, r = i >> shift, word = i & ((1 << shift) - 1), e0 = word * 8;
+      if (i >= total) continue;
+      float x[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = 0.f;
+      if (r < n && e0 < dk) {
+        if (wide) {
+          unpack8(raw[b], x);
+          if (!ROTATED && silu) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] = rounded_to<bf16>(quick_silu(x[e]));
+          }
+          if (ROTATED && e0 < 2 * rot_half) {
+            const bool low = e0 < rot_half;
+            float y[8];
+            unpack8(other[ROTATED ? b : 0], y);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float4 a = cs[ROTATED ? b : 0][e];
+              x[2 * e] = x[2 * e] * a.x + y[2 * e] * (low ? -a.y : a.y);
+              x[2 * e + 1] = x[2 * e + 1] * a.z + y[2 * e + 1] * (low ? -a.w : a.w);
+            }
+          }
+        } else {
+          const bf16* src = proj + (start + r) * stride + col0;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const int j = e0 + e;
+            if (j >= dk) continue;
+            float v = to_f32(src[j]);
+            if (!ROTATED && silu) v = rounded_to<bf16>(quick_silu(v));
+            if (ROTATED && j < 2 * rot_half) {
+              const bool low = j < rot_half;
+              const float2 a = turns[(start + r) * rot_half + (low ? j : j - rot_half)];
+              v = v * a.x + to_f32(src[low ? j + rot_half : j - rot_half]) * (low ? -a.y : a.y);
+            }
+            x[e] = v;
+          }
+        }
+        const float by = WEIGHTED ? scale * exp2f(log2_decay * (float)(n - 1 - r)) : scale;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] *= by;
+      }
+      put_terms(x, hi, lo, operand_offset(r, word, BLOCK_BYTES));
+    }
   }
 }
 
-// A chunk's values, columns v0 .. v0 + padded - 1 of one head, zeros beyond row n and column dv.
+// A chunk's values, columns v0 .. of one head in `blocks` blocks of 64 elements, zeros beyond row n and column dv.
 __device__ __forceinline__ void stage_values(const bf16* __restrict__ proj, int64_t stride, int64_t start, int n, int col0, int v0, int dv,
-                                             int padded, int silu, uint8_t* vs) {
-  const int words = padded / 8;
+                                             int blocks, int silu, uint8_t* vs) {
+  constexpr int BATCH = 4;
+  const int shift = blocks == 1 ? 3 : 4, total = CHUNK << shift;
   const bool wide = dv % 8 == 0 && stride % 8 == 0 && col0 % 8 == 0;
-  for (int i = threadIdx.x; i < CHUNK * words; i += CHUNK_THREADS) {
-    const int r = i / words, word = i - r * words, e0 = word * 8;
-    uint4 raw = make_uint4(0, 0, 0, 0);
-    if (r < n && v0 + e0 < dv) {
-      const bf16* src = proj + (start + r) * stride + col0 + v0 + e0;
-      bf16* x = reinterpret_cast<bf16*>(&raw);
-      if (wide) {
-        raw = *reinterpret_cast<const uint4*>(src);
-      } else {
+  for (int i0 = threadIdx.x; i0 < total; i0 += BATCH * CHUNK_THREADS) {
+    uint4 raw[BATCH];
 #pragma unroll
-        for (int e = 0; e < 8; ++e)
-          if (v0 + e0 + e < dv) x[e] = src[e];
-      }
-      if (silu) {
+    for (int b = 0; b < BATCH; ++b) {
+      const int i = i0 + b * CHUNK_THREADS, r = i >> shift, e0 = (i & ((1 << shift) - 1)) * 8;
+      raw[b] = make_uint4(0, 0, 0, 0);
+      if (r < n && v0 + e0 < dv) {
+        const bf16* src = proj + (start + r) * stride + col0 + v0 + e0;
+        if (wide) {
+          raw[b] = *reinterpret_cast<const uint4*>(src);
+        } else {
+          bf16* x = reinterpret_cast<bf16*>(&raw[b]);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = __float2bfloat16_rn(silu_of(__bfloat162float(x[e])));
+          for (int e = 0; e < 8; ++e)
+            if (v0 + e0 + e < dv) x[e] = src[e];
+        }
       }
     }
-    *reinterpret_cast<uint4*>(vs + operand_offset(r, word, BLOCK_BYTES)) = raw;
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b) {
+      const int i = i0 + b * CHUNK_THREADS, r = i >> shift, word = i & ((1 << shift) - 1);
+      if (i >= total) continue;
+      if (silu) {
+        float x[8];
+        unpack8(raw[b], x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = quick_silu(x[e]);
+        raw[b] = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+      }
+      *reinterpret_cast<uint4*>(vs + operand_offset(r, word, BLOCK_BYTES)) = raw[b];
+    }
   }
 }
 
@@ -394,6 +426,7 @@ __device__ __forceinline__ void tensor_leave(uint32_t tmem, uint32_t cols, volat
 constexpr uint32_t STATE_TMEM = 128;
 
 // grid (chunks, heads, value tiles): U[dk, dv] = K^T V, the head's key channels on the MMA's M side (128, zeros beyond dk).
+template <bool ROTATED>
 __global__ void __launch_bounds__(CHUNK_THREADS, 2)
 decay_chunk_state_kernel(const Projection p, const Recurrence c, const Chunks k, unsigned* status) {
   extern __shared__ uint8_t chunk_raw[];
@@ -414,8 +447,8 @@ decay_chunk_state_kernel(const Projection p, const Recurrence c, const Chunks k,
   tensor_setup(done, &tmem_holder, &abort_flag, STATE_TMEM);
   const uint32_t tmem = tmem_holder;
   const bf16* proj = reinterpret_cast<const bf16*>(p.data);
-  stage_rows<true>(proj, p.stride, start, n, p.off_k + h * dk, dk, 128, c.silu, k.turns, c.rot_half, c.key_scale, c.log2_decay[h], kh, kl);
-  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, 64 * vblocks, c.silu, vs);
+  stage_rows<true, ROTATED>(proj, p.stride, start, n, p.off_k + h * dk, dk, 2, c.silu, k.turns, c.rot_half, c.key_scale, c.log2_decay[h], kh, kl);
+  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, vblocks, c.silu, vs);
   operands_ready();
   if (threadIdx.x == 0) {
     const uint32_t idesc = instr_both_mn(64 * vblocks);
@@ -536,8 +569,8 @@ decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, f
   const uint32_t tmem = tmem_holder;
   const bf16* proj = reinterpret_cast<const bf16*>(p.data);
   const float l2d = c.log2_decay[h];
-  stage_rows<false>(proj, p.stride, start, n, p.off_q + h * dk, dk, 64 * kblocks, c.silu, k.turns, c.rot_half, 1.f, 0.f, qh, LO ? ql : nullptr);
-  stage_rows<false>(proj, p.stride, start, n, p.off_k + h * dk, dk, 64 * kblocks, c.silu, k.turns, c.rot_half, c.key_scale, 0.f, kh, LO ? kl : nullptr);
+  stage_rows<false, LO>(proj, p.stride, start, n, p.off_q + h * dk, dk, kblocks, c.silu, k.turns, c.rot_half, 1.f, 0.f, qh, LO ? ql : nullptr);
+  stage_rows<false, LO>(proj, p.stride, start, n, p.off_k + h * dk, dk, kblocks, c.silu, k.turns, c.rot_half, c.key_scale, 0.f, kh, LO ? kl : nullptr);
   operands_ready();
   if (threadIdx.x == 0) {
     const uint32_t idesc = umma_instr_desc(CHUNK, CHUNK, false);
@@ -553,34 +586,42 @@ decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, f
   // the state before the chunk and the values, while the scores are made
   {
     const float* S = k.states + ((int64_t)chunk * c.heads + h) * dk * dv + v0;
-    const int words = 8 * vblocks, rows = 64 * kblocks;
+    constexpr int BATCH = 4;
+    const int shift = vblocks == 1 ? 3 : 4, total = 64 * kblocks << shift;
     const bool wide = dv % 4 == 0;
-    for (int i = threadIdx.x; i < rows * words; i += CHUNK_THREADS) {
-      const int r = i / words, word = i - r * words, e0 = word * 8;
-      float x[8];
+    for (int i0 = threadIdx.x; i0 < total; i0 += BATCH * CHUNK_THREADS) {
+      float x[BATCH][8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] = 0.f;
-      if (r < dk) {
-        const float* src = S + (int64_t)r * dv + e0;
-        if (wide) {
-          if (v0 + e0 < dv) {
-            const float4 a = *reinterpret_cast<const float4*>(src);
-            x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w;
-          }
-          if (v0 + e0 + 4 < dv) {
-            const float4 a = *reinterpret_cast<const float4*>(src + 4);
-            x[4] = a.x; x[5] = a.y; x[6] = a.z; x[7] = a.w;
-          }
-        } else {
+      for (int b = 0; b < BATCH; ++b) {
+        const int i = i0 + b * CHUNK_THREADS, r = i >> shift, e0 = (i & ((1 << shift) - 1)) * 8;
 #pragma unroll
-          for (int e = 0; e < 8; ++e)
-            if (v0 + e0 + e < dv) x[e] = src[e];
+        for (int e = 0; e < 8; ++e) x[b][e] = 0.f;
+        if (r < dk) {                                  // (dk <= 64 * kblocks: words beyond the total are left out too)
+          const float* src = S + (int64_t)r * dv + e0;
+          if (wide) {
+            if (v0 + e0 < dv) {
+              const float4 a = *reinterpret_cast<const float4*>(src);
+              x[b][0] = a.x; x[b][1] = a.y; x[b][2] = a.z; x[b][3] = a.w;
+            }
+            if (v0 + e0 + 4 < dv) {
+              const float4 a = *reinterpret_cast<const float4*>(src + 4);
+              x[b][4] = a.x; x[b][5] = a.y; x[b][6] = a.z; x[b][7] = a.w;
+            }
+          } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+              if (v0 + e0 + e < dv) x[b][e] = src[e];
+          }
         }
       }
-      put_terms(x, sh, sl, operand_offset(r, word, s_block));
+#pragma unroll
+      for (int b = 0; b < BATCH; ++b) {
+        const int i = i0 + b * CHUNK_THREADS;
+        if (i < total) put_terms(x[b], sh, sl, operand_offset(i >> shift, i & ((1 << shift) - 1), s_block));
+      }
     }
   }
-  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, 64 * vblocks, c.silu, vs);
+  stage_values(proj, p.stride, start, n, p.off_v + h * dv, v0, dv, vblocks, c.silu, vs);
   operands_ready();
   const uint32_t idesc_v = umma_instr_desc(CHUNK, 64 * vblocks, true);
   if (threadIdx.x == 0) {
@@ -606,7 +647,7 @@ decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, f
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         const int back = row - (c0 + 8 * w + e);
-        x[e] = back >= 0 ? __uint_as_float(r[8 * w + e]) * exp2f(l2d * (float)back) : 0.f;
+        x[e] = back >= 0 ? __uint_as_float(r[8 * w + e]) * fast_exp2(l2d * (float)back) : 0.f;
       }
       put_terms(x, ph, pl, operand_offset(row, c0 / 8 + w, BLOCK_BYTES));
     }
@@ -664,13 +705,13 @@ decay_chunk_out_kernel(const Projection p, const Recurrence c, const Chunks k, f
             uint32_t v[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e)
-              v[e] = pack_bf16(o[8 * w + 2 * e] * inv * gate_value(g[2 * e], fin.gate_silu), o[8 * w + 2 * e + 1] * inv * gate_value(g[2 * e + 1], fin.gate_silu));
+              v[e] = pack_bf16(o[8 * w + 2 * e] * inv * quick_gate(g[2 * e], fin.gate_silu), o[8 * w + 2 * e + 1] * inv * quick_gate(g[2 * e + 1], fin.gate_silu));
             *reinterpret_cast<uint4*>(dst + 8 * w) = make_uint4(v[0], v[1], v[2], v[3]);
           }
         } else {
 #pragma unroll
           for (int e = 0; e < 8; ++e)
-            if (c0 + 8 * w + e < dv) dst[8 * w + e] = __float2bfloat16_rn(o[8 * w + e] * inv * gate_value(to_f32(proj[at + 8 * w + e]), fin.gate_silu));
+            if (c0 + 8 * w + e < dv) dst[8 * w + e] = __float2bfloat16_rn(o[8 * w + e] * inv * quick_gate(to_f32(proj[at + 8 * w + e]), fin.gate_silu));
         }
       }
     }
@@ -888,13 +929,15 @@ VOSTI_API int vosti_decay_chunks(const void* proj, int64_t stride, int tokens, i
   const HeadOut fin = {(bf16*)y, eps, gate_silu};
   static bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(decay_chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)state_smem(VT));
+    cudaFuncSetAttribute(decay_chunk_state_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)state_smem(VT));
+    cudaFuncSetAttribute(decay_chunk_state_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)state_smem(VT));
     cudaFuncSetAttribute(decay_chunk_out_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem(CHUNK_MAX_DK, VT, true));
     cudaFuncSetAttribute(decay_chunk_out_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out_smem(CHUNK_MAX_DK, VT, false));
     configured = true;
   }
   const dim3 grid(chunks, heads, (dv + VT - 1) / VT);
-  vosti_launch(decay_chunk_state_kernel, grid, dim3(CHUNK_THREADS), state_smem(dv), stream, p, c, k, status);
+  if (rot_half > 0) vosti_launch(decay_chunk_state_kernel<true>, grid, dim3(CHUNK_THREADS), state_smem(dv), stream, p, c, k, status);
+  else vosti_launch(decay_chunk_state_kernel<false>, grid, dim3(CHUNK_THREADS), state_smem(dv), stream, p, c, k, status);
   const int64_t size = (int64_t)dk * dv;
   if (size % 4 == 0)
     vosti_launch(decay_chunk_scan_kernel<4>, dim3((unsigned)((size / 4 + 255) / 256), heads, requests), dim3(256), 0, stream, c, long_requests, long_chunk0, states);

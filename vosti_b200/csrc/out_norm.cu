@@ -160,11 +160,18 @@ out_norm_stream_kernel(const OutNorm a, TO* __restrict__ out, unsigned* status) 
     const float inv1 = 1.f / sqrtf(block_sum(ss[1], scratch) / (float)width + a.branch_eps);
     float sum = 0.f;
     for (int i = first; i < width; i += step) {
-#pragma unroll
-      for (int e = 0; e < V; ++e) {
-        const float y = 0.5f * (rows_smem[i + e] * inv0 * load_flex(a.branch_w[0], a.branch_f32, i + e) +
-                                rows_smem[width + i + e] * inv1 * load_flex(a.branch_w[1], a.branch_f32, i + e));
-        rows_smem[i + e] = y;
+      if (V == 4) {
+        const float4 w0 = flex4(a.branch_w[0], a.branch_f32, i), w1 = flex4(a.branch_w[1], a.branch_f32, i);
+        float4 y = *reinterpret_cast<const float4*>(rows_smem + i);
+        const float4 z = *reinterpret_cast<const float4*>(rows_smem + width + i);
+        y = make_float4(0.5f * (y.x * inv0 * w0.x + z.x * inv1 * w1.x), 0.5f * (y.y * inv0 * w0.y + z.y * inv1 * w1.y),
+                        0.5f * (y.z * inv0 * w0.z + z.z * inv1 * w1.z), 0.5f * (y.w * inv0 * w0.w + z.w * inv1 * w1.w));
+        *reinterpret_cast<float4*>(rows_smem + i) = y;
+        sum += dot4(y);
+      } else {
+        const float y = 0.5f * (rows_smem[i] * inv0 * load_flex(a.branch_w[0], a.branch_f32, i) +
+                                rows_smem[width + i] * inv1 * load_flex(a.branch_w[1], a.branch_f32, i));
+        rows_smem[i] = y;
         sum += y * y;
       }
     }
@@ -243,9 +250,10 @@ VOSTI_API int vosti_out_norm_stream(const void* const* ys, const int* y_f32, con
   a.w = w; a.w_f32 = w_f32; a.offset = offset; a.eps = eps;
   a.scale = scale; a.scale_f32 = scale_f32;
   a.width = width;
-  // few rows: a thread a 16-byte word, so that a row's loads are all in flight at once
-  int threads = 256;
-  if (rows <= 64) threads = width / 4 >= 1024 ? 1024 : ((width / 4 + 31) / 32 * 32 > 128 ? (width / 4 + 31) / 32 * 32 : 128);
+  // few rows: a thread a 16-byte word, so that a row's loads are all in flight at once; many: four words, and small
+  // blocks, of which an SM holds more (measured at widths of 2,048 and 4,096)
+  const int wanted = (width / (rows <= 64 ? 4 : 16) + 31) / 32 * 32, most = rows <= 64 ? 1024 : 256;
+  const int threads = wanted > most ? most : wanted < 128 ? 128 : wanted;
   cudaError_t e;
   if (width % 4 == 0) e = launch_out_norm<bf16, 4>(a, out, rows, threads, smem, status, stream_id);
   else e = launch_out_norm<bf16, 1>(a, out, rows, threads, smem, status, stream_id);

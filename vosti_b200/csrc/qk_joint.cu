@@ -158,8 +158,9 @@ VOSTI_API int vosti_qk_joint(const void* proj, int proj_f32, int splits, int64_t
   const bool words = dk % 4 == 0 && stride % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
                      (bias == nullptr || (reinterpret_cast<uintptr_t>(bias) & 15) == 0) && (reinterpret_cast<uintptr_t>(q_norm) & 15) == 0 &&
                      (reinterpret_cast<uintptr_t>(k_norm) & 15) == 0;
-  int threads = 256;
-  if (tokens <= 64) threads = wide / 4 >= 1024 ? 1024 : ((wide / 4 + 31) / 32 * 32 > 128 ? (wide / 4 + 31) / 32 * 32 : 128);
+  // few tokens: a thread a 16-byte word; many: small blocks, of which an SM holds more
+  const int wanted = (wide / 4 + 31) / 32 * 32, most = tokens <= 64 ? 1024 : 128;
+  const int threads = wanted > most ? most : wanted < 128 ? 128 : wanted;
   cudaError_t e;
 #define VOSTI_JOINT_ARGS a, q_out, k_cache, v_cache, tokens, threads, smem, status, stream
   if (is_f32) e = words ? launch_qk_joint<float, 4>(VOSTI_JOINT_ARGS) : launch_qk_joint<float, 1>(VOSTI_JOINT_ARGS);

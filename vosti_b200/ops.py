@@ -1768,7 +1768,7 @@ def decay_attention(proj, offsets: dict, state: torch.Tensor, ctx, *, heads: int
     if chunked:
         turns = None
         if half:
-            # one table of angles a step and set of frequencies, shared by the layers that rotate alike
+            # one table of angles a step and layer, shared by the layer's runs
             key = ("rotation_table", freq.data_ptr())
             turns = ctx.extras.get(key)
             if turns is None:
